@@ -6,15 +6,22 @@
 // work in the latent space (the up-projections are absorbed into the query and applied to the output by the
 // caller, as per-head products):
 //   score(t, s, h) = (q_lat[h, t] . c_s + q_rot[t, h] . k_rot_s) * scale          q_lat = W_uk[h]^T q_nope
-//   p = exp(score - m) / (sum_s exp(score - m) + exp(sink_h - m))                  causal: s <= t
+//   p = exp(score - m) / (sum_s exp(score - m) + exp(sink_h - m))                  causal: s <= t; with a window: t - s < window
 //   out_lat[h, t] = sum_s p_s c_s                                                  (value = W_uv[h] out_lat)
 //
 // latent_kv_prep   from the projected row [dq (q_rank) | dkv (rank) | k_rot (dr)]: weighted RMS norms of the two
 //                  latents, the rotation of k_rot, and the page write, in one kernel.
 // latent_q_prep    from the projected queries [H, dn + dr]: the unrotated parts head-major (for the per-head
 //                  products) and the rotated parts, rotated.
-// Rotation: pairs (2i, 2i+1), i < dims/2, by the angle position * inv_freq[i] in 32-bit; entries from `dims` on pass.
+// Rotation: pairs (2i, 2i+1), or with `halves` (i, i + dims/2), i < dims/2, by the angle position * inv_freq[i] in 32-bit;
+// entries from `dims` on pass.
 #include "common.cuh"
+
+// The two entries that rotate together as pair i.
+__device__ __forceinline__ void rot_pair(int i, int rot_dims, int halves, int* a, int* b) {
+  *a = halves ? i : 2 * i;
+  *b = halves ? i + (rot_dims >> 1) : 2 * i + 1;
+}
 
 __device__ __forceinline__ float row_sum_splits(const float* p, int splits, long long stride) {
   float s = 0.f;
@@ -28,14 +35,13 @@ __global__ void latent_kv_prep_kernel(const float* __restrict__ proj, int splits
                                       const float* __restrict__ inv_freq, int rot_dims, TO* __restrict__ cq, TO* __restrict__ pages,
                                       const int* __restrict__ block_table, int bt_stride, const int* __restrict__ req_of_token,
                                       const int* __restrict__ positions, int q_rank, int rank, int dr, int page_size,
-                                      int num_pages, int* status) {
+                                      int num_pages, int ld, int halves, int* status) {
   JLX_TL(TL_ROPE);
   pdl_launch_dependents_if_small();
   pdl_wait();
   __shared__ float scratch[33];
   const int n = blockIdx.x;
-  const int C = q_rank + rank + dr;
-  const float* row = proj + (size_t)n * C;
+  const float* row = proj + (size_t)n * ld;
   // the query's latent
   float ss = 0.f;
   for (int i = threadIdx.x; i < q_rank; i += blockDim.x) {
@@ -67,9 +73,11 @@ __global__ void latent_kv_prep_kernel(const float* __restrict__ proj, int splits
   for (int i = threadIdx.x; i < rot_dims / 2; i += blockDim.x) {
     float sn, cs;
     sincosf((float)p * inv_freq[i], &sn, &cs);
-    const float u = row_sum_splits(kr + 2 * i, splits, split_stride), v = row_sum_splits(kr + 2 * i + 1, splits, split_stride);
-    dst[rank + 2 * i] = from_f32<TO>(u * cs - v * sn);
-    dst[rank + 2 * i + 1] = from_f32<TO>(v * cs + u * sn);
+    int ia, ib;
+    rot_pair(i, rot_dims, halves, &ia, &ib);
+    const float u = row_sum_splits(kr + ia, splits, split_stride), v = row_sum_splits(kr + ib, splits, split_stride);
+    dst[rank + ia] = from_f32<TO>(u * cs - v * sn);
+    dst[rank + ib] = from_f32<TO>(v * cs + u * sn);
   }
   for (int i = rot_dims + threadIdx.x; i < dr; i += blockDim.x) dst[rank + i] = from_f32<TO>(row_sum_splits(kr + i, splits, split_stride));
 }
@@ -77,16 +85,17 @@ __global__ void latent_kv_prep_kernel(const float* __restrict__ proj, int splits
 JLX_API int jlx_latent_kv_prep(const float* proj, int splits, long long split_stride, const float* q_norm_w,
                                const float* kv_norm_w, float eps, const float* inv_freq, int rot_dims, void* cq, void* pages,
                                int dtype, const int* block_table, int bt_stride, const int* req_of_token, const int* positions,
-                               int N, int q_rank, int rank, int dr, int page_size, int num_pages, int* status,
-                               cudaStream_t stream) {
+                               int N, int q_rank, int rank, int dr, int page_size, int num_pages, int ld, int halves,
+                               int* status, cudaStream_t stream) {
   JLX_REQUIRE(N >= 0 && q_rank > 0 && rank > 0 && dr >= 0 && splits >= 1, "latent_kv_prep: bad sizes");
   JLX_REQUIRE(rot_dims >= 0 && rot_dims <= dr && rot_dims % 2 == 0, "latent_kv_prep: %d rotated entries of %d", rot_dims, dr);
   JLX_REQUIRE(eps > 0.f, "latent_kv_prep: eps must be positive");
+  JLX_REQUIRE(ld >= q_rank + rank + dr, "latent_kv_prep: rows of %d entries do not hold %d + %d + %d", ld, q_rank, rank, dr);
   if (N == 0) return 0;
   JLX_DISPATCH_DTYPE(dtype, TO, {
     JLX_CUDA(jlx_launch_pdl(latent_kv_prep_kernel<TO>, dim3(N), dim3(128), 0, stream, proj, splits, split_stride, q_norm_w, kv_norm_w,
                             eps, inv_freq, rot_dims, (TO*)cq, (TO*)pages, block_table, bt_stride, req_of_token, positions, q_rank,
-                            rank, dr, page_size, num_pages, status));
+                            rank, dr, page_size, num_pages, ld, halves, status));
   });
   JLX_LAUNCH_CHECK("latent_kv_prep");
   return 0;
@@ -98,7 +107,7 @@ template <typename TO>
 __global__ void latent_q_prep_kernel(const float* __restrict__ q, int splits, long long split_stride,
                                      const float* __restrict__ inv_freq, int rot_dims, const int* __restrict__ positions,
                                      TO* __restrict__ q_nope, float* __restrict__ q_rot, TO* __restrict__ q_full, int N, int H,
-                                     int dn, int dr) {
+                                     int dn, int dr, int halves) {
   JLX_TL(TL_ROPE);
   pdl_launch_dependents_if_small();
   pdl_wait();
@@ -116,11 +125,13 @@ __global__ void latent_q_prep_kernel(const float* __restrict__ q, int splits, lo
   for (int i = threadIdx.x; i < rot_dims / 2; i += blockDim.x) {
     float sn, cs;
     sincosf((float)p * inv_freq[i], &sn, &cs);
-    const float u = row_sum_splits(qr + 2 * i, splits, split_stride), v = row_sum_splits(qr + 2 * i + 1, splits, split_stride);
+    int ia, ib;
+    rot_pair(i, rot_dims, halves, &ia, &ib);
+    const float u = row_sum_splits(qr + ia, splits, split_stride), v = row_sum_splits(qr + ib, splits, split_stride);
     const float a = u * cs - v * sn, b = v * cs + u * sn;
-    dst[2 * i] = a;
-    dst[2 * i + 1] = b;
-    if (full) { full[dn + 2 * i] = from_f32<TO>(a); full[dn + 2 * i + 1] = from_f32<TO>(b); }
+    dst[ia] = a;
+    dst[ib] = b;
+    if (full) { full[dn + ia] = from_f32<TO>(a); full[dn + ib] = from_f32<TO>(b); }
   }
   for (int i = rot_dims + threadIdx.x; i < dr; i += blockDim.x) {
     const float v = row_sum_splits(qr + i, splits, split_stride);
@@ -131,14 +142,14 @@ __global__ void latent_q_prep_kernel(const float* __restrict__ q, int splits, lo
 
 JLX_API int jlx_latent_q_prep(const float* q, int splits, long long split_stride, const float* inv_freq, int rot_dims,
                               const int* positions, void* q_nope, int dtype, float* q_rot, void* q_full, int N, int H, int dn,
-                              int dr, cudaStream_t stream) {
+                              int dr, int halves, cudaStream_t stream) {
   JLX_REQUIRE(N >= 0 && H > 0 && dn > 0 && dr >= 0 && splits >= 1, "latent_q_prep: bad sizes");
   JLX_REQUIRE(rot_dims >= 0 && rot_dims <= dr && rot_dims % 2 == 0, "latent_q_prep: %d rotated entries of %d", rot_dims, dr);
   JLX_REQUIRE(H <= 65535, "latent_q_prep: too many heads (%d)", H);
   if (N == 0) return 0;
   JLX_DISPATCH_DTYPE(dtype, TO, {
     JLX_CUDA(jlx_launch_pdl(latent_q_prep_kernel<TO>, dim3(N, H), dim3(64), 0, stream, q, splits, split_stride, inv_freq, rot_dims,
-                            positions, (TO*)q_nope, q_rot, (TO*)q_full, N, H, dn, dr));
+                            positions, (TO*)q_nope, q_rot, (TO*)q_full, N, H, dn, dr, halves));
   });
   JLX_LAUNCH_CHECK("latent_q_prep");
   return 0;
@@ -150,9 +161,11 @@ JLX_API int jlx_latent_q_prep(const float* q, int splits, long long split_stride
 // products.  All heads share each tile of keys.  Key tiles are aligned to absolute positions (0, 32, 64, ...), so the
 // order of a position's sums depends on the position alone.  The sink opens the running maximum and denominator:
 // m = sink, l = exp(sink - m) = 1.
+// With a window the walk starts at the tile that holds the first visible key; earlier keys of that tile (whose pages may
+// have been given back) are read as zeros and masked.
 // With `rows` the block serves token rows[blockIdx.x] (the single decoded tokens of a step that also holds prompt
-// portions).  With splits > 1 block z takes the keys [z * split_keys, (z + 1) * split_keys) (a multiple of the tile, so
-// tiles stay aligned) and leaves (m, l, unnormalised sums) for the combine kernel; the sink opens split 0.
+// portions).  With splits > 1 block z takes the keys [(s0 + z) split_keys, (s0 + z + 1) split_keys), s0 the first visible key's range (a multiple of
+// the tile, so tiles stay aligned), and leaves (m, l, unnormalised sums) for the combine kernel; the sink opens split 0.
 #define LAT_TILE 32
 #define LAT_WARPS 8
 #define LAT_MAX_R32 32  // latent size up to 1024
@@ -164,7 +177,7 @@ __global__ void attention_latent_kernel(const float* __restrict__ q_lat, const f
                                         const float* __restrict__ sink, TO* __restrict__ out_lat, int N, int H, int rank,
                                         int dr, int page_size, int num_pages, float scale, const int* __restrict__ rows,
                                         int splits, int split_keys, float* __restrict__ part_acc, float* __restrict__ part_ml,
-                                        int ldk, int* status) {
+                                        int ldk, int window, int* status) {
   JLX_TL(TL_ATTN_GENERIC);
   pdl_launch_dependents_if_small();
   pdl_wait();
@@ -194,8 +207,13 @@ __global__ void attention_latent_kernel(const float* __restrict__ q_lat, const f
     for (int i = 0; i < R32; ++i) acc[u][i] = 0.f;
   }
   const int nd = (rank + 31) >> 5;
-  const int t_begin = splits > 1 ? z * split_keys : 0;
-  const int t_end = splits > 1 ? min(p, (z + 1) * split_keys - 1) : p;  // last key of this block
+  const int lo = window > 0 ? max(0, p - window + 1) : 0;  // the first visible key
+  int t_begin = lo / LAT_TILE * LAT_TILE, t_end = p;         // first tile and last key of this block
+  if (splits > 1) {
+    const int range = (lo / split_keys + z) * split_keys;
+    t_begin = max(t_begin, range);
+    t_end = min(p, range + split_keys - 1);
+  }
 
   // 16-byte loads of the cached rows where their size and the pool's address allow
   constexpr int VEC = 16 / (int)sizeof(TC);
@@ -207,8 +225,8 @@ __global__ void attention_latent_kernel(const float* __restrict__ q_lat, const f
     const int cnt = min(LAT_TILE, t_end - t0 + 1);
     if (threadIdx.x < cnt) {  // where the tile's rows lie
       const int pos = t0 + threadIdx.x;
-      int page = block_table[(size_t)r * bt_stride + pos / page_size];
-      if (page < 0 || page >= num_pages) { bad_page = true; page = -1; }
+      int page = pos >= lo ? block_table[(size_t)r * bt_stride + pos / page_size] : -1;
+      if (pos >= lo && (page < 0 || page >= num_pages)) { bad_page = true; page = -1; }
       row_at[threadIdx.x] = page < 0 ? -1 : (long long)page * page_size + pos % page_size;
     }
     __syncthreads();
@@ -236,7 +254,8 @@ __global__ void attention_latent_kernel(const float* __restrict__ q_lat, const f
     float sc[HPW];
 #pragma unroll
     for (int u = 0; u < HPW; ++u) sc[u] = -INFINITY;
-    if (lane < cnt) {
+    const bool seen = lane < cnt && t0 + lane >= lo;
+    if (seen) {
       float dot[HPW];
 #pragma unroll
       for (int u = 0; u < HPW; ++u) dot[u] = 0.f;
@@ -269,7 +288,7 @@ __global__ void attention_latent_kernel(const float* __restrict__ q_lat, const f
     for (int u = 0; u < HPW; ++u) {
       const float m_new = fmaxf(m[u], warp_max(sc[u]));
       const float corr = expf(m[u] - m_new);  // without a sink m is -inf on the first tile: exp(-inf) = 0
-      pj[u] = lane < cnt ? expf(sc[u] - m_new) : 0.f;
+      pj[u] = seen ? expf(sc[u] - m_new) : 0.f;
       l[u] = l[u] * corr + warp_sum(pj[u]);
       m[u] = m_new;
 #pragma unroll
@@ -347,10 +366,10 @@ JLX_API int jlx_attention_latent(const float* q_lat, const float* q_rot, const v
                                  const int* block_table, int bt_stride, const int* req_of_token, const int* positions,
                                  const float* sink, void* out_lat, int out_dtype, int N, int H, int rank, int dr,
                                  int page_size, int num_pages, float scale, const int* rows, int n_rows, int splits,
-                                 int split_keys, float* part_acc, float* part_ml, int* status, cudaStream_t stream) {
+                                 int split_keys, float* part_acc, float* part_ml, int window, int* status, cudaStream_t stream) {
   JLX_REQUIRE(N >= 0 && H > 0 && rank > 0 && dr >= 0 && page_size > 0 && num_pages > 0, "attention_latent: bad sizes");
   JLX_REQUIRE(rank <= 32 * LAT_MAX_R32, "attention_latent: latent size %d is above the supported maximum %d", rank, 32 * LAT_MAX_R32);
-  JLX_REQUIRE(splits >= 1 && splits <= 65535, "attention_latent: bad split count %d", splits);
+  JLX_REQUIRE(splits >= 1 && splits <= 65535 && window >= 0, "attention_latent: bad split count %d or window %d", splits, window);
   JLX_REQUIRE(splits == 1 || (split_keys > 0 && split_keys % LAT_TILE == 0 && part_acc && part_ml),
               "attention_latent: splits need a key count that is a multiple of %d, and scratch", LAT_TILE);
   const int served = rows ? n_rows : N;
@@ -377,7 +396,7 @@ JLX_API int jlx_attention_latent(const float* q_lat, const float* q_rot, const v
     JLX_CUDA(jlx_launch_pdl(attention_latent_kernel<TC, TO, HPW, R32>, dim3(served, hb, splits), dim3(nwarp * 32), smem, stream, \
                             q_lat, q_rot, (const TC*)pages, block_table, bt_stride, req_of_token, positions, sink, (TO*)out_lat, \
                             N, H, rank, dr, page_size, num_pages, scale, rows, splits, split_keys, part_acc, part_ml, ldk,  \
-                            status));                                                                                      \
+                            window, status));                                                                                      \
   } while (0)
   JLX_DISPATCH_DTYPE(cache_dtype, TC, JLX_DISPATCH_DTYPE(out_dtype, TO, {
     if (big) LAT_GO(2, 32);
@@ -400,28 +419,30 @@ JLX_API int jlx_attention_latent(const float* q_lat, const float* q_rot, const v
 // from the library), around three kernels of this file: the request's cached rows gathered into two dense matrices,
 // the keys put together per head, and the softmax with its causal edge and its sink.
 
-// c[t, :] = cache row t's first `rank` entries, kr[t, :] = its last dr, t < L, for the request of block-table row r.
+// c[t, :] = the first `rank` entries of the cache row of position first + t, kr[t, :] = its last dr, t < L, for the
+// request of one block-table row.
 template <typename T>
 __global__ void latent_gather_kernel(const T* __restrict__ pages, const int* __restrict__ bt_row, T* __restrict__ c,
-                                     T* __restrict__ kr, int rank, int dr, int page_size, int num_pages, int* status) {
+                                     T* __restrict__ kr, int first, int rank, int dr, int page_size, int num_pages,
+                                     int* status) {
   JLX_TL(TL_OTHER);
-  const int t = blockIdx.x;
-  const int page = bt_row[t / page_size];
+  const int t = blockIdx.x, pos = first + t;
+  const int page = bt_row[pos / page_size];
   if (page < 0 || page >= num_pages) {
     if (threadIdx.x == 0) atomicOr(status, JLX_STATUS_BAD_PAGE);
     return;
   }
-  const T* src = pages + ((size_t)page * page_size + t % page_size) * (rank + dr);
+  const T* src = pages + ((size_t)page * page_size + pos % page_size) * (rank + dr);
   for (int i = threadIdx.x; i < rank; i += blockDim.x) c[(size_t)t * rank + i] = src[i];
   for (int i = threadIdx.x; i < dr; i += blockDim.x) kr[(size_t)t * dr + i] = src[rank + i];
 }
 
-JLX_API int jlx_latent_gather(const void* pages, int dtype, const int* bt_row, void* c, void* kr, int L, int rank, int dr,
+JLX_API int jlx_latent_gather(const void* pages, int dtype, const int* bt_row, void* c, void* kr, int first, int L, int rank, int dr,
                               int page_size, int num_pages, int* status, cudaStream_t stream) {
-  JLX_REQUIRE(L >= 0 && rank > 0 && dr >= 0 && page_size > 0, "latent_gather: bad sizes");
+  JLX_REQUIRE(L >= 0 && first >= 0 && rank > 0 && dr >= 0 && page_size > 0, "latent_gather: bad sizes");
   if (L == 0) return 0;
   JLX_DISPATCH_DTYPE(dtype, T, {
-    latent_gather_kernel<T><<<L, 128, 0, stream>>>((const T*)pages, bt_row, (T*)c, (T*)kr, rank, dr, page_size, num_pages, status);
+    latent_gather_kernel<T><<<L, 128, 0, stream>>>((const T*)pages, bt_row, (T*)c, (T*)kr, first, rank, dr, page_size, num_pages, status);
   });
   JLX_LAUNCH_CHECK("latent_gather");
   return 0;
@@ -450,38 +471,43 @@ JLX_API int jlx_latent_key_assemble(const void* kv_up, long long ld_up, const vo
   return 0;
 }
 
-// p[h, i, j] = exp(scale * s[h, i, j] - m) / (sum over visible j + exp(sink_h - m)) for j <= q_start + i, else 0.
+// p[h, i, j] = exp(scale * s[h, i, j] - m) / (sum over visible j + exp(sink_h - m)) for visible j, else 0.  Column j is the
+// key at position k_start + j, row i the query at q_start + i: it sees keys up to itself, with a window only the last
+// `window` of them.
 // s: float32 [H, T, L]; p: [H, T, L] in the activations' type.  One block per (query row, head); 32-bit throughout.
 // With `staged` the visible part of the row is read once into shared memory (L floats) and the three passes run there.
 template <typename TO>
 __global__ void causal_sink_softmax_kernel(const float* __restrict__ s, const float* __restrict__ sink, float scale,
-                                           int q_start, TO* __restrict__ p, int T, int L, int staged) {
+                                           int q_start, int k_start, int window, TO* __restrict__ p, int T, int L,
+                                           int staged) {
   JLX_TL(TL_OTHER);
   extern __shared__ __align__(16) float stage[];
   __shared__ float scratch[33];
   const int i = blockIdx.x, h = blockIdx.y;
   const float* row = s + ((size_t)h * T + i) * L;
   TO* out = p + ((size_t)h * T + i) * L;
-  const int visible = min(L, q_start + i + 1);
+  const int own = q_start + i - k_start;                             // the query's own column
+  const int visible = min(L, own + 1);                               // columns [first, visible) are seen
+  const int first = window > 0 ? max(0, own - window + 1) : 0;
   float m = sink ? sink[h] : -INFINITY;
   if (staged) {
     if ((L & 3) == 0) {  // rows start on 16-byte boundaries
-      for (int j = threadIdx.x * 4; j < visible; j += blockDim.x * 4) {
+      for (int j = (first & ~3) + threadIdx.x * 4; j < visible; j += blockDim.x * 4) {
         float4 v = *reinterpret_cast<const float4*>(row + j);
         v.x *= scale; v.y *= scale; v.z *= scale; v.w *= scale;
         *reinterpret_cast<float4*>(stage + j) = v;
-        m = fmaxf(m, v.x);
-        if (j + 1 < visible) m = fmaxf(m, v.y);
-        if (j + 2 < visible) m = fmaxf(m, v.z);
-        if (j + 3 < visible) m = fmaxf(m, v.w);
+        if (j >= first) m = fmaxf(m, v.x);
+        if (j + 1 >= first && j + 1 < visible) m = fmaxf(m, v.y);
+        if (j + 2 >= first && j + 2 < visible) m = fmaxf(m, v.z);
+        if (j + 3 >= first && j + 3 < visible) m = fmaxf(m, v.w);
       }
     } else {
-      for (int j = threadIdx.x; j < visible; j += blockDim.x) { stage[j] = row[j] * scale; m = fmaxf(m, stage[j]); }
+      for (int j = first + threadIdx.x; j < visible; j += blockDim.x) { stage[j] = row[j] * scale; m = fmaxf(m, stage[j]); }
     }
     row = stage;
     scale = 1.f;
   } else {
-    for (int j = threadIdx.x; j < visible; j += blockDim.x) m = fmaxf(m, row[j] * scale);
+    for (int j = first + threadIdx.x; j < visible; j += blockDim.x) m = fmaxf(m, row[j] * scale);
   }
   // the block's maximum: warp maxima, then every thread takes the largest
   m = warp_max(m);
@@ -491,43 +517,60 @@ __global__ void causal_sink_softmax_kernel(const float* __restrict__ s, const fl
   m = scratch[0];
   for (int w = 1; w < (blockDim.x >> 5); ++w) m = fmaxf(m, scratch[w]);
   float l = 0.f;
-  for (int j = threadIdx.x; j < visible; j += blockDim.x) l += expf(row[j] * scale - m);
+  for (int j = first + threadIdx.x; j < visible; j += blockDim.x) l += expf(row[j] * scale - m);
   l = block_sum(l, scratch) + (sink ? expf(sink[h] - m) : 0.f);
-  for (int j = threadIdx.x; j < L; j += blockDim.x) out[j] = from_f32<TO>(j < visible ? expf(row[j] * scale - m) / l : 0.f);
+  for (int j = threadIdx.x; j < L; j += blockDim.x) out[j] = from_f32<TO>(j >= first && j < visible ? expf(row[j] * scale - m) / l : 0.f);
 }
 
-JLX_API int jlx_causal_sink_softmax(const float* s, const float* sink, float scale, int q_start, void* p, int dtype, int H,
-                                    int T, int L, cudaStream_t stream) {
-  JLX_REQUIRE(H > 0 && T >= 0 && L > 0 && q_start >= 0 && H <= 65535, "causal_sink_softmax: bad sizes");
+JLX_API int jlx_causal_sink_softmax(const float* s, const float* sink, float scale, int q_start, int k_start, int window, void* p,
+                                    int dtype, int H, int T, int L, cudaStream_t stream) {
+  JLX_REQUIRE(H > 0 && T >= 0 && L > 0 && q_start >= 0 && k_start >= 0 && k_start <= q_start && window >= 0 && H <= 65535, "causal_sink_softmax: bad sizes");
   if (T == 0) return 0;
   const int staged = (size_t)L * 4 <= 160 * 1024;
   const size_t smem = staged ? (size_t)(L + 4) * 4 : 0;
   JLX_DISPATCH_DTYPE(dtype, TO, {
     if (smem > 48 * 1024)
       JLX_CUDA(cudaFuncSetAttribute(causal_sink_softmax_kernel<TO>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
-    causal_sink_softmax_kernel<TO><<<dim3(T, H), 256, smem, stream>>>(s, sink, scale, q_start, (TO*)p, T, L, staged);
+    causal_sink_softmax_kernel<TO><<<dim3(T, H), 256, smem, stream>>>(s, sink, scale, q_start, k_start, window, (TO*)p, T, L, staged);
   });
   JLX_LAUNCH_CHECK("causal_sink_softmax");
   return 0;
 }
 
-// [H, N, d] -> [N, H * d]: the per-head products' rows back into token rows.
+// [H, N, d] -> [N, H * d]: the per-head products' rows back into token rows, with `gate` (float32 rows, possibly split-K
+// partials) through a gate per token and head: out[n, h d + c] = sigmoid(gate[n, h]) * in[h, n, c].
+struct GateRowsView {
+  const float* p;
+  long long split_stride;
+  long long ld;
+  int splits;
+  int pad_;
+};
+
 template <typename T>
-__global__ void heads_to_rows_kernel(const T* __restrict__ in, T* __restrict__ out, int N, int H, int d) {
+__global__ void heads_to_rows_kernel(const T* __restrict__ in, T* __restrict__ out, int N, int H, int d, GateRowsView gate) {
   JLX_TL(TL_OTHER);
   pdl_launch_dependents_if_small();
   pdl_wait();
   const int n = blockIdx.x;
   for (int i = threadIdx.x; i < H * d; i += blockDim.x) {
     const int h = i / d, c = i - h * d;
-    out[(size_t)n * H * d + i] = in[((size_t)h * N + n) * d + c];
+    T v = in[((size_t)h * N + n) * d + c];
+    if (gate.p) {
+      const float s = row_sum_splits(gate.p + (size_t)n * gate.ld + h, gate.splits, gate.split_stride);
+      v = from_f32<T>(to_f32<T>(v) / (1.f + expf(-s)));
+    }
+    out[(size_t)n * H * d + i] = v;
   }
 }
 
-JLX_API int jlx_heads_to_rows(const void* in, void* out, int dtype, int N, int H, int d, cudaStream_t stream) {
+JLX_API int jlx_heads_to_rows(const void* in, void* out, int dtype, int N, int H, int d, const GateRowsView* gate, cudaStream_t stream) {
   JLX_REQUIRE(N >= 0 && H > 0 && d > 0, "heads_to_rows: bad sizes");
   if (N == 0) return 0;
-  JLX_DISPATCH_DTYPE(dtype, T, { JLX_CUDA(jlx_launch_pdl(heads_to_rows_kernel<T>, dim3(N), dim3(256), 0, stream, (const T*)in, (T*)out, N, H, d)); });
+  const GateRowsView none = {nullptr, 0, 0, 1, 0};
+  JLX_DISPATCH_DTYPE(dtype, T, {
+    JLX_CUDA(jlx_launch_pdl(heads_to_rows_kernel<T>, dim3(N), dim3(256), 0, stream, (const T*)in, (T*)out, N, H, d, gate ? *gate : none));
+  });
   JLX_LAUNCH_CHECK("heads_to_rows");
   return 0;
 }

@@ -24,6 +24,7 @@
 
 #include "common.cuh"
 #include "mbarrier.cuh"
+#include "softcap.cuh"
 
 #define KT 64            // keys per tile
 #define SPLIT_UNIT 64    // decode splits are multiples of this many keys (one tile), aligned to absolute positions
@@ -74,7 +75,8 @@ struct AttnParams {
   const int* positions;
   bf16* out;            // [N, Hq, DH]
   int Hq, Hkv, page_size, num_pages;
-  float scale_log2;     // dh^-0.5 * log2(e)
+  float scale_log2;     // the score scale * log2(e); with a cap: the score scale / cap
+  float cap_log2;       // cap * log2(e) for soft-capped scores cap * tanh(s / cap), 0: none
   int chunk, window;
   float attn_scale, floor_scale;
   int* status;
@@ -100,6 +102,12 @@ __device__ __forceinline__ int first_key(int p, int chunk, int window) {
   if (chunk > 0) s = p - p % chunk;
   if (window > 0) s = max(s, p - window + 1);
   return s;
+}
+
+// A raw product as a base-2 score: `sc` is scale_log2 times the query's temperature.
+__device__ __forceinline__ float scaled_score(const AttnParams& P, float raw, float sc) {
+  const float s = raw * sc;
+  return P.cap_log2 > 0.f ? P.cap_log2 * cap_tanh(s) : s;
 }
 
 __device__ __forceinline__ float temperature(int p, float attn_scale, float floor_scale) {
@@ -225,7 +233,7 @@ __global__ void __launch_bounds__(128) attention_decode_kernel(const AttnParams 
       for (int e = 0; e < 4; ++e) {
         const int key = tile_key + warp * 16 + nt * 8 + (lane & 3) * 2 + (e & 1);
         const bool ok = key >= lo && key <= p;
-        s[nt][e] = ok ? fmaf(-sl[e >> 1], (float)(p - key), s[nt][e] * sc) : NEG_BIG;
+        s[nt][e] = ok ? fmaf(-sl[e >> 1], (float)(p - key), scaled_score(P, s[nt][e], sc)) : NEG_BIG;
         mx[e >> 1] = fmaxf(mx[e >> 1], s[nt][e]);
       }
 #pragma unroll
@@ -442,7 +450,7 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map, const AttnP
       for (int e = 0; e < 4; ++e) {
         const int key = tile_key + warp * 16 + nt * 8 + (lane & 3) * 2 + (e & 1);
         const bool in = key >= lo && key <= p;
-        s[nt][e] = in ? fmaf(-sl[e >> 1], (float)(p - key), s[nt][e] * sc) : NEG_BIG;
+        s[nt][e] = in ? fmaf(-sl[e >> 1], (float)(p - key), scaled_score(P, s[nt][e], sc)) : NEG_BIG;
         mx[e >> 1] = fmaxf(mx[e >> 1], s[nt][e]);
       }
 #pragma unroll
@@ -668,7 +676,7 @@ __global__ void __launch_bounds__(256) attention_prefill_kernel(const AttnParams
         for (int e = 0; e < 4; ++e) {
           const int key = tile_key + nt * 8 + (lane & 3) * 2 + (e & 1);
           const bool ok = (e < 2) ? (row0 && key >= lo0 && key <= p0) : (row1 && key >= lo1 && key <= p1);
-          s[nt][e] = ok ? fmaf(-slope, (float)(((e < 2) ? p0 : p1) - key), s[nt][e] * ((e < 2) ? sc0 : sc1)) : NEG_BIG;
+          s[nt][e] = ok ? fmaf(-slope, (float)(((e < 2) ? p0 : p1) - key), scaled_score(P, s[nt][e], (e < 2) ? sc0 : sc1)) : NEG_BIG;
           mx[e >> 1] = fmaxf(mx[e >> 1], s[nt][e]);
         }
 #pragma unroll
@@ -852,7 +860,7 @@ attention_prefill_tma_kernel(const __grid_constant__ CUtensorMap map, const Attn
           bool in = true;
           const int key = tile_key + half * 32 + nt * 8 + (lane & 3) * 2 + (e & 1);
           if (need_mask) in = (e < 2) ? (row0 && key >= lo0 && key <= p0) : (row1 && key >= lo1 && key <= p1);
-          s[nt][e] = in ? fmaf(-slope, (float)(((e < 2) ? p0 : p1) - key), s[nt][e] * ((e < 2) ? sc0 : sc1)) : NEG_BIG;
+          s[nt][e] = in ? fmaf(-slope, (float)(((e < 2) ? p0 : p1) - key), scaled_score(P, s[nt][e], (e < 2) ? sc0 : sc1)) : NEG_BIG;
           mx[e >> 1] = fmaxf(mx[e >> 1], s[nt][e]);
         }
 #pragma unroll
@@ -922,15 +930,18 @@ attention_prefill_tma_kernel(const __grid_constant__ CUtensorMap map, const Attn
 static int fill_params(AttnParams& P, const void* q, const void* pages, const int* block_table, int bt_stride,
                        const int* req_of_token, const int* positions, void* out, int Hq, int Hkv, int dh, int page_size,
                        int num_pages, float scale, int chunk, int window, float attn_scale, float floor_scale, const float* sink, const float* slopes,
-                       int* status) {
+                       float softcap, int* status) {
   JLX_REQUIRE(Hq > 0 && Hkv > 0 && Hq % Hkv == 0, "attention: %d query heads are no multiple of %d KV heads", Hq, Hkv);
   JLX_REQUIRE(dh == 64 || dh == 128, "attention_mma: head size %d is not built (64 and 128 are); use the generic kernel", dh);
   JLX_REQUIRE(page_size > 0 && num_pages > 0 && bt_stride > 0, "attention: bad cache sizes");
+  JLX_REQUIRE(softcap >= 0.f, "attention: the score cap must be positive (0: none)");
   JLX_REQUIRE(attn_scale == 0.f || floor_scale > 0.f, "attention: floor_scale must be positive");
   JLX_REQUIRE(((uintptr_t)q & 15) == 0 && ((uintptr_t)pages & 15) == 0, "attention: q and pages must be 16-byte aligned");
   P.q = (const bf16*)q; P.pages = (const bf16*)pages; P.block_table = block_table; P.bt_stride = bt_stride;
   P.req_of_token = req_of_token; P.positions = positions; P.out = (bf16*)out; P.Hq = Hq; P.Hkv = Hkv;
-  P.page_size = page_size; P.num_pages = num_pages; P.scale_log2 = scale * 1.4426950408889634f;
+  P.page_size = page_size; P.num_pages = num_pages; 
+  P.scale_log2 = softcap > 0.f ? scale / softcap : scale * 1.4426950408889634f;
+  P.cap_log2 = softcap > 0.f ? softcap * 1.4426950408889634f : 0.f;
   P.chunk = chunk; P.window = window; P.attn_scale = attn_scale; P.floor_scale = floor_scale; P.status = status;
   P.tiles = nullptr; P.part_o = nullptr; P.part_ml = nullptr; P.max_splits = 0; P.split_keys = SPLIT_UNIT; P.rows = nullptr;
   P.sink = sink;
@@ -1016,10 +1027,10 @@ JLX_API int jlx_attention_decode(const void* q, const void* pages, const int* bl
                                  const int* req_of_token, const int* positions, void* out, int N, int Hq, int Hkv, int dh,
                                  int page_size, int num_pages, float scale, int chunk, int window, float attn_scale,
                                  float floor_scale, float* part_o, float* part_ml, int max_splits, int split_keys,
-                                 const int* rows, const float* sink, const float* slopes, int* status, cudaStream_t stream) {
+                                 const int* rows, const float* sink, const float* slopes, float softcap, int* status, cudaStream_t stream) {
   AttnParams P;
   if (fill_params(P, q, pages, block_table, bt_stride, req_of_token, positions, out, Hq, Hkv, dh, page_size, num_pages,
-                  scale, chunk, window, attn_scale, floor_scale, sink, slopes, status)) return 1;
+                  scale, chunk, window, attn_scale, floor_scale, sink, slopes, softcap, status)) return 1;
   JLX_REQUIRE(Hq / Hkv <= 16, "attention_decode: %d query heads per KV head; up to 16 are supported", Hq / Hkv);
   JLX_REQUIRE(part_o && part_ml && max_splits > 0, "attention_decode: scratch for the partial results is missing");
   JLX_REQUIRE(split_keys > 0 && split_keys % SPLIT_UNIT == 0, "attention_decode: split size %d is no multiple of %d", split_keys, SPLIT_UNIT);
@@ -1066,10 +1077,11 @@ JLX_API int jlx_attention_decode(const void* q, const void* pages, const int* bl
 JLX_API int jlx_attention_prefill(const void* q, const void* pages, const int* block_table, int bt_stride,
                                   const int* req_of_token, const int* positions, void* out, const int* tiles, int n_tiles,
                                   int Hq, int Hkv, int dh, int page_size, int num_pages, float scale, int chunk, int window,
-                                  float attn_scale, float floor_scale, const float* sink, const float* slopes, int* status, cudaStream_t stream) {
+                                  float attn_scale, float floor_scale, const float* sink, const float* slopes, float softcap, int* status,
+                                  cudaStream_t stream) {
   AttnParams P;
   if (fill_params(P, q, pages, block_table, bt_stride, req_of_token, positions, out, Hq, Hkv, dh, page_size, num_pages,
-                  scale, chunk, window, attn_scale, floor_scale, sink, slopes, status)) return 1;
+                  scale, chunk, window, attn_scale, floor_scale, sink, slopes, softcap, status)) return 1;
   const int G = Hq / Hkv;
   JLX_REQUIRE(G <= 8, "attention_prefill: %d query heads per KV head; up to 8 are supported", G);
   JLX_REQUIRE(Hkv <= 65535, "attention_prefill: too many KV heads");

@@ -28,6 +28,7 @@
 
 #include "common.cuh"
 #include "mbarrier.cuh"
+#include "softcap.cuh"
 
 #define DH 128
 #define BQ 128           // query rows per block
@@ -108,6 +109,47 @@ __device__ __forceinline__ float fast_exp2(float x) {
 __device__ __forceinline__ void tmem_ld_wait() { asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory"); }
 __device__ __forceinline__ void tmem_st_wait() { asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory"); }
 
+// Two float32 operations per instruction (IEEE, as their one-value forms).
+__device__ __forceinline__ uint64_t pack2(float a, float b) { return (uint64_t)__float_as_uint(a) | ((uint64_t)__float_as_uint(b) << 32); }
+__device__ __forceinline__ uint64_t mul2(uint64_t a, uint64_t b) {
+  uint64_t d;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+  return d;
+}
+__device__ __forceinline__ uint64_t fma2(uint64_t a, uint64_t b, uint64_t c) {
+  uint64_t d;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
+  return d;
+}
+
+// v <- tanh(v * in) for a thread's CP raw scores: the polynomial on pairs of scores; when any score of the warp lies
+// outside its range, the warp reads its scores from tensor memory again (`s_addr`) and takes the general form.
+__device__ __forceinline__ void cap_scores(uint32_t* v, float in, uint32_t s_addr) {
+  const uint64_t in2 = pack2(in, in);
+  float far = 0.f;
+#pragma unroll
+  for (int c = 0; c < CP; c += 2) {
+    const uint64_t x = mul2(pack2(__uint_as_float(v[c]), __uint_as_float(v[c + 1])), in2);
+    const uint64_t u = mul2(x, x);
+    uint64_t p = fma2(pack2(CAP_C5, CAP_C5), u, pack2(CAP_C4, CAP_C4));
+    p = fma2(p, u, pack2(CAP_C3, CAP_C3));
+    p = fma2(p, u, pack2(CAP_C2, CAP_C2));
+    p = fma2(p, u, pack2(CAP_C1, CAP_C1));
+    p = fma2(p, u, pack2(CAP_C0, CAP_C0));
+    p = mul2(p, x);
+    far = fmaxf(far, fmaxf(__uint_as_float((uint32_t)u), __uint_as_float((uint32_t)(u >> 32))));
+    v[c] = (uint32_t)p;
+    v[c + 1] = (uint32_t)(p >> 32);
+  }
+  if (__any_sync(0xffffffffu, far > 1.f)) {
+#pragma unroll
+    for (int c = 0; c < CP; c += 32) tmem_ld32(s_addr + c, v + c);
+    tmem_ld_wait();
+#pragma unroll
+    for (int c = 0; c < CP; ++c) v[c] = __float_as_uint(cap_tanh(__uint_as_float(v[c]) * in));
+  }
+}
+
 // Shared-memory matrix descriptors for tiles whose rows are 128 bytes (64 bfloat16) with the 128-byte
 // swizzle, 8-row groups 1024 bytes apart.  K-major: the 64 elements of a row run along K.  MN-major: they run
 // along the operand's M/N direction and rows are K steps; blocks of 64 along M/N are `lbo_bytes` apart.
@@ -131,7 +173,8 @@ struct TcParams {
   bf16* out;            // [N, Hq, DH]
   const int* tiles;     // [n_tiles][2] = (first token row, count <= 128), one request each
   int Hq, Hkv, page_size, num_pages;
-  float scale_log2;
+  float scale_log2;     // the score scale * log2(e); with a cap: the score scale / cap
+  float cap_log2;       // cap * log2(e) for soft-capped scores cap * tanh(s / cap), 0: none
   int chunk, window;
   float attn_scale, floor_scale;
   int* status;
@@ -360,6 +403,10 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
       const int lo_last = first_key(it.p_last, P.chunk, P.window);
       float sc = P.scale_log2;  // positive: raw scores and scaled scores have their maximum at the same key
       if (P.attn_scale != 0.f) sc *= 1.f + P.attn_scale * log1pf(floorf(((float)p_row + 1.f) / P.floor_scale));
+      // With a cap the raw scores are replaced by tanh(raw * cap_in) as they are read, and cap * log2(e) takes the scale's place.
+      const bool capped = P.cap_log2 > 0.f;
+      const float cap_in = sc;
+      if (capped) sc = P.cap_log2;
       // A distance bias in units of the RAW score (sc > 0): raw - bias_raw * (p - key) times sc is the biased scaled score,
       // so the maximum and the exponents below work on it as they do on raw scores.
       const bool biased = P.slopes != nullptr;
@@ -380,6 +427,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
 #pragma unroll
         for (int c = 0; c < CP; c += 32) tmem_ld32(s_addr + c, v + c);
         tmem_ld_wait();
+        if (capped) cap_scores(v, cap_in, s_addr);
         float mx4[4] = {NEG_BIG, NEG_BIG, NEG_BIG, NEG_BIG};  // four chains instead of one long chain of dependent steps
         if (need_mask) {
 #pragma unroll
@@ -556,8 +604,8 @@ JLX_API int jlx_attention_prefill_tc_supported(int Hq, int Hkv, int dh, int page
 JLX_API int jlx_attention_prefill_tc(const void* q, const void* pages, const int* block_table, int bt_stride,
                                      const int* req_of_token, const int* positions, void* out, const int* tiles,
                                      int n_tiles, int N, int Hq, int Hkv, int dh, int page_size, int num_pages, float scale,
-                                     int chunk, int window, float attn_scale, float floor_scale, const float* sink, const float* slopes, int* status,
-                                     cudaStream_t stream) {
+                                     int chunk, int window, float attn_scale, float floor_scale, const float* sink, const float* slopes,
+                                     float softcap, int* status, cudaStream_t stream) {
   JLX_REQUIRE(jlx_attention_prefill_tc_supported(Hq, Hkv, dh, page_size),
               "attention_prefill_tc: needs head size 128 and pages of a multiple of 64 tokens (got %d, %d)", dh, page_size);
   JLX_REQUIRE(N > 0 && num_pages > 0 && bt_stride > 0, "attention_prefill_tc: bad sizes");
@@ -566,6 +614,7 @@ JLX_API int jlx_attention_prefill_tc(const void* q, const void* pages, const int
               "attention_prefill_tc: q, pages and out must be 16-byte aligned");
   JLX_REQUIRE(attn_scale == 0.f || floor_scale > 0.f, "attention: floor_scale must be positive");
   JLX_REQUIRE(Hq <= 65535, "attention_prefill_tc: too many heads");
+  JLX_REQUIRE(softcap >= 0.f, "attention: the score cap must be positive (0: none)");
   if (n_tiles == 0) return 0;
   EncodeTiledFn fn = encode_fn();
   JLX_REQUIRE(fn != nullptr, "attention_prefill_tc: the driver does not offer cuTensorMapEncodeTiled");
@@ -593,7 +642,9 @@ JLX_API int jlx_attention_prefill_tc(const void* q, const void* pages, const int
   TcParams P;
   P.block_table = block_table; P.bt_stride = bt_stride; P.req_of_token = req_of_token; P.positions = positions;
   P.out = (bf16*)out; P.tiles = tiles; P.Hq = Hq; P.Hkv = Hkv; P.page_size = page_size; P.num_pages = num_pages;
-  P.scale_log2 = scale * 1.4426950408889634f; P.chunk = chunk; P.window = window; P.attn_scale = attn_scale;
+  P.scale_log2 = softcap > 0.f ? scale / softcap : scale * 1.4426950408889634f;
+  P.cap_log2 = softcap > 0.f ? softcap * 1.4426950408889634f : 0.f;
+  P.chunk = chunk; P.window = window; P.attn_scale = attn_scale;
   P.floor_scale = floor_scale; P.status = status; P.sink = sink; P.slopes = slopes;
   const size_t smem = 5 * (size_t)TILE_BYTES + 1024;
   static bool cfg = false;

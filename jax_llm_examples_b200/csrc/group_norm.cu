@@ -12,6 +12,55 @@
 // Every sum runs in an order that depends on the row alone (not on the batch or on how a prompt was cut).
 #include "common.cuh"
 
+// Where a row's delta lies.  Without `index`: row r of `delta`.  With it, the delta is an expert layer's output still in
+// expert order: the sum over j < k of weights[r k + j] (null: 1) times row index[r k + j], j ascending.  In both cases
+// `splits` partials of a row are added first, ascending.
+struct DeltaRows {
+  const float* p;
+  long long split_stride;
+  const int* index;
+  const float* weights;
+  int splits, k;
+};
+
+__device__ __forceinline__ float delta_at(const DeltaRows& t, size_t r, int D, int d) {
+  if (!t.index) {
+    float s = 0.f;
+    for (int z = 0; z < t.splits; ++z) s += t.p[(size_t)z * t.split_stride + r * D + d];
+    return s;
+  }
+  float s = 0.f;
+  for (int j = 0; j < t.k; ++j) {
+    const float* p = t.p + (size_t)t.index[r * t.k + j] * D + d;
+    float e = 0.f;
+    for (int z = 0; z < t.splits; ++z) e += p[(size_t)z * t.split_stride];
+    s = fmaf(t.weights ? t.weights[r * t.k + j] : 1.f, e, s);
+  }
+  return s;
+}
+
+__device__ __forceinline__ float4 delta_at4(const DeltaRows& t, size_t r, int D, int d) {  // entries d .. d + 3
+  float4 s = make_float4(0.f, 0.f, 0.f, 0.f);
+  if (!t.index) {
+    for (int z = 0; z < t.splits; ++z) {
+      const float4 v = *reinterpret_cast<const float4*>(t.p + (size_t)z * t.split_stride + r * D + d);
+      s.x += v.x; s.y += v.y; s.z += v.z; s.w += v.w;
+    }
+    return s;
+  }
+  for (int j = 0; j < t.k; ++j) {
+    const float* p = t.p + (size_t)t.index[r * t.k + j] * D + d;
+    float4 e = make_float4(0.f, 0.f, 0.f, 0.f);
+    for (int z = 0; z < t.splits; ++z) {
+      const float4 v = *reinterpret_cast<const float4*>(p + (size_t)z * t.split_stride);
+      e.x += v.x; e.y += v.y; e.z += v.z; e.w += v.w;
+    }
+    const float w = t.weights ? t.weights[r * t.k + j] : 1.f;
+    s.x = fmaf(w, e.x, s.x); s.y = fmaf(w, e.y, s.y); s.z = fmaf(w, e.z, s.z); s.w = fmaf(w, e.w, s.w);
+  }
+  return s;
+}
+
 // 1 / rms of every group of row[0..D) into inv[0..groups): warp w takes groups w, w + nwarp, ...
 __device__ __forceinline__ void group_rms(const float* row, int D, int groups, float eps, float* rms) {
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarp = blockDim.x >> 5;
@@ -27,7 +76,7 @@ __device__ __forceinline__ void group_rms(const float* row, int D, int groups, f
 
 // One block per row.  Source row r = row_index ? row_index[n] : n (then x is not written back).
 template <typename TO>
-__global__ void group_norm_kernel(float* __restrict__ x, const float* __restrict__ delta, int splits, long long split_stride,
+__global__ void group_norm_kernel(float* __restrict__ x, const DeltaRows delta,
                                   const float* __restrict__ delta_bias, const float* __restrict__ post_w, int post_groups,
                                   int post_norm, float mult, const float* __restrict__ pre_w, int pre_groups, int pre_norm, float eps,
                                   TO* __restrict__ out, long long ld_out, float* __restrict__ out32,
@@ -41,10 +90,9 @@ __global__ void group_norm_kernel(float* __restrict__ x, const float* __restrict
   const int n = blockIdx.x;
   const size_t r = row_index ? (size_t)row_index[n] : (size_t)n;
   float* xr = x + r * D;
-  if (delta) {
+  if (delta.p) {
     for (int d = threadIdx.x; d < D; d += blockDim.x) {
-      float s = 0.f;
-      for (int z = 0; z < splits; ++z) s += delta[(size_t)z * split_stride + r * D + d];
+      float s = delta_at(delta, r, D, d);
       if (delta_bias) s += delta_bias[d];
       row[d] = s;
     }
@@ -100,7 +148,7 @@ template <> __device__ __forceinline__ void store4<bf16>(bf16* p, float4 v) {
 // The same row, four values per access: for widths and groups that are multiples of 4 and 16-byte aligned tensors.
 // Every value goes through the same operations as in the kernel above.
 template <typename TO>
-__global__ void group_norm_x4_kernel(float* __restrict__ x, const float* __restrict__ delta, int splits, long long split_stride,
+__global__ void group_norm_x4_kernel(float* __restrict__ x, const DeltaRows delta,
                                      const float* __restrict__ delta_bias, const float* __restrict__ post_w, int post_groups,
                                      int post_norm, float mult, const float* __restrict__ pre_w, int pre_groups, int pre_norm, float eps,
                                      TO* __restrict__ out, long long ld_out, float* __restrict__ out32,
@@ -115,13 +163,9 @@ __global__ void group_norm_x4_kernel(float* __restrict__ x, const float* __restr
   const int n = blockIdx.x, D4 = D >> 2;
   const size_t r = row_index ? (size_t)row_index[n] : (size_t)n;
   float4* xr4 = reinterpret_cast<float4*>(x + r * D);
-  if (delta) {
+  if (delta.p) {
     for (int d = threadIdx.x; d < D4; d += blockDim.x) {
-      float4 s = make_float4(0.f, 0.f, 0.f, 0.f);
-      for (int z = 0; z < splits; ++z) {
-        const float4 v = *reinterpret_cast<const float4*>(delta + (size_t)z * split_stride + r * D + 4 * d);
-        s.x += v.x; s.y += v.y; s.z += v.z; s.w += v.w;
-      }
+      float4 s = delta_at4(delta, r, D, 4 * d);
       if (delta_bias) {
         const float4 b = reinterpret_cast<const float4*>(delta_bias)[d];
         s.x += b.x; s.y += b.y; s.z += b.z; s.w += b.w;
@@ -187,9 +231,12 @@ __global__ void group_norm_x4_kernel(float* __restrict__ x, const float* __restr
 JLX_API int jlx_group_norm(float* x, const float* delta, int splits, long long split_stride, const float* delta_bias,
                            const float* post_w, int post_groups, int post_norm, float mult, const float* pre_w,
                            int pre_groups, int pre_norm, float eps, void* out, int out_dtype, long long ld_out, float* out32,
-                           const int* row_index, int N, int D, cudaStream_t stream) {
+                           const int* row_index, int N, int D, const int* delta_index, const float* delta_weights, int delta_k,
+                           cudaStream_t stream) {
   JLX_REQUIRE(N >= 0 && D > 0 && splits >= 1, "group_norm: bad sizes N=%d D=%d splits=%d", N, D, splits);
   JLX_REQUIRE(eps > 0.f, "group_norm: eps must be positive");
+  JLX_REQUIRE(!delta_index || (delta && delta_k >= 1), "group_norm: gathered rows need the rows and how many a token adds");
+  const DeltaRows rows = {delta, split_stride, delta_index, delta_weights, splits, delta_k};
   if (!post_norm) post_groups = 1;
   JLX_REQUIRE(!post_w || (post_groups >= 1 && D % post_groups == 0), "group_norm: %d groups do not divide the width %d", post_groups, D);
   JLX_REQUIRE(!pre_norm || (pre_groups >= 1 && D % pre_groups == 0), "group_norm: %d groups do not divide the width %d", pre_groups, D);
@@ -208,7 +255,7 @@ JLX_API int jlx_group_norm(float* x, const float* delta, int splits, long long s
       if (smem > 48 * 1024)
         JLX_CUDA(cudaFuncSetAttribute(group_norm_x4_kernel<TO>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
       JLX_CUDA(jlx_launch_pdl(group_norm_x4_kernel<TO>, dim3(N), dim3(D >= 8192 ? 512 : (D >= 2048 ? 256 : 128)), smem, stream,
-                              x, delta, splits, split_stride, delta_bias, post_w, post_groups, post_norm, mult, pre_w, pre_groups, pre_norm,
+                              x, rows, delta_bias, post_w, post_groups, post_norm, mult, pre_w, pre_groups, pre_norm,
                               eps, (TO*)out, ld_out, out32, row_index, D));
     });
     JLX_LAUNCH_CHECK("group_norm");
@@ -217,7 +264,7 @@ JLX_API int jlx_group_norm(float* x, const float* delta, int splits, long long s
   JLX_DISPATCH_DTYPE(out_dtype, TO, {
     if (smem > 48 * 1024)
       JLX_CUDA(cudaFuncSetAttribute(group_norm_kernel<TO>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
-    JLX_CUDA(jlx_launch_pdl(group_norm_kernel<TO>, dim3(N), dim3(threads), smem, stream, x, delta, splits, split_stride, delta_bias,
+    JLX_CUDA(jlx_launch_pdl(group_norm_kernel<TO>, dim3(N), dim3(threads), smem, stream, x, rows, delta_bias,
                             post_w, post_groups, post_norm, mult, pre_w, pre_groups, pre_norm, eps, (TO*)out, ld_out, out32, row_index, D));
   });
   JLX_LAUNCH_CHECK("group_norm");

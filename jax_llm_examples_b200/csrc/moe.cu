@@ -14,7 +14,7 @@
 // One block per token.  Warp w computes the scores of experts w, w + nwarp, ...: a fixed order of
 // the D products per (token, expert), so a token's routing does not depend on the batch.
 // bias (null: none) is added to the scores before the choice.  weight_form 0: sigmoid of the chosen score;
-// 1: softmax over the chosen scores only; 2: see RouterChoice.
+// 1: softmax over the chosen scores only; 2, 3: see RouterChoice.
 __device__ __forceinline__ void softmax_of_chosen(float* w, int k) {
   float m = -INFINITY, sum = 0.f;
   for (int j = 0; j < k; ++j) m = fmaxf(m, w[j]);
@@ -22,30 +22,36 @@ __device__ __forceinline__ void softmax_of_chosen(float* w, int k) {
   for (int j = 0; j < k; ++j) w[j] = expf(w[j] - m) / sum;
 }
 
-// What the choice needs beyond the scores, for weight_form 2 ("softmax over all, the chosen shares normalised"):
-// s = softmax(z) over all E outputs; the choice is made on s + correction, and only among the `keep` best of `groups`
-// equal groups of neighbouring outputs (a group's score: its largest s + correction; the others count as -inf, not
-// 0: corrections may be negative); the weights are the chosen s, divided by their sum (+ 1e-20), times `scale`.
+// What the choice needs beyond the scores, for the corrected forms: weight_form 2, s = softmax(z) over all E outputs, and
+// weight_form 3, s = sigmoid(z).  The choice is made on s + correction, and only among the `keep` best of `groups`
+// equal groups of neighbouring outputs (a group's score: the sum of its `group_top` largest s + correction, one or two;
+// the others count as -inf, not 0: corrections may be negative); the weights are the chosen s, with `normalize` divided
+// by their sum (+ 1e-20), times `scale`.
 struct RouterChoice {
   const float* correction;  // [E] or null
   int groups, keep;         // groups <= 1: no limit
   float scale;
+  int group_top, normalize;
 };
 
 // One thread: the k largest scores in order (strict comparison: the lower index wins a tie), their weights by form.
 // `sc` (shared memory, E entries) is used up.
 __device__ __forceinline__ void choose_experts(float* sc, int E, int k, int* __restrict__ idx, float* __restrict__ w, int weight_form,
                                                const RouterChoice& ch) {
-  if (weight_form == 2) {
+  if (weight_form >= 2) {
     // the shares once (E exponentials), in place; after that the choice only compares and adds
-    float m = -INFINITY, sum = 0.f;
-    for (int e = 0; e < E; ++e) m = fmaxf(m, sc[e]);
-    for (int e = 0; e < E; ++e) {
-      const float x = expf(sc[e] - m);
-      sc[e] = x;
-      sum += x;
+    if (weight_form == 3) {
+      for (int e = 0; e < E; ++e) sc[e] = 1.f / (1.f + expf(-sc[e]));
+    } else {
+      float m = -INFINITY, sum = 0.f;
+      for (int e = 0; e < E; ++e) m = fmaxf(m, sc[e]);
+      for (int e = 0; e < E; ++e) {
+        const float x = expf(sc[e] - m);
+        sc[e] = x;
+        sum += x;
+      }
+      for (int e = 0; e < E; ++e) sc[e] = sc[e] / sum;
     }
-    for (int e = 0; e < E; ++e) sc[e] = sc[e] / sum;
     const int per = ch.groups > 1 ? E / ch.groups : E;
     unsigned long long allowed = ~0ull;  // bit g: group g may be chosen from (up to 64 groups)
     if (ch.groups > 1 && ch.keep < ch.groups) {
@@ -55,8 +61,13 @@ __device__ __forceinline__ void choose_experts(float* sc, int E, int k, int* __r
         float bv = 0.f;
         for (int g = 0; g < ch.groups; ++g) {
           if ((allowed >> g) & 1ull) continue;
-          float gv = -INFINITY;
-          for (int e = g * per; e < (g + 1) * per; ++e) gv = fmaxf(gv, sc[e] + (ch.correction ? ch.correction[e] : 0.f));
+          float gv = -INFINITY, second = -INFINITY;
+          for (int e = g * per; e < (g + 1) * per; ++e) {
+            const float v = sc[e] + (ch.correction ? ch.correction[e] : 0.f);
+            second = fmaxf(second, fminf(gv, v));
+            gv = fmaxf(gv, v);
+          }
+          if (ch.group_top == 2 && per > 1) gv += second;
           if (bg < 0 || gv > bv) {
             bg = g;
             bv = gv;
@@ -87,7 +98,7 @@ __device__ __forceinline__ void choose_experts(float* sc, int E, int k, int* __r
       total += bs;
       taken[best >> 6] |= 1ull << (best & 63);
     }
-    for (int j = 0; j < k; ++j) w[j] = w[j] / (total + 1e-20f) * ch.scale;
+    for (int j = 0; j < k; ++j) w[j] = (ch.normalize ? w[j] / (total + 1e-20f) : w[j]) * ch.scale;
     return;
   }
   for (int j = 0; j < k; ++j) {
@@ -117,9 +128,9 @@ __global__ void router_kernel(const float* __restrict__ h, const float* __restri
   const int n = blockIdx.x;
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarp = blockDim.x >> 5;
   const float* hr = h + (size_t)n * D;
-  // The newest weight form reads four columns per access with four sums under way (the walk below is a chain of
+  // The corrected forms read four columns per access with four sums under way (the walk below is a chain of
   // loads that wait on one another); the older forms keep the order of their sums.
-  const bool wide = weight_form == 2 && (D & 3) == 0 && (((uintptr_t)h | (uintptr_t)w_router) & 15) == 0;
+  const bool wide = weight_form >= 2 && (D & 3) == 0 && (((uintptr_t)h | (uintptr_t)w_router) & 15) == 0;
   for (int e = warp; e < E; e += nwarp) {
     const float* wr = w_router + (size_t)e * D;
     float s = 0.f;
@@ -202,11 +213,12 @@ router_rows_kernel(const float* __restrict__ h, const float* __restrict__ w_rout
 // one-token kernel's: a caller whose results must not depend on the batch uses one of the two throughout).
 JLX_API int jlx_router(const float* h, const float* w_router, int* topk_idx, float* topk_w, float* scores_out, int N,
                        int D, int E, int k, int many_rows, const float* bias, int weight_form, const float* correction,
-                       int groups, int keep, float scale, cudaStream_t stream) {
-  JLX_REQUIRE(weight_form >= 0 && weight_form <= 2, "router: unknown weight form %d", weight_form);
-  JLX_REQUIRE(groups <= 1 || (weight_form == 2 && groups <= 64 && E % groups == 0 && keep >= 1 && keep <= groups),
-              "router: %d groups (keep %d) of %d outputs: the softmax-over-all form, equal groups, up to 64, keep in 1..groups", groups, keep, E);
-  const RouterChoice choice = {correction, groups, keep, scale};
+                       int groups, int keep, float scale, int group_top, int normalize, cudaStream_t stream) {
+  JLX_REQUIRE(weight_form >= 0 && weight_form <= 3, "router: unknown weight form %d", weight_form);
+  JLX_REQUIRE(groups <= 1 || (weight_form >= 2 && groups <= 64 && E % groups == 0 && keep >= 1 && keep <= groups),
+              "router: %d groups (keep %d) of %d outputs: a corrected form, equal groups, up to 64, keep in 1..groups", groups, keep, E);
+  JLX_REQUIRE(group_top == 1 || group_top == 2, "router: a group's score sums its %d largest; 1 or 2 are supported", group_top);
+  const RouterChoice choice = {correction, groups, keep, scale, group_top, normalize};
   JLX_REQUIRE(N >= 0 && D > 0, "router: bad sizes N=%d D=%d", N, D);
   JLX_REQUIRE(E >= 1 && E <= ROUTER_MAX_E, "router: %d experts; supported 1..%d", E, ROUTER_MAX_E);
   JLX_REQUIRE(k >= 1 && k <= E && k <= ROUTER_MAX_K, "router: top-%d of %d experts; supported k in 1..min(E, %d)", k, E, ROUTER_MAX_K);

@@ -413,7 +413,8 @@ __global__ void rope_half_kv_store_kernel(RopeRowsView proj, int k_col, int v_co
                                           const int* __restrict__ positions, const float* __restrict__ q_norm_w,
                                           const float* __restrict__ k_norm_w, float eps, const float* __restrict__ inv_freq,
                                           int rot, int pairing, int norm_mode, int Hq, int Hkv, int dk, int dv, int dpad,
-                                          int page_size, int num_pages, int store, int* status, float amplitude) {
+                                          int page_size, int num_pages, int store, int* status, float amplitude, const float* __restrict__ q_scale,
+                                          int v_norm) {
   JLX_TL(TL_ROPE);
   pdl_launch_dependents_if_small();
   __shared__ float whole_part[2][8];
@@ -474,7 +475,7 @@ __global__ void rope_half_kv_store_kernel(RopeRowsView proj, int k_col, int v_co
       ss = fmaf(s, s, ss);
     }
     const float* w = is_q ? q_norm_w : (is_k ? k_norm_w : nullptr);
-    if (qk && norm_mode == ROPE_NORM_BEFORE) {
+    if ((qk && norm_mode == ROPE_NORM_BEFORE) || (!qk && v_norm)) {
       ss = warp_sum(ss);
       const float rms = sqrtf(ss / (float)d + eps);
       __syncwarp();
@@ -510,11 +511,13 @@ __global__ void rope_half_kv_store_kernel(RopeRowsView proj, int k_col, int v_co
       rms_turned = sqrtf(ss2 / (float)d + eps);
     }
     __syncwarp();
+    const float qs = is_q && q_scale ? q_scale[hh] : 1.f;
     for (int i = lane; i < dpad; i += 32) {
       float y = 0.f;
       if (i < d) {
         y = turned[i];
         if (after) y = w ? y / rms_turned * w[i] : y / rms_turned;
+        y *= qs;
       }
       dst[i] = from_f32<T>(y);
     }
@@ -524,12 +527,14 @@ __global__ void rope_half_kv_store_kernel(RopeRowsView proj, int k_col, int v_co
 
 // proj: float32 rows (see RopeRowsView; p points at the first q column).  pages: [P, 2, Hkv, page_size, dpad] or null.
 // pairing: which entries turn together; norm_mode: no q/k norm, before the rotation, or after it (a null weight: the
-// norm without one).  v_col == k_col with dv == dk stores the keys as projected (neither normed nor turned) as values.
+// norm without one).  v_norm: each value head is divided by its root mean square over dv (no weight).  q_scale [Hq] (or
+// null): every query head is multiplied by its number, last.  v_col == k_col with dv == dk stores the keys as projected (neither normed nor turned) as values.
 JLX_API int jlx_rope_half_kv_store(const RopeRowsView* proj, int k_col, int v_col, void* q_out, void* pages, int dtype,
                                    const int* block_table, int bt_stride, const int* req_of_token, const int* positions,
                                    const float* q_norm_w, const float* k_norm_w, float eps, const float* inv_freq, int rot,
                                    int pairing, int norm_mode, int N, int Hq, int Hkv, int dk, int dv, int dpad, int page_size,
-                                   int num_pages, int store, int* status, float amplitude, cudaStream_t stream) {
+                                   int num_pages, int store, int* status, float amplitude, const float* q_scale, int v_norm,
+                                   cudaStream_t stream) {
   JLX_REQUIRE(N >= 0 && Hq > 0 && Hkv > 0 && dk > 0 && dv > 0, "rope_half: bad sizes");
   JLX_REQUIRE(dpad >= dk && dpad >= dv, "rope_half: the padded head size %d is below the key or value size (%d, %d)", dpad, dk, dv);
   JLX_REQUIRE(rot >= 0 && rot % 2 == 0 && rot <= dk, "rope_half: %d rotated entries of %d", rot, dk);
@@ -546,7 +551,8 @@ JLX_API int jlx_rope_half_kv_store(const RopeRowsView* proj, int k_col, int v_co
   JLX_DISPATCH_DTYPE(dtype, T, {
     JLX_CUDA(jlx_launch_pdl(rope_half_kv_store_kernel<T>, dim3(N, by), dim3(nwarp * 32), smem, stream, *proj, k_col, v_col,
                             (T*)q_out, (T*)pages, block_table, bt_stride, req_of_token, positions, q_norm_w, k_norm_w, eps,
-                            inv_freq, rot, pairing, norm_mode, Hq, Hkv, dk, dv, dpad, page_size, num_pages, store, status, amplitude));
+                            inv_freq, rot, pairing, norm_mode, Hq, Hkv, dk, dv, dpad, page_size, num_pages, store, status, amplitude,
+                            q_scale, v_norm));
   });
   JLX_LAUNCH_CHECK("rope_half_kv_store");
   return 0;

@@ -256,15 +256,21 @@ def group_norm(x: torch.Tensor, delta: torch.Tensor | None = None, delta_splits:
                post_weight: torch.Tensor | None = None, post_groups: int = 1, mult: float = 1.0,
                pre_weight: torch.Tensor | None = None, pre_groups: int = 1, pre_norm: bool = True, eps: float = 1e-6,
                out: torch.Tensor | None = None, out32: torch.Tensor | None = None, row_index: torch.Tensor | None = None,
-               post_norm: bool = True) -> None:
+               post_norm: bool = True, delta_index: torch.Tensor | None = None, delta_k: int = 1,
+               delta_weights: torch.Tensor | None = None) -> None:
     """One pass over each row of the float32 residual x [N, D]:
     x += mult * post_weight * groupnorm(delta + delta_bias) (``delta``: float32 [N, D] or ``delta_splits`` partials of
     it; without post_weight the sum is added as it is; with ``post_norm`` False post_weight is a plain scale per
     channel: x += mult * post_weight * delta), then out / out32 = pre_weight * groupnorm(x) (``pre_norm``
     False: x itself).  groupnorm divides each of ``groups`` equal consecutive parts of a row by
     sqrt(mean(part^2) + eps).  ``out`` may be a view whose rows are longer than D (its row stride is kept).  With
-    row_index, row n reads source row row_index[n] and x is not written back."""
-    _contig(x, delta, delta_bias, post_weight, pre_weight, out32, row_index)
+    row_index, row n reads source row row_index[n] and x is not written back.  With ``delta_index`` (int32 [rows *
+    delta_k]) the delta is an expert layer's output in expert order: row r's is the sum over j < delta_k of
+    ``delta_weights[r, j]`` (float32; None: 1) times row delta_index[r * delta_k + j] of ``delta``."""
+    _contig(x, delta, delta_bias, post_weight, pre_weight, out32, row_index, delta_index, delta_weights)
+    if delta_index is not None and (delta_index.dtype != torch.int32 or delta_index.numel() < x.shape[0] * delta_k or (
+            delta_weights is not None and (delta_weights.dtype != torch.float32 or delta_weights.numel() < x.shape[0] * delta_k))):
+        raise KernelError(f"group_norm: {x.shape[0]} gathered rows need {delta_k} int32 indices and float32 weights each")
     N, D = (row_index.numel() if row_index is not None else x.shape[0]), x.shape[1]
     if x.dtype != torch.float32 or any(t is not None and t.dtype != torch.float32 for t in (delta, delta_bias, post_weight, pre_weight)):
         raise KernelError("group_norm: the residual stream, what is added to it and the norm weights must be float32")
@@ -277,7 +283,7 @@ def group_norm(x: torch.Tensor, delta: torch.Tensor | None = None, delta_splits:
     _run("group_norm", "jlx_group_norm", _ptr(x), _ptr(delta), c_int(sp), c_longlong(stride), _ptr(delta_bias),
          _ptr(post_weight), c_int(post_groups), c_int(int(post_norm)), c_float(mult), _ptr(pre_weight), c_int(pre_groups), c_int(int(pre_norm)),
          c_float(eps), _ptr(out), c_int(code(out.dtype) if out is not None else F32), c_longlong(ld_out), _ptr(out32),
-         _ptr(row_index), c_int(N), c_int(D), _stream())
+         _ptr(row_index), c_int(N), c_int(D), _ptr(delta_index), _ptr(delta_weights), c_int(delta_k), _stream())
 
 
 def bias_act(rows: torch.Tensor, out: torch.Tensor, bias: torch.Tensor | None = None, add: torch.Tensor | None = None,
@@ -377,9 +383,10 @@ def hgrn2_scan(qfv: torch.Tensor, splits: int, f_bias: torch.Tensor, lower: torc
 def latent_kv_prep(proj: torch.Tensor, splits: int, q_norm_weight: torch.Tensor, kv_norm_weight: torch.Tensor, eps: float,
                    inv_freq: torch.Tensor, rot_dims: int, cq: torch.Tensor, pages: torch.Tensor | None,
                    block_table: torch.Tensor | None, req_of_token: torch.Tensor, positions: torch.Tensor,
-                   q_rank: int, rank: int, dr: int, status: torch.Tensor) -> None:
-    """From projected rows [N, q_rank + rank + dr] (float32, or partials): cq = weighted RMS norm of the first q_rank
-    entries; the page row of the token = [weighted RMS norm of the next rank entries | the last dr entries, rotated].
+                   q_rank: int, rank: int, dr: int, status: torch.Tensor, pairing: str = "pairs") -> None:
+    """From projected rows whose first entries are [q_rank | rank | dr] (float32 [N, >= that], or partials): cq = weighted RMS norm of the first q_rank
+    entries; the page row of the token = [weighted RMS norm of the next rank entries | the next dr entries, rotated
+    (``pairing`` "pairs": entry 2i with 2i + 1; "halves": i with i + rot_dims / 2)].
     pages: [P, 1, 1, page_size, rank + dr]."""
     _contig(proj, q_norm_weight, kv_norm_weight, inv_freq, cq, pages, block_table)
     N = cq.shape[0]
@@ -391,11 +398,12 @@ def latent_kv_prep(proj: torch.Tensor, splits: int, q_norm_weight: torch.Tensor,
          _ptr(kv_norm_weight), c_float(eps), _ptr(inv_freq), c_int(rot_dims), _ptr(cq), _ptr(pages), c_int(code(cq.dtype)),
          _ptr(block_table), c_int(block_table.shape[1] if store else 0), _ptr(req_of_token), _ptr(positions), c_int(N),
          c_int(q_rank), c_int(rank), c_int(dr), c_int(pages.shape[3] if store else 0), c_int(pages.shape[0] if store else 0),
-         _ptr(status), _stream())
+         c_int(proj.shape[-1]), c_int(int(pairing == "halves")), _ptr(status), _stream())
 
 
 def latent_q_prep(q: torch.Tensor, splits: int, inv_freq: torch.Tensor, rot_dims: int, positions: torch.Tensor,
-                  q_nope: torch.Tensor, q_rot: torch.Tensor, heads: int, dn: int, dr: int, q_full: torch.Tensor | None = None) -> None:
+                  q_nope: torch.Tensor, q_rot: torch.Tensor, heads: int, dn: int, dr: int, q_full: torch.Tensor | None = None,
+                  pairing: str = "pairs") -> None:
     """q: float32 [N, H (dn + dr)] (or partials) -> q_nope [H, N, dn] (head-major), q_rot float32 [N, H, dr], rotated,
     and optionally q_full [H, N, dn + dr] (both parts, in q_nope's type)."""
     _contig(q, inv_freq, q_nope, q_rot, q_full)
@@ -403,7 +411,7 @@ def latent_q_prep(q: torch.Tensor, splits: int, inv_freq: torch.Tensor, rot_dims
     sp, stride = _splits(q, splits)
     _run("attention_latent", "jlx_latent_q_prep", _ptr(q), c_int(sp), c_longlong(stride), _ptr(inv_freq), c_int(rot_dims),
          _ptr(positions), _ptr(q_nope), c_int(code(q_nope.dtype)), _ptr(q_rot), _ptr(q_full), c_int(N), c_int(heads), c_int(dn),
-         c_int(dr), _stream())
+         c_int(dr), c_int(int(pairing == "halves")), _stream())
 
 
 LATENT_KEY_TILE = 32  # keys per tile of the latent attention kernel: split sizes are multiples of it
@@ -412,11 +420,13 @@ LATENT_KEY_TILE = 32  # keys per tile of the latent attention kernel: split size
 def attention_latent(q_lat: torch.Tensor, q_rot: torch.Tensor, pages: torch.Tensor, block_table: torch.Tensor,
                      req_of_token: torch.Tensor, positions: torch.Tensor, sink: torch.Tensor | None, out_lat: torch.Tensor,
                      scale: float, status: torch.Tensor, rows: torch.Tensor | None = None, n_rows: int = 0, splits: int = 1,
-                     split_keys: int = 0, part_acc: torch.Tensor | None = None, part_ml: torch.Tensor | None = None) -> None:
-    """Causal attention in the latent space with an optional per-head sink.  q_lat: float32 [H, N, rank]; q_rot:
+                     split_keys: int = 0, part_acc: torch.Tensor | None = None, part_ml: torch.Tensor | None = None,
+                     window: int = 0) -> None:
+    """Causal attention in the latent space with an optional per-head sink and window (a query sees itself and the
+    window - 1 keys before it; 0: all).  q_lat: float32 [H, N, rank]; q_rot:
     float32 [N, H, dr]; pages: [P, 1, 1, page_size, rank + dr]; out_lat: [H, N, rank].
     rows / n_rows: serve these token rows only (int32).  splits > 1: the keys are cut into ranges of ``split_keys``
-    (a multiple of LATENT_KEY_TILE), a block each, and a second kernel adds the ranges' results; part_acc: float32
+    (a multiple of LATENT_KEY_TILE; ranges are counted from the first visible key's), a block each, and a second kernel adds the ranges' results; part_acc: float32
     [served * H * splits * rank], part_ml: float32 [served * H * splits * 2]."""
     _contig(q_lat, q_rot, pages, block_table, sink, out_lat, rows, part_acc, part_ml)
     H, N, rank = q_lat.shape
@@ -434,19 +444,21 @@ def attention_latent(q_lat: torch.Tensor, q_rot: torch.Tensor, pages: torch.Tens
          _ptr(block_table), c_int(block_table.shape[1]), _ptr(req_of_token), _ptr(positions), _ptr(sink), _ptr(out_lat),
          c_int(code(out_lat.dtype)), c_int(N), c_int(H), c_int(rank), c_int(dr), c_int(pages.shape[3]), c_int(pages.shape[0]),
          c_float(scale), _ptr(rows), c_int(n_rows), c_int(splits), c_int(split_keys), _ptr(part_acc), _ptr(part_ml),
-         _ptr(status), _stream())
+         c_int(window), _ptr(status), _stream())
     _launches += int(splits > 1)  # the combine kernel
 
 
-def latent_gather(pages: torch.Tensor, block_table_row: torch.Tensor, c: torch.Tensor, kr: torch.Tensor, status: torch.Tensor) -> None:
-    """The first L cached rows of one request (its block-table row) as two dense matrices: c [L, rank], kr [L, dr]."""
+def latent_gather(pages: torch.Tensor, block_table_row: torch.Tensor, c: torch.Tensor, kr: torch.Tensor, status: torch.Tensor,
+                  first: int = 0) -> None:
+    """The cached rows of positions first .. first + L - 1 of one request (its block-table row) as two dense matrices:
+    c [L, rank], kr [L, dr]."""
     _contig(pages, block_table_row, c, kr)
     L, rank = c.shape
     dr = kr.shape[1]
     if pages.shape[4] != rank + dr or c.dtype != pages.dtype or kr.dtype != pages.dtype:
         raise KernelError("latent_gather: cache rows and outputs disagree")
     _run("attention_latent", "jlx_latent_gather", _ptr(pages), c_int(code(pages.dtype)), _ptr(block_table_row), _ptr(c), _ptr(kr),
-         c_int(L), c_int(rank), c_int(dr), c_int(pages.shape[3]), c_int(pages.shape[0]), _ptr(status), _stream())
+         c_int(first), c_int(L), c_int(rank), c_int(dr), c_int(pages.shape[3]), c_int(pages.shape[0]), _ptr(status), _stream())
 
 
 def latent_key_assemble(kv_up: torch.Tensor, kr: torch.Tensor, k: torch.Tensor, heads: int, dn: int) -> None:
@@ -459,26 +471,30 @@ def latent_key_assemble(kv_up: torch.Tensor, kr: torch.Tensor, k: torch.Tensor, 
          c_int(code(k.dtype)), c_int(L), c_int(heads), c_int(dn), c_int(dr), _stream())
 
 
-def causal_sink_softmax(scores: torch.Tensor, sink: torch.Tensor | None, scale: float, q_start: int, probs: torch.Tensor) -> None:
-    """probs[h, i, j] = softmax over j <= q_start + i of scale * scores[h, i, j], the denominator also holding
-    exp(sink[h]); 0 beyond the causal edge.  scores: float32 [H, T, L]; probs: [H, T, L]."""
+def causal_sink_softmax(scores: torch.Tensor, sink: torch.Tensor | None, scale: float, q_start: int, probs: torch.Tensor,
+                        k_start: int = 0, window: int = 0) -> None:
+    """probs[h, i, j] = softmax over the visible columns of scale * scores[h, i, j], the denominator also holding
+    exp(sink[h]); 0 elsewhere.  Column j is the key at position k_start + j, row i the query at q_start + i: it sees the
+    keys up to itself, with ``window`` > 0 the last so many of them.  scores: float32 [H, T, L]; probs: [H, T, L]."""
     _contig(scores, sink, probs)
     H, T, L = scores.shape
     if scores.dtype != torch.float32 or probs.shape != scores.shape:
         raise KernelError("causal_sink_softmax: float32 scores and probabilities of the same shape are needed")
-    _run("attention_latent", "jlx_causal_sink_softmax", _ptr(scores), _ptr(sink), c_float(scale), c_int(q_start), _ptr(probs),
-         c_int(code(probs.dtype)), c_int(H), c_int(T), c_int(L), _stream())
+    _run("attention_latent", "jlx_causal_sink_softmax", _ptr(scores), _ptr(sink), c_float(scale), c_int(q_start), c_int(k_start),
+         c_int(window), _ptr(probs), c_int(code(probs.dtype)), c_int(H), c_int(T), c_int(L), _stream())
 
 
-def heads_to_rows(x: torch.Tensor, out: torch.Tensor) -> None:
-    """x: [H, N, d] -> out: [N, H * d]."""
+def heads_to_rows(x: torch.Tensor, out: torch.Tensor, gate: "_RowsView | None" = None) -> None:
+    """x: [H, N, d] -> out: [N, H * d]; with ``gate`` (projected rows, column h of row n for head h of token n) every head
+    is multiplied by sigmoid(gate[n, h])."""
     _contig(x, out)
     H, N, d = x.shape
-    _run("attention_latent", "jlx_heads_to_rows", _ptr(x), _ptr(out), c_int(code(x.dtype)), c_int(N), c_int(H), c_int(d), _stream())
+    _run("attention_latent", "jlx_heads_to_rows", _ptr(x), _ptr(out), c_int(code(x.dtype)), c_int(N), c_int(H), c_int(d),
+         ctypes.byref(gate) if gate is not None else None, _stream())
 
 
 # ------------------------------------------------------ linear attention with a decay per key channel
-class _RowsView(ctypes.Structure):  # RowsView in csrc/decay_scan.cu, RopeRowsView in csrc/rope_kv.cu
+class _RowsView(ctypes.Structure):  # RowsView in csrc/decay_scan.cu, RopeRowsView in csrc/rope_kv.cu, GateRowsView in csrc/attention_latent.cu
     _fields_ = [("p", c_void_p), ("split_stride", c_longlong), ("ld", c_longlong), ("splits", c_int), ("pad_", c_int)]
 
 
@@ -631,14 +647,19 @@ def rope_norm_kv_store(proj: _RowsView, k_col: int, v_col: int, q_out: torch.Ten
                        block_table: torch.Tensor | None, req_of_token: torch.Tensor, positions: torch.Tensor,
                        q_norm_weight: torch.Tensor | None, k_norm_weight: torch.Tensor | None, eps: float,
                        inv_freq: torch.Tensor | None, rot_dims: int, Hq: int, Hkv: int, dk: int, dv: int, status: torch.Tensor,
-                       pairing: str = "halves", norm: str = "before", amplitude: float = 1.0) -> None:
+                       pairing: str = "halves", norm: str = "before", amplitude: float = 1.0,
+                       q_head_scale: torch.Tensor | None = None, v_norm: bool = False) -> None:
     """From projected float32 rows (q heads from the view's first column, k heads from column k_col, v heads of dv
     entries from v_col; v_col = k_col stores the keys as projected as values): q and k RMS-normed over dk (``norm``:
     "none", "before" or "after" the rotation; with a weight where one is given), their first rot_dims entries rotated
     (``pairing`` "halves": entry i with i + rot_dims / 2; "pairs": entry 2i with 2i + 1); q into q_out [N, Hq, dpad],
     k and v into the token's cache row (pages [P, 2, Hkv, page_size, dpad]), all padded with zeros to dpad.
     ``norm`` "whole": before the rotation, over all heads of q (of k) at once, the weights [Hq dk] and [Hkv dk].
-    ``amplitude`` multiplies both the cosine and the sine of every angle."""
+    ``amplitude`` multiplies both the cosine and the sine of every angle.  ``v_norm``: every value head is divided by its
+    root mean square over dv.  ``q_head_scale`` (float32 [Hq]): every query head is multiplied by its number, last."""
+    if q_head_scale is not None and (q_head_scale.dtype != torch.float32 or q_head_scale.numel() != Hq):
+        raise KernelError(f"rope_norm_kv_store: the queries' factors must be float32 [{Hq}]")
+    _contig(q_head_scale)
     _contig(q_out, pages, block_table, q_norm_weight, k_norm_weight, inv_freq)
     N, _, dpad = q_out.shape
     if norm == "whole" and (q_norm_weight is None or k_norm_weight is None or q_norm_weight.numel() != Hq * dk or k_norm_weight.numel() != Hkv * dk):
@@ -651,7 +672,7 @@ def rope_norm_kv_store(proj: _RowsView, k_col: int, v_col: int, q_out: torch.Ten
          _ptr(positions), _ptr(q_norm_weight), _ptr(k_norm_weight), c_float(eps), _ptr(inv_freq), c_int(rot_dims),
          c_int(ROPE_PAIRINGS[pairing]), c_int(ROPE_NORMS[norm]), c_int(N), c_int(Hq), c_int(Hkv), c_int(dk), c_int(dv), c_int(dpad),
          c_int(pages.shape[3] if store else 0), c_int(pages.shape[0] if store else 0), c_int(int(store)), _ptr(status),
-         c_float(amplitude), _stream())
+         c_float(amplitude), _ptr(q_head_scale), c_int(int(v_norm)), _stream())
 
 
 def rope_half_kv_store(proj: _RowsView, k_col: int, v_col: int, q_out: torch.Tensor, pages: torch.Tensor | None,
@@ -708,10 +729,11 @@ def kv_store(k: torch.Tensor, v: torch.Tensor, pages: torch.Tensor, block_table:
 def attention_generic(q: torch.Tensor, pages: torch.Tensor, block_table: torch.Tensor, req_of_token: torch.Tensor,
                       positions: torch.Tensor, out: torch.Tensor, scale: float, chunk: int, window: int,
                       attn_scale: float, floor_scale: float, status: torch.Tensor, sink: torch.Tensor | None = None,
-                      slopes: torch.Tensor | None = None) -> None:
+                      slopes: torch.Tensor | None = None, softcap: float = 0.0) -> None:
     """q: [N, Hq, dh]; pages: [P, 2, Hkv, page, dh]; out: [N, Hq, dh].  ``sink``: float32 [Hq] or None; with it the
     softmax's denominator has one more term exp(sink[h]) that carries no value.  ``slopes``: float32 [Hq] or None; with
-    it slopes[h] * (query position - key position) is taken off every scaled score (all four attention kernels take both)."""
+    it slopes[h] * (query position - key position) is taken off every scaled score.  ``softcap`` > 0: a scaled score s
+    becomes softcap * tanh(s / softcap) first (all four attention kernels take all three)."""
     _contig(q, pages, block_table, out)
     _check_sink(sink, q.shape[1])
     _check_sink(slopes, q.shape[1], "slopes")
@@ -722,7 +744,7 @@ def attention_generic(q: torch.Tensor, pages: torch.Tensor, block_table: torch.T
     _run("attention_generic", "jlx_attention_generic", _ptr(q), _ptr(pages), c_int(code(q.dtype)), _ptr(block_table),
          c_int(block_table.shape[1]), _ptr(req_of_token), _ptr(positions), _ptr(out), c_int(N), c_int(Hq), c_int(Hkv),
          c_int(dh), c_int(page_size), c_int(P), c_float(scale), c_int(chunk), c_int(window), c_float(attn_scale),
-         c_float(floor_scale), _ptr(sink), _ptr(slopes), _ptr(status), _stream())
+         c_float(floor_scale), _ptr(sink), _ptr(slopes), c_float(softcap), _ptr(status), _stream())
 
 
 def _check_sink(sink: torch.Tensor | None, Hq: int, what: str = "sink") -> None:
@@ -747,7 +769,7 @@ def attention_decode(q: torch.Tensor, pages: torch.Tensor, block_table: torch.Te
                      positions: torch.Tensor, out: torch.Tensor, scale: float, chunk: int, window: int, attn_scale: float,
                      floor_scale: float, part_o: torch.Tensor, part_ml: torch.Tensor, max_splits: int, split_keys: int,
                      status: torch.Tensor, rows: torch.Tensor | None = None, n_rows: int = 0,
-                     sink: torch.Tensor | None = None, slopes: torch.Tensor | None = None) -> None:
+                     sink: torch.Tensor | None = None, slopes: torch.Tensor | None = None, softcap: float = 0.0) -> None:
     """Split-KV attention for one query token per request (tensor cores, bfloat16).
     part_o: float32 [N * Hq * max_splits * dh]; part_ml: float32 [N * Hq * max_splits * 2].
     rows / n_rows: work on these token rows only (int32, the first n_rows entries): the single decoded tokens of
@@ -764,13 +786,14 @@ def attention_decode(q: torch.Tensor, pages: torch.Tensor, block_table: torch.Te
     _run("attention_mma", "jlx_attention_decode", _ptr(q), _ptr(pages), _ptr(block_table), c_int(block_table.shape[1]),
          _ptr(req_of_token), _ptr(positions), _ptr(out), c_int(N), c_int(Hq), c_int(Hkv), c_int(dh), c_int(page_size),
          c_int(P), c_float(scale), c_int(chunk), c_int(window), c_float(attn_scale), c_float(floor_scale), _ptr(part_o),
-         _ptr(part_ml), c_int(max_splits), c_int(split_keys), _ptr(rows), _ptr(sink), _ptr(slopes), _ptr(status), _stream())
+         _ptr(part_ml), c_int(max_splits), c_int(split_keys), _ptr(rows), _ptr(sink), _ptr(slopes),
+         c_float(softcap), _ptr(status), _stream())
 
 
 def attention_prefill(q: torch.Tensor, pages: torch.Tensor, block_table: torch.Tensor, req_of_token: torch.Tensor,
                       positions: torch.Tensor, out: torch.Tensor, tiles: torch.Tensor, n_tiles: int, scale: float,
                       chunk: int, window: int, attn_scale: float, floor_scale: float, status: torch.Tensor,
-                      sink: torch.Tensor | None = None, slopes: torch.Tensor | None = None) -> None:
+                      sink: torch.Tensor | None = None, slopes: torch.Tensor | None = None, softcap: float = 0.0) -> None:
     """Flash attention over the paged cache for prompt portions (tensor cores, bfloat16).
     tiles: int32 [n_tiles, 2] = (first token row, count <= 16), each within one request."""
     _contig(q, pages, block_table, out, tiles)
@@ -781,7 +804,7 @@ def attention_prefill(q: torch.Tensor, pages: torch.Tensor, block_table: torch.T
     _run("attention_mma", "jlx_attention_prefill", _ptr(q), _ptr(pages), _ptr(block_table), c_int(block_table.shape[1]),
          _ptr(req_of_token), _ptr(positions), _ptr(out), _ptr(tiles), c_int(n_tiles), c_int(Hq), c_int(Hkv), c_int(dh),
          c_int(page_size), c_int(P), c_float(scale), c_int(chunk), c_int(window), c_float(attn_scale),
-         c_float(floor_scale), _ptr(sink), _ptr(slopes), _ptr(status), _stream())
+         c_float(floor_scale), _ptr(sink), _ptr(slopes), c_float(softcap), _ptr(status), _stream())
 
 
 def attention_prefill_tc_supported(q_dtype: torch.dtype, Hq: int, Hkv: int, dh: int, page_size: int) -> bool:
@@ -793,7 +816,7 @@ def attention_prefill_tc_supported(q_dtype: torch.dtype, Hq: int, Hkv: int, dh: 
 def attention_prefill_tc(q: torch.Tensor, pages: torch.Tensor, block_table: torch.Tensor, req_of_token: torch.Tensor,
                          positions: torch.Tensor, out: torch.Tensor, tiles: torch.Tensor, n_tiles: int, scale: float,
                          chunk: int, window: int, attn_scale: float, floor_scale: float, status: torch.Tensor,
-                         sink: torch.Tensor | None = None, slopes: torch.Tensor | None = None) -> None:
+                         sink: torch.Tensor | None = None, slopes: torch.Tensor | None = None, softcap: float = 0.0) -> None:
     """Flash attention for prompt portions on tcgen05 (bfloat16, head size 128, pages of a multiple of 64).
     tiles: int32 [n_tiles, 2] = (first token row, count <= 128), each within one request; only the rows
     of these tiles are written."""
@@ -805,7 +828,7 @@ def attention_prefill_tc(q: torch.Tensor, pages: torch.Tensor, block_table: torc
     _run("attention_tc", "jlx_attention_prefill_tc", _ptr(q), _ptr(pages), _ptr(block_table), c_int(block_table.shape[1]),
          _ptr(req_of_token), _ptr(positions), _ptr(out), _ptr(tiles), c_int(n_tiles), c_int(N), c_int(Hq), c_int(Hkv),
          c_int(dh), c_int(page_size), c_int(P), c_float(scale), c_int(chunk), c_int(window), c_float(attn_scale),
-         c_float(floor_scale), _ptr(sink), _ptr(slopes), _ptr(status), _stream())
+         c_float(floor_scale), _ptr(sink), _ptr(slopes), c_float(softcap), _ptr(status), _stream())
 
 
 # ------------------------------------------------------------------------------------- GEMMs
@@ -874,19 +897,21 @@ def gemm_stream(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, status: tor
 
 
 # --------------------------------------------------------------------------------------- MoE
-ROUTER_WEIGHT_FORMS = {"sigmoid": 0, "softmax_of_chosen": 1, "softmax_normalized": 2}  # csrc/moe.cu
+ROUTER_WEIGHT_FORMS = {"sigmoid": 0, "softmax_of_chosen": 1, "softmax_normalized": 2, "sigmoid_corrected": 3}  # csrc/moe.cu
 ROUTER_MAX_GROUPS = 64
 
 
 def router(h32: torch.Tensor, w_router: torch.Tensor, topk_idx: torch.Tensor, topk_w: torch.Tensor,
            scores_out: torch.Tensor | None = None, many_rows: bool = False, bias: torch.Tensor | None = None,
            weight_form: str = "sigmoid", correction: torch.Tensor | None = None, groups: int = 1, keep: int = 1,
-           scale: float = 1.0) -> None:
+           scale: float = 1.0, group_top: int = 1, normalize: bool | None = None) -> None:
     """Scores h32 @ w_router^T (+ bias) in 32-bit, top-k of the scores (lower index wins ties); the weights are the
     sigmoid of each chosen score, or (``weight_form`` "softmax_of_chosen") the softmax over the chosen scores only.
     "softmax_normalized": s = softmax of the scores over ALL outputs; the choice is made on s + ``correction`` (float32
-    [E]), among the ``keep`` best of ``groups`` equal groups of neighbouring outputs only (a group's score is its largest
-    choice score); the weights are the chosen s divided by their sum and multiplied by ``scale``.
+    [E]), among the ``keep`` best of ``groups`` equal groups of neighbouring outputs only (a group's score is the sum of its
+    ``group_top`` largest choice scores, 1 or 2); the weights are the chosen s divided by their sum and multiplied by ``scale``.
+    "sigmoid_corrected": the same with s = sigmoid of the scores, the chosen s not divided by their sum.  ``normalize``
+    says otherwise in either form.
     ``many_rows``: the kernel that shares each router row among eight tokens (for prompt portions; its sums
     run in another order than the one-token kernel's)."""
     _contig(h32, w_router, topk_idx, topk_w, scores_out, bias)
@@ -898,7 +923,8 @@ def router(h32: torch.Tensor, w_router: torch.Tensor, topk_idx: torch.Tensor, to
         raise KernelError("router: scores are computed from float32 input, weight, bias and correction (one number per output)")
     _run("moe", "jlx_router", _ptr(h32), _ptr(w_router), _ptr(topk_idx), _ptr(topk_w), _ptr(scores_out), c_int(N),
          c_int(D), c_int(E), c_int(k), c_int(int(many_rows)), _ptr(bias), c_int(ROUTER_WEIGHT_FORMS[weight_form]),
-         _ptr(correction), c_int(groups), c_int(keep), c_float(scale), _stream())
+         _ptr(correction), c_int(groups), c_int(keep), c_float(scale), c_int(group_top),
+         c_int(int(weight_form == "softmax_normalized" if normalize is None else normalize)), _stream())
 
 
 def expert_sort(topk_idx: torch.Tensor, offsets: torch.Tensor, sorted_pair: torch.Tensor, sorted_pos: torch.Tensor,

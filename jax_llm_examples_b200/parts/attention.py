@@ -76,6 +76,7 @@ class PagedAttention(Mixer):
         self.scale = float(head_dim) ** -0.5 if scale is None else float(scale)  # model.py:774
 
     sink: torch.Tensor | None = None
+    softcap: float = 0.0  # > 0: a scaled score s becomes softcap * tanh(s / softcap)
     slopes: torch.Tensor | None = None  # [Hq]: slopes[h] * (query position - key position) is taken off the scaled scores
 
     @staticmethod
@@ -133,7 +134,7 @@ class PagedAttention(Mixer):
         part_ml = ctx.workspace.get("attn_part_ml", n * 2, torch.float32)
         K.attention_decode(q, cache.pages, cache.block_table, ctx.req_of_token, ctx.positions, out, self.scale,
                            chunk, window, attn_scale, floor_scale, part_o, part_ml, splits, split_keys, ctx.status,
-                           rows, n_rows, self.sink, self.slopes)
+                           rows, n_rows, self.sink, self.slopes, self.softcap)
 
     def attend(self, ctx: StepContext, q, cache: LayerCache, out, attn_scale: float, floor_scale: float) -> None:
         """Tensor-core kernels where they are built (bfloat16, head size 64 or 128, small groups): split-KV for
@@ -159,16 +160,17 @@ class PagedAttention(Mixer):
                     # long portions on the tcgen05 kernel (128-token tiles), the short ones below
                     K.attention_prefill_tc(q, cache.pages, cache.block_table, ctx.req_of_token, ctx.positions, out,
                                            ctx.arrays["attn_tiles_long"], count["attn_tiles_long"], self.scale, chunk, window,
-                                           attn_scale, floor_scale, ctx.status, self.sink, self.slopes)
+                                           attn_scale, floor_scale, ctx.status, self.sink, self.slopes, self.softcap)
                     tiles, n_tiles = ctx.arrays["attn_tiles_short"], count["attn_tiles_short"]
                     kinds = ("tc", "flash" if n_tiles else "", "split_kv" if count["attn_single_rows"] else "")
                     ctx.scratch.setdefault("attention_kernels", set()).add(tuple(k for k in kinds if k))
                 if n_tiles:
                     K.attention_prefill(q, cache.pages, cache.block_table, ctx.req_of_token, ctx.positions, out, tiles,
-                                        n_tiles, self.scale, chunk, window, attn_scale, floor_scale, ctx.status, self.sink, self.slopes)
+                                        n_tiles, self.scale, chunk, window, attn_scale, floor_scale, ctx.status, self.sink, self.slopes,
+                                        self.softcap)
                 return
         K.attention_generic(q, cache.pages, cache.block_table, ctx.req_of_token, ctx.positions, out, self.scale,
-                            self.chunk or 0, self.window or 0, attn_scale, floor_scale, ctx.status, self.sink, self.slopes)
+                            self.chunk or 0, self.window or 0, attn_scale, floor_scale, ctx.status, self.sink, self.slopes, self.softcap)
 
 
 register_part("mixer", "paged_attention", PagedAttention)
@@ -192,7 +194,10 @@ class GatedPagedAttention(ProjectedMixer, PagedAttention):
     [Hq dk] and [Hkv dk].  ``rot_amplitude`` multiplies the cosine and the sine of every angle (a rotation that also
     stretches the rotated entries).  ``slopes`` [Hq]: slopes[h] * (i - j) is taken off the scaled score of query i and key
     j.  ``query_temperature`` (coef, every): queries at position p are multiplied by 1 + coef * ln(floor((p + 1) / every)
-    + 1).  ``keep_window``: pages are kept for a window of at least this many positions (a layer with a longer window
+    + 1); ``head_temperature`` [Hq]: every head's scores are multiplied by its number (its queries are, before they are
+    rounded).  ``softcap``: a scaled score s becomes softcap * tanh(s / softcap), before a bias and the sink.
+    ``value_norm``: every value head is divided by its root mean square (no weight) before it is cached.
+    ``keep_window``: pages are kept for a window of at least this many positions (a layer with a longer window
     reads them; 0: for good).  ``window``: a query
     sees itself and the window - 1 positions before it; ``chunk``: the positions of its own chunk.  Keys, queries and
     values are kept at one padded size (``padded_dim`` >= max(dk, dv), zeros beyond their own): one page layout, and the
@@ -208,7 +213,8 @@ class GatedPagedAttention(ProjectedMixer, PagedAttention):
                  gated: bool = True, padded_dim: int | None = None, sink: torch.Tensor | None = None, pairing: str = "halves",
                  norm: str | None = None, values_are_keys: bool = False, gate: str | None = None,
                  rot_amplitude: float = 1.0, slopes: torch.Tensor | None = None, query_temperature: tuple[float, float] | None = None,
-                 projects_kv: bool = True, keep_window: int | None = None):
+                 projects_kv: bool = True, keep_window: int | None = None, head_temperature: torch.Tensor | None = None,
+                 softcap: float | None = None, value_norm: bool = False):
         if n_heads % n_kv_heads:
             raise ValueError(f"{n_heads} query heads are no multiple of {n_kv_heads} KV heads")
         gate = ("head" if gated else "none") if gate is None else gate
@@ -255,6 +261,10 @@ class GatedPagedAttention(ProjectedMixer, PagedAttention):
         if self.q_temperature[0] != 0.0 and self.q_temperature[1] <= 0:
             raise ValueError("the query temperature's period must be positive")
         self.projects_kv, self.keep_window = bool(projects_kv), keep_window
+        self.head_temperature = self._sink_vector(head_temperature, n_heads, "vector of head temperatures")
+        self.softcap, self.value_norm = 0.0 if softcap is None else float(softcap), bool(value_norm)
+        if self.softcap < 0:
+            raise ValueError("the score cap must be positive")
         self.position, self.qk_norm_eps = None, None
 
     def kv_need(self) -> KVNeed:
@@ -293,7 +303,7 @@ class GatedPagedAttention(ProjectedMixer, PagedAttention):
                                  cache.pages if cache.writes else None, cache.block_table if cache.writes else None,
                                  ctx.req_of_token, ctx.positions, self.q_norm_weight, self.k_norm_weight, self.eps,
                                  self.inv_freq, self.rot_dims, Hq, Hkv, dk, dv, ctx.status, self.pairing, self.norm,
-                                 self.rot_amplitude)
+                                 self.rot_amplitude, self.head_temperature, self.value_norm)
         attn = torch.empty_like(q)
         with scope("attention"):
             self.attend(ctx, q, cache, attn, *self.q_temperature)

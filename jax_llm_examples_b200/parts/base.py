@@ -64,13 +64,15 @@ class Rows:
     slices the consumer adds in ascending order (saving the launch that would add them).
 
     As a term of a :class:`RowSum` the rows may also lie elsewhere in ``data``: token r's row is ``base + r``, or,
-    with ``index`` (int32 [N * k]), the sum of the k rows ``index[r * k + j]``, j ascending."""
+    with ``index`` (int32 [N * k]), the sum of the k rows ``index[r * k + j]``, j ascending, each times
+    ``weights[r, j]`` (float32 [N, k]) if there are weights."""
 
     data: torch.Tensor
     splits: int = 1
     index: torch.Tensor | None = None
     k: int = 1
     base: int = 0
+    weights: torch.Tensor | None = None
 
 
 @dataclasses.dataclass
@@ -97,12 +99,18 @@ class PostNormed:
     mult: float
     bias: torch.Tensor | None = None  # float32 [D], added to the rows before the norm (a biased product's bias)
 
+    def gather(self) -> dict:
+        """The group-norm kernel's arguments for rows that lie in expert order (``Rows.index``)."""
+        return dict(delta_index=self.rows.index, delta_k=self.rows.k, delta_weights=self.rows.weights)
+
     def materialize(self) -> torch.Tensor:
         from ..kernels import api as K
 
-        n, d = self.rows.data.shape[-2], self.rows.data.shape[-1]
+        n = self.rows.data.shape[-2] if self.rows.index is None else self.rows.index.numel() // self.rows.k
+        d = self.rows.data.shape[-1]
         zero = torch.zeros((n, d), dtype=torch.float32, device=self.weight.device)
-        K.group_norm(zero, self.rows.data, self.rows.splits, self.bias, self.weight, self.groups, self.mult, eps=self.eps)
+        K.group_norm(zero, self.rows.data, self.rows.splits, self.bias, self.weight, self.groups, self.mult, eps=self.eps,
+                     **self.gather())
         return zero
 
 

@@ -127,6 +127,62 @@ class SandwichNormBlock(Block):
         return self._closing(self.norm2b, y, getattr(self.feed_forward, "bias_out", None))
 
 
+class PostNormBlock(Block):
+    """A block that norms each sublayer's OUTPUT only; the sublayers read the residual rows themselves:
+
+        x += norm1(mixer(x));   x += norm2(feed_forward(x))
+
+    The feed-forward (with norm2) may be missing.  A sublayer's output goes on as a :class:`PostNormed` delta; the kernel
+    that closes it (norm, residual sum) also writes the rows that the next sublayer reads, in the activations' type.
+    A routed feed-forward may hand on its rows in expert order, with their weights: that kernel gathers them too."""
+
+    kernel_libraries = ("group_norm",)
+
+    def __init__(self, norm1: Norm, mixer: Mixer, norm2: Norm | None = None, feed_forward: FeedForward | None = None):
+        if (feed_forward is None) != (norm2 is None):
+            raise ValueError("a feed-forward comes with its norm, or not at all")
+        self.norm1, self.mixer, self.norm2, self.feed_forward = norm1, mixer, norm2, feed_forward
+
+    def sub_parts(self):
+        return tuple(p for p in (self.norm1, self.mixer, self.norm2, self.feed_forward) if p is not None)
+
+    @staticmethod
+    def _closing(norm: Norm, y, bias=None):
+        from .base import PostNormed, RowSum, as_rows
+
+        if isinstance(y, RowSum) and len(y.terms) == 1 and y.terms[0].base == 0 and y.terms[0].data.dtype == torch.float32:
+            rows = y.terms[0]
+        else:
+            rows = as_rows(y)
+        return PostNormed(rows, norm.weight, norm.eps, norm.groups, 1.0, bias)
+
+    @staticmethod
+    def _open(ctx: StepContext, x: torch.Tensor, delta, eps: float) -> torch.Tensor:
+        """x += delta; the new x in the activations' type."""
+        from .norms import add_to_residual
+
+        if ctx.runtime.dtype == torch.float32:  # the rows themselves serve (nothing changes them before their readers ran)
+            if delta is not None:
+                add_to_residual(x, delta, pre_norm=False, eps=eps)
+            return x
+        h = torch.empty(x.shape, dtype=ctx.runtime.dtype, device=x.device)
+        add_to_residual(x, delta, pre_norm=False, eps=eps, out=h)
+        return h
+
+    def forward(self, ctx: StepContext, x: torch.Tensor, delta, cache: LayerCache):
+        with scope("attn_pre_norm"):
+            h = self._open(ctx, x, delta, self.norm1.eps)
+        y = self.mixer.forward(ctx, None, cache, h32=x) if self.mixer.needs_f32_input else self.mixer.forward(ctx, h, cache)
+        pending = self._closing(self.norm1, y)
+        if self.feed_forward is None:
+            return pending
+        with scope("attn_post_norm"):
+            h = self._open(ctx, x, pending, self.norm1.eps)
+        with scope("ffn"):
+            y = self.feed_forward.forward(ctx, h, x if self.feed_forward.needs_f32_input else None, None)
+        return self._closing(self.norm2, y, getattr(self.feed_forward, "bias_out", None))
+
+
 class ReinjectionBlock(Block):
     """Feeds the embedding's output into the stream again:  x <- W [x; x0] + step,  x0 = what the embedding put out
     for the token, W: [D, 2D] (x's half first), ``step``: a vector of this entry (one per pass of a loop over layers).
@@ -247,5 +303,6 @@ class HyperConnectionBlock(Block):
 
 register_part("block", "hyper_connection", HyperConnectionBlock)
 register_part("block", "sandwich_norm", SandwichNormBlock)
+register_part("block", "post_norm", PostNormBlock)
 register_part("block", "reinjection", ReinjectionBlock)
 register_part("block", "embedding_reentry", EmbeddingReentryBlock)

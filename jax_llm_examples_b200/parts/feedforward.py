@@ -237,45 +237,75 @@ class DenseBiasedMLP(FeedForward):
 register_part("feed_forward", "dense_biased", DenseBiasedMLP)
 
 
-class SoftmaxRoutedMLPExperts(FeedForward):
-    """Experts of the form down(act(up h)) chosen by a biased router, their OUTPUTS weighted:
+class RoutedMLPExperts(FeedForward):
+    """Experts of the form down(act(up h)), their OUTPUTS weighted:
 
-        z = W_router h + b (float32);  the top-k experts by z;  weights = softmax over the chosen z only;
-        out = sum_j weight_j * expert_j(h)  (+ shared(h): an expert of the same form that takes every token).
+        out = sum_j weight_j * expert_j(h)  (+ shared(h): an expert of the same form that takes every token),
 
-    ``w_router``: [E, D]; ``router_bias``: [E]; ``we_up``: [E, F, D]; ``we_down``: [E, D, F]; ``activation``: a name
-    of ``K.ACTIVATIONS``.  The tokens' rows are gathered in expert order (unscaled), both products run as grouped
-    products over that order, and the kernel that brings the rows back applies the weights and adds the shared expert."""
+    chosen by a router of one of two families (``weight_form``), z = W_router h (+ bias) in float32:
+
+    * "softmax_of_chosen": the top-k experts by z; weights = softmax over the chosen z only;
+    * "sigmoid_corrected": s = sigmoid(z); the choice is made on s + ``correction``, among the ``keep`` best of ``groups``
+      equal groups of neighbouring experts (a group's score is the sum of its ``group_top`` largest choice scores); weights
+      = the chosen s (``normalize``: divided by their sum), times ``route_scale``.
+
+    ``w_router``: [E, D]; ``router_bias``, ``correction``: [E] or None; ``we_up``: [E, F, D]; ``we_down``: [E, D, F];
+    ``activation``: a name of ``K.ACTIVATIONS``.  The tokens' rows are gathered in expert order (unscaled), both products
+    run as grouped products over that order.  The result is a :class:`RowSum` of one term, the rows in expert order with
+    their weights, for a consumer that gathers them in its own kernel; else one kernel brings them back, weights them and
+    adds the shared expert."""
 
     kernel_libraries = ("moe", "group_norm", "gemm_simt")
     kernel_libraries_bf16 = ("gemm_stream",)
     needs_f32_input = True
+    MANY_ROWS = 64  # above this many rows (bfloat16) a corrected router shares each of its rows among eight tokens
 
     def __init__(self, w_router: torch.Tensor, router_bias: torch.Tensor | None, we_up: torch.Tensor, we_down: torch.Tensor,
-                 top_k: int, activation: str = "relu2", shared: "DenseBiasedMLP | None" = None):
+                 top_k: int, activation: str = "relu2", shared: "DenseBiasedMLP | None" = None, weight_form: str = "softmax_of_chosen",
+                 correction: torch.Tensor | None = None, groups: int = 1, keep: int = 1, group_top: int = 1, normalize: bool = False,
+                 route_scale: float = 1.0):
         E = w_router.shape[0]
         if we_up.shape[0] != E or we_down.shape[0] != E or we_up.shape[1] != we_down.shape[2] or we_up.shape[2] != we_down.shape[1] \
-                or w_router.shape[1] != we_down.shape[1] or (router_bias is not None and router_bias.numel() != E):
+                or w_router.shape[1] != we_down.shape[1] or any(t is not None and t.numel() != E for t in (router_bias, correction)):
             raise ValueError(f"expert weights do not fit: router {tuple(w_router.shape)}, up {tuple(we_up.shape)}, down {tuple(we_down.shape)}")
-        if not 1 <= top_k <= E:
-            raise ValueError(f"top-{top_k} of {E} experts")
+        if weight_form not in ("softmax_of_chosen", "sigmoid_corrected"):
+            raise ValueError(f"unknown weight form {weight_form!r}")
+        if weight_form == "softmax_of_chosen" and (correction is not None or groups != 1):
+            raise ValueError("a softmax over the chosen scores has neither a correction nor groups")
+        if groups < 1 or E % groups or not 1 <= keep <= groups or groups > K.ROUTER_MAX_GROUPS or group_top not in (1, 2):
+            raise ValueError(f"{groups} groups (keep {keep}, {group_top} scores each) do not divide {E} experts evenly")
+        if not 1 <= top_k <= E // groups * keep:
+            raise ValueError(f"top-{top_k} of {E // groups * keep} experts")
         if activation not in K.ACTIVATIONS:
             raise ValueError(f"unknown activation {activation!r}; known: {sorted(K.ACTIVATIONS)}")
         self.w_router = w_router.to(torch.float32).contiguous()
         self.router_bias = None if router_bias is None else router_bias.to(torch.float32).contiguous()
+        self.correction = None if correction is None else correction.to(torch.float32).contiguous()
         self.we_up, self.we_down = we_up.contiguous(), we_down.contiguous()
         self.top_k, self.num_experts, self.activation, self.shared = top_k, E, activation, shared
+        self.weight_form, self.groups, self.keep, self.group_top = weight_form, int(groups), int(keep), int(group_top)
+        self.normalize, self.route_scale = bool(normalize), float(route_scale)
 
     def sub_parts(self):
         return () if self.shared is None else (self.shared,)
+
+    def route(self, ctx: StepContext, h32: torch.Tensor):
+        n, k, dev = h32.shape[0], self.top_k, h32.device
+        topk_idx = torch.empty((n, k), dtype=torch.int32, device=dev)
+        topk_w = torch.empty((n, k), dtype=torch.float32, device=dev)
+        if self.weight_form == "softmax_of_chosen":
+            K.router(h32, self.w_router, topk_idx, topk_w, bias=self.router_bias, weight_form=self.weight_form)
+        else:
+            K.router(h32, self.w_router, topk_idx, topk_w, many_rows=ctx.runtime.dtype == torch.bfloat16 and n > self.MANY_ROWS,
+                     bias=self.router_bias, weight_form=self.weight_form, correction=self.correction, groups=self.groups,
+                     keep=self.keep, scale=self.route_scale, group_top=self.group_top, normalize=self.normalize)
+        return topk_idx, topk_w
 
     def forward(self, ctx: StepContext, h, h32, routing=None):
         rt = ctx.runtime
         n, D = h32.shape
         k, E, dev = self.top_k, self.num_experts, h32.device
-        topk_idx = torch.empty((n, k), dtype=torch.int32, device=dev)
-        topk_w = torch.empty((n, k), dtype=torch.float32, device=dev)
-        K.router(h32, self.w_router, topk_idx, topk_w, bias=self.router_bias, weight_form="softmax_of_chosen")
+        topk_idx, topk_w = self.route(ctx, h32)
         if "record_routing" in ctx.scratch:
             ctx.scratch["record_routing"].append(topk_idx)
         with scope("moe_routed_expert"):
@@ -303,14 +333,25 @@ class SoftmaxRoutedMLPExperts(FeedForward):
         if self.shared is not None:
             with scope("moe_shared_expert"):
                 shared = as_rows(self.shared.forward(ctx, h, None))
-        delta = torch.empty((n, D), dtype=torch.float32, device=dev)
-        with scope("unpermute"):
-            K.moe_combine(y.data, None if shared is None else shared.data, sorted_pos, delta, k,
-                          1 if shared is None else shared.splits, y.splits, -1, pair_weights=topk_w)
-        return delta
+
+        def combine() -> torch.Tensor:
+            delta = torch.empty((n, D), dtype=torch.float32, device=dev)
+            with scope("unpermute"):
+                K.moe_combine(y.data, None if shared is None else shared.data, sorted_pos, delta, k,
+                              1 if shared is None else shared.splits, y.splits, -1, pair_weights=topk_w)
+            return delta
+
+        if shared is not None:
+            return combine()
+        return RowSum([Rows(y.data, y.splits, sorted_pos, k, 0, topk_w)], combine)
+
+
+class SoftmaxRoutedMLPExperts(RoutedMLPExperts):
+    """The form with a biased router and a softmax over the chosen logits (see :class:`RoutedMLPExperts`)."""
 
 
 register_part("feed_forward", "softmax_routed_mlp", SoftmaxRoutedMLPExperts)
+register_part("feed_forward", "routed_mlp", RoutedMLPExperts)
 
 
 class GroupLimitedGLUExperts(FeedForward):

@@ -48,9 +48,12 @@ class LatentAttention(InputConvMixer):
     Only [c | k_rot] is cached (``planes`` = 1, one "head" of rank + dr).  The kernels work in the latent space:
     q_lat = W_uk[h]^T q_nope (a product per head), scores and weighted sums against the cached rows, then
     v = W_uv[h] out_lat (a product per head).  Rotation: the first ``rot_dims`` entries of the rotated part, in pairs
-    (2i, 2i+1), by position * rot_base^(-2i / rot_dims).
+    (``pairing`` "pairs": entry 2i with 2i+1; "halves": i with i + rot_dims / 2), by position * rot_base^(-2i / rot_dims).
+    ``window``: a query sees itself and the window - 1 positions before it.  ``gated``: every head's output is multiplied
+    by sigmoid(W_g h)_h.
 
-    ``w_down``: [q_rank + rank + dr, D] = W_dq over W_dkv.  ``w_uk``: [H dn, rank]; ``w_uv``: [H dv, rank]."""
+    ``w_down``: [q_rank + rank + dr (+ H), D] = W_dq over W_dkv (over W_g).  ``w_uk``: [H dn, rank]; ``w_uv``: [H dv, rank].
+    Without ``input_conv`` the mixer reads the rows in the activations' type; with it, the unrounded ones."""
 
     kernel_libraries = ("attention_latent", "gemm_simt")
     kernel_libraries_bf16 = ("gemm_stream",)
@@ -58,9 +61,11 @@ class LatentAttention(InputConvMixer):
     def __init__(self, w_down: torch.Tensor, q_norm_weight: torch.Tensor, w_uq: torch.Tensor, kv_norm_weight: torch.Tensor,
                  w_uk: torch.Tensor, w_uv: torch.Tensor, w_o: torch.Tensor, sink: torch.Tensor | None, heads: int, dim: int,
                  rot_dim: int, vdim: int, q_rank: int, kv_rank: int, scale: float, rot_base: float, rot_dims: int, eps: float,
-                 input_conv: ResidualShortConv | None = None):
+                 input_conv: ResidualShortConv | None = None, window: int | None = None, pairing: str = "pairs", gated: bool = False):
         H, dn, dr, dv = heads, dim, rot_dim, vdim
-        ok = (w_down.shape[0] == q_rank + kv_rank + dr and tuple(w_uq.shape) == (H * (dn + dr), q_rank)
+        if pairing not in K.ROPE_PAIRINGS or (window is not None and window < 1):
+            raise ValueError(f"pairing {pairing!r} (halves, pairs) is unknown or the window {window} is not positive")
+        ok = (w_down.shape[0] == q_rank + kv_rank + dr + (H if gated else 0) and tuple(w_uq.shape) == (H * (dn + dr), q_rank)
               and tuple(w_uk.shape) == (H * dn, kv_rank) and tuple(w_uv.shape) == (H * dv, kv_rank)
               and w_o.shape[1] == H * dv and q_norm_weight.numel() == q_rank and kv_norm_weight.numel() == kv_rank
               and (sink is None or sink.numel() == H))
@@ -83,10 +88,13 @@ class LatentAttention(InputConvMixer):
         self.inv_freq = rotary_frequencies(rot_base, rot_dims).to(w_down.device) if rot_dims else \
             torch.zeros(1, dtype=torch.float32, device=w_down.device)
         self.input_conv = input_conv
+        self.needs_f32_input = input_conv is not None
+        self.window, self.pairing, self.gated = window, pairing, bool(gated)
         self._planner = plan_head_groups(H)
 
     def kv_need(self) -> KVNeed:
-        return KVNeed(1, self.kv_rank + self.rot_dim, Retention.all(), planes=1)
+        keep = Retention.all() if self.window is None else Retention.window(self.window)
+        return KVNeed(1, self.kv_rank + self.rot_dim, keep, planes=1)
 
     def step_planners(self):
         # the attention part's planner gives the rows of the single decoded tokens of a mixed step
@@ -107,48 +115,55 @@ class LatentAttention(InputConvMixer):
         blocks = served * -(-H // per_block)
         want = max(1, (self.SPLIT_ROUNDS * K.sm_count()) // max(blocks, 1))
         tile = K.LATENT_KEY_TILE
-        per_split = -(-ctx.max_kv_len // want)  # keys each range would hold, rounded up to whole tiles below
+        seen = ctx.max_kv_len if self.window is None else min(ctx.max_kv_len, self.window)
+        per_split = -(-seen // want)  # keys each range would hold, rounded up to whole tiles below
         split_keys = max(self.MIN_SPLIT_KEYS, -(-per_split // tile) * tile)
-        splits = -(-ctx.max_kv_len // split_keys)
+        splits = -(-ctx.max_kv_len // split_keys)  # ranges are aligned to absolute positions: a window can straddle one more
+        if self.window is not None:
+            splits = min(splits, (seen - 1) // split_keys + 2)
         part_acc = part_ml = None
         if splits > 1:
             part_acc = ctx.workspace.get("latent_part_acc", served * H * splits * self.kv_rank, torch.float32)
             part_ml = ctx.workspace.get("latent_part_ml", served * H * splits * 2, torch.float32)
         K.attention_latent(q_lat, q_rot, cache.pages, cache.block_table, ctx.req_of_token, ctx.positions, self.sink, out_lat,
-                           self.scale, ctx.status, rows, n_rows, splits, split_keys, part_acc, part_ml)
+                           self.scale, ctx.status, rows, n_rows, splits, split_keys, part_acc, part_ml, self.window or 0)
 
-    def _portion(self, ctx: StepContext, cache: LayerCache, r: int, n0: int, T: int, start: int, q_full, rows_out) -> None:
+    def _portion(self, ctx: StepContext, cache: LayerCache, r: int, n0: int, T: int, start: int, q_full, rows_out, gate) -> None:
         """One request's prompt portion (rows n0 .. n0 + T, positions start ..) on the tensor cores: the request's cached
         rows gathered, every head's keys and values up-projected from them (the library's product), scores and weighted
         sums as per-head products (the library's, bfloat16 in, 32-bit sums), and between them this package's softmax
-        with the causal edge and the sink, in 32-bit."""
+        with the causal edge, the window and the sink, in 32-bit.  ``gate``: (rows, first column) of the heads' gates, or None."""
         dt, dev = q_full.dtype, q_full.device
         H, dn, dr, dv = self.heads, self.dim, self.rot_dim, self.vdim
-        keys = start + T
+        k0 = 0 if self.window is None else max(0, start - self.window + 1)  # the first key the portion sees
+        keys = start + T - k0
         L = -(-keys // 8) * 8  # rows in multiples of 8 for the products; the padding is zero and no query sees it
         c = torch.empty((L, self.kv_rank), dtype=dt, device=dev)
         kr = torch.empty((L, dr), dtype=dt, device=dev)
         c[keys:].zero_()
         kr[keys:].zero_()
-        K.latent_gather(cache.pages, cache.block_table[r], c[:keys], kr[:keys], ctx.status)
+        K.latent_gather(cache.pages, cache.block_table[r], c[:keys], kr[:keys], ctx.status, k0)
         kv_up = linear(ctx, c, self.w_ukv, dt)  # [L, H dn + H dv]
         k = torch.empty((H, L, dn + dr), dtype=dt, device=dev)
         K.latent_key_assemble(kv_up, kr, k, H, dn)
         v = kv_up[:, H * dn:].unflatten(1, (H, dv)).permute(1, 0, 2)  # [H, L, dv], a view
-        # query tiles: each sees the keys up to its own last row only (the rest of the causal triangle is not computed)
+        # query tiles: each sees the keys from its first row's window to its own last row only (the rest of the causal
+        # triangle is not computed)
         tile = max(16, min(self.QUERY_TILE, self.SCORE_TILE_BYTES // (4 * H * L)))
         for t0 in range(0, T, tile):
             t1 = min(T, t0 + tile)
-            Lt = min(L, -(-(start + t1) // 8) * 8)
-            scores = torch.bmm(q_full[:, n0 + t0:n0 + t1], k[:, :Lt].transpose(1, 2), out_dtype=torch.float32)  # [H, t, Lt]
+            lo = 0 if self.window is None else max(0, start + t0 - self.window + 1 - k0) // 8 * 8
+            hi = min(L, -(-(start + t1 - k0) // 8) * 8)
+            scores = torch.bmm(q_full[:, n0 + t0:n0 + t1], k[:, lo:hi].transpose(1, 2), out_dtype=torch.float32)  # [H, t, hi - lo]
             probs = torch.empty(scores.shape, dtype=dt, device=dev)
-            K.causal_sink_softmax(scores, self.sink, self.scale, start + t0, probs)
-            o = torch.bmm(probs, v[:, :Lt])  # [H, t, dv]
-            K.heads_to_rows(o, rows_out[n0 + t0:n0 + t1])
+            K.causal_sink_softmax(scores, self.sink, self.scale, start + t0, probs, k0 + lo, self.window or 0)
+            o = torch.bmm(probs, v[:, lo:hi])  # [H, t, dv]
+            K.heads_to_rows(o, rows_out[n0 + t0:n0 + t1], None if gate is None else K.rows_view(*gate, row=n0 + t0))
 
     def forward(self, ctx: StepContext, h, cache: LayerCache, h32: torch.Tensor | None = None):
-        dt, dev = ctx.runtime.dtype, h32.device
-        a, _ = self.read_input(ctx, h32, cache)
+        dt = ctx.runtime.dtype
+        a = h if self.input_conv is None and h is not None else self.read_input(ctx, h32, cache)[0]
+        dev = a.device
         n, H = a.shape[0], self.heads
         offsets = ctx.arrays[self._planner.array_name]
         # prompt portions in bfloat16 go to the tensor cores, request by request (their sizes are read on the host: such
@@ -160,7 +175,8 @@ class LatentAttention(InputConvMixer):
         with scope("rope"):  # both latents' norms, the shared key part's rotation and the page write in one kernel
             K.latent_kv_prep(down.data, down.splits, self.q_norm_weight, self.kv_norm_weight, self.eps, self.inv_freq,
                              self.rot_dims, cq, cache.pages if cache.writes else None, cache.block_table if cache.writes else None,
-                             ctx.req_of_token, ctx.positions, self.q_rank, self.kv_rank, self.rot_dim, ctx.status)
+                             ctx.req_of_token, ctx.positions, self.q_rank, self.kv_rank, self.rot_dim, ctx.status, self.pairing)
+        gate = (down.data, down.splits, self.q_rank + self.kv_rank + self.rot_dim) if self.gated else None
         with scope("qkv_matmul"):
             q = as_rows(linear(ctx, cq, self.w_uq, torch.float32, partials=True))
         q_nope = torch.empty((H, n, self.dim), dtype=dt, device=dev)
@@ -168,7 +184,7 @@ class LatentAttention(InputConvMixer):
         q_full = torch.empty((H, n, self.dim + self.rot_dim), dtype=dt, device=dev) if portions else None
         with scope("rope"):
             K.latent_q_prep(q.data, q.splits, self.inv_freq, self.rot_dims, ctx.positions, q_nope, q_rot, H, self.dim,
-                            self.rot_dim, q_full)
+                            self.rot_dim, q_full, self.pairing)
         rows = torch.empty((n, H * self.vdim), dtype=dt, device=dev)
         with scope("attention"):
             singles = len(ctx.host_arrays["attn_single_rows"]) if portions else n
@@ -181,12 +197,12 @@ class LatentAttention(InputConvMixer):
                 else:
                     self._latent_space(ctx, q_lat.view(H, n, self.kv_rank), q_rot, cache, out_lat)
                 v = grouped_linear(ctx, out_lat.view(H * n, self.kv_rank), self.w_uv, offsets, dt, largest_group=n)
-                K.heads_to_rows(v.view(H, n, self.vdim), rows)
+                K.heads_to_rows(v.view(H, n, self.vdim), rows, None if gate is None else K.rows_view(*gate))
             if portions:
                 n0 = 0
                 for r, (T, start) in enumerate(zip(ctx.host_q_lens, ctx.host_q_start)):
                     if T > 1:
-                        self._portion(ctx, cache, r, n0, T, start, q_full, rows)
+                        self._portion(ctx, cache, r, n0, T, start, q_full, rows, gate)
                     n0 += T
         with scope("projection"):
             return linear(ctx, rows, self.w_o, torch.float32, partials=True)

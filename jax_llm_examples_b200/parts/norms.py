@@ -28,7 +28,7 @@ class RMSNorm(Norm):
         out32 = torch.empty((n, x.shape[1]), dtype=torch.float32, device=dev) if want_f32 else None
         # a sum of terms (an expert layer's rows still in expert order) is added term by term in the kernel
         # (the kernel takes so many terms, rows per token and partials; beyond that the sum is made by its producer)
-        if isinstance(delta, RowSum) and len(delta.terms) <= K.DELTA_MAX_TERMS and all(t.k <= 16 for t in delta.terms) and \
+        if isinstance(delta, RowSum) and len(delta.terms) <= K.DELTA_MAX_TERMS and all(t.k <= 16 and t.weights is None for t in delta.terms) and \
                 sum((t.k if t.index is not None else 1) * t.splits for t in delta.terms) <= K.DELTA_MAX_STREAMS:
             terms = [(t.data, t.splits, t.index, t.k, t.base) for t in delta.terms]
         else:
@@ -107,7 +107,7 @@ def add_to_residual(x: torch.Tensor, delta, *, pre_weight=None, pre_groups: int 
             delta = Rows(delta.materialize(), 1)
         else:
             K.group_norm(x, delta.rows.data, delta.rows.splits, delta.bias, delta.weight, delta.groups, delta.mult,
-                         pre_weight, pre_groups, pre_norm, eps, out, out32, row_index)
+                         pre_weight, pre_groups, pre_norm, eps, out, out32, row_index, **delta.gather())
             return
     d = as_rows(delta)
     if d is not None and d.data.dtype != torch.float32:
