@@ -480,12 +480,16 @@ def run_compare(args) -> dict:
     feed-forward size.
     --compare koduzen: the same for Koduzen beside Makisun (the closest: windowed attention over the same pages, a
     recurrence on the same decay-scan kernel, routed experts whose outputs are weighted), both with a dense feed-forward
-    and with 16 routed experts in every second layer, at equal width, depth, head count and feed-forward size."""
+    and with 16 routed experts in every second layer, at equal width, depth, head count and feed-forward size.
+    --compare marinex: the same for Marinex (16 experts in every layer) beside the three models that have its mechanisms'
+    nearest relatives: Koduzen with 16 experts (group-limited experts, attention behind a weighted norm and a rotation),
+    Tebivik (latent attention, norms on the sublayers' outputs) and a dense Llama-4-style decoder (attention over all
+    earlier positions), at equal width, depth, head count and feed-forward size."""
     import torch
 
     import jax_llm_examples_b200 as J
     from jax_llm_examples_b200 import tracing
-    from jax_llm_examples_b200.config.presets import dense_llama_sized, koduzen_sized, makisun_sized, tebivik_sized, vofusun_sized
+    from jax_llm_examples_b200.config.presets import dense_llama_sized, koduzen_sized, makisun_sized, marinex_sized, tebivik_sized, vofusun_sized
 
     peaks, peak_src = _peaks()
     hbm, tflops = peaks["hbm_gbs"] * 1e9, peaks["bf16_tflops"] * 1e12
@@ -496,7 +500,8 @@ def run_compare(args) -> dict:
     if args.layers:
         sizes = [(w, args.layers, h, f) for w, _, h, f in sizes]
     what = {"tebivik": "Tebivik beside a dense Llama-4-style decoder", "makisun": "Makisun beside Tebivik",
-            "vofusun": "Vofusun beside Makisun", "koduzen": "Koduzen beside Makisun"}[args.compare]
+            "vofusun": "Vofusun beside Makisun", "koduzen": "Koduzen beside Makisun",
+            "marinex": "Marinex beside Koduzen, Tebivik and a dense Llama-4-style decoder"}[args.compare]
     out = {"metric": "prefill and decode throughput, " + what, "unit": "tok/s", "n_gpus": 1,
            "dtype": "bf16", "data": "synthetic (random weights and tokens)", "peaks": peaks, "peaks_source": peak_src,
            "config": {"prefill_tokens": P, "decode_batch": B, "decode_context": C, "l2": "a 256 MiB buffer is written between timed steps"},
@@ -661,6 +666,62 @@ def run_compare(args) -> dict:
         }
         out["sizes"].append({"width": width, "layers": layers, "heads": heads, "ff": ff, "koduzen": k, "makisun": m,
                              "koduzen_16_experts": kx, "makisun_16_experts": mx, "fraction_of_measured_roofline": roof})
+    for width, layers, heads, ff in sizes if args.compare == "marinex" else ():
+        x, k = measure(marinex_sized(width, layers, heads, ff)), measure(koduzen_sized(width, layers, heads, ff, experts=16))
+        t, l = measure(tebivik_sized(width, layers, heads, ff)), measure(dense_llama_sized(width, layers, heads, ff))
+        # Marinex's layers in turn: attention over all positions, latent attention over a window
+        n_att, n_lat = (layers + 1) // 2, layers // 2
+        t_runs = layers + layers // 2  # the first half of Tebivik's layers runs twice
+        t_lat = sum(1 for i in range(layers) if i % 2 == 0) + sum(1 for i in range(layers // 2) if i % 2 == 0)
+        k_ret = sum(1 for i in range(layers) if i % 4 == 2)
+        k_own = sum(1 for i in range(layers) if i % 4 in (0, 3))
+        k_moe = layers // 2
+        dh, hkv, window, rank, dr, fe, S = 128, max(heads // 4, 1), 1024, 512, 64, ff // 4, 2
+        seen = sum(i + 1 for i in range(P))
+        tiles = lambda lo: sum(min(512, P - t0) * (min(P, t0 + 512) - lo(t0)) for t0 in range(0, P, 512))  # scores of a portion's query tiles
+        score_bytes = lambda runs, lo: runs * heads * tiles(lo) * 6  # float32 in, bfloat16 out
+        in_window = lambda t0: max(0, t0 - window + 1) // 8 * 8
+        experts_b = 16 * (1 - (1 - 2 / 16) ** B)  # experts that B tokens' choices touch, on average
+        norm = lambda runs, n: (2 * runs + 1) * n * width * 14
+        rope = lambda n_full, n_q: P * (n_full * (heads + 2 * hkv) + n_q * heads) * dh * 6
+        pm = lambda m, name: m["prefill_kernels_ms"].get(name, 0)  # noqa: E731
+        dm = lambda m, name: m["decode_kernels_ms"].get(name, 0)  # noqa: E731
+        roof = {
+            "decode": {
+                "marinex attention_decode": frac(dm(x, "jlx_attention_decode"), n_att * B * C * 2 * hkv * dh * 2),
+                "llama attention_decode": frac(dm(l, "jlx_attention_decode"), layers * B * C * 2 * hkv * dh * 2),
+                "marinex attention_latent": frac(dm(x, "jlx_attention_latent"), n_lat * B * min(C, window) * (rank + dr) * 2),
+                "tebivik attention_latent": frac(dm(t, "jlx_attention_latent"), t_lat * B * C * (rank + dr) * 2),
+                "marinex group_norm": frac(dm(x, "jlx_group_norm"), norm(layers, B)),
+                "tebivik group_norm": frac(dm(t, "jlx_group_norm"), norm(t_runs, B)),
+                "marinex router": frac(dm(x, "jlx_router"), layers * (B + 16) * width * 4),
+                "koduzen router": frac(dm(k, "jlx_router"), k_moe * (B + 18) * width * 4),
+                "marinex rope_half_kv_store": frac(dm(x, "jlx_rope_half_kv_store"), rope(n_att, 0) / P * B),
+                "koduzen rope_half_kv_store": frac(dm(k, "jlx_rope_half_kv_store"), rope(k_own, layers - k_ret - k_own) / P * B),
+                "marinex gemm_stream (all weights of the step)": frac(dm(x, "jlx_gemm_stream"), x["weights_gb"] * 1e9 - 32768 * width * 2 - layers * (16 - experts_b) * 2 * width * fe * 2),
+                "koduzen gemm_stream (all weights of the step)": frac(dm(k, "jlx_gemm_stream"), k["weights_gb"] * 1e9 - k_moe * (16 - experts_b) * 3 * width * fe * 2),
+            },
+            "prefill": {
+                "marinex attention_prefill_tc": frac(pm(x, "jlx_attention_prefill_tc"), 0, n_att * heads * seen * 4 * dh),
+                "llama attention_prefill_tc": frac(pm(l, "jlx_attention_prefill_tc"), 0, layers * heads * seen * 4 * dh),
+                "marinex causal_sink_softmax": frac(pm(x, "jlx_causal_sink_softmax"), score_bytes(n_lat, in_window)),
+                "tebivik causal_sink_softmax": frac(pm(t, "jlx_causal_sink_softmax"), score_bytes(t_lat, lambda t0: 0)),
+                "marinex group_norm": frac(pm(x, "jlx_group_norm"), norm(layers, P)),
+                "tebivik group_norm": frac(pm(t, "jlx_group_norm"), norm(t_runs, P)),
+                "marinex rope_half_kv_store": frac(pm(x, "jlx_rope_half_kv_store"), rope(n_att, 0)),
+                "koduzen rope_half_kv_store": frac(pm(k, "jlx_rope_half_kv_store"), rope(k_own, layers - k_ret - k_own)),
+                "marinex router": frac(pm(x, "jlx_router"), layers * P * width * 4),
+                "koduzen router": frac(pm(k, "jlx_router"), k_moe * P * width * 4),
+                "marinex experts gemm_stream": frac(pm(x, "jlx_gemm_stream"), 0, layers * P * 2 * 2 * width * fe * 2),
+                "koduzen experts gemm_stream": frac(pm(k, "jlx_gemm_stream"), 0, k_moe * P * 2 * 3 * width * fe * 2),
+                "marinex permute_scale": frac(pm(x, "jlx_permute_scale"), layers * P * width * (4 + 2 * 2)),
+                "koduzen permute_scale": frac(pm(k, "jlx_permute_scale"), k_moe * P * width * (4 + 2 * 2)),
+                "marinex bias_act": frac(pm(x, "jlx_bias_act"), layers * P * 2 * fe * 6),
+                "tebivik bias_act": frac(pm(t, "jlx_bias_act"), t_runs * P * ff * 6),
+            },
+        }
+        out["sizes"].append({"width": width, "layers": layers, "heads": heads, "ff": ff, "marinex": x, "koduzen_16_experts": k, "tebivik": t,
+                             "dense_llama": l, "fraction_of_measured_roofline": roof})
     for width, layers, heads, ff in sizes if args.compare == "makisun" else ():
         m, t = measure(makisun_sized(width, layers, heads, ff)), measure(tebivik_sized(width, layers, heads, ff))
         routed = measure(makisun_sized(width, layers, heads, ff, experts=16))
@@ -744,7 +805,7 @@ def main() -> int:
     ap.add_argument("--long-tokens", type=int, default=32768)
     ap.add_argument("--skip-e2e", action="store_true", help="skip the end-to-end run (for profiling captures)")
     ap.add_argument("--skip-prefill", action="store_true", help="skip the prefill measurement (for profiling captures)")
-    ap.add_argument("--compare", default=None, choices=["tebivik", "makisun", "vofusun", "koduzen"],
+    ap.add_argument("--compare", default=None, choices=["tebivik", "makisun", "vofusun", "koduzen", "marinex"],
                     help="instead of the benchmark: throughput of this architecture at real layer sizes beside the closest "
                     "model the framework had before (with --prefill-tokens, --batch, --context up to 4096, --layers)")
     args = ap.parse_args()

@@ -198,6 +198,37 @@ PRESETS["koduzen_tiny"] = {
                    "rot": {"base": 10000.0, "dims": 16, "scaling": {"factor": 4.0, "original": 64, "fast": 8.0, "slow": 1.0}}}},
     ],
 }
+def marinex_sized(width: int, layers: int, heads: int, ff: int, vocab: int = 32768, experts: int = 16) -> dict[str, Any]:
+    """A Marinex configuration at the layer sizes of a real model: soft-capped attention over all earlier positions (head
+    size 128, four query heads per key head, half of each head rotated) and latent attention over a window of 1024 (head
+    size 128 + 64 rotated, latent 512, query latent 3/8 of the width) in turn; in every layer a mixture of ``experts``
+    experts (top 2, in two groups of which one is kept, each expert a quarter of ``ff``)."""
+    moe = {"kind": "moe", "expert": {"ff": ff // 4}, "router": {"experts": experts, "top": 2, "groups": {"count": 2, "keep": 1}}}
+    att = {"type": "attention", "mlp": moe,
+           "mixer": {"heads": heads, "kv_heads": max(heads // 4, 1), "dim": 128, "vdim": 128, "rot": {"base": 250000.0, "dims": 64},
+                     "scale": 128 ** -0.5, "softcap": 20.0}}
+    lat = {"type": "latent_attention", "mlp": moe,
+           "mixer": {"heads": heads, "dim": 128, "rot_dim": 64, "vdim": 128, "q_rank": 3 * width // 8, "kv_rank": 512,
+                     "mask": {"size": 1024}, "scale": 192 ** -0.5, "rot": {"base": 10000.0, "dims": 64}}}
+    return {"architecture": "Marinex", "vocab": vocab, "width": width, "norm": {"eps": 1e-6},
+            "layers": [dict(att if i % 2 == 0 else lat) for i in range(layers)]}
+
+
+# Marinex, tiny: values of another size than keys, part of the head rotated, groups of experts, a layer without a feed-forward.
+PRESETS["marinex_tiny"] = {
+    "architecture": "Marinex", "vocab": 256, "width": 64, "norm": {"eps": 1e-5},
+    "layers": [
+        {"type": "attention", "mlp": {"kind": "moe", "expert": {"ff": 32}, "router": {"experts": 6, "top": 2, "groups": {"count": 3, "keep": 2}}},
+         "mixer": {"heads": 4, "kv_heads": 2, "dim": 16, "vdim": 24, "rot": {"base": 10000.0, "dims": 8}, "scale": 0.25, "softcap": 8.0}},
+        {"type": "latent_attention", "mlp": {"kind": "moe", "expert": {"ff": 24}, "router": {"experts": 4, "top": 1}},
+         "mixer": {"heads": 4, "dim": 16, "rot_dim": 8, "vdim": 16, "q_rank": 24, "kv_rank": 32, "mask": {"size": 24}, "scale": 0.2,
+                   "rot": {"base": 10000.0, "dims": 8}}},
+        {"type": "attention", "mlp": None,
+         "mixer": {"heads": 2, "kv_heads": 1, "dim": 32, "vdim": 32, "rot": {"base": 500.0, "dims": 32}, "scale": 0.2, "softcap": 12.0}},
+    ],
+}
+PRESETS["marinex_2k"] = marinex_sized(2048, 8, 16, 8192)
+PRESETS["marinex_4k"] = marinex_sized(4096, 8, 32, 14336)
 PRESETS["koduzen_2k"] = koduzen_sized(2048, 8, 16, 8192)
 PRESETS["koduzen_4k"] = koduzen_sized(4096, 8, 32, 14336)
 PRESETS["vofusun_2k"] = vofusun_sized(2048, 8, 16, 8192)
