@@ -16,6 +16,8 @@
 // Rotation: pairs (2i, 2i+1), or with `halves` (i, i + dims/2), i < dims/2, by the angle position * inv_freq[i] in 32-bit;
 // entries from `dims` on pass.
 #include "common.cuh"
+#include "mbarrier.cuh"
+#include "mma_sync.cuh"
 
 // The two entries that rotate together as pair i.
 __device__ __forceinline__ void rot_pair(int i, int rot_dims, int halves, int* a, int* b) {
@@ -39,19 +41,21 @@ __global__ void latent_kv_prep_kernel(const float* __restrict__ proj, int splits
   JLX_TL(TL_ROPE);
   pdl_launch_dependents_if_small();
   pdl_wait();
+  extern __shared__ float sums[];  // the latent's entries, split-K partials added
   __shared__ float scratch[33];
   const int n = blockIdx.x;
   const float* row = proj + (size_t)n * ld;
-  // the query's latent
-  float ss = 0.f;
-  for (int i = threadIdx.x; i < q_rank; i += blockDim.x) {
-    const float v = row_sum_splits(row + i, splits, split_stride);
-    ss = fmaf(v, v, ss);
+  if (blockIdx.y == 0) {  // the query's latent
+    float ss = 0.f;
+    for (int i = threadIdx.x; i < q_rank; i += blockDim.x) {
+      const float v = row_sum_splits(row + i, splits, split_stride);
+      sums[i] = v;
+      ss = fmaf(v, v, ss);
+    }
+    const float rms = sqrtf(block_sum(ss, scratch) / (float)q_rank + eps);
+    for (int i = threadIdx.x; i < q_rank; i += blockDim.x) cq[(size_t)n * q_rank + i] = from_f32<TO>(sums[i] / rms * q_norm_w[i]);
+    return;
   }
-  float rms = sqrtf(block_sum(ss, scratch) / (float)q_rank + eps);
-  for (int i = threadIdx.x; i < q_rank; i += blockDim.x)
-    cq[(size_t)n * q_rank + i] = from_f32<TO>(row_sum_splits(row + i, splits, split_stride) / rms * q_norm_w[i]);
-  if (!pages) return;
   const int p = positions[n], r = req_of_token[n];
   const int page = block_table[(size_t)r * bt_stride + p / page_size];
   if (page < 0 || page >= num_pages) {
@@ -60,14 +64,12 @@ __global__ void latent_kv_prep_kernel(const float* __restrict__ proj, int splits
   }
   TO* dst = pages + ((size_t)page * page_size + p % page_size) * (rank + dr);
   // the keys' and values' latent
-  ss = 0.f;
+  float ss = 0.f;
   for (int i = threadIdx.x; i < rank; i += blockDim.x) {
     const float v = row_sum_splits(row + q_rank + i, splits, split_stride);
+    sums[i] = v;
     ss = fmaf(v, v, ss);
   }
-  rms = sqrtf(block_sum(ss, scratch) / (float)rank + eps);
-  for (int i = threadIdx.x; i < rank; i += blockDim.x)
-    dst[i] = from_f32<TO>(row_sum_splits(row + q_rank + i, splits, split_stride) / rms * kv_norm_w[i]);
   // the shared rotated key part
   const float* kr = row + q_rank + rank;
   for (int i = threadIdx.x; i < rot_dims / 2; i += blockDim.x) {
@@ -80,6 +82,8 @@ __global__ void latent_kv_prep_kernel(const float* __restrict__ proj, int splits
     dst[rank + ib] = from_f32<TO>(v * cs + u * sn);
   }
   for (int i = rot_dims + threadIdx.x; i < dr; i += blockDim.x) dst[rank + i] = from_f32<TO>(row_sum_splits(kr + i, splits, split_stride));
+  const float rms = sqrtf(block_sum(ss, scratch) / (float)rank + eps);
+  for (int i = threadIdx.x; i < rank; i += blockDim.x) dst[i] = from_f32<TO>(sums[i] / rms * kv_norm_w[i]);
 }
 
 JLX_API int jlx_latent_kv_prep(const float* proj, int splits, long long split_stride, const float* q_norm_w,
@@ -91,9 +95,12 @@ JLX_API int jlx_latent_kv_prep(const float* proj, int splits, long long split_st
   JLX_REQUIRE(rot_dims >= 0 && rot_dims <= dr && rot_dims % 2 == 0, "latent_kv_prep: %d rotated entries of %d", rot_dims, dr);
   JLX_REQUIRE(eps > 0.f, "latent_kv_prep: eps must be positive");
   JLX_REQUIRE(ld >= q_rank + rank + dr, "latent_kv_prep: rows of %d entries do not hold %d + %d + %d", ld, q_rank, rank, dr);
+  const int widest = q_rank > rank ? q_rank : rank;
+  JLX_REQUIRE((size_t)widest * 4 <= 48 * 1024, "latent_kv_prep: a latent of %d entries does not fit shared memory", widest);
   if (N == 0) return 0;
   JLX_DISPATCH_DTYPE(dtype, TO, {
-    JLX_CUDA(jlx_launch_pdl(latent_kv_prep_kernel<TO>, dim3(N), dim3(128), 0, stream, proj, splits, split_stride, q_norm_w, kv_norm_w,
+    // a block for the query's latent and one for the cached row
+    JLX_CUDA(jlx_launch_pdl(latent_kv_prep_kernel<TO>, dim3(N, pages ? 2 : 1), dim3(widest >= 512 ? 256 : 128), sizeof(float) * (size_t)widest, stream, proj, splits, split_stride, q_norm_w, kv_norm_w,
                             eps, inv_freq, rot_dims, (TO*)cq, (TO*)pages, block_table, bt_stride, req_of_token, positions, q_rank,
                             rank, dr, page_size, num_pages, ld, halves, status));
   });
@@ -169,6 +176,7 @@ JLX_API int jlx_latent_q_prep(const float* q, int splits, long long split_stride
 #define LAT_TILE 32
 #define LAT_WARPS 8
 #define LAT_MAX_R32 32  // latent size up to 1024
+#define LAT_COMBINE_CACHE 512
 
 template <typename TC, typename TO, int HPW, int R32>
 __global__ void attention_latent_kernel(const float* __restrict__ q_lat, const float* __restrict__ q_rot,
@@ -332,6 +340,225 @@ __global__ void attention_latent_kernel(const float* __restrict__ q_lat, const f
   }
 }
 
+// ---- the same on the tensor cores (mma.sync), for a bfloat16 cache: the decoded tokens of a step
+// One block of four warps serves one query token, up to 16 heads (the M rows of the products) and one range of keys.
+// Tiles of 32 keys come by cp.async, found row by row through the block table, two in flight; a key's row [c | k_rot] in
+// shared memory is padded by 16 bytes so that ldmatrix meets no bank twice.
+//   scores   warp w takes keys [8 w, 8 w + 8) of the tile: the whole row against all 16 queries (bfloat16, 32-bit sums)
+//   softmax  the scores meet in shared memory; every warp keeps the same running maximum and sum per head (32-bit)
+//   values   warp w takes the latent's 16-column pieces w, w + 4, ...: P (bfloat16) times the tile's rows
+// When every served token is its request's only one of the step (`single`), everything but its own row is older than the
+// step: tiles that end below it are asked for before the wait for the predecessor.  Rows outside [lo, t_end] are zeros in shared memory and masked.
+#define LATM_KEYS LAT_TILE
+#define LATM_THREADS 128
+
+template <typename TO, int PIECES>
+__global__ void __launch_bounds__(LATM_THREADS)
+attention_latent_mma_kernel(const float* __restrict__ q_lat, const float* __restrict__ q_rot, const bf16* __restrict__ pages,
+                            const int* __restrict__ block_table, int bt_stride, const int* __restrict__ req_of_token,
+                            const int* __restrict__ positions, const float* __restrict__ sink, TO* __restrict__ out_lat, int N,
+                            int H, int rank, int dr, int page_size, int num_pages, float scale, const int* __restrict__ rows,
+                            int splits, int split_keys, float* __restrict__ part_acc, float* __restrict__ part_ml, int ldk,
+                            int window, int single, int* status) {
+  JLX_TL(TL_ATTN_GENERIC);
+  extern __shared__ __align__(16) uint8_t smem_bytes[];
+  __shared__ float sc[2][16][LATM_KEYS + 1];
+  const int dk = rank + dr, dkp = (dk + 15) & ~15;  // products take 16 columns at a time: the rest of a row is zero
+  bf16* qs = reinterpret_cast<bf16*>(smem_bytes);   // [16][ldk]
+  bf16* ks = qs + 16 * ldk;                          // [2][LATM_KEYS][ldk]
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const int n = rows ? rows[blockIdx.x] : blockIdx.x, h0 = blockIdx.y * 16, z = blockIdx.z;
+  const int p = positions[n], r = req_of_token[n];
+  const int lo = window > 0 ? max(0, p - window + 1) : 0;
+  int t_begin = lo / LATM_KEYS * LATM_KEYS, t_end = p;
+  if (splits > 1) {
+    const int range = (lo / split_keys + z) * split_keys;
+    t_begin = max(t_begin, range);
+    t_end = min(p, range + split_keys - 1);
+  }
+  const int n_tiles = t_begin <= t_end ? (t_end - t_begin) / LATM_KEYS + 1 : 0;
+  const int* table = block_table + (size_t)r * bt_stride;
+  const int chunks = dk >> 3;  // 16-byte pieces of a row
+  bool bad_page = false;
+  auto load = [&](int t) {  // a warp copies a row with neighbouring lanes
+    bf16* dst = ks + (size_t)(t & 1) * LATM_KEYS * ldk;
+    for (int j = warp; j < LATM_KEYS; j += LATM_THREADS / 32) {
+      const int pos = t_begin + t * LATM_KEYS + j;
+      bool valid = pos >= lo && pos <= t_end;
+      const bf16* src = pages;
+      if (valid) {
+        const int page = table[pos / page_size];
+        if (page < 0 || page >= num_pages) { bad_page = true; valid = false; }
+        else src = pages + ((size_t)page * page_size + pos % page_size) * dk;
+      }
+      for (int c = lane; c < chunks; c += 32) cp_async16(smem_u32(dst + (size_t)j * ldk + c * 8), valid ? src + c * 8 : pages, valid);
+    }
+  };
+  // zeros behind every row up to a multiple of 16 columns, once
+  if (dkp > dk)
+    for (int i = threadIdx.x; i < (2 * LATM_KEYS + 16) * 8; i += LATM_THREADS) qs[(size_t)(i >> 3) * ldk + dk + (i & 7)] = __float2bfloat16_rn(0.f);
+  auto old_tile = [&](int t) { return t_begin + (t + 1) * LATM_KEYS <= p; };  // ends below the token's own row
+  const bool early0 = single && n_tiles > 0 && old_tile(0), early1 = early0 && n_tiles > 1 && old_tile(1);
+  if (early0) load(0);
+  if (early0) cp_async_commit();
+  if (early1) load(1);
+  if (early1) cp_async_commit();
+  pdl_launch_dependents_if_small();
+  pdl_wait();
+  if (n_tiles > 0 && !early0) { load(0); cp_async_commit(); }
+  if (!early1) {
+    if (n_tiles > 1) load(1);
+    cp_async_commit();  // (maybe empty: the waits below count groups)
+  }
+  for (int u = warp; u < 16; u += LATM_THREADS / 32) {  // heads beyond H get a zero query: they run along and write nothing
+    const int h = h0 + u;
+    for (int d = lane; d < dk; d += 32) {
+      float v = 0.f;
+      if (h < H) v = d < rank ? q_lat[((size_t)h * N + n) * rank + d] : q_rot[((size_t)n * H + h) * dr + (d - rank)];
+      qs[(size_t)u * ldk + d] = __float2bfloat16_rn(v);
+    }
+  }
+  const int g0 = lane >> 2, g1 = g0 + 8;  // this thread's two heads
+  const float sc2 = scale * 1.4426950408889634f;
+  const bool has_sink = sink != nullptr && z == 0;
+  float m[2], l[2];  // base-2 running maximum and sum
+#pragma unroll
+  for (int u = 0; u < 2; ++u) {
+    const int h = h0 + (u ? g1 : g0);
+    m[u] = has_sink && h < H ? sink[h] * 1.4426950408889634f : -INFINITY;
+    l[u] = has_sink ? 1.f : 0.f;
+  }
+  float o[PIECES][2][4];
+#pragma unroll
+  for (int i = 0; i < PIECES; ++i)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) o[i][0][e] = o[i][1][e] = 0.f;
+
+  for (int t = 0; t < n_tiles; ++t) {
+    if (t == 0) cp_async_wait<1>();
+    else cp_async_wait<0>();
+    __syncthreads();  // tile t has landed for everyone; everyone is done with tile t - 1
+    if (t > 0) {
+      if (t + 1 < n_tiles) load(t + 1);
+      cp_async_commit();
+    }
+    const bf16* kt = ks + (size_t)(t & 1) * LATM_KEYS * ldk;
+    // scores of this warp's 8 keys; two chains of sums
+    float s0[4] = {0.f, 0.f, 0.f, 0.f}, s1[4] = {0.f, 0.f, 0.f, 0.f};
+    const uint32_t qa = smem_u32(qs + (size_t)(lane & 15) * ldk + (lane >> 4) * 8);
+    const uint32_t ka = smem_u32(kt + (size_t)(warp * 8 + (lane & 7)) * ldk + (lane >> 3) * 8);
+    int d = 0;
+    for (; d + 32 <= dkp; d += 32) {
+      uint32_t a[4], b[4], c[4];
+      ldmatrix_x4(qa + d * 2, a[0], a[1], a[2], a[3]);
+      ldmatrix_x4(qa + d * 2 + 32, c[0], c[1], c[2], c[3]);
+      ldmatrix_x4(ka + d * 2, b[0], b[1], b[2], b[3]);
+      mma_bf16(s0, a, b[0], b[1]);
+      mma_bf16(s1, c, b[2], b[3]);
+    }
+    if (d < dkp) {  // 16 columns are left (lanes 16.. read columns that are in the row's padding or the next row: unused)
+      uint32_t a[4], b[4];
+      ldmatrix_x4(qa + d * 2, a[0], a[1], a[2], a[3]);
+      ldmatrix_x4(smem_u32(kt + (size_t)(warp * 8 + (lane & 7)) * ldk + ((lane >> 3) & 1) * 8) + d * 2, b[0], b[1], b[2], b[3]);
+      mma_bf16(s0, a, b[0], b[1]);
+    }
+    {
+      float* w0 = &sc[t & 1][g0][warp * 8 + (lane & 3) * 2];
+      float* w1 = &sc[t & 1][g1][warp * 8 + (lane & 3) * 2];
+      w0[0] = s0[0] + s1[0]; w0[1] = s0[1] + s1[1];
+      w1[0] = s0[2] + s1[2]; w1[1] = s0[3] + s1[3];
+    }
+    __syncthreads();
+    // every warp: the 32 keys' weights of its lanes' two heads, in the layout of the product's A operand
+    float pv[2][2][4];  // [16-key step][head][columns 2 (lane & 3) + {0, 1, 8, 9}]
+    float mx[2] = {m[0], m[1]};
+    const int tile_key = t_begin + t * LATM_KEYS;
+#pragma unroll
+    for (int st = 0; st < 2; ++st)
+#pragma unroll
+      for (int u = 0; u < 2; ++u)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const int j = st * 16 + (lane & 3) * 2 + (e & 1) + (e >> 1) * 8;
+          const bool seen = tile_key + j >= lo && tile_key + j <= t_end;
+          const float s = seen ? sc[t & 1][u ? g1 : g0][j] * sc2 : -INFINITY;
+          pv[st][u][e] = s;
+          mx[u] = fmaxf(mx[u], s);
+        }
+    float corr[2], rs[2] = {0.f, 0.f};
+#pragma unroll
+    for (int u = 0; u < 2; ++u) {
+      mx[u] = fmaxf(mx[u], __shfl_xor_sync(0xffffffffu, mx[u], 1));
+      mx[u] = fmaxf(mx[u], __shfl_xor_sync(0xffffffffu, mx[u], 2));  // a tile has a visible key: never -infinity
+      corr[u] = exp2f(m[u] - mx[u]);
+    }
+#pragma unroll
+    for (int st = 0; st < 2; ++st)
+#pragma unroll
+      for (int u = 0; u < 2; ++u)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          pv[st][u][e] = exp2f(pv[st][u][e] - mx[u]);
+          rs[u] += pv[st][u][e];
+        }
+#pragma unroll
+    for (int u = 0; u < 2; ++u) {
+      rs[u] += __shfl_xor_sync(0xffffffffu, rs[u], 1);
+      rs[u] += __shfl_xor_sync(0xffffffffu, rs[u], 2);
+      l[u] = l[u] * corr[u] + rs[u];
+      m[u] = mx[u];
+    }
+    uint32_t pa[2][4];
+#pragma unroll
+    for (int st = 0; st < 2; ++st) {
+      pa[st][0] = pack_bf16(pv[st][0][0], pv[st][0][1]);
+      pa[st][1] = pack_bf16(pv[st][1][0], pv[st][1][1]);
+      pa[st][2] = pack_bf16(pv[st][0][2], pv[st][0][3]);
+      pa[st][3] = pack_bf16(pv[st][1][2], pv[st][1][3]);
+    }
+#pragma unroll
+    for (int i = 0; i < PIECES; ++i) {
+      const int col = (warp + i * 4) * 16;
+      if (col >= rank) break;
+#pragma unroll
+      for (int q = 0; q < 2; ++q) {
+        o[i][q][0] *= corr[0]; o[i][q][1] *= corr[0]; o[i][q][2] *= corr[1]; o[i][q][3] *= corr[1];
+      }
+#pragma unroll
+      for (int st = 0; st < 2; ++st) {
+        uint32_t b0, b1, b2, b3;
+        ldmatrix_x4_trans(smem_u32(kt + (size_t)(st * 16 + ((lane >> 3) & 1) * 8 + (lane & 7)) * ldk + col + (lane >> 4) * 8), b0, b1, b2, b3);
+        mma_bf16(o[i][0], pa[st], b0, b1);
+        mma_bf16(o[i][1], pa[st], b2, b3);
+      }
+    }
+  }
+  cp_async_wait<0>();
+  if (bad_page) atomicOr(status, JLX_STATUS_BAD_PAGE);
+#pragma unroll
+  for (int u = 0; u < 2; ++u) {
+    const int h = h0 + (u ? g1 : g0);
+    if (h >= H) continue;
+    const size_t slot = ((size_t)blockIdx.x * H + h) * splits + z;
+    if (splits > 1 && warp == 0 && (lane & 3) == 0) {
+      part_ml[2 * slot] = m[u] * 0.6931471805599453f;  // the combine kernel works with natural exponentials
+      part_ml[2 * slot + 1] = l[u];
+    }
+    const float inv = 1.f / l[u];
+#pragma unroll
+    for (int i = 0; i < PIECES; ++i)
+#pragma unroll
+      for (int q = 0; q < 2; ++q)
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+          const int c = (warp + i * 4) * 16 + q * 8 + (lane & 3) * 2 + e;
+          if (c >= rank) continue;
+          if (splits > 1) part_acc[slot * rank + c] = o[i][q][u * 2 + e];
+          else out_lat[((size_t)h * N + n) * rank + c] = from_f32<TO>(o[i][q][u * 2 + e] * inv);
+        }
+  }
+}
+
 // out = sum_z acc_z exp(m_z - m) / sum_z l_z exp(m_z - m), m = max_z m_z, the splits in ascending order.
 template <typename TO>
 __global__ void attention_latent_combine_kernel(const float* __restrict__ part_acc, const float* __restrict__ part_ml,
@@ -343,6 +570,7 @@ __global__ void attention_latent_combine_kernel(const float* __restrict__ part_a
   const int b = blockIdx.x, h = blockIdx.y;
   const int n = rows ? rows[b] : b;
   const size_t slot0 = ((size_t)b * H + h) * splits;
+  __shared__ float wgt[LAT_COMBINE_CACHE];  // the ranges' shares of the sum
   float m = -INFINITY;
   for (int z = 0; z < splits; ++z) m = fmaxf(m, part_ml[2 * (slot0 + z)]);
   float l = 0.f;
@@ -350,23 +578,47 @@ __global__ void attention_latent_combine_kernel(const float* __restrict__ part_a
     const float mz = part_ml[2 * (slot0 + z)];
     if (mz > -INFINITY) l += part_ml[2 * (slot0 + z) + 1] * expf(mz - m);
   }
+  const bool cached = splits <= LAT_COMBINE_CACHE;
+  if (cached) {
+    for (int z = threadIdx.x; z < splits; z += blockDim.x) {
+      const float mz = part_ml[2 * (slot0 + z)];
+      wgt[z] = mz > -INFINITY ? expf(mz - m) : 0.f;
+    }
+    __syncthreads();
+  }
   for (int d = threadIdx.x; d < rank; d += blockDim.x) {
     float a = 0.f;
+#pragma unroll 4
     for (int z = 0; z < splits; ++z) {
-      const float mz = part_ml[2 * (slot0 + z)];
-      if (mz > -INFINITY) a = fmaf(part_acc[(slot0 + z) * rank + d], expf(mz - m), a);
+      const float mz = cached ? 0.f : part_ml[2 * (slot0 + z)];
+      const float w = cached ? wgt[z] : (mz > -INFINITY ? expf(mz - m) : 0.f);
+      a = fmaf(part_acc[(slot0 + z) * rank + d], w, a);  // (a range without keys left zeros)
     }
     out_lat[((size_t)h * N + n) * rank + d] = from_f32<TO>(a / l);
   }
 }
 
+static int latent_combine(const float* part_acc, const float* part_ml, void* out_lat, int out_dtype, const int* rows, int served, int N,
+                          int H, int rank, int splits, cudaStream_t stream) {
+  if (splits == 1) return 0;
+  JLX_DISPATCH_DTYPE(out_dtype, TO, {
+    JLX_CUDA(jlx_launch_pdl(attention_latent_combine_kernel<TO>, dim3(served, H), dim3(128), 0, stream, part_acc, part_ml, (TO*)out_lat,
+                            rows, N, H, rank, splits));
+  });
+  JLX_LAUNCH_CHECK("attention_latent_combine");
+  return 0;
+}
+
+// use_mma: 0 keeps a bfloat16 cache on the 32-bit kernel too.  single: every served token is its request's only one of
+// the step.
 // rows / n_rows: serve these token rows only (N stays the row count of q and out).  splits > 1: part_acc float32
 // [n_rows * H * splits * rank], part_ml float32 [n_rows * H * splits * 2].
 JLX_API int jlx_attention_latent(const float* q_lat, const float* q_rot, const void* pages, int cache_dtype,
                                  const int* block_table, int bt_stride, const int* req_of_token, const int* positions,
                                  const float* sink, void* out_lat, int out_dtype, int N, int H, int rank, int dr,
                                  int page_size, int num_pages, float scale, const int* rows, int n_rows, int splits,
-                                 int split_keys, float* part_acc, float* part_ml, int window, int* status, cudaStream_t stream) {
+                                 int split_keys, float* part_acc, float* part_ml, int window, int use_mma, int single, int* status,
+                                 cudaStream_t stream) {
   JLX_REQUIRE(N >= 0 && H > 0 && rank > 0 && dr >= 0 && page_size > 0 && num_pages > 0, "attention_latent: bad sizes");
   JLX_REQUIRE(rank <= 32 * LAT_MAX_R32, "attention_latent: latent size %d is above the supported maximum %d", rank, 32 * LAT_MAX_R32);
   JLX_REQUIRE(splits >= 1 && splits <= 65535 && window >= 0, "attention_latent: bad split count %d or window %d", splits, window);
@@ -375,6 +627,30 @@ JLX_API int jlx_attention_latent(const float* q_lat, const float* q_rot, const v
   const int served = rows ? n_rows : N;
   if (served == 0) return 0;
   const int dk = rank + dr;
+  // a bfloat16 cache whose rows are whole 16-byte pieces: on the tensor cores
+  if (use_mma && cache_dtype == JLX_BF16 && rank % 8 == 0 && dr % 8 == 0 && ((uintptr_t)pages & 15) == 0) {
+    const int ldm = ((dk + 15) & ~15) + 8;  // rows an odd number of 16-byte pieces apart
+    const size_t smem_m = sizeof(bf16) * (size_t)(2 * LATM_KEYS + 16) * ldm;
+    const int hb = (H + 15) / 16;
+    if (smem_m <= 220 * 1024 && hb <= 65535) {
+#define LATM_GO(PIECES)                                                                                                        \
+  do {                                                                                                                         \
+    if (smem_m > 48 * 1024)                                                                                                    \
+      JLX_CUDA(cudaFuncSetAttribute(attention_latent_mma_kernel<TO, PIECES>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem_m)); \
+    JLX_CUDA(jlx_launch_pdl(attention_latent_mma_kernel<TO, PIECES>, dim3(served, hb, splits), dim3(LATM_THREADS), smem_m, stream, q_lat, \
+                            q_rot, (const bf16*)pages, block_table, bt_stride, req_of_token, positions, sink, (TO*)out_lat, N, H, rank, \
+                            dr, page_size, num_pages, scale, rows, splits, split_keys, part_acc, part_ml, ldm, window, single, status)); \
+  } while (0)
+      JLX_DISPATCH_DTYPE(out_dtype, TO, {
+        if (rank <= 128) LATM_GO(2);
+        else if (rank <= 512) LATM_GO(8);
+        else LATM_GO(16);
+      });
+#undef LATM_GO
+      JLX_LAUNCH_CHECK("attention_latent_mma");
+      return latent_combine(part_acc, part_ml, out_lat, out_dtype, rows, served, N, H, rank, splits, stream);
+    }
+  }
   // a key's row in shared memory: padded so that 16-byte reads of a quarter warp's rows fall into different banks
   // (rows a multiple of 4 floats apart with an odd count of 16-byte pieces), else by one float
   const int ldk = (dk & 3) == 0 ? (((dk >> 2) & 1) ? dk : dk + 4) : dk + 1;
@@ -404,14 +680,7 @@ JLX_API int jlx_attention_latent(const float* q_lat, const float* q_rot, const v
   }));
 #undef LAT_GO
   JLX_LAUNCH_CHECK("attention_latent");
-  if (splits > 1) {
-    JLX_DISPATCH_DTYPE(out_dtype, TO, {
-      JLX_CUDA(jlx_launch_pdl(attention_latent_combine_kernel<TO>, dim3(served, H), dim3(128), 0, stream, (const float*)part_acc,
-                              (const float*)part_ml, (TO*)out_lat, rows, N, H, rank, splits));
-    });
-    JLX_LAUNCH_CHECK("attention_latent_combine");
-  }
-  return 0;
+  return latent_combine(part_acc, part_ml, out_lat, out_dtype, rows, served, N, H, rank, splits, stream);
 }
 
 // ------------------------------------------------------------------------------------------------ prompt portions

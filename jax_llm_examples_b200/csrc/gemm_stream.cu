@@ -21,6 +21,7 @@
 // own copies, frees its tensor memory and returns.
 #include <cuda.h>
 
+#include "activation.cuh"
 #include "common.cuh"
 #include "mbarrier.cuh"
 
@@ -145,6 +146,7 @@ struct StreamArgs {
   int out_is_f32;
   int silu;              // 1: rows come in blocks of [16 gate, 16 up]; out[m, j] = silu(gate_j) * up_j, [rows, N / 2]
   float glu_alpha, glu_limit, glu_shift;  // the gated activation's form: g sigmoid(alpha g) (u + shift), g and u clipped at +-limit (g from above only) when limit > 0
+  int act;               // an activation's number (activation.cuh), applied to every finished sum; 0: none
   int splits;
   int k_per_split;       // multiple of BK
   int offsets_settled;   // grouped: offsets and tile list were complete before the kernel in front of this one began its work
@@ -207,6 +209,7 @@ __device__ __forceinline__ void stream_epilogue(const StreamArgs& args, int warp
           for (int j = 0; j < 16; ++j) {
             const int m = row_lo + c0 + j;
             if (m < row_hi) {
+              if (args.act) r[j] = __float_as_uint(activate(__uint_as_float(r[j]), args.act));
               if (args.out_is_f32 || args.splits > 1)
                 ((float*)args.out)[split_off + (size_t)m * args.N + n] = __uint_as_float(r[j]);
               else
@@ -623,6 +626,7 @@ JLX_API int jlx_gemm_stream_token_tile(int rows_hint) { return pick_bt(rows_hint
 // mode 2: fused SwiGLU epilogue: weight rows are interleaved in blocks of [16 gate, 16 up], out is
 //         [rows, N / 2] = silu(gate) * up; no split-K.  In general g sigmoid(glu_alpha g) (u + glu_shift) with
 //         g = min(gate, glu_limit), u = clamp(up, +-glu_limit) when glu_limit > 0; (1, 0, 0) is silu(gate) * up.
+// mode 3: an activation in the epilogue, out = act(sum) by its number `act` (activation.cuh); no split-K.
 // tile_list / n_tiles (optional, grouped only): the row tiles that have rows, made by jlx_expert_sort for the
 // tile width jlx_gemm_stream_token_tile(rows_hint); without them every block walks the offsets.
 // offsets_settled (grouped only): the caller's word that the kernel launched just before this one on the stream is a
@@ -631,15 +635,16 @@ JLX_API int jlx_gemm_stream_token_tile(int rows_hint) { return pick_bt(rows_hint
 JLX_API int jlx_gemm_stream(const void* A, const void* W, void* out, int out_is_f32, int rows, int N, int K,
                             const int* offsets, int E, int rows_hint, int splits, float* scratch, int mode,
                             const int* tile_list, const int* n_tiles, int offsets_settled, int* splits_used, int* status,
-                            float glu_alpha, float glu_limit, float glu_shift, cudaStream_t stream) {
+                            float glu_alpha, float glu_limit, float glu_shift, int act, cudaStream_t stream) {
   JLX_REQUIRE(rows >= 0 && N > 0 && K > 0, "gemm_stream: bad sizes rows=%d N=%d K=%d", rows, N, K);
   JLX_REQUIRE(K % 8 == 0, "gemm_stream: K = %d is no multiple of 8 (TMA needs 16-byte row strides); use the SIMT product", K);
   JLX_REQUIRE(((uintptr_t)A & 15) == 0 && ((uintptr_t)W & 15) == 0, "gemm_stream: operands must be 16-byte aligned");
   JLX_REQUIRE(!offsets || E > 0, "gemm_stream: a grouped product needs a group count");
   JLX_REQUIRE(!tile_list || n_tiles, "gemm_stream: a tile list needs its count");
-  JLX_REQUIRE(mode >= 0 && mode <= 2, "gemm_stream: unknown mode %d", mode);
+  JLX_REQUIRE(mode >= 0 && mode <= 3, "gemm_stream: unknown mode %d", mode);
   JLX_REQUIRE(splits >= 1 && (splits == 1 || mode == 1 || scratch), "gemm_stream: split-K needs scratch memory");
   JLX_REQUIRE(mode != 2 || (splits == 1 && N % 32 == 0), "gemm_stream: the SwiGLU epilogue needs N %% 32 == 0 and no split-K");
+  JLX_REQUIRE(mode != 3 || (splits == 1 && act >= ACT_NONE && act <= ACT_TANH), "gemm_stream: unknown activation %d, or one with split-K", act);
   JLX_REQUIRE(mode != 1 || out_is_f32, "gemm_stream: partials are float32");
   if (splits_used) *splits_used = 1;
   if (rows == 0) return 0;
@@ -659,6 +664,7 @@ JLX_API int jlx_gemm_stream(const void* A, const void* W, void* out, int out_is_
   a.tile_list = offsets ? tile_list : nullptr; a.n_tiles = n_tiles;
   a.out = (splits > 1 && mode == 0) ? (void*)scratch : out;
   a.out_is_f32 = out_is_f32; a.silu = mode == 2; a.glu_alpha = glu_alpha; a.glu_limit = glu_limit; a.glu_shift = glu_shift; a.splits = splits; a.k_per_split = kps; a.status = status;
+  a.act = mode == 3 ? act : 0;
   a.offsets_settled = offsets && offsets_settled;
   // Row tiles to launch blocks for.  Grouped: a group of r rows has ceil(r / bt) <= r / bt + 1 tiles and only a group
   // with rows has any, so there are at most rows / bt + min(E, rows) of them.  (A looser bound costs time: a block

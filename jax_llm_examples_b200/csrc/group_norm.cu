@@ -10,61 +10,34 @@
 //                last taps - 1 inputs of every request kept as its state.
 //
 // Every sum runs in an order that depends on the row alone (not on the batch or on how a prompt was cut).
+#include "activation.cuh"
 #include "common.cuh"
+#include "delta_rows.cuh"
 
-// Where a row's delta lies.  Without `index`: row r of `delta`.  With it, the delta is an expert layer's output still in
-// expert order: the sum over j < k of weights[r k + j] (null: 1) times row index[r k + j], j ascending.  In both cases
-// `splits` partials of a row are added first, ascending.
-struct DeltaRows {
-  const float* p;
-  long long split_stride;
-  const int* index;
-  const float* weights;
-  int splits, k;
-};
-
-__device__ __forceinline__ float delta_at(const DeltaRows& t, size_t r, int D, int d) {
-  if (!t.index) {
-    float s = 0.f;
-    for (int z = 0; z < t.splits; ++z) s += t.p[(size_t)z * t.split_stride + r * D + d];
-    return s;
-  }
-  float s = 0.f;
-  for (int j = 0; j < t.k; ++j) {
-    const float* p = t.p + (size_t)t.index[r * t.k + j] * D + d;
-    float e = 0.f;
-    for (int z = 0; z < t.splits; ++z) e += p[(size_t)z * t.split_stride];
-    s = fmaf(t.weights ? t.weights[r * t.k + j] : 1.f, e, s);
-  }
-  return s;
-}
-
-__device__ __forceinline__ float4 delta_at4(const DeltaRows& t, size_t r, int D, int d) {  // entries d .. d + 3
-  float4 s = make_float4(0.f, 0.f, 0.f, 0.f);
-  if (!t.index) {
-    for (int z = 0; z < t.splits; ++z) {
-      const float4 v = *reinterpret_cast<const float4*>(t.p + (size_t)z * t.split_stride + r * D + d);
-      s.x += v.x; s.y += v.y; s.z += v.z; s.w += v.w;
-    }
-    return s;
-  }
-  for (int j = 0; j < t.k; ++j) {
-    const float* p = t.p + (size_t)t.index[r * t.k + j] * D + d;
-    float4 e = make_float4(0.f, 0.f, 0.f, 0.f);
-    for (int z = 0; z < t.splits; ++z) {
-      const float4 v = *reinterpret_cast<const float4*>(p + (size_t)z * t.split_stride);
-      e.x += v.x; e.y += v.y; e.z += v.z; e.w += v.w;
-    }
-    const float w = t.weights ? t.weights[r * t.k + j] : 1.f;
-    s.x = fmaf(w, e.x, s.x); s.y = fmaf(w, e.y, s.y); s.z = fmaf(w, e.z, s.z); s.w = fmaf(w, e.w, s.w);
-  }
-  return s;
-}
-
-// 1 / rms of every group of row[0..D) into inv[0..groups): warp w takes groups w, w + nwarp, ...
+// The root mean square of every group of row[0..D) into rms[0..groups), the block's warps dealt out evenly: with fewer
+// groups than warps several warps share a group and thread g adds their parts in order; else a warp takes every
+// nwarp-th group.  Called by the whole block; the caller synchronises before it reads rms.
 __device__ __forceinline__ void group_rms(const float* row, int D, int groups, float eps, float* rms) {
+  __shared__ float part[32];
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarp = blockDim.x >> 5;
   const int gs = D / groups;
+  if (2 * groups <= nwarp) {
+    const int per = nwarp / groups, g = warp / per, w = warp - g * per;
+    if (g < groups) {
+      const float* p = row + (size_t)g * gs;
+      float s = 0.f;
+      for (int i = w * 32 + lane; i < gs; i += 32 * per) s = fmaf(p[i], p[i], s);
+      s = warp_sum(s);
+      if (lane == 0) part[warp] = s;
+    }
+    __syncthreads();
+    if (threadIdx.x < groups) {
+      float s = 0.f;
+      for (int u = 0; u < per; ++u) s += part[threadIdx.x * per + u];
+      rms[threadIdx.x] = sqrtf(s / (float)gs + eps);
+    }
+    return;
+  }
   for (int g = warp; g < groups; g += nwarp) {
     const float* p = row + (size_t)g * gs;
     float s = 0.f;
@@ -272,19 +245,6 @@ JLX_API int jlx_group_norm(float* x, const float* delta, int splits, long long s
 }
 
 // ------------------------------------------------------------------------------------------------ bias + activation
-enum { ACT_NONE = 0, ACT_RELU2 = 1, ACT_SILU = 2, ACT_GELU_TANH = 3, ACT_GELU = 4, ACT_TANH = 5 };
-
-__device__ __forceinline__ float activate(float z, int act) {
-  switch (act) {
-    case ACT_RELU2: { const float r = fmaxf(z, 0.f); return r * r; }
-    case ACT_SILU: return z / (1.f + expf(-z));
-    case ACT_GELU: return 0.5f * z * (1.f + erff(z * 0.7071067811865476f));
-    case ACT_TANH: return tanhf(z);
-    case ACT_GELU_TANH: return 0.5f * z * (1.f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
-    default: return z;
-  }
-}
-
 template <typename TI, typename TO>
 __global__ void bias_act_kernel(const TI* __restrict__ in, int splits, long long split_stride, const float* __restrict__ bias,
                                 const float* __restrict__ add, int act, TO* __restrict__ out, int F) {

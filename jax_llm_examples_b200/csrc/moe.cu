@@ -7,9 +7,7 @@
 // model.py:1139 (add the shared expert).  Ties go to the lower expert index (jax.lax.top_k order).
 #include "common.cuh"
 #include "expert_sort.cuh"
-
-#define ROUTER_MAX_E 256
-#define ROUTER_MAX_K 16
+#include "router_choice.cuh"
 
 // One block per token.  Warp w computes the scores of experts w, w + nwarp, ...: a fixed order of
 // the D products per (token, expert), so a token's routing does not depend on the batch.
@@ -22,85 +20,9 @@ __device__ __forceinline__ void softmax_of_chosen(float* w, int k) {
   for (int j = 0; j < k; ++j) w[j] = expf(w[j] - m) / sum;
 }
 
-// What the choice needs beyond the scores, for the corrected forms: weight_form 2, s = softmax(z) over all E outputs, and
-// weight_form 3, s = sigmoid(z).  The choice is made on s + correction, and only among the `keep` best of `groups`
-// equal groups of neighbouring outputs (a group's score: the sum of its `group_top` largest s + correction, one or two;
-// the others count as -inf, not 0: corrections may be negative); the weights are the chosen s, with `normalize` divided
-// by their sum (+ 1e-20), times `scale`.
-struct RouterChoice {
-  const float* correction;  // [E] or null
-  int groups, keep;         // groups <= 1: no limit
-  float scale;
-  int group_top, normalize;
-};
-
-// One thread: the k largest scores in order (strict comparison: the lower index wins a tie), their weights by form.
+// One thread: the k largest scores in order (strict comparison: the lower index wins a tie), their weights by form (0, 1).
 // `sc` (shared memory, E entries) is used up.
-__device__ __forceinline__ void choose_experts(float* sc, int E, int k, int* __restrict__ idx, float* __restrict__ w, int weight_form,
-                                               const RouterChoice& ch) {
-  if (weight_form >= 2) {
-    // the shares once (E exponentials), in place; after that the choice only compares and adds
-    if (weight_form == 3) {
-      for (int e = 0; e < E; ++e) sc[e] = 1.f / (1.f + expf(-sc[e]));
-    } else {
-      float m = -INFINITY, sum = 0.f;
-      for (int e = 0; e < E; ++e) m = fmaxf(m, sc[e]);
-      for (int e = 0; e < E; ++e) {
-        const float x = expf(sc[e] - m);
-        sc[e] = x;
-        sum += x;
-      }
-      for (int e = 0; e < E; ++e) sc[e] = sc[e] / sum;
-    }
-    const int per = ch.groups > 1 ? E / ch.groups : E;
-    unsigned long long allowed = ~0ull;  // bit g: group g may be chosen from (up to 64 groups)
-    if (ch.groups > 1 && ch.keep < ch.groups) {
-      allowed = 0ull;
-      for (int t = 0; t < ch.keep; ++t) {
-        int bg = -1;
-        float bv = 0.f;
-        for (int g = 0; g < ch.groups; ++g) {
-          if ((allowed >> g) & 1ull) continue;
-          float gv = -INFINITY, second = -INFINITY;
-          for (int e = g * per; e < (g + 1) * per; ++e) {
-            const float v = sc[e] + (ch.correction ? ch.correction[e] : 0.f);
-            second = fmaxf(second, fminf(gv, v));
-            gv = fmaxf(gv, v);
-          }
-          if (ch.group_top == 2 && per > 1) gv += second;
-          if (bg < 0 || gv > bv) {
-            bg = g;
-            bv = gv;
-          }
-        }
-        allowed |= 1ull << bg;
-      }
-    }
-    unsigned long long taken[ROUTER_MAX_E / 64] = {0ull, 0ull, 0ull, 0ull};
-    float total = 0.f;
-    for (int j = 0; j < k; ++j) {
-      int best = -1;
-      float bv = 0.f;
-      for (int e = 0; e < E; ++e) {
-        if (((taken[e >> 6] >> (e & 63)) & 1ull) || !((allowed >> (ch.groups > 1 ? e / per : 0)) & 1ull)) continue;
-        const float v = sc[e] + (ch.correction ? ch.correction[e] : 0.f);
-        if (isnan(v)) continue;
-        if (best < 0 || v > bv) {  // strict: the lower index wins a tie
-          best = e;
-          bv = v;
-        }
-      }
-      float bs = 0.f;
-      if (best < 0) best = j;  // fewer allowed outputs than k, or all NaN: still a valid index, with no weight
-      else bs = sc[best];
-      idx[j] = best;
-      w[j] = bs;
-      total += bs;
-      taken[best >> 6] |= 1ull << (best & 63);
-    }
-    for (int j = 0; j < k; ++j) w[j] = (ch.normalize ? w[j] / (total + 1e-20f) : w[j]) * ch.scale;
-    return;
-  }
+__device__ __forceinline__ void choose_experts(float* sc, int E, int k, int* __restrict__ idx, float* __restrict__ w, int weight_form) {
   for (int j = 0; j < k; ++j) {
     int best = -1;
     float bv = 0.f;
@@ -151,7 +73,11 @@ __global__ void router_kernel(const float* __restrict__ h, const float* __restri
   __syncthreads();
   if (scores_out)
     for (int e = threadIdx.x; e < E; e += blockDim.x) scores_out[(size_t)n * E + e] = scores[e];
-  if (threadIdx.x == 0) choose_experts(scores, E, k, topk_idx + (size_t)n * k, topk_w + (size_t)n * k, weight_form, choice);
+  if (weight_form >= 2) {
+    if (warp == 0) choose_experts_corrected(scores, E, k, topk_idx + (size_t)n * k, topk_w + (size_t)n * k, weight_form, choice);
+  } else if (threadIdx.x == 0) {
+    choose_experts(scores, E, k, topk_idx + (size_t)n * k, topk_w + (size_t)n * k, weight_form);
+  }
 }
 
 // Many tokens (prompt portions): a block takes ROWS tokens, so that a router row that a warp fetches serves all
@@ -203,9 +129,12 @@ router_rows_kernel(const float* __restrict__ h, const float* __restrict__ w_rout
       }
   }
   __syncthreads();
-  if (threadIdx.x < rows) {
+  if (weight_form >= 2) {  // (eight warps, up to eight rows)
+    const size_t n = (size_t)n0 + warp;
+    if (warp < rows) choose_experts_corrected(scores[warp], E, k, topk_idx + n * k, topk_w + n * k, weight_form, choice);
+  } else if (threadIdx.x < rows) {
     const size_t n = (size_t)n0 + threadIdx.x;
-    choose_experts(scores[threadIdx.x], E, k, topk_idx + n * k, topk_w + n * k, weight_form, choice);
+    choose_experts(scores[threadIdx.x], E, k, topk_idx + n * k, topk_w + n * k, weight_form);
   }
 }
 

@@ -286,6 +286,45 @@ def group_norm(x: torch.Tensor, delta: torch.Tensor | None = None, delta_splits:
          _ptr(row_index), c_int(N), c_int(D), _ptr(delta_index), _ptr(delta_weights), c_int(delta_k), _stream())
 
 
+def close_route_supported(n: int, D: int, E: int, k: int) -> bool:
+    """Whether ``close_route`` takes a step of n rows (a decode step's few, widths that are multiples of 4)."""
+    return bool(library("close_route").jlx_close_route_supported(c_int(n), c_int(D), c_int(E), c_int(k)))
+
+
+def close_route(x: torch.Tensor, delta: torch.Tensor, delta_splits: int, post_weight: torch.Tensor, mult: float, eps: float,
+                out: torch.Tensor | None, router, topk_idx: torch.Tensor, topk_w: torch.Tensor, dispatch,
+                delta_index: torch.Tensor | None = None, delta_k: int = 1, delta_weights: torch.Tensor | None = None) -> None:
+    """x += mult * post_weight * rms_norm(delta); out = x rounded; then the router on x, the sort of the choices by expert and
+    the gather of the rows in that order: ``group_norm`` + ``router`` + ``expert_sort`` + ``permute_scale`` in one launch for the
+    few rows of a decode step (:func:`close_route_supported`).  ``delta``: float32 [N, D], partials of it, or gathered rows
+    as in :func:`group_norm`.  ``router``: an object with w_router, bias, correction, weight_form (a corrected one), groups,
+    keep, group_top, normalize and scale.  ``dispatch``: an object with offsets, sorted_pair, sorted_pos, tiles (a pair or
+    None), tile_rows, a_sorted and status, as ``add_rmsnorm`` takes it (extra_rows 0)."""
+    tile_list, n_tiles = dispatch.tiles if dispatch.tiles is not None else (None, None)
+    _contig(x, delta, post_weight, out, router.w_router, router.bias, router.correction, topk_idx, topk_w, delta_index, delta_weights,
+            dispatch.offsets, dispatch.sorted_pair, dispatch.sorted_pos, dispatch.a_sorted, tile_list, n_tiles)
+    N, D = x.shape
+    E, k = router.w_router.shape[0], topk_idx.shape[1]
+    if any(t is not None and t.dtype != torch.float32 for t in (x, delta, post_weight, router.w_router, router.bias, router.correction, topk_w, delta_weights)):
+        raise KernelError("close_route: rows, norm weight and router must be float32")
+    if out is not None and out.dtype != dispatch.a_sorted.dtype:
+        raise KernelError("close_route: the gathered rows must have the output's type")
+    if dispatch.extra_rows or tuple(dispatch.a_sorted.shape) != (N * k, D) or dispatch.offsets.numel() < E + 1 or router.w_router.shape[1] != D:
+        raise KernelError(f"close_route: shapes do not fit {N} rows of {D}, top-{k} of {E}")
+    if delta_index is not None and delta_index.numel() < N * delta_k:
+        raise KernelError("close_route: too few indices of gathered rows")
+    if tile_list is not None and tile_list.numel() < 2 * (-(-N * k // dispatch.tile_rows) + E):
+        raise KernelError("close_route: tile list too short")
+    sp, stride = _splits(delta, delta_splits)
+    _run("close_route", "jlx_close_route", _ptr(x), _ptr(delta), c_int(sp), c_longlong(stride), _ptr(delta_index), _ptr(delta_weights),
+         c_int(delta_k), _ptr(post_weight), c_float(mult), c_float(eps), _ptr(out), c_int(code(dispatch.a_sorted.dtype)),
+         _ptr(router.w_router), _ptr(router.bias), c_int(ROUTER_WEIGHT_FORMS[router.weight_form]), _ptr(router.correction),
+         c_int(router.groups), c_int(router.keep), c_int(router.group_top), c_int(int(router.normalize)), c_float(router.scale),
+         _ptr(topk_idx), _ptr(topk_w), _ptr(dispatch.offsets), _ptr(dispatch.sorted_pair), _ptr(dispatch.sorted_pos),
+         c_int(dispatch.tile_rows if tile_list is not None else 0), _ptr(tile_list), _ptr(n_tiles), _ptr(dispatch.a_sorted), c_int(N),
+         c_int(D), c_int(E), c_int(k), _ptr(dispatch.status), _stream())
+
+
 def bias_act(rows: torch.Tensor, out: torch.Tensor, bias: torch.Tensor | None = None, add: torch.Tensor | None = None,
              activation: str = "none", splits: int = 1) -> None:
     """out = activation(rows + bias + add).  rows: [N, F] or ``splits`` float32 partials [splits, N, F]; bias: float32
@@ -421,9 +460,11 @@ def attention_latent(q_lat: torch.Tensor, q_rot: torch.Tensor, pages: torch.Tens
                      req_of_token: torch.Tensor, positions: torch.Tensor, sink: torch.Tensor | None, out_lat: torch.Tensor,
                      scale: float, status: torch.Tensor, rows: torch.Tensor | None = None, n_rows: int = 0, splits: int = 1,
                      split_keys: int = 0, part_acc: torch.Tensor | None = None, part_ml: torch.Tensor | None = None,
-                     window: int = 0) -> None:
+                     window: int = 0, tensor_cores: bool = True, single_tokens: bool = False) -> None:
     """Causal attention in the latent space with an optional per-head sink and window (a query sees itself and the
-    window - 1 keys before it; 0: all).  q_lat: float32 [H, N, rank]; q_rot:
+    window - 1 keys before it; 0: all).  A bfloat16 cache whose rows are whole 16-byte pieces goes to the tensor cores
+    (queries and weights rounded to bfloat16, sums in 32-bit) unless ``tensor_cores`` is False.  ``single_tokens``: every
+    served token is its request's only one of the step, so that older keys may be fetched ahead of the predecessor.  q_lat: float32 [H, N, rank]; q_rot:
     float32 [N, H, dr]; pages: [P, 1, 1, page_size, rank + dr]; out_lat: [H, N, rank].
     rows / n_rows: serve these token rows only (int32).  splits > 1: the keys are cut into ranges of ``split_keys``
     (a multiple of LATENT_KEY_TILE; ranges are counted from the first visible key's), a block each, and a second kernel adds the ranges' results; part_acc: float32
@@ -444,7 +485,7 @@ def attention_latent(q_lat: torch.Tensor, q_rot: torch.Tensor, pages: torch.Tens
          _ptr(block_table), c_int(block_table.shape[1]), _ptr(req_of_token), _ptr(positions), _ptr(sink), _ptr(out_lat),
          c_int(code(out_lat.dtype)), c_int(N), c_int(H), c_int(rank), c_int(dr), c_int(pages.shape[3]), c_int(pages.shape[0]),
          c_float(scale), _ptr(rows), c_int(n_rows), c_int(splits), c_int(split_keys), _ptr(part_acc), _ptr(part_ml),
-         c_int(window), _ptr(status), _stream())
+         c_int(window), c_int(int(tensor_cores)), c_int(int(single_tokens)), _ptr(status), _stream())
     _launches += int(splits > 1)  # the combine kernel
 
 
@@ -853,7 +894,7 @@ def gemm_stream_supported(a: torch.Tensor, w: torch.Tensor) -> bool:
             and a.data_ptr() % 16 == 0 and w.data_ptr() % 16 == 0)
 
 
-GEMM_PLAIN, GEMM_PARTIALS, GEMM_SWIGLU = 0, 1, 2
+GEMM_PLAIN, GEMM_PARTIALS, GEMM_SWIGLU, GEMM_ACT = 0, 1, 2, 3
 
 
 def gemm_stream_token_tile(rows_hint: int) -> int:
@@ -864,13 +905,15 @@ def gemm_stream_token_tile(rows_hint: int) -> int:
 def gemm_stream(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, status: torch.Tensor,
                 offsets: torch.Tensor | None = None, rows_hint: int = 0, splits: int = 1,
                 scratch: torch.Tensor | None = None, mode: int = GEMM_PLAIN,
-                tiles: tuple[torch.Tensor, torch.Tensor] | None = None, offsets_settled: bool = False, glu=SILU_GLU) -> int:
+                tiles: tuple[torch.Tensor, torch.Tensor] | None = None, offsets_settled: bool = False, glu=SILU_GLU,
+                activation: str = "none") -> int:
     """a @ w^T on the tcgen05 tensor cores (bfloat16 in, float32 accumulate).  a: [M, K]; w: [N, K] or,
     with row-group offsets [E + 1], [E, N, K].
     GEMM_PLAIN: out [M, N] bfloat16 or float32; splits > 1 cuts K across blocks (scratch: float32
     [splits * M * N]) and adds the partials.  GEMM_PARTIALS: out is float32 [splits, M, N], left for the
     consumer to add.  GEMM_SWIGLU: w's rows are interleaved [16 gate, 16 up]; out [M, N / 2] =
-    silu(gate) * up, or the gated activation ``glu`` (see :func:`glu_form`).  ``tiles`` = (tile_list, n_tiles) from
+    silu(gate) * up, or the gated activation ``glu`` (see :func:`glu_form`).  GEMM_ACT: out [M, N] = ``activation`` (a name
+    of ACTIVATIONS) of the sums.  ``tiles`` = (tile_list, n_tiles) from
     expert_sort for the same rows_hint.
     ``offsets_settled``: the kernel launched just before this call on the stream was a grouped gemm_stream over the
     same offsets and tiles (this one then finds its tile and asks for its weights without waiting for that one).
@@ -881,7 +924,7 @@ def gemm_stream(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, status: tor
     N = w.shape[-2]
     if w.shape[-1] != K or (offsets is None) != (w.dim() == 2):
         raise KernelError(f"gemm_stream: shapes do not fit: a {tuple(a.shape)}, w {tuple(w.shape)}")
-    want = {GEMM_PLAIN: M * N, GEMM_PARTIALS: splits * M * N, GEMM_SWIGLU: M * (N // 2)}[mode]
+    want = {GEMM_PLAIN: M * N, GEMM_PARTIALS: splits * M * N, GEMM_SWIGLU: M * (N // 2), GEMM_ACT: M * N}[mode]
     if out.numel() < want:
         raise KernelError(f"gemm_stream: out has {out.numel()} elements, {want} are needed")
     if a.dtype != torch.bfloat16 or w.dtype != torch.bfloat16 or out.dtype not in (torch.bfloat16, torch.float32):
@@ -892,7 +935,7 @@ def gemm_stream(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, status: tor
     _run("gemm_stream", "jlx_gemm_stream", _ptr(a), _ptr(w), _ptr(out), c_int(int(out.dtype == torch.float32)), c_int(M),
          c_int(N), c_int(K), _ptr(offsets), c_int(E), c_int(rows_hint), c_int(splits), _ptr(scratch), c_int(mode),
          _ptr(tiles[0]) if tiles else None, _ptr(tiles[1]) if tiles else None, c_int(int(offsets_settled and offsets is not None)),
-         ctypes.byref(used), _ptr(status), c_float(glu[0]), c_float(glu[1]), c_float(glu[2]), _stream())
+         ctypes.byref(used), _ptr(status), c_float(glu[0]), c_float(glu[1]), c_float(glu[2]), c_int(ACTIVATIONS[activation]), _stream())
     return used.value
 
 

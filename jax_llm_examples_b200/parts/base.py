@@ -303,7 +303,7 @@ class Dispatch:
     them offers the buffers through ``router_request()``; a norm that routes for it may fill them in the same kernel
     and hands them back with the routing, which saves a decode step two dependent launches per layer."""
 
-    counter: torch.Tensor  # int32 [1], zero between launches
+    counter: torch.Tensor | None  # int32 [1], zero between launches (None: the kernel that fills this keeps none)
     offsets: torch.Tensor  # int32 [groups + 1]
     sorted_pair: torch.Tensor  # int32 [pairs]
     sorted_pos: torch.Tensor  # int32 [pairs]
@@ -312,6 +312,24 @@ class Dispatch:
     extra_rows: int  # rows of a group appended after the experts (a shared expert that takes every token)
     tile_rows: int
     status: torch.Tensor
+
+
+@dataclasses.dataclass
+class CorrectedRouter:
+    """A corrected, group-limited router (``K.router``'s forms of that kind) as a routed feed-forward describes it to whoever
+    may route for it, with ``dispatch(ctx, n_rows)`` for the buffers of its sort and gather."""
+
+    w_router: torch.Tensor  # float32 [E, D]
+    bias: torch.Tensor | None
+    correction: torch.Tensor | None
+    weight_form: str
+    groups: int
+    keep: int
+    group_top: int
+    normalize: bool
+    scale: float
+    top_k: int
+    dispatch: Callable[["StepContext", int], Dispatch]
 
 
 class Norm(Part):
@@ -403,6 +421,11 @@ class FeedForward(Part):
     def router_request(self):
         """(w_router, top_k) if the preceding norm may route the tokens for this part, else None; optionally a third
         element, see Norm.forward."""
+        return None
+
+    def corrected_router(self) -> "CorrectedRouter | None":
+        """The part's router, if it is of the corrected kind and a block may route for it in the kernel that closes the
+        sublayer before (``PostNormBlock`` does in decode steps)."""
         return None
 
     def forward(self, ctx: StepContext, h: torch.Tensor, h32: torch.Tensor | None, routing=None) -> "torch.Tensor | Rows":

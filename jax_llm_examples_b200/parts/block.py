@@ -134,9 +134,12 @@ class PostNormBlock(Block):
 
     The feed-forward (with norm2) may be missing.  A sublayer's output goes on as a :class:`PostNormed` delta; the kernel
     that closes it (norm, residual sum) also writes the rows that the next sublayer reads, in the activations' type.
-    A routed feed-forward may hand on its rows in expert order, with their weights: that kernel gathers them too."""
+    A routed feed-forward may hand on its rows in expert order, with their weights: that kernel gathers them too.  In a
+    decode step (bfloat16, few rows) the kernel in front of a feed-forward with a corrected router also routes, sorts and
+    gathers for it."""
 
     kernel_libraries = ("group_norm",)
+    kernel_libraries_bf16 = ("close_route",)
 
     def __init__(self, norm1: Norm, mixer: Mixer, norm2: Norm | None = None, feed_forward: FeedForward | None = None):
         if (feed_forward is None) != (norm2 is None):
@@ -169,6 +172,25 @@ class PostNormBlock(Block):
         add_to_residual(x, delta, pre_norm=False, eps=eps, out=h)
         return h
 
+    def _open_and_route(self, ctx: StepContext, x: torch.Tensor, pending):
+        """x += pending, the rows for the feed-forward and its routing, sort and gather in one launch; None where the step is
+        not of that kind.  Returns ((expert indices, weights, Dispatch), rows)."""
+        from ..kernels import api as K
+
+        router = self.feed_forward.corrected_router()
+        if router is None or ctx.runtime.dtype != torch.bfloat16 or pending.groups != 1 or pending.bias is not None \
+                or pending.rows.data.dtype != torch.float32 or ctx.max_q_len != 1 \
+                or not K.close_route_supported(x.shape[0], x.shape[1], router.w_router.shape[0], router.top_k):
+            return None
+        n = x.shape[0]
+        idx = torch.empty((n, router.top_k), dtype=torch.int32, device=x.device)
+        wt = torch.empty((n, router.top_k), dtype=torch.float32, device=x.device)
+        h = torch.empty(x.shape, dtype=ctx.runtime.dtype, device=x.device)
+        dispatch = router.dispatch(ctx, n)
+        K.close_route(x, pending.rows.data, pending.rows.splits, pending.weight, pending.mult, pending.eps, h, router, idx, wt, dispatch,
+                      **pending.gather())
+        return (idx, wt, dispatch), h
+
     def forward(self, ctx: StepContext, x: torch.Tensor, delta, cache: LayerCache):
         with scope("attn_pre_norm"):
             h = self._open(ctx, x, delta, self.norm1.eps)
@@ -177,9 +199,10 @@ class PostNormBlock(Block):
         if self.feed_forward is None:
             return pending
         with scope("attn_post_norm"):
-            h = self._open(ctx, x, pending, self.norm1.eps)
+            routing = self._open_and_route(ctx, x, pending)
+            h = routing[1] if routing is not None else self._open(ctx, x, pending, self.norm1.eps)
         with scope("ffn"):
-            y = self.feed_forward.forward(ctx, h, x if self.feed_forward.needs_f32_input else None, None)
+            y = self.feed_forward.forward(ctx, h, x if self.feed_forward.needs_f32_input else None, None if routing is None else routing[0])
         return self._closing(self.norm2, y, getattr(self.feed_forward, "bias_out", None))
 
 

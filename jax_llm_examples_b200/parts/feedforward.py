@@ -7,8 +7,8 @@ import torch
 from ..kernels import api as K
 from ..tracing import active as tracing_active
 from ..tracing import scope
-from .base import Dispatch, FeedForward, Rows, RowSum, StepContext, as_rows, register_part
-from .linear import (STREAM_MAX_ROWS, group_rows_hint, grouped_linear, grouped_swiglu_linear, grouped_swiglu_streams,
+from .base import CorrectedRouter, Dispatch, FeedForward, Rows, RowSum, StepContext, as_rows, register_part
+from .linear import (STREAM_MAX_ROWS, group_rows_hint, grouped_act_linear, grouped_linear, grouped_swiglu_linear, grouped_swiglu_streams,
                      interleave_gate_up, linear,
                      swiglu_linear)
 
@@ -289,6 +289,23 @@ class RoutedMLPExperts(FeedForward):
     def sub_parts(self):
         return () if self.shared is None else (self.shared,)
 
+    def corrected_router(self) -> CorrectedRouter | None:
+        if self.weight_form != "sigmoid_corrected":
+            return None
+        return CorrectedRouter(self.w_router, self.router_bias, self.correction, self.weight_form, self.groups, self.keep, self.group_top,
+                               self.normalize, self.route_scale, self.top_k, self.sort_buffers)
+
+    def sort_buffers(self, ctx: StepContext, n: int) -> Dispatch:
+        """The buffers of a step's sort and gather, not yet filled."""
+        k, E, dev = self.top_k, self.num_experts, self.w_router.device
+        i32 = lambda size: torch.empty(size, dtype=torch.int32, device=dev)  # noqa: E731
+        tiles, tile_rows = None, 0
+        if self.we_up.dtype == torch.bfloat16 and ctx.runtime.dtype == torch.bfloat16:
+            tile_rows = K.gemm_stream_token_tile(group_rows_hint(n * k, E))
+            tiles = (i32(2 * (-(-n * k // tile_rows) + E)), i32(1))
+        a_sorted = torch.empty((n * k, self.w_router.shape[1]), dtype=ctx.runtime.dtype, device=dev)
+        return Dispatch(None, i32(E + 1), i32(n * k), i32(n * k), tiles, a_sorted, 0, tile_rows, ctx.status)
+
     def route(self, ctx: StepContext, h32: torch.Tensor):
         n, k, dev = h32.shape[0], self.top_k, h32.device
         topk_idx = torch.empty((n, k), dtype=torch.int32, device=dev)
@@ -305,30 +322,23 @@ class RoutedMLPExperts(FeedForward):
         rt = ctx.runtime
         n, D = h32.shape
         k, E, dev = self.top_k, self.num_experts, h32.device
-        topk_idx, topk_w = self.route(ctx, h32)
+        # the block may have routed, sorted and gathered already (CorrectedRouter)
+        topk_idx, topk_w, *dispatched = routing if routing is not None else self.route(ctx, h32)
         if "record_routing" in ctx.scratch:
             ctx.scratch["record_routing"].append(topk_idx)
         with scope("moe_routed_expert"):
-            with scope("permute"):
-                offsets = torch.empty(E + 1, dtype=torch.int32, device=dev)
-                sorted_pair = torch.empty(n * k, dtype=torch.int32, device=dev)
-                sorted_pos = torch.empty(n * k, dtype=torch.int32, device=dev)
-                tiles = None
-                if self.we_up.dtype == torch.bfloat16 and rt.dtype == torch.bfloat16:
-                    tile_rows = K.gemm_stream_token_tile(group_rows_hint(n * k, E))
-                    tiles = (torch.empty(2 * (-(-n * k // tile_rows) + E), dtype=torch.int32, device=dev),
-                             torch.empty(1, dtype=torch.int32, device=dev))
-                    K.expert_sort(topk_idx, offsets, sorted_pair, sorted_pos, E, ctx.status, 0, tile_rows, *tiles)
-                else:
-                    K.expert_sort(topk_idx, offsets, sorted_pair, sorted_pos, E, ctx.status)
-                a_sorted = torch.empty((n * k, D), dtype=rt.dtype, device=dev)
-                K.permute_scale(h32, sorted_pair, None, a_sorted, k)
+            done = dispatched[0] if dispatched else self.sort_buffers(ctx, n)
+            offsets, sorted_pos, tiles, a_sorted = done.offsets, done.sorted_pos, done.tiles, done.a_sorted
+            if not dispatched:
+                with scope("permute"):
+                    K.expert_sort(topk_idx, offsets, done.sorted_pair, sorted_pos, E, ctx.status, 0,
+                                  *((done.tile_rows, *tiles) if tiles is not None else ()))
+                    K.permute_scale(h32, done.sorted_pair, None, a_sorted, k)
             with scope("we_gate_up"):
-                up = as_rows(grouped_linear(ctx, a_sorted, self.we_up, offsets, torch.float32, partials=True, tiles=tiles))
-                act = torch.empty((n * k, self.we_up.shape[1]), dtype=rt.dtype, device=dev)
-                K.bias_act(up.data, act, None, None, self.activation, up.splits)
+                act, one_product = grouped_act_linear(ctx, a_sorted, self.we_up, offsets, self.activation, rt.dtype, tiles)
             with scope("we_down"):
-                y = as_rows(grouped_linear(ctx, act, self.we_down, offsets, torch.float32, partials=True, tiles=tiles))
+                y = as_rows(grouped_linear(ctx, act, self.we_down, offsets, torch.float32, partials=True, tiles=tiles,
+                                           after_grouped=one_product and not tracing_active()))
         shared = None
         if self.shared is not None:
             with scope("moe_shared_expert"):

@@ -111,7 +111,9 @@ class LatentAttention(InputConvMixer):
         ranges so that about two rounds of blocks fill the GPU; a second kernel adds the ranges."""
         H = self.heads
         served = n_rows if rows is not None else q_rot.shape[0]
-        per_block = 8 * (2 if self.kv_rank > 512 else 4)  # heads a block of the kernel serves (csrc/attention_latent.cu)
+        # heads a block of the kernel serves (csrc/attention_latent.cu): the tensor-core form, or the 32-bit one
+        tensor_cores = ctx.runtime.dtype == torch.bfloat16 and self.kv_rank % 8 == 0 and self.rot_dim % 8 == 0
+        per_block = 16 if tensor_cores else 8 * (2 if self.kv_rank > 512 else 4)
         blocks = served * -(-H // per_block)
         want = max(1, (self.SPLIT_ROUNDS * K.sm_count()) // max(blocks, 1))
         tile = K.LATENT_KEY_TILE
@@ -126,7 +128,8 @@ class LatentAttention(InputConvMixer):
             part_acc = ctx.workspace.get("latent_part_acc", served * H * splits * self.kv_rank, torch.float32)
             part_ml = ctx.workspace.get("latent_part_ml", served * H * splits * 2, torch.float32)
         K.attention_latent(q_lat, q_rot, cache.pages, cache.block_table, ctx.req_of_token, ctx.positions, self.sink, out_lat,
-                           self.scale, ctx.status, rows, n_rows, splits, split_keys, part_acc, part_ml, self.window or 0)
+                           self.scale, ctx.status, rows, n_rows, splits, split_keys, part_acc, part_ml, self.window or 0,
+                           single_tokens=rows is not None or ctx.max_q_len == 1)
 
     def _portion(self, ctx: StepContext, cache: LayerCache, r: int, n0: int, T: int, start: int, q_full, rows_out, gate) -> None:
         """One request's prompt portion (rows n0 .. n0 + T, positions start ..) on the tensor cores: the request's cached

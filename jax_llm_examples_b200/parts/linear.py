@@ -137,6 +137,22 @@ def grouped_linear(ctx: StepContext, a_sorted: torch.Tensor, w: torch.Tensor, of
     return Rows(out, 1) if partials else out
 
 
+def grouped_act_linear(ctx: StepContext, a_sorted: torch.Tensor, w: torch.Tensor, offsets: torch.Tensor, activation: str,
+                       out_dtype: torch.dtype, tiles=None) -> "tuple[torch.Tensor, bool]":
+    """activation(rows [offsets[e], offsets[e+1]) of a_sorted times w[e]^T): in the product's epilogue where the streaming
+    kernel runs and does not cut K, else on its partial sums by a kernel of its own (few groups with rows: the cuts fill
+    the GPU).  Returns the rows and whether the product was one streaming launch with nothing after it."""
+    rows, E, N = a_sorted.shape[0], w.shape[0], w.shape[1]
+    act = torch.empty((rows, N), dtype=out_dtype, device=a_sorted.device)
+    if _streams(a_sorted, w, False) and (rows > STREAM_MAX_ROWS or _splits_for(N, a_sorted.shape[1], min(E, rows)) == 1):
+        K.gemm_stream(a_sorted, w, act, ctx.status, offsets=offsets, rows_hint=_group_rows_hint(rows, E), mode=K.GEMM_ACT, tiles=tiles,
+                      activation=activation)
+        return act, True
+    up = grouped_linear(ctx, a_sorted, w, offsets, torch.float32, partials=True, tiles=tiles)
+    K.bias_act(up.data, act, None, None, activation, up.splits)
+    return act, False
+
+
 def grouped_swiglu_streams(a_sorted: torch.Tensor, w_gate_up: torch.Tensor, interleaved: bool) -> bool:
     """Whether ``grouped_swiglu_linear`` runs as ONE streaming product (activation in its epilogue), nothing after it."""
     return interleaved and _streams(a_sorted, w_gate_up, False)
