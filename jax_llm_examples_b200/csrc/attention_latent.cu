@@ -40,11 +40,14 @@ __global__ void latent_kv_prep_kernel(const float* __restrict__ proj, int splits
                                       int num_pages, int ld, int halves, int* status) {
   JLX_TL(TL_ROPE);
   pdl_launch_dependents_if_small();
-  pdl_wait();
   extern __shared__ float sums[];  // the latent's entries, split-K partials added
   __shared__ float scratch[33];
   const int n = blockIdx.x;
   const float* row = proj + (size_t)n * ld;
+  // the step's description is older than the step: the token's place is looked up before the wait for the projected rows
+  const int p = positions[n];
+  const int page = blockIdx.y ? block_table[(size_t)req_of_token[n] * bt_stride + p / page_size] : 0;
+  pdl_wait();
   if (blockIdx.y == 0) {  // the query's latent
     float ss = 0.f;
     for (int i = threadIdx.x; i < q_rank; i += blockDim.x) {
@@ -56,8 +59,6 @@ __global__ void latent_kv_prep_kernel(const float* __restrict__ proj, int splits
     for (int i = threadIdx.x; i < q_rank; i += blockDim.x) cq[(size_t)n * q_rank + i] = from_f32<TO>(sums[i] / rms * q_norm_w[i]);
     return;
   }
-  const int p = positions[n], r = req_of_token[n];
-  const int page = block_table[(size_t)r * bt_stride + p / page_size];
   if (page < 0 || page >= num_pages) {
     if (threadIdx.x == 0) atomicOr(status, JLX_STATUS_BAD_PAGE);
     return;
@@ -108,56 +109,56 @@ JLX_API int jlx_latent_kv_prep(const float* proj, int splits, long long split_st
   return 0;
 }
 
-// q: float32 [N, H, dn + dr] (or partials).  q_nope: [H, N, dn] in the activation type; q_rot: float32 [N, H, dr];
-// q_full (optional): [H, N, dn + dr] in the activation type, the rotated part rotated (for per-head score products).
-template <typename TO>
+// q: float32 [rows, H, dn + dr] (or partials); row b of the outputs is row rows[b] of q (rows null: row b).  q_nope: [H, N, dn]
+// in the activation type and q_rot: [N, H, dr] (both or neither); q_full (optional): [H, N, dn + dr], the rotated part rotated
+// (for per-head score products).
+template <typename TO, typename TR>
 __global__ void latent_q_prep_kernel(const float* __restrict__ q, int splits, long long split_stride,
                                      const float* __restrict__ inv_freq, int rot_dims, const int* __restrict__ positions,
-                                     TO* __restrict__ q_nope, float* __restrict__ q_rot, TO* __restrict__ q_full, int N, int H,
-                                     int dn, int dr, int halves) {
+                                     TO* __restrict__ q_nope, TR* __restrict__ q_rot, TO* __restrict__ q_full, int N, int H,
+                                     int dn, int dr, int halves, const int* __restrict__ rows) {
   JLX_TL(TL_ROPE);
   pdl_launch_dependents_if_small();
+  const int b = blockIdx.x, h = blockIdx.y;
+  const int n = rows ? rows[b] : b, p = positions[n];
   pdl_wait();
-  const int n = blockIdx.x, h = blockIdx.y;
   const float* row = q + ((size_t)n * H + h) * (dn + dr);
-  TO* full = q_full ? q_full + ((size_t)h * N + n) * (dn + dr) : nullptr;
+  TO* full = q_full ? q_full + ((size_t)h * N + b) * (dn + dr) : nullptr;
   for (int i = threadIdx.x; i < dn; i += blockDim.x) {
     const TO v = from_f32<TO>(row_sum_splits(row + i, splits, split_stride));
-    q_nope[((size_t)h * N + n) * dn + i] = v;
+    if (q_nope) q_nope[((size_t)h * N + b) * dn + i] = v;
     if (full) full[i] = v;
   }
   const float* qr = row + dn;
-  float* dst = q_rot + ((size_t)n * H + h) * dr;
-  const int p = positions[n];
+  TR* dst = q_rot ? q_rot + ((size_t)b * H + h) * dr : nullptr;
   for (int i = threadIdx.x; i < rot_dims / 2; i += blockDim.x) {
     float sn, cs;
     sincosf((float)p * inv_freq[i], &sn, &cs);
     int ia, ib;
     rot_pair(i, rot_dims, halves, &ia, &ib);
     const float u = row_sum_splits(qr + ia, splits, split_stride), v = row_sum_splits(qr + ib, splits, split_stride);
-    const float a = u * cs - v * sn, b = v * cs + u * sn;
-    dst[ia] = a;
-    dst[ib] = b;
-    if (full) { full[dn + ia] = from_f32<TO>(a); full[dn + ib] = from_f32<TO>(b); }
+    const float a = u * cs - v * sn, c = v * cs + u * sn;
+    if (dst) { dst[ia] = from_f32<TR>(a); dst[ib] = from_f32<TR>(c); }
+    if (full) { full[dn + ia] = from_f32<TO>(a); full[dn + ib] = from_f32<TO>(c); }
   }
   for (int i = rot_dims + threadIdx.x; i < dr; i += blockDim.x) {
     const float v = row_sum_splits(qr + i, splits, split_stride);
-    dst[i] = v;
+    if (dst) dst[i] = from_f32<TR>(v);
     if (full) full[dn + i] = from_f32<TO>(v);
   }
 }
 
 JLX_API int jlx_latent_q_prep(const float* q, int splits, long long split_stride, const float* inv_freq, int rot_dims,
-                              const int* positions, void* q_nope, int dtype, float* q_rot, void* q_full, int N, int H, int dn,
-                              int dr, int halves, cudaStream_t stream) {
+                              const int* positions, void* q_nope, int dtype, void* q_rot, int rot_dtype, void* q_full, int N,
+                              int H, int dn, int dr, int halves, const int* rows, cudaStream_t stream) {
   JLX_REQUIRE(N >= 0 && H > 0 && dn > 0 && dr >= 0 && splits >= 1, "latent_q_prep: bad sizes");
   JLX_REQUIRE(rot_dims >= 0 && rot_dims <= dr && rot_dims % 2 == 0, "latent_q_prep: %d rotated entries of %d", rot_dims, dr);
   JLX_REQUIRE(H <= 65535, "latent_q_prep: too many heads (%d)", H);
   if (N == 0) return 0;
-  JLX_DISPATCH_DTYPE(dtype, TO, {
-    JLX_CUDA(jlx_launch_pdl(latent_q_prep_kernel<TO>, dim3(N, H), dim3(64), 0, stream, q, splits, split_stride, inv_freq, rot_dims,
-                            positions, (TO*)q_nope, q_rot, (TO*)q_full, N, H, dn, dr, halves));
-  });
+  JLX_DISPATCH_DTYPE(dtype, TO, JLX_DISPATCH_DTYPE(rot_dtype, TR, {
+    JLX_CUDA(jlx_launch_pdl(latent_q_prep_kernel<TO, TR>, dim3(N, H), dim3(64), 0, stream, q, splits, split_stride, inv_freq, rot_dims,
+                            positions, (TO*)q_nope, (TR*)q_rot, (TO*)q_full, N, H, dn, dr, halves, rows));
+  }));
   JLX_LAUNCH_CHECK("latent_q_prep");
   return 0;
 }
@@ -170,7 +171,7 @@ JLX_API int jlx_latent_q_prep(const float* q, int splits, long long split_stride
 // m = sink, l = exp(sink - m) = 1.
 // With a window the walk starts at the tile that holds the first visible key; earlier keys of that tile (whose pages may
 // have been given back) are read as zeros and masked.
-// With `rows` the block serves token rows[blockIdx.x] (the single decoded tokens of a step that also holds prompt
+// With `rows` block b serves token rows[b], whose query and output are row b of theirs (the single decoded tokens of a step that also holds prompt
 // portions).  With splits > 1 block z takes the keys [(s0 + z) split_keys, (s0 + z + 1) split_keys), s0 the first visible key's range (a multiple of
 // the tile, so tiles stay aligned), and leaves (m, l, unnormalised sums) for the combine kernel; the sink opens split 0.
 #define LAT_TILE 32
@@ -196,14 +197,15 @@ __global__ void attention_latent_kernel(const float* __restrict__ q_lat, const f
   float* qs = smem;                     // [nwarp * HPW][dk]
   float* ks = qs + nwarp * HPW * dk;    // [LAT_TILE][ldk]
   const int n = rows ? rows[blockIdx.x] : blockIdx.x;
+  const int b = blockIdx.x;  // queries, outputs and partial results are numbered as the blocks are
   const int h0 = (blockIdx.y * nwarp + warp) * HPW;  // the warp's first head
   const int z = blockIdx.z;
   const int p = positions[n], r = req_of_token[n];
   for (int u = 0; u < HPW; ++u) {  // heads beyond H get a zero query: they run along and write nothing
     const int h = h0 + u;
     float* q = qs + (warp * HPW + u) * dk;
-    for (int d = lane; d < rank; d += 32) q[d] = h < H ? q_lat[((size_t)h * N + n) * rank + d] : 0.f;
-    for (int d = lane; d < dr; d += 32) q[rank + d] = h < H ? q_rot[((size_t)n * H + h) * dr + d] : 0.f;
+    for (int d = lane; d < rank; d += 32) q[d] = h < H ? q_lat[((size_t)h * N + b) * rank + d] : 0.f;
+    for (int d = lane; d < dr; d += 32) q[rank + d] = h < H ? q_rot[((size_t)b * H + h) * dr + d] : 0.f;
   }
   const bool has_sink = sink != nullptr && z == 0;
   float m[HPW], l[HPW], acc[HPW][R32];
@@ -334,7 +336,7 @@ __global__ void attention_latent_kernel(const float* __restrict__ q_lat, const f
 #pragma unroll
       for (int i = 0; i < R32; ++i) {
         const int d = lane + 32 * i;
-        if (i < nd && d < rank) out_lat[((size_t)h * N + n) * rank + d] = from_f32<TO>(acc[u][i] / l[u]);
+        if (i < nd && d < rank) out_lat[((size_t)h * N + b) * rank + d] = from_f32<TO>(acc[u][i] / l[u]);
       }
     }
   }
@@ -354,7 +356,7 @@ __global__ void attention_latent_kernel(const float* __restrict__ q_lat, const f
 
 template <typename TO, int PIECES>
 __global__ void __launch_bounds__(LATM_THREADS)
-attention_latent_mma_kernel(const float* __restrict__ q_lat, const float* __restrict__ q_rot, const bf16* __restrict__ pages,
+attention_latent_mma_kernel(const bf16* __restrict__ q_lat, const bf16* __restrict__ q_rot, const bf16* __restrict__ pages,
                             const int* __restrict__ block_table, int bt_stride, const int* __restrict__ req_of_token,
                             const int* __restrict__ positions, const float* __restrict__ sink, TO* __restrict__ out_lat, int N,
                             int H, int rank, int dr, int page_size, int num_pages, float scale, const int* __restrict__ rows,
@@ -399,24 +401,23 @@ attention_latent_mma_kernel(const float* __restrict__ q_lat, const float* __rest
     for (int i = threadIdx.x; i < (2 * LATM_KEYS + 16) * 8; i += LATM_THREADS) qs[(size_t)(i >> 3) * ldk + dk + (i & 7)] = __float2bfloat16_rn(0.f);
   auto old_tile = [&](int t) { return t_begin + (t + 1) * LATM_KEYS <= p; };  // ends below the token's own row
   const bool early0 = single && n_tiles > 0 && old_tile(0), early1 = early0 && n_tiles > 1 && old_tile(1);
-  if (early0) load(0);
-  if (early0) cp_async_commit();
-  if (early1) load(1);
-  if (early1) cp_async_commit();
+  if (early0) { load(0); cp_async_commit(); }
+  if (early1) { load(1); cp_async_commit(); }
   pdl_launch_dependents_if_small();
   pdl_wait();
-  if (n_tiles > 0 && !early0) { load(0); cp_async_commit(); }
-  if (!early1) {
-    if (n_tiles > 1) load(1);
-    cp_async_commit();  // (maybe empty: the waits below count groups)
-  }
   for (int u = warp; u < 16; u += LATM_THREADS / 32) {  // heads beyond H get a zero query: they run along and write nothing
     const int h = h0 + u;
-    for (int d = lane; d < dk; d += 32) {
-      float v = 0.f;
-      if (h < H) v = d < rank ? q_lat[((size_t)h * N + n) * rank + d] : q_rot[((size_t)n * H + h) * dr + (d - rank)];
-      qs[(size_t)u * ldk + d] = __float2bfloat16_rn(v);
-    }
+    const bool valid = h < H;
+    const bf16* a = q_lat + ((size_t)(valid ? h : 0) * N + blockIdx.x) * rank;
+    const bf16* c = q_rot + ((size_t)blockIdx.x * H + (valid ? h : 0)) * dr;
+    const uint32_t dst = smem_u32(qs + (size_t)u * ldk);
+    for (int i = lane; i < chunks; i += 32) cp_async16(dst + i * 16, i * 8 < rank ? a + i * 8 : c + (i * 8 - rank), valid);
+  }
+  if (n_tiles > 0 && !early0) load(0);
+  cp_async_commit();
+  if (!early1) {
+    if (n_tiles > 1) load(1);
+    cp_async_commit();  // (maybe empty: the first wait counts groups)
   }
   const int g0 = lane >> 2, g1 = g0 + 8;  // this thread's two heads
   const float sc2 = scale * 1.4426950408889634f;
@@ -435,7 +436,7 @@ attention_latent_mma_kernel(const float* __restrict__ q_lat, const float* __rest
     for (int e = 0; e < 4; ++e) o[i][0][e] = o[i][1][e] = 0.f;
 
   for (int t = 0; t < n_tiles; ++t) {
-    if (t == 0) cp_async_wait<1>();
+    if (t == 0 && !early1) cp_async_wait<1>();  // all but tile 1
     else cp_async_wait<0>();
     __syncthreads();  // tile t has landed for everyone; everyone is done with tile t - 1
     if (t > 0) {
@@ -554,7 +555,7 @@ attention_latent_mma_kernel(const float* __restrict__ q_lat, const float* __rest
           const int c = (warp + i * 4) * 16 + q * 8 + (lane & 3) * 2 + e;
           if (c >= rank) continue;
           if (splits > 1) part_acc[slot * rank + c] = o[i][q][u * 2 + e];
-          else out_lat[((size_t)h * N + n) * rank + c] = from_f32<TO>(o[i][q][u * 2 + e] * inv);
+          else out_lat[((size_t)h * N + blockIdx.x) * rank + c] = from_f32<TO>(o[i][q][u * 2 + e] * inv);
         }
   }
 }
@@ -562,58 +563,59 @@ attention_latent_mma_kernel(const float* __restrict__ q_lat, const float* __rest
 // out = sum_z acc_z exp(m_z - m) / sum_z l_z exp(m_z - m), m = max_z m_z, the splits in ascending order.
 template <typename TO>
 __global__ void attention_latent_combine_kernel(const float* __restrict__ part_acc, const float* __restrict__ part_ml,
-                                                TO* __restrict__ out_lat, const int* __restrict__ rows, int N, int H, int rank,
-                                                int splits) {
+                                                TO* __restrict__ out_lat, int N, int H, int rank, int splits) {
   JLX_TL(TL_ATTN_COMBINE);
   pdl_launch_dependents_if_small();
   pdl_wait();
   const int b = blockIdx.x, h = blockIdx.y;
-  const int n = rows ? rows[b] : b;
   const size_t slot0 = ((size_t)b * H + h) * splits;
-  __shared__ float wgt[LAT_COMBINE_CACHE];  // the ranges' shares of the sum
-  float m = -INFINITY;
-  for (int z = 0; z < splits; ++z) m = fmaxf(m, part_ml[2 * (slot0 + z)]);
-  float l = 0.f;
-  for (int z = 0; z < splits; ++z) {
-    const float mz = part_ml[2 * (slot0 + z)];
-    if (mz > -INFINITY) l += part_ml[2 * (slot0 + z) + 1] * expf(mz - m);
-  }
+  __shared__ float ms[LAT_COMBINE_CACHE], wgt[LAT_COMBINE_CACHE];  // the ranges' maxima; their sums, then their shares
   const bool cached = splits <= LAT_COMBINE_CACHE;
+  const float2* ml = reinterpret_cast<const float2*>(part_ml) + slot0;
+  float m = -INFINITY, l = 0.f;
   if (cached) {
     for (int z = threadIdx.x; z < splits; z += blockDim.x) {
-      const float mz = part_ml[2 * (slot0 + z)];
-      wgt[z] = mz > -INFINITY ? expf(mz - m) : 0.f;
+      const float2 v = ml[z];
+      ms[z] = v.x;
+      wgt[z] = v.y;
     }
     __syncthreads();
+    for (int z = 0; z < splits; ++z) m = fmaxf(m, ms[z]);
+    for (int z = 0; z < splits; ++z) l += ms[z] > -INFINITY ? wgt[z] * expf(ms[z] - m) : 0.f;
+    __syncthreads();
+    for (int z = threadIdx.x; z < splits; z += blockDim.x) wgt[z] = ms[z] > -INFINITY ? expf(ms[z] - m) : 0.f;
+    __syncthreads();
+  } else {
+    for (int z = 0; z < splits; ++z) m = fmaxf(m, ml[z].x);
+    for (int z = 0; z < splits; ++z) l += ml[z].x > -INFINITY ? ml[z].y * expf(ml[z].x - m) : 0.f;
   }
   for (int d = threadIdx.x; d < rank; d += blockDim.x) {
     float a = 0.f;
-#pragma unroll 4
+#pragma unroll 8
     for (int z = 0; z < splits; ++z) {
-      const float mz = cached ? 0.f : part_ml[2 * (slot0 + z)];
-      const float w = cached ? wgt[z] : (mz > -INFINITY ? expf(mz - m) : 0.f);
+      const float w = cached ? wgt[z] : (ml[z].x > -INFINITY ? expf(ml[z].x - m) : 0.f);
       a = fmaf(part_acc[(slot0 + z) * rank + d], w, a);  // (a range without keys left zeros)
     }
-    out_lat[((size_t)h * N + n) * rank + d] = from_f32<TO>(a / l);
+    out_lat[((size_t)h * N + b) * rank + d] = from_f32<TO>(a / l);
   }
 }
 
-static int latent_combine(const float* part_acc, const float* part_ml, void* out_lat, int out_dtype, const int* rows, int served, int N,
-                          int H, int rank, int splits, cudaStream_t stream) {
+static int latent_combine(const float* part_acc, const float* part_ml, void* out_lat, int out_dtype, int served, int N, int H, int rank,
+                          int splits, cudaStream_t stream) {
   if (splits == 1) return 0;
   JLX_DISPATCH_DTYPE(out_dtype, TO, {
-    JLX_CUDA(jlx_launch_pdl(attention_latent_combine_kernel<TO>, dim3(served, H), dim3(128), 0, stream, part_acc, part_ml, (TO*)out_lat,
-                            rows, N, H, rank, splits));
+    JLX_CUDA(jlx_launch_pdl(attention_latent_combine_kernel<TO>, dim3(served, H), dim3(rank > 256 ? 512 : (rank > 128 ? 256 : 128)), 0, stream, part_acc, part_ml, (TO*)out_lat,
+                            N, H, rank, splits));
   });
   JLX_LAUNCH_CHECK("attention_latent_combine");
   return 0;
 }
 
-// use_mma: 0 keeps a bfloat16 cache on the 32-bit kernel too.  single: every served token is its request's only one of
+// use_mma: the queries are bfloat16, for the tensor cores (else float32).  single: every served token is its request's only one of
 // the step.
-// rows / n_rows: serve these token rows only (N stays the row count of q and out).  splits > 1: part_acc float32
+// rows / n_rows: serve these token rows only (N = n_rows: queries and outputs in the list's order).  splits > 1: part_acc float32
 // [n_rows * H * splits * rank], part_ml float32 [n_rows * H * splits * 2].
-JLX_API int jlx_attention_latent(const float* q_lat, const float* q_rot, const void* pages, int cache_dtype,
+JLX_API int jlx_attention_latent(const void* q_lat, const void* q_rot, const void* pages, int cache_dtype,
                                  const int* block_table, int bt_stride, const int* req_of_token, const int* positions,
                                  const float* sink, void* out_lat, int out_dtype, int N, int H, int rank, int dr,
                                  int page_size, int num_pages, float scale, const int* rows, int n_rows, int splits,
@@ -627,29 +629,29 @@ JLX_API int jlx_attention_latent(const float* q_lat, const float* q_rot, const v
   const int served = rows ? n_rows : N;
   if (served == 0) return 0;
   const int dk = rank + dr;
-  // a bfloat16 cache whose rows are whole 16-byte pieces: on the tensor cores
-  if (use_mma && cache_dtype == JLX_BF16 && rank % 8 == 0 && dr % 8 == 0 && ((uintptr_t)pages & 15) == 0) {
+  if (use_mma) {  // on the tensor cores
+    JLX_REQUIRE(cache_dtype == JLX_BF16 && rank % 8 == 0 && dr % 8 == 0 && (((uintptr_t)pages | (uintptr_t)q_lat | (uintptr_t)q_rot) & 15) == 0,
+                "attention_latent: bfloat16 queries need a bfloat16 cache and sizes that are multiples of 8 (got %d + %d)", rank, dr);
     const int ldm = ((dk + 15) & ~15) + 8;  // rows an odd number of 16-byte pieces apart
     const size_t smem_m = sizeof(bf16) * (size_t)(2 * LATM_KEYS + 16) * ldm;
     const int hb = (H + 15) / 16;
-    if (smem_m <= 220 * 1024 && hb <= 65535) {
+    JLX_REQUIRE(smem_m <= 220 * 1024 && hb <= 65535, "attention_latent: a latent of %d + %d or %d heads are too many", rank, dr, H);
 #define LATM_GO(PIECES)                                                                                                        \
   do {                                                                                                                         \
     if (smem_m > 48 * 1024)                                                                                                    \
       JLX_CUDA(cudaFuncSetAttribute(attention_latent_mma_kernel<TO, PIECES>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem_m)); \
-    JLX_CUDA(jlx_launch_pdl(attention_latent_mma_kernel<TO, PIECES>, dim3(served, hb, splits), dim3(LATM_THREADS), smem_m, stream, q_lat, \
-                            q_rot, (const bf16*)pages, block_table, bt_stride, req_of_token, positions, sink, (TO*)out_lat, N, H, rank, \
+    JLX_CUDA(jlx_launch_pdl(attention_latent_mma_kernel<TO, PIECES>, dim3(served, hb, splits), dim3(LATM_THREADS), smem_m, stream, (const bf16*)q_lat, \
+                            (const bf16*)q_rot, (const bf16*)pages, block_table, bt_stride, req_of_token, positions, sink, (TO*)out_lat, N, H, rank, \
                             dr, page_size, num_pages, scale, rows, splits, split_keys, part_acc, part_ml, ldm, window, single, status)); \
   } while (0)
-      JLX_DISPATCH_DTYPE(out_dtype, TO, {
-        if (rank <= 128) LATM_GO(2);
-        else if (rank <= 512) LATM_GO(8);
-        else LATM_GO(16);
-      });
+    JLX_DISPATCH_DTYPE(out_dtype, TO, {
+      if (rank <= 128) LATM_GO(2);
+      else if (rank <= 512) LATM_GO(8);
+      else LATM_GO(16);
+    });
 #undef LATM_GO
-      JLX_LAUNCH_CHECK("attention_latent_mma");
-      return latent_combine(part_acc, part_ml, out_lat, out_dtype, rows, served, N, H, rank, splits, stream);
-    }
+    JLX_LAUNCH_CHECK("attention_latent_mma");
+    return latent_combine(part_acc, part_ml, out_lat, out_dtype, served, N, H, rank, splits, stream);
   }
   // a key's row in shared memory: padded so that 16-byte reads of a quarter warp's rows fall into different banks
   // (rows a multiple of 4 floats apart with an odd count of 16-byte pieces), else by one float
@@ -670,7 +672,7 @@ JLX_API int jlx_attention_latent(const float* q_lat, const float* q_rot, const v
       JLX_CUDA(cudaFuncSetAttribute(attention_latent_kernel<TC, TO, HPW, R32>, cudaFuncAttributeMaxDynamicSharedMemorySize, \
                                     (int)smem));                                                                           \
     JLX_CUDA(jlx_launch_pdl(attention_latent_kernel<TC, TO, HPW, R32>, dim3(served, hb, splits), dim3(nwarp * 32), smem, stream, \
-                            q_lat, q_rot, (const TC*)pages, block_table, bt_stride, req_of_token, positions, sink, (TO*)out_lat, \
+                            (const float*)q_lat, (const float*)q_rot, (const TC*)pages, block_table, bt_stride, req_of_token, positions, sink, (TO*)out_lat, \
                             N, H, rank, dr, page_size, num_pages, scale, rows, splits, split_keys, part_acc, part_ml, ldk,  \
                             window, status));                                                                                      \
   } while (0)
@@ -680,7 +682,7 @@ JLX_API int jlx_attention_latent(const float* q_lat, const float* q_rot, const v
   }));
 #undef LAT_GO
   JLX_LAUNCH_CHECK("attention_latent");
-  return latent_combine(part_acc, part_ml, out_lat, out_dtype, rows, served, N, H, rank, splits, stream);
+  return latent_combine(part_acc, part_ml, out_lat, out_dtype, served, N, H, rank, splits, stream);
 }
 
 // ------------------------------------------------------------------------------------------------ prompt portions
@@ -807,7 +809,8 @@ JLX_API int jlx_causal_sink_softmax(const float* s, const float* sink, float sca
 }
 
 // [H, N, d] -> [N, H * d]: the per-head products' rows back into token rows, with `gate` (float32 rows, possibly split-K
-// partials) through a gate per token and head: out[n, h d + c] = sigmoid(gate[n, h]) * in[h, n, c].
+// partials) through a gate per token and head: out[n, h d + c] = sigmoid(gate[n, h]) * in[h, n, c].  With `rows` row b of
+// the input belongs to token rows[b].
 struct GateRowsView {
   const float* p;
   long long split_stride;
@@ -817,14 +820,15 @@ struct GateRowsView {
 };
 
 template <typename T>
-__global__ void heads_to_rows_kernel(const T* __restrict__ in, T* __restrict__ out, int N, int H, int d, GateRowsView gate) {
+__global__ void heads_to_rows_kernel(const T* __restrict__ in, T* __restrict__ out, int N, int H, int d, GateRowsView gate,
+                                     const int* __restrict__ rows) {
   JLX_TL(TL_OTHER);
   pdl_launch_dependents_if_small();
   pdl_wait();
-  const int n = blockIdx.x;
+  const int b = blockIdx.x, n = rows ? rows[b] : b;
   for (int i = threadIdx.x; i < H * d; i += blockDim.x) {
     const int h = i / d, c = i - h * d;
-    T v = in[((size_t)h * N + n) * d + c];
+    T v = in[((size_t)h * N + b) * d + c];
     if (gate.p) {
       const float s = row_sum_splits(gate.p + (size_t)n * gate.ld + h, gate.splits, gate.split_stride);
       v = from_f32<T>(to_f32<T>(v) / (1.f + expf(-s)));
@@ -833,12 +837,13 @@ __global__ void heads_to_rows_kernel(const T* __restrict__ in, T* __restrict__ o
   }
 }
 
-JLX_API int jlx_heads_to_rows(const void* in, void* out, int dtype, int N, int H, int d, const GateRowsView* gate, cudaStream_t stream) {
+JLX_API int jlx_heads_to_rows(const void* in, void* out, int dtype, int N, int H, int d, const GateRowsView* gate, const int* rows,
+                              cudaStream_t stream) {
   JLX_REQUIRE(N >= 0 && H > 0 && d > 0, "heads_to_rows: bad sizes");
   if (N == 0) return 0;
   const GateRowsView none = {nullptr, 0, 0, 1, 0};
   JLX_DISPATCH_DTYPE(dtype, T, {
-    JLX_CUDA(jlx_launch_pdl(heads_to_rows_kernel<T>, dim3(N), dim3(256), 0, stream, (const T*)in, (T*)out, N, H, d, gate ? *gate : none));
+    JLX_CUDA(jlx_launch_pdl(heads_to_rows_kernel<T>, dim3(N), dim3(256), 0, stream, (const T*)in, (T*)out, N, H, d, gate ? *gate : none, rows));
   });
   JLX_LAUNCH_CHECK("heads_to_rows");
   return 0;

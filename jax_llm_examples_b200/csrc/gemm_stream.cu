@@ -140,6 +140,7 @@ struct StreamArgs {
   int rows;              // token rows in A (upper bound of offsets[E])
   const int* offsets;    // null: one group over all rows
   int E;
+  int uniform;           // > 0: E groups of so many rows each, without offsets
   const int* tile_list;  // optional, with offsets: (group, first row) of every row tile that has rows
   const int* n_tiles;    // ... and how many there are
   void* out;             // [rows, N] (bf16 or f32), or partials [splits][rows][N] f32 when splits > 1
@@ -277,6 +278,11 @@ gemm_stream_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_const
       t -= tiles;
     }
     if (!found) return;
+  } else if (args.uniform) {
+    const int per_group = (args.uniform + BT - 1) / BT;
+    group = blockIdx.y / per_group;
+    row_lo = group * args.uniform + (blockIdx.y - group * per_group) * BT;
+    row_hi = (group + 1) * args.uniform;
   } else {
     row_lo = blockIdx.y * BT;
     row_hi = args.rows;
@@ -430,6 +436,11 @@ gemm_stream_pair_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_
       t -= tiles;
     }
     if (!found) return;
+  } else if (args.uniform) {
+    const int per_group = (args.uniform + BT - 1) / BT;
+    group = blockIdx.y / per_group;
+    row_lo = group * args.uniform + (blockIdx.y - group * per_group) * BT;
+    row_hi = (group + 1) * args.uniform;
   } else {
     row_lo = blockIdx.y * BT;
     row_hi = args.rows;
@@ -627,6 +638,7 @@ JLX_API int jlx_gemm_stream_token_tile(int rows_hint) { return pick_bt(rows_hint
 //         [rows, N / 2] = silu(gate) * up; no split-K.  In general g sigmoid(glu_alpha g) (u + glu_shift) with
 //         g = min(gate, glu_limit), u = clamp(up, +-glu_limit) when glu_limit > 0; (1, 0, 0) is silu(gate) * up.
 // mode 3: an activation in the epilogue, out = act(sum) by its number `act` (activation.cuh); no split-K.
+// uniform_rows > 0 (no offsets): E groups of so many rows each, so that no block has to look for its tile.
 // tile_list / n_tiles (optional, grouped only): the row tiles that have rows, made by jlx_expert_sort for the
 // tile width jlx_gemm_stream_token_tile(rows_hint); without them every block walks the offsets.
 // offsets_settled (grouped only): the caller's word that the kernel launched just before this one on the stream is a
@@ -635,7 +647,7 @@ JLX_API int jlx_gemm_stream_token_tile(int rows_hint) { return pick_bt(rows_hint
 JLX_API int jlx_gemm_stream(const void* A, const void* W, void* out, int out_is_f32, int rows, int N, int K,
                             const int* offsets, int E, int rows_hint, int splits, float* scratch, int mode,
                             const int* tile_list, const int* n_tiles, int offsets_settled, int* splits_used, int* status,
-                            float glu_alpha, float glu_limit, float glu_shift, int act, cudaStream_t stream) {
+                            float glu_alpha, float glu_limit, float glu_shift, int act, int uniform_rows, cudaStream_t stream) {
   JLX_REQUIRE(rows >= 0 && N > 0 && K > 0, "gemm_stream: bad sizes rows=%d N=%d K=%d", rows, N, K);
   JLX_REQUIRE(K % 8 == 0, "gemm_stream: K = %d is no multiple of 8 (TMA needs 16-byte row strides); use the SIMT product", K);
   JLX_REQUIRE(((uintptr_t)A & 15) == 0 && ((uintptr_t)W & 15) == 0, "gemm_stream: operands must be 16-byte aligned");
@@ -648,8 +660,10 @@ JLX_API int jlx_gemm_stream(const void* A, const void* W, void* out, int out_is_
   JLX_REQUIRE(mode != 1 || out_is_f32, "gemm_stream: partials are float32");
   if (splits_used) *splits_used = 1;
   if (rows == 0) return 0;
-  const int groups = offsets ? E : 1;
-  const int bt = pick_bt(rows_hint > 0 ? rows_hint : rows);
+  JLX_REQUIRE(uniform_rows >= 0 && (uniform_rows == 0 || (!offsets && E > 0 && (long long)E * uniform_rows == rows)),
+              "gemm_stream: %d groups of %d rows are not %d rows", E, uniform_rows, rows);
+  const int groups = offsets || uniform_rows ? E : 1;
+  const int bt = pick_bt(uniform_rows ? uniform_rows : (rows_hint > 0 ? rows_hint : rows));
   CUtensorMap mw, ma;
   if (make_map(&mw, W, (long long)groups * N, K, WN)) return 1;
   if (make_map(&ma, A, rows, K, bt)) return 1;
@@ -660,7 +674,7 @@ JLX_API int jlx_gemm_stream(const void* A, const void* W, void* out, int out_is_
   }
   if (splits_used) *splits_used = splits;
   StreamArgs a;
-  a.N = N; a.K = K; a.rows = rows; a.offsets = offsets; a.E = E;
+  a.N = N; a.K = K; a.rows = rows; a.offsets = offsets; a.E = E; a.uniform = uniform_rows;
   a.tile_list = offsets ? tile_list : nullptr; a.n_tiles = n_tiles;
   a.out = (splits > 1 && mode == 0) ? (void*)scratch : out;
   a.out_is_f32 = out_is_f32; a.silu = mode == 2; a.glu_alpha = glu_alpha; a.glu_limit = glu_limit; a.glu_shift = glu_shift; a.splits = splits; a.k_per_split = kps; a.status = status;
@@ -670,7 +684,8 @@ JLX_API int jlx_gemm_stream(const void* A, const void* W, void* out, int out_is_
   // with rows has any, so there are at most rows / bt + min(E, rows) of them.  (A looser bound costs time: a block
   // without a tile returns at once, but with the kernel's shared memory only two blocks fit an SM at a time, and with
   // 128 experts and a handful of rows the blocks without work were a hundred times the blocks with.)
-  const int row_tiles = offsets ? rows / bt + (E < rows ? E : rows) : (rows + bt - 1) / bt;
+  const int row_tiles = offsets ? rows / bt + (E < rows ? E : rows)
+                                : (uniform_rows ? E * ((uniform_rows + bt - 1) / bt) : (rows + bt - 1) / bt);
   JLX_REQUIRE(row_tiles <= 65535, "gemm_stream: too many row tiles");
   int rc;
   // Wide token tiles (prompt portions): a pair of blocks per 256 weight rows, when the rows divide so.

@@ -224,10 +224,15 @@ JLX_API int jlx_group_norm(float* x, const float* delta, int splits, long long s
                   (((uintptr_t)x | (uintptr_t)delta | (uintptr_t)delta_bias | (uintptr_t)post_w | (uintptr_t)pre_w |
                     (uintptr_t)out | (uintptr_t)out32) & 15) == 0;
   if (x4) {
+    // Few rows in bfloat16 (decoding) are bound by latency: a thread per four values.  The block's size fixes the order of
+    // the sums, so in 32-bit output it depends on the width alone.
+    int threads4 = D >= 8192 ? 512 : (D >= 2048 ? 256 : 128);
+    if (N <= 64 && out && out_dtype == JLX_BF16)
+      while (threads4 < 1024 && threads4 * 4 < D) threads4 *= 2;
     JLX_DISPATCH_DTYPE(out_dtype, TO, {
       if (smem > 48 * 1024)
         JLX_CUDA(cudaFuncSetAttribute(group_norm_x4_kernel<TO>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
-      JLX_CUDA(jlx_launch_pdl(group_norm_x4_kernel<TO>, dim3(N), dim3(D >= 8192 ? 512 : (D >= 2048 ? 256 : 128)), smem, stream,
+      JLX_CUDA(jlx_launch_pdl(group_norm_x4_kernel<TO>, dim3(N), dim3(threads4), smem, stream,
                               x, rows, delta_bias, post_w, post_groups, post_norm, mult, pre_w, pre_groups, pre_norm,
                               eps, (TO*)out, ld_out, out32, row_index, D));
     });

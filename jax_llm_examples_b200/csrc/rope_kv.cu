@@ -418,15 +418,23 @@ __global__ void rope_half_kv_store_kernel(RopeRowsView proj, int k_col, int v_co
   JLX_TL(TL_ROPE);
   pdl_launch_dependents_if_small();
   __shared__ float whole_part[2][8];
-  extern __shared__ float buf[];  // [warps][2][max(dk, dv)]: a head's row as projected (and normed), and as rotated
+  extern __shared__ float buf[];  // [warps][2][max(dk, dv)]: a head's row as projected (and normed), and as rotated; the angles
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarp = blockDim.x >> 5;
   const size_t n = blockIdx.x;
   const int dmax = dk > dv ? dk : dv;
   float* row = buf + (size_t)warp * 2 * dmax;
   float* turned = row + dmax;
-  pdl_wait();
+  float* angles = buf + (size_t)nwarp * 2 * dmax;  // [rot / 2][2]: sine and cosine of this token's angles
+  // the step's description is older than the step: the token's place and its angles are made before the wait for the
+  // projected rows
   const int pos = positions[n];
   const int half = rot >> 1;
+  for (int i = threadIdx.x; i < half; i += blockDim.x) {
+    float sn, cs;
+    sincosf((float)pos * inv_freq[i], &sn, &cs);
+    angles[2 * i] = sn * amplitude;
+    angles[2 * i + 1] = cs * amplitude;
+  }
   T* kdst = nullptr;
   if (store) {
     const int page = block_table[(size_t)req_of_token[n] * bt_stride + pos / page_size];
@@ -436,6 +444,8 @@ __global__ void rope_half_kv_store_kernel(RopeRowsView proj, int k_col, int v_co
       kdst = pages + ((size_t)page * 2 * Hkv * page_size + (size_t)(pos % page_size)) * dpad;
     }
   }
+  __syncthreads();
+  pdl_wait();
   const int heads = Hq + (store ? 2 * Hkv : 0);
   float whole_rms[2] = {1.f, 1.f};  // of all q entries, of all k entries
   if (norm_mode == ROPE_NORM_WHOLE) {
@@ -495,10 +505,7 @@ __global__ void rope_half_kv_store_kernel(RopeRowsView proj, int k_col, int v_co
         const bool first = pairing == ROPE_PAIRS_INTERLEAVED ? !(i & 1) : i < half;
         const int f = pairing == ROPE_PAIRS_INTERLEAVED ? i >> 1 : (first ? i : i - half);
         const int partner = pairing == ROPE_PAIRS_INTERLEAVED ? i ^ 1 : (first ? i + half : i - half);
-        float sn, cs;
-        sincosf((float)pos * inv_freq[f], &sn, &cs);
-        sn *= amplitude;
-        cs *= amplitude;
+        const float sn = angles[2 * f], cs = angles[2 * f + 1];
         y = first ? row[i] * cs - row[partner] * sn : row[i] * cs + row[partner] * sn;
       }
       turned[i] = y;
@@ -546,7 +553,7 @@ JLX_API int jlx_rope_half_kv_store(const RopeRowsView* proj, int k_col, int v_co
   const int heads = Hq + (store ? 2 * Hkv : 0);
   const int nwarp = heads < 8 ? heads : 8;
   const int by = N >= 64 ? 1 : (heads + nwarp - 1) / nwarp;
-  const size_t smem = sizeof(float) * 2 * (size_t)nwarp * (dk > dv ? dk : dv);
+  const size_t smem = sizeof(float) * (2 * (size_t)nwarp * (dk > dv ? dk : dv) + rot);
   JLX_REQUIRE(smem <= 48 * 1024, "rope_half: head size too large");
   JLX_DISPATCH_DTYPE(dtype, T, {
     JLX_CUDA(jlx_launch_pdl(rope_half_kv_store_kernel<T>, dim3(N, by), dim3(nwarp * 32), smem, stream, *proj, k_col, v_col,

@@ -441,16 +441,21 @@ def latent_kv_prep(proj: torch.Tensor, splits: int, q_norm_weight: torch.Tensor,
 
 
 def latent_q_prep(q: torch.Tensor, splits: int, inv_freq: torch.Tensor, rot_dims: int, positions: torch.Tensor,
-                  q_nope: torch.Tensor, q_rot: torch.Tensor, heads: int, dn: int, dr: int, q_full: torch.Tensor | None = None,
-                  pairing: str = "pairs") -> None:
-    """q: float32 [N, H (dn + dr)] (or partials) -> q_nope [H, N, dn] (head-major), q_rot float32 [N, H, dr], rotated,
-    and optionally q_full [H, N, dn + dr] (both parts, in q_nope's type)."""
-    _contig(q, inv_freq, q_nope, q_rot, q_full)
-    N = q_rot.shape[0]
+                  q_nope: torch.Tensor | None, q_rot: torch.Tensor | None, heads: int, dn: int, dr: int, q_full: torch.Tensor | None = None,
+                  pairing: str = "pairs", rows: torch.Tensor | None = None) -> None:
+    """q: float32 [N, H (dn + dr)] (or partials) -> q_nope [H, S, dn] (head-major) and q_rot [S, H, dr], rotated (float32 or
+    the activations' type), and / or q_full [H, S, dn + dr] (both parts).  S = N, or the rows listed in ``rows`` (int32)."""
+    _contig(q, inv_freq, q_nope, q_rot, q_full, rows)
+    if (q_nope is None) != (q_rot is None) or (q_nope is None and q_full is None):
+        raise KernelError("latent_q_prep: q_nope comes with q_rot; one of the two forms is needed")
+    N = q_rot.shape[0] if q_rot is not None else q_full.shape[1]
+    dtype = q_nope.dtype if q_nope is not None else q_full.dtype
+    if q_rot is not None and q_rot.dtype not in (torch.float32, dtype):
+        raise KernelError("latent_q_prep: the rotated parts are float32 or of the activations' type")
     sp, stride = _splits(q, splits)
     _run("attention_latent", "jlx_latent_q_prep", _ptr(q), c_int(sp), c_longlong(stride), _ptr(inv_freq), c_int(rot_dims),
-         _ptr(positions), _ptr(q_nope), c_int(code(q_nope.dtype)), _ptr(q_rot), _ptr(q_full), c_int(N), c_int(heads), c_int(dn),
-         c_int(dr), c_int(int(pairing == "halves")), _stream())
+         _ptr(positions), _ptr(q_nope), c_int(code(dtype)), _ptr(q_rot), c_int(code(q_rot.dtype) if q_rot is not None else F32),
+         _ptr(q_full), c_int(N), c_int(heads), c_int(dn), c_int(dr), c_int(int(pairing == "halves")), _ptr(rows), _stream())
 
 
 LATENT_KEY_TILE = 32  # keys per tile of the latent attention kernel: split sizes are multiples of it
@@ -460,23 +465,26 @@ def attention_latent(q_lat: torch.Tensor, q_rot: torch.Tensor, pages: torch.Tens
                      req_of_token: torch.Tensor, positions: torch.Tensor, sink: torch.Tensor | None, out_lat: torch.Tensor,
                      scale: float, status: torch.Tensor, rows: torch.Tensor | None = None, n_rows: int = 0, splits: int = 1,
                      split_keys: int = 0, part_acc: torch.Tensor | None = None, part_ml: torch.Tensor | None = None,
-                     window: int = 0, tensor_cores: bool = True, single_tokens: bool = False) -> None:
+                     window: int = 0, single_tokens: bool = False) -> None:
     """Causal attention in the latent space with an optional per-head sink and window (a query sees itself and the
-    window - 1 keys before it; 0: all).  A bfloat16 cache whose rows are whole 16-byte pieces goes to the tensor cores
-    (queries and weights rounded to bfloat16, sums in 32-bit) unless ``tensor_cores`` is False.  ``single_tokens``: every
-    served token is its request's only one of the step, so that older keys may be fetched ahead of the predecessor.  q_lat: float32 [H, N, rank]; q_rot:
-    float32 [N, H, dr]; pages: [P, 1, 1, page_size, rank + dr]; out_lat: [H, N, rank].
-    rows / n_rows: serve these token rows only (int32).  splits > 1: the keys are cut into ranges of ``split_keys``
+    window - 1 keys before it; 0: all).  Queries in bfloat16 (a bfloat16 cache, rank and dr multiples of 8) go to the tensor
+    cores (sums in 32-bit); there ``single_tokens`` says that every served token is its request's only one of the step, so
+    that older keys may be fetched ahead of the predecessor.  q_lat: [H, S, rank]; q_rot:
+    [S, H, dr]; pages: [P, 1, 1, page_size, rank + dr]; out_lat: [H, S, rank];
+    S = N tokens.  rows / n_rows: serve these token rows only (int32; S = n_rows: queries and outputs in the list's order).  splits > 1: the keys are cut into ranges of ``split_keys``
     (a multiple of LATENT_KEY_TILE; ranges are counted from the first visible key's), a block each, and a second kernel adds the ranges' results; part_acc: float32
     [served * H * splits * rank], part_ml: float32 [served * H * splits * 2]."""
     _contig(q_lat, q_rot, pages, block_table, sink, out_lat, rows, part_acc, part_ml)
     H, N, rank = q_lat.shape
     dr = q_rot.shape[2]
-    if q_lat.dtype != torch.float32 or q_rot.dtype != torch.float32 or (sink is not None and sink.dtype != torch.float32):
-        raise KernelError("attention_latent: queries and sinks must be float32")
+    tensor_cores = q_lat.dtype == torch.bfloat16
+    if q_rot.dtype != q_lat.dtype or (q_lat.dtype != torch.float32 and not tensor_cores) or (sink is not None and sink.dtype != torch.float32):
+        raise KernelError("attention_latent: queries are float32 or bfloat16, sinks float32")
+    if rows is not None and N != n_rows:
+        raise KernelError(f"attention_latent: {n_rows} listed rows need {n_rows} queries, not {N}")
     if pages.shape[4] != rank + dr:
         raise KernelError("attention_latent: cache rows and queries disagree in size")
-    served = n_rows if rows is not None else N
+    served = N
     if splits > 1 and (part_acc is None or part_ml is None or part_acc.numel() < served * H * splits * rank
                        or part_ml.numel() < served * H * splits * 2):
         raise KernelError("attention_latent: scratch for the partial results is missing or too small")
@@ -485,7 +493,7 @@ def attention_latent(q_lat: torch.Tensor, q_rot: torch.Tensor, pages: torch.Tens
          _ptr(block_table), c_int(block_table.shape[1]), _ptr(req_of_token), _ptr(positions), _ptr(sink), _ptr(out_lat),
          c_int(code(out_lat.dtype)), c_int(N), c_int(H), c_int(rank), c_int(dr), c_int(pages.shape[3]), c_int(pages.shape[0]),
          c_float(scale), _ptr(rows), c_int(n_rows), c_int(splits), c_int(split_keys), _ptr(part_acc), _ptr(part_ml),
-         c_int(window), c_int(int(tensor_cores)), c_int(int(single_tokens)), _ptr(status), _stream())
+         c_int(window), c_int(int(tensor_cores)), c_int(int(single_tokens and tensor_cores)), _ptr(status), _stream())
     _launches += int(splits > 1)  # the combine kernel
 
 
@@ -525,13 +533,13 @@ def causal_sink_softmax(scores: torch.Tensor, sink: torch.Tensor | None, scale: 
          c_int(window), _ptr(probs), c_int(code(probs.dtype)), c_int(H), c_int(T), c_int(L), _stream())
 
 
-def heads_to_rows(x: torch.Tensor, out: torch.Tensor, gate: "_RowsView | None" = None) -> None:
+def heads_to_rows(x: torch.Tensor, out: torch.Tensor, gate: "_RowsView | None" = None, rows: torch.Tensor | None = None) -> None:
     """x: [H, N, d] -> out: [N, H * d]; with ``gate`` (projected rows, column h of row n for head h of token n) every head
-    is multiplied by sigmoid(gate[n, h])."""
-    _contig(x, out)
+    is multiplied by sigmoid(gate[n, h]).  ``rows`` (int32 [N]): x's row i goes to (and takes its gate from) row rows[i]."""
+    _contig(x, out, rows)
     H, N, d = x.shape
     _run("attention_latent", "jlx_heads_to_rows", _ptr(x), _ptr(out), c_int(code(x.dtype)), c_int(N), c_int(H), c_int(d),
-         ctypes.byref(gate) if gate is not None else None, _stream())
+         ctypes.byref(gate) if gate is not None else None, _ptr(rows), _stream())
 
 
 # ------------------------------------------------------ linear attention with a decay per key channel
@@ -906,23 +914,24 @@ def gemm_stream(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, status: tor
                 offsets: torch.Tensor | None = None, rows_hint: int = 0, splits: int = 1,
                 scratch: torch.Tensor | None = None, mode: int = GEMM_PLAIN,
                 tiles: tuple[torch.Tensor, torch.Tensor] | None = None, offsets_settled: bool = False, glu=SILU_GLU,
-                activation: str = "none") -> int:
+                activation: str = "none", uniform_rows: int = 0) -> int:
     """a @ w^T on the tcgen05 tensor cores (bfloat16 in, float32 accumulate).  a: [M, K]; w: [N, K] or,
     with row-group offsets [E + 1], [E, N, K].
     GEMM_PLAIN: out [M, N] bfloat16 or float32; splits > 1 cuts K across blocks (scratch: float32
     [splits * M * N]) and adds the partials.  GEMM_PARTIALS: out is float32 [splits, M, N], left for the
     consumer to add.  GEMM_SWIGLU: w's rows are interleaved [16 gate, 16 up]; out [M, N / 2] =
     silu(gate) * up, or the gated activation ``glu`` (see :func:`glu_form`).  GEMM_ACT: out [M, N] = ``activation`` (a name
-    of ACTIVATIONS) of the sums.  ``tiles`` = (tile_list, n_tiles) from
+    of ACTIVATIONS) of the sums.  ``uniform_rows`` > 0 (instead of offsets): w's
+    groups have so many rows each.  ``tiles`` = (tile_list, n_tiles) from
     expert_sort for the same rows_hint.
     ``offsets_settled``: the kernel launched just before this call on the stream was a grouped gemm_stream over the
     same offsets and tiles (this one then finds its tile and asks for its weights without waiting for that one).
     Returns the split count used."""
     _contig(a, w, out, offsets, scratch)
     M, K = a.shape
-    E = w.shape[0] if offsets is not None else 0
+    E = w.shape[0] if offsets is not None or uniform_rows else 0
     N = w.shape[-2]
-    if w.shape[-1] != K or (offsets is None) != (w.dim() == 2):
+    if w.shape[-1] != K or (E == 0) != (w.dim() == 2):
         raise KernelError(f"gemm_stream: shapes do not fit: a {tuple(a.shape)}, w {tuple(w.shape)}")
     want = {GEMM_PLAIN: M * N, GEMM_PARTIALS: splits * M * N, GEMM_SWIGLU: M * (N // 2), GEMM_ACT: M * N}[mode]
     if out.numel() < want:
@@ -935,7 +944,7 @@ def gemm_stream(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, status: tor
     _run("gemm_stream", "jlx_gemm_stream", _ptr(a), _ptr(w), _ptr(out), c_int(int(out.dtype == torch.float32)), c_int(M),
          c_int(N), c_int(K), _ptr(offsets), c_int(E), c_int(rows_hint), c_int(splits), _ptr(scratch), c_int(mode),
          _ptr(tiles[0]) if tiles else None, _ptr(tiles[1]) if tiles else None, c_int(int(offsets_settled and offsets is not None)),
-         ctypes.byref(used), _ptr(status), c_float(glu[0]), c_float(glu[1]), c_float(glu[2]), c_int(ACTIVATIONS[activation]), _stream())
+         ctypes.byref(used), _ptr(status), c_float(glu[0]), c_float(glu[1]), c_float(glu[2]), c_int(ACTIVATIONS[activation]), c_int(uniform_rows), _stream())
     return used.value
 
 

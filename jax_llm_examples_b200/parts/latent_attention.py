@@ -25,13 +25,14 @@ def rotary_frequencies(base: float, dims: int) -> torch.Tensor:
 
 @functools.lru_cache(maxsize=None)
 def plan_head_groups(heads: int):
-    """The step planner for per-head products over head-major rows [H, N, ...]: the row offsets h * N of the heads'
-    groups (one planner per head count; mixers with the same count share it)."""
+    """The step planner for per-head products over head-major rows [H, S, ...]: the row offsets h * S of the heads' groups
+    for all of a step's tokens, and for its single tokens alone (one planner per head count; mixers with the same count
+    share it)."""
     name = f"head_group_offsets_{heads}"
 
     def planner(shape: StepShape) -> dict[str, np.ndarray]:
-        n = int(sum(shape.q_lens))
-        return {name: np.arange(heads + 1, dtype=np.int32) * n}
+        heads_at = np.arange(heads + 1, dtype=np.int32)
+        return {name: heads_at * int(sum(shape.q_lens)), name + "_single": heads_at * int(sum(n == 1 for n in shape.q_lens))}
 
     planner.array_name = name
     return planner
@@ -112,8 +113,7 @@ class LatentAttention(InputConvMixer):
         H = self.heads
         served = n_rows if rows is not None else q_rot.shape[0]
         # heads a block of the kernel serves (csrc/attention_latent.cu): the tensor-core form, or the 32-bit one
-        tensor_cores = ctx.runtime.dtype == torch.bfloat16 and self.kv_rank % 8 == 0 and self.rot_dim % 8 == 0
-        per_block = 16 if tensor_cores else 8 * (2 if self.kv_rank > 512 else 4)
+        per_block = 16 if q_lat.dtype == torch.bfloat16 else 8 * (2 if self.kv_rank > 512 else 4)
         blocks = served * -(-H // per_block)
         want = max(1, (self.SPLIT_ROUNDS * K.sm_count()) // max(blocks, 1))
         tile = K.LATENT_KEY_TILE
@@ -168,7 +168,6 @@ class LatentAttention(InputConvMixer):
         a = h if self.input_conv is None and h is not None else self.read_input(ctx, h32, cache)[0]
         dev = a.device
         n, H = a.shape[0], self.heads
-        offsets = ctx.arrays[self._planner.array_name]
         # prompt portions in bfloat16 go to the tensor cores, request by request (their sizes are read on the host: such
         # a step is never captured in a graph, only steps of single tokens are)
         portions = dt == torch.bfloat16 and ctx.max_q_len > 1 and self.w_ukv is not None
@@ -182,25 +181,32 @@ class LatentAttention(InputConvMixer):
         gate = (down.data, down.splits, self.q_rank + self.kv_rank + self.rot_dim) if self.gated else None
         with scope("qkv_matmul"):
             q = as_rows(linear(ctx, cq, self.w_uq, torch.float32, partials=True))
-        q_nope = torch.empty((H, n, self.dim), dtype=dt, device=dev)
-        q_rot = torch.empty((n, H, self.rot_dim), dtype=torch.float32, device=dev)
+        # which rows the latent-space kernel serves: all, or the single tokens beside the portions (a list of their rows)
+        singles = len(ctx.host_arrays["attn_single_rows"]) if portions else n
+        listed = ctx.arrays["attn_single_rows"] if portions else None
+        # queries in bfloat16 run on the tensor cores where the cached rows are whole 16-byte pieces
+        q_type = torch.bfloat16 if dt == torch.bfloat16 and self.kv_rank % 8 == 0 and self.rot_dim % 8 == 0 else torch.float32
+        q_nope = torch.empty((H, singles, self.dim), dtype=dt, device=dev)
+        q_rot = torch.empty((singles, H, self.rot_dim), dtype=q_type, device=dev)
         q_full = torch.empty((H, n, self.dim + self.rot_dim), dtype=dt, device=dev) if portions else None
         with scope("rope"):
-            K.latent_q_prep(q.data, q.splits, self.inv_freq, self.rot_dims, ctx.positions, q_nope, q_rot, H, self.dim,
-                            self.rot_dim, q_full, self.pairing)
+            if portions:
+                K.latent_q_prep(q.data, q.splits, self.inv_freq, self.rot_dims, ctx.positions, None, None, H, self.dim, self.rot_dim,
+                                q_full, self.pairing)
+            if singles:
+                K.latent_q_prep(q.data, q.splits, self.inv_freq, self.rot_dims, ctx.positions, q_nope, q_rot, H, self.dim, self.rot_dim,
+                                None, self.pairing, listed)
         rows = torch.empty((n, H * self.vdim), dtype=dt, device=dev)
         with scope("attention"):
-            singles = len(ctx.host_arrays["attn_single_rows"]) if portions else n
             if singles:
-                q_lat = grouped_linear(ctx, q_nope.view(H * n, self.dim), self.w_uk_t, offsets, torch.float32, largest_group=n)
-                out_lat = torch.empty((H, n, self.kv_rank), dtype=dt, device=dev)
-                if portions:  # only the single tokens' rows mean anything; the portions' rows are overwritten below
-                    out_lat.zero_()
-                    self._latent_space(ctx, q_lat.view(H, n, self.kv_rank), q_rot, cache, out_lat, ctx.arrays["attn_single_rows"], singles)
-                else:
-                    self._latent_space(ctx, q_lat.view(H, n, self.kv_rank), q_rot, cache, out_lat)
-                v = grouped_linear(ctx, out_lat.view(H * n, self.kv_rank), self.w_uv, offsets, dt, largest_group=n)
-                K.heads_to_rows(v.view(H, n, self.vdim), rows, None if gate is None else K.rows_view(*gate))
+                offsets = ctx.arrays[self._planner.array_name + ("_single" if portions else "")]
+                q_lat = grouped_linear(ctx, q_nope.view(H * singles, self.dim), self.w_uk_t, offsets, q_type, largest_group=singles,
+                                       uniform_rows=singles)
+                out_lat = torch.empty((H, singles, self.kv_rank), dtype=dt, device=dev)
+                self._latent_space(ctx, q_lat.view(H, singles, self.kv_rank), q_rot, cache, out_lat, listed, singles if portions else 0)
+                v = grouped_linear(ctx, out_lat.view(H * singles, self.kv_rank), self.w_uv, offsets, dt, largest_group=singles,
+                                   uniform_rows=singles)
+                K.heads_to_rows(v.view(H, singles, self.vdim), rows, None if gate is None else K.rows_view(*gate), listed)
             if portions:
                 n0 = 0
                 for r, (T, start) in enumerate(zip(ctx.host_q_lens, ctx.host_q_start)):

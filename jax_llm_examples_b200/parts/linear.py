@@ -114,12 +114,18 @@ def group_rows_hint(rows: int, groups: int, largest_group: int = 0) -> int:
 
 
 def grouped_linear(ctx: StepContext, a_sorted: torch.Tensor, w: torch.Tensor, offsets: torch.Tensor,
-                   out_dtype: torch.dtype, partials: bool = False, largest_group: int = 0, tiles=None, after_grouped: bool = False):
+                   out_dtype: torch.dtype, partials: bool = False, largest_group: int = 0, tiles=None, after_grouped: bool = False,
+                   uniform_rows: int = 0):
     """Rows [offsets[e], offsets[e+1]) of a_sorted times w[e]^T.  w: [E, N, K].  With ``partials`` the result
     is float32 :class:`Rows`; few rows (few groups in use) then get K cut across blocks to fill the GPU.
     ``after_grouped``: a_sorted was made by the call just before this one, ``grouped_swiglu_linear`` over the same
-    offsets and tiles, which ran as one streaming product (``grouped_swiglu_streams``; see ``K.gemm_stream``)."""
+    offsets and tiles, which ran as one streaming product (``grouped_swiglu_streams``; see ``K.gemm_stream``).
+    ``uniform_rows`` > 0: every group has so many rows (the streaming kernel then needs no offsets; no partials)."""
     rows, E, N = a_sorted.shape[0], w.shape[0], w.shape[1]
+    if uniform_rows and _streams(a_sorted, w, False):
+        out = torch.empty((rows, N), dtype=out_dtype, device=a_sorted.device)
+        K.gemm_stream(a_sorted, w, out, ctx.status, uniform_rows=uniform_rows)
+        return out
     if _streams(a_sorted, w, False):
         hint = _group_rows_hint(rows, E, largest_group)
         if partials:

@@ -76,7 +76,7 @@ def main(argv=None) -> int:
         recorded.append(timeline.launches())
     eng.check_status()
     rows = DeviceTimeline.summary(recorded)
-    print(f"# one decode step, {args.preset}, {model.config.num_hidden_layers} layers, batch {b}, context {args.context}: "
+    print(f"# one decode step, {args.preset}, {len(model.schedule)} layers, batch {b}, context {args.context}: "
           f"{len(rows)} launches, {sum(r['adds'] for r in rows):.1f} us (medians of {args.repeat} steps, in us)")
     print(DeviceTimeline.table(rows))
     return 0
@@ -108,7 +108,7 @@ def _prompt_steps(J, model, args, page) -> int:
         recorded.append(timeline.launches())
     eng.check_status()
     rows = DeviceTimeline.summary(recorded)
-    print(f"# one step of a {T}-token prompt, {args.preset}, {model.config.num_hidden_layers} layers: {len(rows)} stamped launches "
+    print(f"# one step of a {T}-token prompt, {args.preset}, {len(model.schedule)} layers: {len(rows)} stamped launches "
           f"(medians of {args.repeat} steps, in us)")
     print(DeviceTimeline.table(rows))
     return 0
