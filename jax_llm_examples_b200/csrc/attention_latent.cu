@@ -826,6 +826,23 @@ __global__ void heads_to_rows_kernel(const T* __restrict__ in, T* __restrict__ o
   pdl_launch_dependents_if_small();
   pdl_wait();
   const int b = blockIdx.x, n = rows ? rows[b] : b;
+  constexpr int VEC = 16 / (int)sizeof(T);
+  if (d % VEC == 0 && (((uintptr_t)in | (uintptr_t)out) & 15) == 0) {  // 16 bytes per access
+    const int per = d / VEC;
+    for (int i = threadIdx.x; i < H * per; i += blockDim.x) {
+      const int h = i / per, c = i - h * per;
+      uint4 raw = *reinterpret_cast<const uint4*>(in + ((size_t)h * N + b) * d + c * VEC);
+      if (gate.p) {
+        const float s = row_sum_splits(gate.p + (size_t)n * gate.ld + h, gate.splits, gate.split_stride);
+        const float den = 1.f + expf(-s);
+        T* e = reinterpret_cast<T*>(&raw);
+#pragma unroll
+        for (int u = 0; u < VEC; ++u) e[u] = from_f32<T>(to_f32<T>(e[u]) / den);
+      }
+      *reinterpret_cast<uint4*>(out + (size_t)n * H * d + (size_t)i * VEC) = raw;
+    }
+    return;
+  }
   for (int i = threadIdx.x; i < H * d; i += blockDim.x) {
     const int h = i / d, c = i - h * d;
     T v = in[((size_t)h * N + b) * d + c];

@@ -210,7 +210,10 @@ __device__ __forceinline__ void stream_epilogue(const StreamArgs& args, int warp
           for (int j = 0; j < 16; ++j) {
             const int m = row_lo + c0 + j;
             if (m < row_hi) {
-              if (args.act) r[j] = __float_as_uint(activate(__uint_as_float(r[j]), args.act));
+              if (args.act) {
+                const float v = __uint_as_float(r[j]);
+                r[j] = __float_as_uint(args.act == ACT_GELU && !args.out_is_f32 ? gelu_for_bf16(v) : activate(v, args.act));
+              }
               if (args.out_is_f32 || args.splits > 1)
                 ((float*)args.out)[split_off + (size_t)m * args.N + n] = __uint_as_float(r[j]);
               else

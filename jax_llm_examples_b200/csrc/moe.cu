@@ -225,6 +225,63 @@ __global__ void expert_sort_kernel(const int* __restrict__ topk_idx, int* __rest
   }
 }
 
+// The same sort for many pairs (prompt portions): every warp takes a stretch of the pairs and counts its experts 32 pairs at a
+// time (lanes with the same expert find one another by a match), a scan over the warps gives each its places, and a second
+// walk writes them: a pair is touched twice, not twice per expert.
+#define SORT_WARPS 32
+__global__ void __launch_bounds__(SORT_WARPS * 32)
+expert_sort_many_kernel(const int* __restrict__ topk_idx, int* __restrict__ offsets, int* __restrict__ sorted_pair,
+                        int* __restrict__ sorted_pos, int P, int E, int extra_rows, int tile_rows, int* __restrict__ tile_list,
+                        int* __restrict__ n_tiles, int* status, int tile_groups) {
+  JLX_TL(TL_SORT);
+  __shared__ int counts[ROUTER_MAX_E + 1];
+  extern __shared__ int held[];  // [SORT_WARPS][E]: a warp's pairs per expert, then its next place among them
+  pdl_launch_dependents();
+  pdl_wait();
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const int per = ((P + SORT_WARPS - 1) / SORT_WARPS + 31) & ~31;
+  const int lo = min(P, warp * per), hi = min(P, lo + per);
+  int* mine = held + warp * E;
+  for (int e = lane; e < E; e += 32) mine[e] = 0;
+  __syncwarp();
+  for (int base = lo; base < hi; base += 32) {
+    const int i = base + lane;
+    const int v = i < hi ? topk_idx[i] : -1;
+    const unsigned same = __match_any_sync(0xffffffffu, v);
+    if (v >= 0 && v < E && (same & ((1u << lane) - 1u)) == 0) mine[v] += __popc(same);
+    __syncwarp();
+  }
+  __syncthreads();
+  for (int e = threadIdx.x; e < E; e += blockDim.x) {  // an expert's pairs, warp by warp
+    int run = 0;
+    for (int w = 0; w < SORT_WARPS; ++w) {
+      const int c = held[w * E + e];
+      held[w * E + e] = run;
+      run += c;
+    }
+    counts[e] = run;
+  }
+  __syncthreads();
+  if (warp == 0) expert_offsets_and_tiles(counts, E, P, extra_rows, tile_rows, offsets, tile_list, n_tiles, status, true, tile_groups);
+  __syncthreads();
+  for (int base = lo; base < hi; base += 32) {
+    const int i = base + lane;
+    const int v = i < hi ? topk_idx[i] : -1;
+    const unsigned same = __match_any_sync(0xffffffffu, v);
+    const unsigned before = same & ((1u << lane) - 1u);
+    const bool ok = v >= 0 && v < E;
+    const int at = ok ? mine[v] : 0;
+    __syncwarp();
+    if (ok) {
+      const int dst = counts[v] + at + __popc(before);
+      sorted_pair[dst] = i;
+      sorted_pos[i] = dst;
+      if (before == 0) mine[v] = at + __popc(same);
+    }
+    __syncwarp();
+  }
+}
+
 // tile_list: int [(ceil((P + extra_rows) / tile_rows) + groups) * 2]; n_tiles: int [1]; both unused if tile_rows == 0.
 JLX_API int jlx_expert_sort(const int* topk_idx, int* offsets, int* sorted_pair, int* sorted_pos, int P, int E,
                             int extra_rows, int tile_rows, int* tile_list, int* n_tiles, int* status, int tile_groups,
@@ -232,6 +289,11 @@ JLX_API int jlx_expert_sort(const int* topk_idx, int* offsets, int* sorted_pair,
   JLX_REQUIRE(tile_rows == 0 || (tile_list && n_tiles), "expert_sort: tile list outputs missing");
   JLX_REQUIRE(tile_groups >= 0 && (tile_groups == 0 || extra_rows == 0), "expert_sort: tiles for the first groups only, without an appended group");
   JLX_REQUIRE(P >= 0 && E >= 1 && E <= ROUTER_MAX_E && extra_rows >= 0, "expert_sort: bad sizes P=%d E=%d", P, E);
+  if (P >= 1024) {
+    JLX_CUDA(jlx_launch_pdl(expert_sort_many_kernel, dim3(1), dim3(SORT_WARPS * 32), (size_t)SORT_WARPS * E * sizeof(int), stream, topk_idx,
+                            offsets, sorted_pair, sorted_pos, P, E, extra_rows, tile_rows, tile_list, n_tiles, status, tile_groups));
+    return 0;
+  }
   const int warps = E < 32 ? E : 32;
   const int in_smem = (size_t)P * sizeof(int) <= 40 * 1024;
   JLX_CUDA(jlx_launch_pdl(expert_sort_kernel, dim3(1), dim3(warps * 32), in_smem ? (size_t)P * sizeof(int) : 0, stream, topk_idx,

@@ -114,6 +114,140 @@ def test_softmax_of_a_portion_with_a_window(window, H_, T, q_start, k_start, L):
         _close(p[a], plain.softmax_with_sink(s[a].double().cpu() * 0.7, mask, float(sink[a])), 3e-6)
 
 
+@pytest.mark.parametrize("P, E, extra, tile_rows, tile_groups", [(1024, 16, 0, 128, 0), (4096, 256, 0, 32, 0), (5003, 7, 0, 0, 0), (2048, 3, 100, 64, 0),
+                                                                 (1500, 1, 0, 16, 0), (3000, 40, 0, 96, 33), (8192, 128, 0, 160, 0)])
+def test_sort_of_many_pairs(P, E, extra, tile_rows, tile_groups):
+    """The sort by expert of a prompt portion's pairs: offsets, stable order, places, and the products' row tiles."""
+    from jax_llm_examples_b200.kernels import api as K
+
+    torch.manual_seed(P)
+    idx = torch.randint(0, E, (P,), dtype=torch.int32)
+    idx[torch.rand(P) < 0.3] = E // 2  # one crowded expert
+    groups = E + (extra > 0)
+    i32 = lambda n: torch.full((n,), -7, dtype=torch.int32, device=DEV)  # noqa: E731
+    off, pair, pos, st = i32(E + 2), i32(P), i32(P), torch.zeros(1, dtype=torch.int32, device=DEV)
+    tiles = (i32(2 * (-(-(P + extra) // tile_rows) + groups)), i32(1)) if tile_rows else ()
+    K.expert_sort(idx.to(DEV), off, pair, pos, E, st, extra, tile_rows, *tiles, **({"tile_groups": tile_groups} if tile_groups else {}))
+    order = torch.sort(idx.long(), stable=True).indices
+    assert torch.equal(pair.cpu().long(), order) and torch.equal(pos.cpu().long()[order], torch.arange(P))
+    want = [0] + torch.cumsum(torch.bincount(idx.long(), minlength=E), 0).tolist() + ([P + extra] if extra else [])
+    assert off.cpu()[:len(want)].tolist() == want and int(st) == 0
+    if tile_rows:
+        listed = [(g, r) for g in range(tile_groups or groups) for r in range(want[g], want[g + 1], tile_rows)]
+        n = int(tiles[1])
+        assert n == len(listed) and tiles[0].cpu()[:2 * n].view(n, 2).tolist() == [list(t) for t in listed]
+
+
+@pytest.mark.parametrize("E, N, Kd, rows", [(16, 256, 128, 40), (4, 96, 64, 3), (3, 200, 72, 700)])
+def test_activation_in_the_grouped_products_epilogue(E, N, Kd, rows):
+    """gelu(a W^T) finished inside the streaming product, against float64: bfloat16 and float32 results, values far out."""
+    from jax_llm_examples_b200.kernels import api as K
+
+    torch.manual_seed(rows)
+    a, w = (torch.randn(rows, Kd, device=DEV) * 1.5).bfloat16(), (torch.randn(E, N, Kd, device=DEV) * 0.3).bfloat16()
+    cuts = sorted(random.Random(rows).choices(range(rows + 1), k=E - 1))
+    off = torch.tensor([0] + cuts + [rows], dtype=torch.int32, device=DEV)
+    st = torch.zeros(1, dtype=torch.int32, device=DEV)
+    at = off.tolist()
+    ref = torch.cat([a[at[e]:at[e + 1]].double() @ w[e].double().T for e in range(E)])
+    for act, fn in (("gelu", plain.gelu_exact), ("relu2", lambda z: torch.relu(z) ** 2), ("silu", lambda z: z * torch.sigmoid(z)), ("none", lambda z: z)):
+        for dt, tol in ((torch.float32, 4e-6), (torch.bfloat16, 4e-3)):
+            out = torch.empty(rows, N, device=DEV, dtype=dt)
+            K.gemm_stream(a, w, out, st, offsets=off, rows_hint=max(rows // E, 1), mode=K.GEMM_ACT, activation=act)
+            err = (out.double() - fn(ref)).abs() / (1.0 + fn(ref).abs())
+            assert float(err.max()) < tol, (act, dt, float(err.max()))
+    assert int(st) == 0
+
+
+@pytest.mark.parametrize("E, N, Kd, u", [(16, 512, 128, 8), (3, 40, 64, 1), (5, 128, 72, 17), (2, 256, 512, 300)])
+def test_equal_groups_need_no_offsets(E, N, Kd, u):
+    from jax_llm_examples_b200.kernels import api as K
+
+    torch.manual_seed(u)
+    a, w = torch.randn(E * u, Kd, device=DEV).bfloat16(), torch.randn(E, N, Kd, device=DEV).bfloat16()
+    out, st = torch.full((E * u, N), float("nan"), device=DEV), torch.zeros(1, dtype=torch.int32, device=DEV)
+    K.gemm_stream(a, w, out, st, uniform_rows=u)
+    _close(out.view(E, u, N), torch.einsum("eud,end->eun", a.double().view(E, u, Kd), w.double()), 2e-6)
+    assert int(st) == 0
+
+
+@pytest.mark.parametrize("N", [1, 2, 7, 8, 9, 16])
+@pytest.mark.parametrize("D, E, k, groups, keep, splits, gathered", [(64, 6, 2, 3, 2, 1, False), (2048, 16, 2, 2, 1, 4, False), (512, 40, 5, 8, 3, 2, True),
+                                                                     (4096, 256, 8, 1, 1, 1, False), (132, 5, 1, 1, 1, 3, True), (256, 64, 16, 64, 40, 1, False)])
+def test_closing_norm_router_sort_and_gather_in_one_launch(N, D, E, k, groups, keep, splits, gathered):
+    """What the one kernel of a decode step leaves is what the four kernels leave: residual rows, rounded rows, choices and
+    weights, sorted pairs, tile list, gathered rows; both corrected weight forms."""
+    from jax_llm_examples_b200.kernels import api as K
+    from jax_llm_examples_b200.parts.base import CorrectedRouter, Dispatch
+
+    assert K.close_route_supported(N, D, E, k)
+    torch.manual_seed(N * D)
+    kk = 3
+    x = torch.randn(N, D, device=DEV)
+    y = torch.randn(splits, N * kk if gathered else N, D, device=DEV)
+    extra = dict(delta_index=torch.randperm(N * kk).to(torch.int32).to(DEV), delta_k=kk, delta_weights=torch.rand(N, kk, device=DEV)) if gathered else {}
+    gamma, w, corr = torch.randn(D, device=DEV), torch.randn(E, D, device=DEV) * D ** -0.5, torch.randn(E, device=DEV) - 0.5
+    i32 = lambda *s: torch.full(s, -7, dtype=torch.int32, device=DEV)  # noqa: E731
+    st, tile = torch.zeros(1, dtype=torch.int32, device=DEV), 16
+    for form, norm in (("sigmoid_corrected", False), ("softmax_normalized", True)):
+        r = CorrectedRouter(w, None, corr, form, groups, keep, 2, norm, 1.5, k, None)
+        d = Dispatch(None, i32(E + 1), i32(N * k), i32(N * k), (i32(2 * (-(-N * k // tile) + E)), i32(1)),
+                     torch.zeros(N * k, D, device=DEV, dtype=torch.bfloat16), 0, tile, st)
+        x1, h1, idx1, w1 = x.clone(), torch.empty(N, D, device=DEV, dtype=torch.bfloat16), i32(N, k), torch.empty(N, k, device=DEV)
+        K.close_route(x1, y, splits, gamma, 0.7, 1e-5, h1, r, idx1, w1, d, **extra)
+        x2, h2, idx2, w2 = x.clone(), torch.empty_like(h1), i32(N, k), torch.empty(N, k, device=DEV)
+        K.group_norm(x2, y, splits, None, gamma, 1, 0.7, pre_norm=False, eps=1e-5, out=h2, **extra)
+        K.router(x1, w, idx2, w2, weight_form=form, correction=corr, groups=groups, keep=keep, scale=1.5, group_top=2, normalize=norm)
+        off, pair, pos, tl, nt = i32(E + 1), i32(N * k), i32(N * k), i32(2 * (-(-N * k // tile) + E)), i32(1)
+        K.expert_sort(idx1, off, pair, pos, E, st, 0, tile, tl, nt)
+        _close(x1, x2, 2e-6, "residual")
+        assert torch.equal(h1, x1.bfloat16())
+        assert torch.equal(idx1, idx2)
+        _close(w1, w2, 2e-6, "weights")
+        assert torch.equal(d.offsets, off) and torch.equal(d.sorted_pair, pair) and torch.equal(d.sorted_pos, pos)
+        assert torch.equal(d.tiles[1], nt) and torch.equal(d.tiles[0][:2 * int(nt)], tl[:2 * int(nt)])
+        assert torch.equal(d.a_sorted, h1[(pair.long() // k)])
+        assert int(st) == 0
+
+
+@pytest.mark.parametrize("rank, dr, heads, window", [(64, 16, 4, 0), (512, 64, 16, 100), (200, 24, 18, 33), (528, 8, 3, 0), (1024, 64, 2, 7), (16, 8, 1, 1)])
+def test_latent_attention_on_the_tensor_cores_equals_the_32_bit_kernel(rank, dr, heads, window):
+    """The same bfloat16 queries and cache through both kernels: contexts of one token to hundreds, whole and cut into
+    ranges, all rows and listed ones (which come in the list's order)."""
+    from jax_llm_examples_b200.kernels import api as K
+
+    torch.manual_seed(rank)
+    page, lens = 16, [1, 17, 32, 33, 100, 299, 300, 64]
+    R = len(lens)
+    width = 300 // page + 1
+    pages = torch.randn(R * width, 1, 1, page, rank + dr, device=DEV).bfloat16()
+    table = torch.randperm(R * width).to(torch.int32).view(R, width).to(DEV)
+    if window:
+        for r, n in enumerate(lens):
+            table[r, :max(0, n - window) // page] = -1
+    pos, req = torch.tensor([n - 1 for n in lens], dtype=torch.int32, device=DEV), torch.arange(R, dtype=torch.int32, device=DEV)
+    q, qr, sink = torch.randn(heads, R, rank, device=DEV).bfloat16(), torch.randn(R, heads, dr, device=DEV).bfloat16(), torch.randn(heads, device=DEV)
+    st, scale = torch.zeros(1, dtype=torch.int32, device=DEV), 2.0 * (rank + dr) ** -0.5
+    want = torch.empty(heads, R, rank, device=DEV)
+    K.attention_latent(q.float(), qr.float(), pages, table, req, pos, sink, want, scale, st, window=window)
+    for splits, keys in ((1, 0), (5, 64), (10, 32)):
+        n = R * heads * splits
+        pa, pm = torch.empty(n * rank, device=DEV), torch.empty(n * 2, device=DEV)
+        for single in (False, True):
+            got = torch.full_like(want, float("nan"))
+            K.attention_latent(q, qr, pages, table, req, pos, sink, got, scale, st, splits=splits, split_keys=keys, part_acc=pa, part_ml=pm,
+                               window=window, single_tokens=single)
+            _close(got, want, 6e-3, f"{splits} ranges")
+        rows = torch.tensor([5, 0, 3], dtype=torch.int32, device=DEV)
+        at = rows.long()
+        for cast in (torch.bfloat16, torch.float32):
+            got = torch.full((heads, 3, rank), float("nan"), device=DEV)
+            K.attention_latent(q[:, at].to(cast).contiguous(), qr[at].to(cast).contiguous(), pages, table, req, pos, sink, got, scale, st, rows, 3,
+                               splits, keys, pa, pm, window, single_tokens=True)
+            _close(got, want[:, at], 6e-3, f"listed rows, {splits} ranges")
+    assert int(st) == 0
+
+
 # --------------------------------------------------------------------------------------------- parts alone
 def _attention_part(wd, m, eps, dtype):
     from jax_llm_examples_b200.parts import GatedPagedAttention, rotary_frequencies
