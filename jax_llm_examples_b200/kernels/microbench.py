@@ -5,6 +5,8 @@
     python -m jax_llm_examples_b200.kernels.microbench gemm --rows 8 --n 16384 --k 5120 [--experts 16] [--swiglu]
     python -m jax_llm_examples_b200.kernels.microbench decay_scan --tokens 2048 --requests 1 --heads 16 [--read-before]
     python -m jax_llm_examples_b200.kernels.microbench delta_scan --tokens 2048 --requests 1 --heads 16 [--key-heads 8]
+    python -m jax_llm_examples_b200.kernels.microbench latent_decode --batch 8 --context 4096 --heads 16 [--window 1024] [--float32-queries]
+    python -m jax_llm_examples_b200.kernels.microbench close_route --rows 8 --width 2048 --experts 16 [--unfused]
 
 The reference benchmarks its kernels the same way, from ``__main__`` blocks in the kernel files
 (llama4/llama4_jax/ragged_attention.py:299-418, llama4/llama4_jax/decode_ragged_dot.py:239-291).
@@ -63,7 +65,7 @@ def attention_decode(a) -> dict:
 
     def run():
         K.attention_decode(q, pages, table, req, pos, out, a.head_dim ** -0.5, a.chunk, 0, 0.0, 1.0, part_o, part_ml, splits,
-                           keys, status)
+                           keys, status, softcap=a.softcap)
 
     t = _time(run, a.reps, _flush(a))
     nbytes = a.batch * a.context * 2 * a.kv_heads * a.head_dim * 2
@@ -86,7 +88,7 @@ def attention_prefill(a) -> dict:
     fn = K.attention_prefill_tc if a.tc else K.attention_prefill
 
     def run():
-        fn(q, pages, table, req, pos, out, tiles, tiles.shape[0], a.head_dim ** -0.5, a.chunk, 0, 0.0, 1.0, status)
+        fn(q, pages, table, req, pos, out, tiles, tiles.shape[0], a.head_dim ** -0.5, a.chunk, 0, 0.0, 1.0, status, softcap=a.softcap)
 
     t = _time(run, a.reps, _flush(a))
     flops = 4 * a.heads * a.head_dim * T * (T + 1) / 2
@@ -222,6 +224,63 @@ def stream_mix_norm(a) -> dict:
             "GB/s": round(moved / t / 1e9, 1)}
 
 
+def latent_decode(a) -> dict:
+    """Latent attention of one token per request over a bfloat16 cache, the key ranges as ``LatentAttention`` cuts them."""
+    dev = "cuda"
+    page, row = 64, a.rank + a.rot
+    per = -(-a.context // page)
+    pages = (torch.randn(a.batch * per, 1, 1, page, row, device=dev) * 0.5).bfloat16()
+    table = torch.arange(a.batch * per, device=dev, dtype=torch.int32).view(a.batch, per).contiguous()
+    dt = torch.float32 if a.float32_queries else torch.bfloat16
+    q, qr = torch.randn(a.heads, a.batch, a.rank, device=dev).to(dt), torch.randn(a.batch, a.heads, a.rot, device=dev).to(dt)
+    out = torch.empty(a.heads, a.batch, a.rank, device=dev, dtype=torch.bfloat16)
+    pos = torch.full((a.batch,), a.context - 1, device=dev, dtype=torch.int32)
+    req, status = torch.arange(a.batch, device=dev, dtype=torch.int32), torch.zeros(1, device=dev, dtype=torch.int32)
+    seen = min(a.context, a.window) if a.window else a.context
+    want = max(1, 2 * K.sm_count() // (a.batch * -(-a.heads // (32 if a.float32_queries else 16))))
+    keys = max(64, -(-(-(-seen // want)) // 32) * 32)
+    splits = min(-(-a.context // keys), (seen - 1) // keys + 2)
+    pa, pm = torch.empty(a.batch * a.heads * splits * a.rank, device=dev), torch.empty(a.batch * a.heads * splits * 2, device=dev)
+
+    def run():
+        K.attention_latent(q, qr, pages, table, req, pos, None, out, row ** -0.5, status, splits=splits, split_keys=keys, part_acc=pa,
+                           part_ml=pm, window=a.window, single_tokens=True)
+
+    t = _time(run, a.reps, _flush(a))
+    assert int(status) == 0
+    nbytes = a.batch * seen * row * 2
+    return {"kernel": "attention_latent" + (" (32-bit)" if a.float32_queries else " (tensor cores)") + " + combine", "batch": a.batch,
+            "context": a.context, "window": a.window, "heads": a.heads, "splits": splits, "us": round(t * 1e6, 1), "GB": round(nbytes / 1e9, 4),
+            "GB/s": round(nbytes / t / 1e9, 1)}
+
+
+def close_route(a) -> dict:
+    """The closing norm, corrected router, sort and gather of a decode step in one launch, or (``--unfused``) in four."""
+    from ..parts.base import CorrectedRouter, Dispatch
+
+    dev, N, D, E, k, tile = "cuda", a.rows, a.width, a.experts, a.top, 16
+    x, y = torch.randn(N, D, device=dev), torch.randn(a.splits, N, D, device=dev)
+    gamma, w, corr = torch.ones(D, device=dev), torch.randn(E, D, device=dev) * D ** -0.5, torch.zeros(E, device=dev)
+    i32 = lambda *s: torch.zeros(s, dtype=torch.int32, device=dev)  # noqa: E731
+    r = CorrectedRouter(w, None, corr, "sigmoid_corrected", 2, 1, 2, False, 1.0, k, None)
+    d = Dispatch(None, i32(E + 1), i32(N * k), i32(N * k), (i32(2 * (-(-N * k // tile) + E)), i32(1)),
+                 torch.zeros(N * k, D, device=dev, dtype=torch.bfloat16), 0, tile, i32(1))
+    h, idx, wt = torch.empty(N, D, device=dev, dtype=torch.bfloat16), i32(N, k), torch.empty(N, k, device=dev)
+
+    def fused():
+        K.close_route(x, y, a.splits, gamma, 1.0, 1e-6, h, r, idx, wt, d)
+
+    def unfused():
+        K.group_norm(x, y, a.splits, None, gamma, 1, 1.0, pre_norm=False, out=h)
+        K.router(x, w, idx, wt, weight_form="sigmoid_corrected", correction=corr, groups=2, keep=1, group_top=2)
+        K.expert_sort(idx, d.offsets, d.sorted_pair, d.sorted_pos, E, d.status, 0, tile, *d.tiles)
+        K.permute_scale(x, d.sorted_pair, None, d.a_sorted, k)
+
+    t = _time(unfused if a.unfused else fused, a.reps, _flush(a))
+    return {"kernel": "group_norm + router + expert_sort + permute_scale" if a.unfused else "close_route", "rows": N, "width": D, "experts": E,
+            "top": k, "us": round(t * 1e6, 1)}
+
+
 def _flush(a):
     return None if a.no_flush else torch.empty(256 * 1024 * 1024 // 4, device="cuda")
 
@@ -229,7 +288,8 @@ def _flush(a):
 def main(argv=None) -> int:
     ap = argparse.ArgumentParser(description=__doc__.split("\n\n")[0])
     sub = ap.add_subparsers(dest="what", required=True)
-    for name in ("attention_decode", "attention_prefill", "gemm", "decay_scan", "delta_scan", "conv_unit_prep", "stream_mix_norm"):
+    for name in ("attention_decode", "attention_prefill", "gemm", "decay_scan", "delta_scan", "conv_unit_prep", "stream_mix_norm",
+                 "latent_decode", "close_route"):
         p = sub.add_parser(name)
         p.add_argument("--reps", type=int, default=10)
         p.add_argument("--no-flush", action="store_true", help="do not flush L2 between launches")
@@ -252,7 +312,16 @@ def main(argv=None) -> int:
             p.add_argument("--vdim", type=int, default=128)
         if name == "decay_scan":
             p.add_argument("--read-before", action="store_true", help="o from the state before the update, with a bonus (time mixing)")
+        if name == "latent_decode":
+            for flag, value in (("batch", 8), ("context", 4096), ("heads", 16), ("rank", 512), ("rot", 64), ("window", 0)):
+                p.add_argument(f"--{flag}", type=int, default=value)
+            p.add_argument("--float32-queries", action="store_true", help="the 32-bit kernel instead of the tensor-core one")
+        if name == "close_route":
+            for flag, value in (("rows", 8), ("width", 2048), ("experts", 16), ("top", 2), ("splits", 4)):
+                p.add_argument(f"--{flag}", type=int, default=value)
+            p.add_argument("--unfused", action="store_true")
         if name.startswith("attention"):
+            p.add_argument("--softcap", type=float, default=0.0, help="cap * tanh(score / cap)")
             p.add_argument("--heads", type=int, default=40)
             p.add_argument("--kv-heads", type=int, default=8)
             p.add_argument("--head-dim", type=int, default=128)
@@ -275,7 +344,8 @@ def main(argv=None) -> int:
             p.add_argument("--swiglu", action="store_true", help="fused SiLU(gate) * up epilogue")
     a = ap.parse_args(argv)
     print(json.dumps({"attention_decode": attention_decode, "attention_prefill": attention_prefill, "gemm": gemm, "decay_scan": decay_scan,
-                      "delta_scan": delta_scan, "conv_unit_prep": conv_unit_prep, "stream_mix_norm": stream_mix_norm}[a.what](a)))
+                      "delta_scan": delta_scan, "conv_unit_prep": conv_unit_prep, "stream_mix_norm": stream_mix_norm,
+                      "latent_decode": latent_decode, "close_route": close_route}[a.what](a)))
     return 0
 
 
