@@ -57,7 +57,7 @@ CONFIGS = {
     "wide": {
         "architecture": "Marinex", "vocab": 96, "width": 128, "norm": {"eps": 1e-6},
         "layers": [attention(4, 1, 64, 64, 0.3, 6.0, (10000.0, 64)),
-                   latent(4, 32, 16, 24, 48, 64, 40, 0.15, 10000.0, moe(8, 2, 64, (4, 2))),
+                   latent(4, 40, 16, 24, 48, 64, 36, 0.15, 10000.0, moe(8, 2, 64, (4, 2))),
                    attention(2, 2, 128, 128, 0.2, 12.0, (500000.0, 32), moe(6, 4, 32, (2, 2))),
                    latent(6, 16, 32, 40, 40, 96, 24, 0.2, 300.0, moe(8, 3, 48, (2, 1)))],
     },
