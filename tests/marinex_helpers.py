@@ -182,7 +182,7 @@ TOL = {"float32": 3e-5, "bfloat16": 1.2e-1}
 TOL_MEAN = {"float32": 1e-5, "bfloat16": 3e-2}
 # The share of choices that may differ from the plain router's: two scores that tie within the precision go either way; a
 # fault in the routing (a group, a correction, a tie rule) changes tens of percent.
-OTHER_CHOICES = {"float32": 0.004, "bfloat16": 0.06}
+OTHER_CHOICES = {"float32": 0.004, "bfloat16": 0.04}
 
 
 def row_err(got: np.ndarray, ref: np.ndarray) -> float:
@@ -209,23 +209,42 @@ def compare(folder, requests: dict, got: dict, routing: dict | None, dtype: str,
                 err = row_err(got[(rid, pos)], ref[pos])
                 assert err < TOL[dtype] * (2 if stray else 1), f"{dtype}: request {rid} position {pos}: relative error {err:.3e}"
                 errs.append(err)
-    other = sum(s * n for s, n in shares) / max(sum(n for _, n in shares), 1)
-    assert other <= OTHER_CHOICES[dtype], f"{dtype}: {other:.2%} of the expert choices differ from the plain router's"
+    total = max(sum(n for _, n in shares), 1)
+    other = sum(s * n for s, n in shares) / total
+    few = 3 / (total * max(len(routed), 1)) if dtype == "bfloat16" else 0.0  # a handful of tokens: three near-ties are no share
+    assert other <= max(OTHER_CHOICES[dtype], few), f"{dtype}: {other:.2%} of the expert choices differ from the plain router's"
     assert sum(e >= TOL[dtype] for e in errs) <= stray, f"{dtype}: more than {stray} rows beyond {TOL[dtype]}"
     mean = float(np.mean(errs))
     assert mean < TOL_MEAN[dtype], f"{dtype}: mean relative error {mean:.3e} over {len(errs)} rows"
     return max(errs)
 
 
-def greedy_checked(folder, prompt, got, dtype: str) -> None:
-    """``got`` must be the plain implementation's greedy continuation, except where its two best logits are closer
-    than the precision tells apart; after such a step the comparison follows the engine's choice."""
-    toks = list(prompt)
+def engine_choices(model, tokens, tail: int) -> dict | None:
+    """The experts the engine takes for every token of a sequence whose last ``tail`` tokens it decodes one by one, in the form
+    that ``plain_logits`` takes as ``forced``."""
+    import jax_llm_examples_b200 as J
+    from tests import helpers as H
+
+    routed = [i for i, L in enumerate(model.config.layers) if L.mlp is not None]
+    if not routed:
+        return None
+    engine = J.Engine(model, max_tokens=-(-len(tokens) // 64) * 64, page_size=64, max_slots=1)
+    _, routing = H.run_trace(engine, H.trace_tail_decode({"a": list(tokens)}, tail), record_routing=True)
+    return {layer: torch.as_tensor(np.stack([routing[("a", p)][j] for p in range(len(tokens))])) for j, layer in enumerate(routed)}
+
+
+def greedy_checked(folder, model, prompt, got, dtype: str) -> None:
+    """``got`` must be the plain implementation's greedy continuation, except where its two best logits are closer than the
+    precision tells apart (the plain implementation follows the engine's tokens).  In bfloat16 it also takes the engine's
+    experts: where two choice scores tie, one token through another expert is another logit, not a rounding."""
+    toks = list(prompt) + list(got)
     tol = 1e-4 if dtype == "float32" else 8e-2
+    forced = engine_choices(model, toks, len(got)) if dtype == "bfloat16" else None
+    logits, other = plain_logits(folder, toks, forced)
+    assert other <= 0.1, f"{dtype}: {other:.1%} of the expert choices differ from the plain router's"
     for step, g in enumerate(got):
-        logits = plain_logits(folder, toks)[0][-1]
-        best = int(np.argmax(logits))
+        row = logits[len(prompt) - 1 + step]
+        best = int(np.argmax(row))
         if g != best:
-            gap = float(logits[best] - logits[g]) / float(np.abs(logits - logits.mean()).max())
+            gap = float(row[best] - row[g]) / float(np.abs(row - row.mean()).max())
             assert gap < tol, f"{dtype}: step {step}: engine chose {g}, plain {best}, relative logit gap {gap:.2e}"
-        toks.append(g)

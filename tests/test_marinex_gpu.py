@@ -727,7 +727,7 @@ def test_greedy_generation_through_the_scheduler(folders, name, dtype):
     got = J.generate(model, prompts, J.SamplingParams(max_new_tokens=10), page_size=16, max_tokens_per_step=16)
     for p, g in zip(prompts, got):
         assert len(g) == 10
-        MX.greedy_checked(folders[name], p, g, dtype)
+        MX.greedy_checked(folders[name], model, p, g, dtype)
 
 
 def test_command_line_generates_from_a_preset_and_from_a_folder(folders, capsys):
@@ -738,7 +738,7 @@ def test_command_line_generates_from_a_preset_and_from_a_folder(folders, capsys)
     assert main(["--model", str(folders["padded"]), "--dtype", "float32", "--prompt-ids", "1,2,3,4,5", "--max-new-tokens", "5",
                  "--page-size", "16"]) == 0
     ids = [int(t) for t in capsys.readouterr().out.splitlines()[1].split()]
-    MX.greedy_checked(folders["padded"], [1, 2, 3, 4, 5], ids, "float32")
+    MX.greedy_checked(folders["padded"], None, [1, 2, 3, 4, 5], ids, "float32")
 
 
 def test_trace_replay_program_on_a_marinex_folder(folders, tmp_path):
