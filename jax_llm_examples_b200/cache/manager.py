@@ -31,10 +31,12 @@ class OutOfSlots(CacheError):
 
 @dataclasses.dataclass(frozen=True)
 class Retention:
-    """Which keys a group's layers can still read: all, those of the query's chunk, or a window."""
+    """Which keys a group's layers can still read: all, those of the query's chunk, or a window, with a window also the
+    sequence's first ``keep`` keys."""
 
     kind: int = KEEP_ALL
     size: int = 0
+    keep: int = 0
 
     @staticmethod
     def all() -> "Retention":
@@ -45,8 +47,8 @@ class Retention:
         return Retention(KEEP_CHUNK, int(size))
 
     @staticmethod
-    def window(size: int) -> "Retention":
-        return Retention(KEEP_WINDOW, int(size))
+    def window(size: int, keep: int = 0) -> "Retention":
+        return Retention(KEEP_WINDOW, int(size), int(keep))
 
 
 _lib = None
@@ -59,7 +61,7 @@ def _host() -> ctypes.CDLL:
         lib.cm_create.restype = c_void_p
         lib.cm_create.argtypes = [c_int, c_int, c_int]
         lib.cm_destroy.argtypes = [c_void_p]
-        lib.cm_add_group.argtypes = [c_void_p, c_int, c_int, c_int]
+        lib.cm_add_group.argtypes = [c_void_p, c_int, c_int, c_int, c_int]
         for f in ("cm_num_groups", "cm_free_slot_count", "cm_alloc_slot", "cm_check"):
             getattr(lib, f).argtypes = [c_void_p]
         for f in ("cm_free_pages", "cm_num_pages"):
@@ -101,7 +103,7 @@ class CacheManager:
 
     # ------------------------------------------------------------------ set-up
     def add_group(self, retention: Retention, num_pages: int) -> int:
-        g = self._lib.cm_add_group(self._h, retention.kind, retention.size, num_pages)
+        g = self._lib.cm_add_group(self._h, retention.kind, retention.size, retention.keep, num_pages)
         if g < 0:
             raise CacheError(f"bad group: {retention} with {num_pages} pages")
         self.groups.append(retention)

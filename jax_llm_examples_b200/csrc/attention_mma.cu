@@ -19,9 +19,12 @@
 //
 // A query at position p reads keys [start(p), p], start(p) = max(chunk ? p - p % chunk : 0,
 // window ? p - window + 1 : 0).  Temperature: scores of a layer with attn_scale != 0 are multiplied by
-// 1 + attn_scale * ln(1 + floor((p + 1) / floor_scale)).
+// 1 + attn_scale * ln(1 + floor((p + 1) / floor_scale)).  With `keep` > 0 the sequence's first `keep` keys are visible
+// besides the window's, and two maps per head may be taken off one another at the end (attention_maps.cuh).
+// A group of more query heads than a block takes is served by several blocks.
 #include <cuda.h>
 
+#include "attention_maps.cuh"
 #include "common.cuh"
 #include "mbarrier.cuh"
 #include "mma_sync.cuh"
@@ -32,6 +35,8 @@
 #define SPLIT_MIN 512    // ... and at least this long: shorter blocks spend their time on set-up
 #define DEC_MAX_BOXES 1024  // block-table entries of a decode split kept in shared memory
 #define DEC_STAGES 3     // key/value tiles in flight per decode block (96 KB at head size 128: two blocks per SM)
+#define DEC_MAX_G 16     // query heads of a KV head per decode block (the M of an mma)
+#define PRE_MAX_G 8      // ... and per prefill block (a warp each); even: two maps of a head stay together
 #define NEG_BIG (-1.0e30f)
 
 // ---- TMA and mbarrier (decode kernel: whole [rows, 64-element] boxes of a page per instruction)
@@ -66,7 +71,20 @@ struct AttnParams {
   int split_keys;       // keys per decode split (a multiple of SPLIT_UNIT)
   const float* sink;    // optional, [Hq]: one more term exp(sink[h]) in the softmax's denominator, without a value
   const float* slopes;  // optional, [Hq]: slopes[h] * (query position - key position) is taken off the scaled score
+  int keep;             // the sequence's first so many keys are visible besides the window's
+  int maps;             // 2: the heads are pairs of maps, `out` gets their differences; 1: plain heads
+  MapDifference diff;
 };
+
+// The query heads that a block serves: KV head hk's heads [h0, h0 + G), at most `most` of its whole group.
+struct BlockHeads {
+  int hk, h0, G;
+};
+__device__ __forceinline__ BlockHeads block_heads(const AttnParams& P, int b, int most) {
+  const int group = P.Hq / P.Hkv, chunks = (group + most - 1) / most;
+  const int hk = b / chunks, off = (b - hk * chunks) * most;
+  return {hk, hk * group + off, min(most, group - off)};
+}
 
 // The slope of query head h in base-2 score units (0 without slopes).
 __device__ __forceinline__ float slope_log2(const AttnParams& P, int h, bool valid) {
@@ -100,7 +118,7 @@ __device__ __forceinline__ float inverse_sum_with_sink(float m, float l, const f
 }
 
 // Loads keys [key0, key0 + KT) of request r, KV head hk, into ks / vs (each [KT][DH], swizzled).
-// Keys outside [lo, hi] or without a page become zeros.  Consecutive threads take consecutive 16-byte
+// Keys outside [lo, hi] (and not among the kept first ones) or without a page become zeros.  Consecutive threads take consecutive 16-byte
 // chunks of a row, so a warp's copy covers whole rows: full 128-byte lines from L2.
 template <int DH>
 __device__ __forceinline__ void load_kv_tile(const AttnParams& P, int r, int hk, int key0, int lo, int hi, bf16* ks, bf16* vs,
@@ -111,7 +129,7 @@ __device__ __forceinline__ void load_kv_tile(const AttnParams& P, int r, int hk,
   const int* table = P.block_table + (size_t)r * P.bt_stride;
   for (int j = threadIdx.x / CH; j < KT; j += NT / CH) {
     const int pos = key0 + j;
-    bool valid = pos >= lo && pos <= hi;
+    bool valid = (pos >= lo || pos < P.keep) && pos <= hi;
     const bf16* src = P.pages;
     if (valid) {
       const int pi = pos / P.page_size;
@@ -142,19 +160,28 @@ __global__ void __launch_bounds__(128) attention_decode_kernel(const AttnParams 
   constexpr int CH = DH / 8;
   bf16* ks = reinterpret_cast<bf16*>(smem);                  // [DEC_STAGES][KT][DH]
   bf16* vs = ks + DEC_STAGES * KT * DH;                      // [DEC_STAGES][KT][DH]
-  const int slot = blockIdx.z, n = P.rows ? P.rows[slot] : slot, hk = blockIdx.y, split = blockIdx.x;
-  const int G = P.Hq / P.Hkv;
+  const int slot = blockIdx.z, n = P.rows ? P.rows[slot] : slot, split = blockIdx.x;
+  const BlockHeads heads = block_heads(P, blockIdx.y, DEC_MAX_G);
+  const int hk = heads.hk, h0 = heads.h0, G = heads.G;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int p = P.positions[n], r = P.req_of_token[n];
   const int lo = first_key(p, P.chunk, P.window);
-  const int key_begin = (lo / P.split_keys + split) * P.split_keys;
+  const int first_split = lo / P.split_keys, key_begin = (first_split + split) * P.split_keys;
   if (key_begin > p) return;
   const int key_end = min(p + 1, key_begin + P.split_keys);
-  const int n_tiles = (key_end - key_begin + KT - 1) / KT;
+  // the splits share the tiles of the kept first keys between them, each walks its own before its stretch of the window
+  int kept_lo = 0, n_kept = 0;
+  if (P.keep > 0) {
+    const int kept = kept_tiles(P.keep, first_split * P.split_keys, KT), n_splits = p / P.split_keys - first_split + 1;
+    kept_lo = split * kept / n_splits;
+    n_kept = (split + 1) * kept / n_splits - kept_lo;
+  }
+  const int n_tiles = n_kept + (key_end - key_begin + KT - 1) / KT;
+  auto tile_first_key = [&](int t) { return t < n_kept ? (kept_lo + t) * KT : key_begin + (t - n_kept) * KT; };
 
 #pragma unroll
   for (int t = 0; t < DEC_STAGES - 1; ++t) {
-    if (t < n_tiles) load_kv_tile<DH>(P, r, hk, key_begin + t * KT, lo, p, ks + t * KT * DH, vs + t * KT * DH, 128);
+    if (t < n_tiles) load_kv_tile<DH>(P, r, hk, tile_first_key(t), lo, p, ks + t * KT * DH, vs + t * KT * DH, 128);
     cp_async_commit();
   }
 
@@ -162,8 +189,8 @@ __global__ void __launch_bounds__(128) attention_decode_kernel(const AttnParams 
   uint32_t qf[DH / 16][4];
   {
     const int g0 = lane >> 2, g1 = g0 + 8, kk = (lane & 3) * 2;
-    const bf16* q0 = P.q + ((size_t)n * P.Hq + hk * G + g0) * DH;
-    const bf16* q1 = P.q + ((size_t)n * P.Hq + hk * G + g1) * DH;
+    const bf16* q0 = P.q + ((size_t)n * P.Hq + h0 + g0) * DH;
+    const bf16* q1 = P.q + ((size_t)n * P.Hq + h0 + g1) * DH;
 #pragma unroll
     for (int s = 0; s < DH / 16; ++s) {
       qf[s][0] = g0 < G ? *reinterpret_cast<const uint32_t*>(q0 + s * 16 + kk) : 0u;
@@ -173,7 +200,7 @@ __global__ void __launch_bounds__(128) attention_decode_kernel(const AttnParams 
     }
   }
   const float sc = P.scale_log2 * temperature(p, P.attn_scale, P.floor_scale);
-  const float sl[2] = {slope_log2(P, hk * G + (lane >> 2), (lane >> 2) < G), slope_log2(P, hk * G + (lane >> 2) + 8, (lane >> 2) + 8 < G)};
+  const float sl[2] = {slope_log2(P, h0 + (lane >> 2), (lane >> 2) < G), slope_log2(P, h0 + (lane >> 2) + 8, (lane >> 2) + 8 < G)};
   float m[2] = {NEG_BIG, NEG_BIG}, l[2] = {0.f, 0.f};
   float o[DH / 8][4];
 #pragma unroll
@@ -184,10 +211,10 @@ __global__ void __launch_bounds__(128) attention_decode_kernel(const AttnParams 
     __syncthreads();                  // ... for every thread, and the stage of tile t - 1 is free
     {
       const int nt = t + DEC_STAGES - 1, st = nt % DEC_STAGES;
-      if (nt < n_tiles) load_kv_tile<DH>(P, r, hk, key_begin + nt * KT, lo, p, ks + st * KT * DH, vs + st * KT * DH, 128);
+      if (nt < n_tiles) load_kv_tile<DH>(P, r, hk, tile_first_key(nt), lo, p, ks + st * KT * DH, vs + st * KT * DH, 128);
       cp_async_commit();
     }
-    const int tile_key = key_begin + t * KT;
+    const int tile_key = tile_first_key(t);
     const bf16* kt = ks + (t % DEC_STAGES) * KT * DH;
     const bf16* vt = vs + (t % DEC_STAGES) * KT * DH;
     // S = Q K^T for this warp's 16 keys: two n-tiles of 8 keys
@@ -208,7 +235,7 @@ __global__ void __launch_bounds__(128) attention_decode_kernel(const AttnParams 
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         const int key = tile_key + warp * 16 + nt * 8 + (lane & 3) * 2 + (e & 1);
-        const bool ok = key >= lo && key <= p;
+        const bool ok = (key >= lo || key < P.keep) && key <= p;
         s[nt][e] = ok ? fmaf(-sl[e >> 1], (float)(p - key), scaled_score(P, s[nt][e], sc)) : NEG_BIG;
         mx[e >> 1] = fmaxf(mx[e >> 1], s[nt][e]);
       }
@@ -283,7 +310,7 @@ __global__ void __launch_bounds__(128) attention_decode_kernel(const AttnParams 
       acc += red[(w * 16 + g) * LD + d] * f;
       ll += red[(w * 16 + g) * LD + DH + 1] * f;
     }
-    const size_t row = ((size_t)slot * P.Hq + hk * G + g) * P.max_splits + split;
+    const size_t row = ((size_t)slot * P.Hq + h0 + g) * P.max_splits + split;
     P.part_o[row * DH + d] = acc;
     if (d == 0) {
       P.part_ml[row * 2] = mm;
@@ -312,15 +339,24 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map, const AttnP
   pdl_launch_dependents();
   // Until pdl_wait() below, only what no kernel of this step writes is read: the step's description (rows,
   // positions, requests, block table: on the device before the step began) and keys and values of earlier steps.
-  const int slot = blockIdx.z, n = P.rows ? P.rows[slot] : slot, hk = blockIdx.y, split = blockIdx.x;
-  const int G = P.Hq / P.Hkv;
+  const int slot = blockIdx.z, n = P.rows ? P.rows[slot] : slot, split = blockIdx.x;
+  const BlockHeads heads = block_heads(P, blockIdx.y, DEC_MAX_G);
+  const int hk = heads.hk, h0 = heads.h0, G = heads.G;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int p = P.positions[n], r = P.req_of_token[n];
   const int lo = first_key(p, P.chunk, P.window);
-  const int key_begin = (lo / P.split_keys + split) * P.split_keys;
+  const int first_split = lo / P.split_keys, key_begin = (first_split + split) * P.split_keys;
   if (key_begin > p) return;
   const int key_end = min(p + 1, key_begin + P.split_keys);
-  const int n_tiles = (key_end - key_begin + KT - 1) / KT;
+  // the splits share the tiles of the kept first keys between them, each walks its own before its stretch of the window
+  int kept_lo = 0, n_kept = 0;
+  if (P.keep > 0) {
+    const int kept = kept_tiles(P.keep, first_split * P.split_keys, KT), n_splits = p / P.split_keys - first_split + 1;
+    kept_lo = split * kept / n_splits;
+    n_kept = (split + 1) * kept / n_splits - kept_lo;
+  }
+  const int n_tiles = n_kept + (key_end - key_begin + KT - 1) / KT;
+  auto tile_first_key = [&](int t) { return t < n_kept ? (kept_lo + t) * KT : key_begin + (t - n_kept) * KT; };
   const int* table = P.block_table + (size_t)r * P.bt_stride;
 
   if (threadIdx.x == 0) {
@@ -337,7 +373,7 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map, const AttnP
   const bool cached = n_boxes <= DEC_MAX_BOXES;
   if (cached) {
     for (int b = threadIdx.x; b < n_boxes; b += blockDim.x) {
-      const int pi = (key_begin + b * box_rows) / P.page_size;
+      const int pi = (tile_first_key(b / boxes_per_tile) + (b % boxes_per_tile) * box_rows) / P.page_size;
       page_of_box[b] = pi < P.bt_stride ? table[pi] : -1;
     }
     __syncthreads();
@@ -348,7 +384,7 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map, const AttnP
     const uint32_t bar = smem_u32(&full_bar[st]);
     const uint32_t dst = base + st * STAGE_BYTES;
     mbar_expect_tx(bar, STAGE_BYTES);
-    const int key0 = key_begin + t * KT;
+    const int key0 = tile_first_key(t);
     for (int b = 0; b < boxes_per_tile; ++b) {
       const int pos = key0 + b * box_rows;
       const int pi = pos / P.page_size;
@@ -369,7 +405,7 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map, const AttnP
   // the tile that holds p, wait for it.
   int issued = 0;
   if (threadIdx.x == 0)
-    for (; issued < DEC_STAGES && issued < n_tiles && key_begin + (issued + 1) * KT <= p; ++issued) issue(issued);
+    for (; issued < DEC_STAGES && issued < n_tiles && tile_first_key(issued) + KT <= p; ++issued) issue(issued);
   pdl_wait();
   if (threadIdx.x == 0)
     for (; issued < DEC_STAGES && issued < n_tiles; ++issued) issue(issued);
@@ -377,8 +413,8 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map, const AttnP
   uint32_t qf[DH / 16][4];
   {
     const int g0 = lane >> 2, g1 = g0 + 8, kk = (lane & 3) * 2;
-    const bf16* q0 = P.q + ((size_t)n * P.Hq + hk * G + g0) * DH;
-    const bf16* q1 = P.q + ((size_t)n * P.Hq + hk * G + g1) * DH;
+    const bf16* q0 = P.q + ((size_t)n * P.Hq + h0 + g0) * DH;
+    const bf16* q1 = P.q + ((size_t)n * P.Hq + h0 + g1) * DH;
 #pragma unroll
     for (int s = 0; s < DH / 16; ++s) {
       qf[s][0] = g0 < G ? *reinterpret_cast<const uint32_t*>(q0 + s * 16 + kk) : 0u;
@@ -389,7 +425,7 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map, const AttnP
   }
   JLX_TL_MARK(0);
   const float sc = P.scale_log2 * temperature(p, P.attn_scale, P.floor_scale);
-  const float sl[2] = {slope_log2(P, hk * G + (lane >> 2), (lane >> 2) < G), slope_log2(P, hk * G + (lane >> 2) + 8, (lane >> 2) + 8 < G)};
+  const float sl[2] = {slope_log2(P, h0 + (lane >> 2), (lane >> 2) < G), slope_log2(P, h0 + (lane >> 2) + 8, (lane >> 2) + 8 < G)};
   float m[2] = {NEG_BIG, NEG_BIG}, l[2] = {0.f, 0.f};
   float o[DH / 8][4];
 #pragma unroll
@@ -407,7 +443,7 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map, const AttnP
       }
       break;
     }
-    const int tile_key = key_begin + t * KT;
+    const int tile_key = tile_first_key(t);
     const uint32_t kt = base + st * STAGE_BYTES, vt = kt + HALVES * HALF_BYTES;
     float s[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
 #pragma unroll
@@ -425,7 +461,7 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map, const AttnP
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         const int key = tile_key + warp * 16 + nt * 8 + (lane & 3) * 2 + (e & 1);
-        const bool in = key >= lo && key <= p;
+        const bool in = (key >= lo || key < P.keep) && key <= p;
         s[nt][e] = in ? fmaf(-sl[e >> 1], (float)(p - key), scaled_score(P, s[nt][e], sc)) : NEG_BIG;
         mx[e >> 1] = fmaxf(mx[e >> 1], s[nt][e]);
       }
@@ -503,7 +539,7 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map, const AttnP
       acc += red[(w * 16 + g) * LD + d] * f;
       ll += red[(w * 16 + g) * LD + DH + 1] * f;
     }
-    const size_t row = ((size_t)slot * P.Hq + hk * G + g) * P.max_splits + split;
+    const size_t row = ((size_t)slot * P.Hq + h0 + g) * P.max_splits + split;
     P.part_o[row * DH + d] = acc;
     if (d == 0) {
       P.part_ml[row * 2] = mm;
@@ -566,6 +602,124 @@ __global__ void attention_combine_kernel(const AttnParams P) {
   }
 }
 
+// The same for heads of two maps: one block combines both maps' splits, takes the second off the first and norms the
+// head's output (attention_maps.cuh) from the unrounded sums.
+template <int DH>
+__global__ void attention_combine_maps_kernel(const AttnParams P) {
+  JLX_TL(TL_ATTN_COMBINE);
+  __shared__ float ms[2][COMBINE_CACHE], wgt[2][COMBINE_CACHE];
+  __shared__ float parts[DH / 32];
+  pdl_launch_dependents();
+  const int slot = blockIdx.x, n = P.rows ? P.rows[slot] : slot, h = blockIdx.y;  // the head: maps 2h and 2h + 1
+  const int p = P.positions[n];
+  const int lo = first_key(p, P.chunk, P.window);
+  const int splits = p / P.split_keys - lo / P.split_keys + 1;
+  const size_t row = ((size_t)slot * P.Hq + 2 * h) * P.max_splits;
+  const float2* ml = reinterpret_cast<const float2*>(P.part_ml) + row;
+  const bool cached = splits <= COMBINE_CACHE;
+  const int d = threadIdx.x;
+  float mm[2] = {NEG_BIG, NEG_BIG}, ll[2] = {0.f, 0.f}, acc[2] = {0.f, 0.f};
+  pdl_wait();
+  if (cached) {
+    for (int i = d; i < 2 * splits; i += DH) {
+      const int m = i >= splits, s = i - m * splits;
+      const float2 v = ml[(size_t)m * P.max_splits + s];
+      ms[m][s] = v.x;
+      wgt[m][s] = v.y;
+    }
+    __syncthreads();
+#pragma unroll
+    for (int m = 0; m < 2; ++m) {
+      for (int s = 0; s < splits; ++s) mm[m] = fmaxf(mm[m], ms[m][s]);
+      for (int s = 0; s < splits; ++s) ll[m] += wgt[m][s] * exp2f(ms[m][s] - mm[m]);
+    }
+    __syncthreads();
+    for (int i = d; i < 2 * splits; i += DH) {
+      const int m = i >= splits, s = i - m * splits;
+      wgt[m][s] = exp2f(ms[m][s] - (m ? mm[1] : mm[0])) / (m ? ll[1] : ll[0]);
+    }
+    __syncthreads();
+  } else {
+#pragma unroll
+    for (int m = 0; m < 2; ++m) {
+      const float2* mlm = ml + (size_t)m * P.max_splits;
+      for (int s = 0; s < splits; ++s) mm[m] = fmaxf(mm[m], mlm[s].x);
+      for (int s = 0; s < splits; ++s) ll[m] += mlm[s].y * exp2f(mlm[s].x - mm[m]);
+    }
+  }
+#pragma unroll
+  for (int m = 0; m < 2; ++m) {
+    const float* po = P.part_o + (row + (size_t)m * P.max_splits) * DH + d;
+    if (cached) {
+#pragma unroll 8
+      for (int s = 0; s < splits; ++s) acc[m] += po[(size_t)s * DH] * wgt[m][s];
+    } else {
+      const float2* mlm = ml + (size_t)m * P.max_splits;
+      for (int s = 0; s < splits; ++s) acc[m] += po[(size_t)s * DH] * (exp2f(mlm[s].x - mm[m]) / ll[m]);
+    }
+  }
+  const bool mine = d < P.diff.out_dim;
+  const float o = mine ? acc[0] - P.diff.weight * acc[1] : 0.f;
+  const float w = warp_sum(o * o);
+  if ((d & 31) == 0) parts[d >> 5] = w;
+  __syncthreads();
+  float ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < DH / 32; ++i) ss += parts[i];
+  const float rms = sqrtf(ss / (float)P.diff.out_dim + P.diff.eps);
+  if (mine) P.out[(size_t)n * P.diff.ld_out + (size_t)h * P.diff.out_dim + d] = __float2bfloat16_rn(o / rms * P.diff.mult);
+}
+
+// The end of a prefill block whose warps hold the finished, unnormalised rows of two maps each: warp w is head h0 + w.
+// Second maps leave their rows in shared memory (float [pairs][16][DH + 4], 16-byte aligned), first maps take them off
+// theirs, norm the difference and store it.  Every thread of the block calls it, after a barrier behind its last read of `smem`.
+template <int DH>
+__device__ __forceinline__ void store_map_difference(const AttnParams& P, float* smem, const float (&o)[DH / 8][4], float i0, float i1, int warp,
+                                                     int lane, bool active, int h0, size_t n0, int t0, int t1, bool row0, bool row1) {
+  constexpr int LD = DH + 4;
+  const int col = (lane & 3) * 2;
+  float* a0 = smem + ((size_t)(warp >> 1) * 16 + t0) * LD + col;
+  float* a1 = smem + ((size_t)(warp >> 1) * 16 + t1) * LD + col;
+  if (active && (warp & 1)) {
+#pragma unroll
+    for (int i = 0; i < DH / 8; ++i) {
+      *reinterpret_cast<float2*>(a0 + i * 8) = make_float2(o[i][0] * i0, o[i][1] * i0);
+      *reinterpret_cast<float2*>(a1 + i * 8) = make_float2(o[i][2] * i1, o[i][3] * i1);
+    }
+  }
+  __syncthreads();
+  if (!active || (warp & 1)) return;
+  float ss0 = 0.f, ss1 = 0.f;  // (entries beyond out_dim are zero: so are the padded values')
+  auto diff0 = [&](int i, int e) { return o[i][e] * i0 - P.diff.weight * a0[i * 8 + e]; };
+  auto diff1 = [&](int i, int e) { return o[i][2 + e] * i1 - P.diff.weight * a1[i * 8 + e]; };
+#pragma unroll
+  for (int i = 0; i < DH / 8; ++i)
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+      ss0 += diff0(i, e) * diff0(i, e);
+      ss1 += diff1(i, e) * diff1(i, e);
+    }
+#pragma unroll
+  for (int x = 1; x <= 2; x <<= 1) {
+    ss0 += __shfl_xor_sync(0xffffffffu, ss0, x);
+    ss1 += __shfl_xor_sync(0xffffffffu, ss1, x);
+  }
+  const float r0 = P.diff.mult / sqrtf(ss0 / (float)P.diff.out_dim + P.diff.eps), r1 = P.diff.mult / sqrtf(ss1 / (float)P.diff.out_dim + P.diff.eps);
+  const size_t head = (size_t)((h0 + warp) >> 1) * P.diff.out_dim;
+  bf16* d0 = P.out + (n0 + t0) * P.diff.ld_out + head;
+  bf16* d1 = P.out + (n0 + t1) * P.diff.ld_out + head;
+#pragma unroll
+  for (int i = 0; i < DH / 8; ++i)
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+      const int c = i * 8 + col + e;
+      if (c < P.diff.out_dim) {
+        if (row0) d0[c] = __float2bfloat16_rn(diff0(i, e) * r0);
+        if (row1) d1[c] = __float2bfloat16_rn(diff1(i, e) * r1);
+      }
+    }
+}
+
 // ----------------------------------------------------------------------------------- prefill
 // grid (Hkv, n_tiles); G warps.  A tile is up to 16 consecutive tokens of one request; warp g owns the
 // 16 x DH rows of query head g.  Key tiles of 64 are double-buffered.
@@ -577,15 +731,19 @@ __global__ void __launch_bounds__(256) attention_prefill_kernel(const AttnParams
   constexpr int STAGES = 2;
   bf16* ks = reinterpret_cast<bf16*>(smem);          // [STAGES][KT][DH]
   bf16* vs = ks + STAGES * KT * DH;
-  const int hk = blockIdx.x, tile = blockIdx.y;
-  const int G = P.Hq / P.Hkv;
+  const int tile = blockIdx.y;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const BlockHeads heads = block_heads(P, blockIdx.x, PRE_MAX_G);
+  const int hk = heads.hk;
+  const bool active = warp < heads.G;  // (a group's last block may have warps to spare; they go along with its last head)
+  const int head = heads.h0 + min(warp, heads.G - 1);
   const int n0 = P.tiles[2 * tile], cnt = P.tiles[2 * tile + 1];
   const int r = P.req_of_token[n0];
   const int p_first = P.positions[n0], p_last = p_first + cnt - 1;
   const int lo_tile = first_key(p_first, P.chunk, P.window);  // start(p) grows with p: the tile's lowest
   const int key_begin = lo_tile / KT * KT;
-  const int n_tiles = (p_last - key_begin) / KT + 1;
+  const int n_kept = P.keep > 0 ? kept_tiles(P.keep, key_begin, KT) : 0;
+  const int n_tiles = n_kept + (p_last - key_begin) / KT + 1;
   const int NT = blockDim.x;
 
   // this thread's two rows: tokens lane/4 and lane/4 + 8 of head `warp`
@@ -596,8 +754,8 @@ __global__ void __launch_bounds__(256) attention_prefill_kernel(const AttnParams
   uint32_t qf[DH / 16][4];
   {
     const int kk = (lane & 3) * 2;
-    const bf16* q0 = P.q + ((size_t)(n0 + min(t0, cnt - 1)) * P.Hq + hk * G + warp) * DH;
-    const bf16* q1 = P.q + ((size_t)(n0 + min(t1, cnt - 1)) * P.Hq + hk * G + warp) * DH;
+    const bf16* q0 = P.q + ((size_t)(n0 + min(t0, cnt - 1)) * P.Hq + head) * DH;
+    const bf16* q1 = P.q + ((size_t)(n0 + min(t1, cnt - 1)) * P.Hq + head) * DH;
 #pragma unroll
     for (int s = 0; s < DH / 16; ++s) {
       qf[s][0] = row0 ? *reinterpret_cast<const uint32_t*>(q0 + s * 16 + kk) : 0u;
@@ -608,28 +766,28 @@ __global__ void __launch_bounds__(256) attention_prefill_kernel(const AttnParams
   }
   const float sc0 = P.scale_log2 * temperature(p0, P.attn_scale, P.floor_scale);
   const float sc1 = P.scale_log2 * temperature(p1, P.attn_scale, P.floor_scale);
-  const float slope = slope_log2(P, hk * G + warp, true);
+  const float slope = slope_log2(P, head, true);
   float m[2] = {NEG_BIG, NEG_BIG}, l[2] = {0.f, 0.f};
   float o[DH / 8][4];
 #pragma unroll
   for (int i = 0; i < DH / 8; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
 
   // prologue: first tile
-  load_kv_tile<DH>(P, r, hk, key_begin, lo_tile, p_last, ks, vs, NT);
+  load_kv_tile<DH>(P, r, hk, walk_key(0, n_kept, key_begin, KT), lo_tile, p_last, ks, vs, NT);
   cp_async_commit();
 
   for (int t = 0; t < n_tiles; ++t) {
     const int buf = t & 1;
     // request the next tile into the other buffer (free since the barrier at the end of the last round)
     if (t + 1 < n_tiles)
-      load_kv_tile<DH>(P, r, hk, key_begin + (t + 1) * KT, lo_tile, p_last, ks + (buf ^ 1) * KT * DH, vs + (buf ^ 1) * KT * DH, NT);
+      load_kv_tile<DH>(P, r, hk, walk_key(t + 1, n_kept, key_begin, KT), lo_tile, p_last, ks + (buf ^ 1) * KT * DH, vs + (buf ^ 1) * KT * DH, NT);
     cp_async_commit();
     cp_async_wait<1>();
     __syncthreads();
-    const int tile_key = key_begin + t * KT;
+    const int tile_key = walk_key(t, n_kept, key_begin, KT);
     const bf16* kt = ks + buf * KT * DH;
     const bf16* vt = vs + buf * KT * DH;
-    if (warp < G) {
+    if (active) {
       float s[KT / 8][4];
 #pragma unroll
       for (int i = 0; i < KT / 8; ++i) s[i][0] = s[i][1] = s[i][2] = s[i][3] = 0.f;
@@ -651,7 +809,8 @@ __global__ void __launch_bounds__(256) attention_prefill_kernel(const AttnParams
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
           const int key = tile_key + nt * 8 + (lane & 3) * 2 + (e & 1);
-          const bool ok = (e < 2) ? (row0 && key >= lo0 && key <= p0) : (row1 && key >= lo1 && key <= p1);
+          const bool kept = key < P.keep;
+          const bool ok = (e < 2) ? (row0 && (kept || key >= lo0) && key <= p0) : (row1 && (kept || key >= lo1) && key <= p1);
           s[nt][e] = ok ? fmaf(-slope, (float)(((e < 2) ? p0 : p1) - key), scaled_score(P, s[nt][e], (e < 2) ? sc0 : sc1)) : NEG_BIG;
           mx[e >> 1] = fmaxf(mx[e >> 1], s[nt][e]);
         }
@@ -700,11 +859,15 @@ __global__ void __launch_bounds__(256) attention_prefill_kernel(const AttnParams
     __syncthreads();  // everyone is done with this buffer before the next round overwrites it
   }
   cp_async_wait<0>();
-  if (warp < G) {
+  const float i0 = inverse_sum_with_sink(m[0], l[0], P.sink, head), i1 = inverse_sum_with_sink(m[1], l[1], P.sink, head);
+  if (P.maps == 2) {
+    store_map_difference<DH>(P, reinterpret_cast<float*>(smem), o, i0, i1, warp, lane, active, heads.h0, (size_t)n0, t0, t1, row0, row1);
+    return;
+  }
+  if (active) {
     const int col = (lane & 3) * 2;
-    const float i0 = inverse_sum_with_sink(m[0], l[0], P.sink, hk * G + warp), i1 = inverse_sum_with_sink(m[1], l[1], P.sink, hk * G + warp);
-    bf16* o0 = P.out + ((size_t)(n0 + t0) * P.Hq + hk * G + warp) * DH;
-    bf16* o1 = P.out + ((size_t)(n0 + t1) * P.Hq + hk * G + warp) * DH;
+    bf16* o0 = P.out + ((size_t)(n0 + t0) * P.Hq + head) * DH;
+    bf16* o1 = P.out + ((size_t)(n0 + t1) * P.Hq + head) * DH;
 #pragma unroll
     for (int i = 0; i < DH / 8; ++i) {
       if (row0) *reinterpret_cast<__nv_bfloat162*>(o0 + i * 8 + col) = __floats2bfloat162_rn(o[i][0] * i0, o[i][1] * i0);
@@ -751,15 +914,19 @@ attention_prefill_tma_kernel(const __grid_constant__ CUtensorMap map, const Attn
   constexpr uint32_t STAGE_BYTES = 2 * HALVES * HALF_BYTES;
   __shared__ __align__(8) uint64_t full_bar[PRE_STAGES];
   const uint32_t base = (smem_u32(smem_raw) + 1023u) & ~1023u;
-  const int hk = blockIdx.x, tile = blockIdx.y;
-  const int G = P.Hq / P.Hkv;
+  const int tile = blockIdx.y;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const BlockHeads heads = block_heads(P, blockIdx.x, PRE_MAX_G);
+  const int hk = heads.hk;
+  const bool active = warp < heads.G;  // (a group's last block may have warps to spare; they go along with its last head)
+  const int head = heads.h0 + min(warp, heads.G - 1);
   const int n0 = P.tiles[2 * tile], cnt = P.tiles[2 * tile + 1];
   const int r = P.req_of_token[n0];
   const int p_first = P.positions[n0], p_last = p_first + cnt - 1;
   const int lo_tile = first_key(p_first, P.chunk, P.window);
   const int key_begin = lo_tile / KT * KT;
-  const int n_tiles = (p_last - key_begin) / KT + 1;
+  const int n_kept = P.keep > 0 ? kept_tiles(P.keep, key_begin, KT) : 0;
+  const int n_tiles = n_kept + (p_last - key_begin) / KT + 1;
   const int* table = P.block_table + (size_t)r * P.bt_stride;
 
   if (threadIdx.x == 0) {
@@ -769,7 +936,7 @@ attention_prefill_tma_kernel(const __grid_constant__ CUtensorMap map, const Attn
   __syncthreads();
   if (threadIdx.x == 0)
     for (int t = 0; t < PRE_STAGES && t < n_tiles; ++t)
-      tma_issue_tile<DH>(&map, P, table, hk, key_begin + t * KT, base + t * STAGE_BYTES, smem_u32(&full_bar[t]), box_rows);
+      tma_issue_tile<DH>(&map, P, table, hk, walk_key(t, n_kept, key_begin, KT), base + t * STAGE_BYTES, smem_u32(&full_bar[t]), box_rows);
 
   const int t0 = lane >> 2, t1 = t0 + 8;
   const int p0 = p_first + min(t0, cnt - 1), p1 = p_first + min(t1, cnt - 1);
@@ -778,8 +945,8 @@ attention_prefill_tma_kernel(const __grid_constant__ CUtensorMap map, const Attn
   uint32_t qf[DH / 16][4];
   {
     const int kk = (lane & 3) * 2;
-    const bf16* q0 = P.q + ((size_t)(n0 + min(t0, cnt - 1)) * P.Hq + hk * G + warp) * DH;
-    const bf16* q1 = P.q + ((size_t)(n0 + min(t1, cnt - 1)) * P.Hq + hk * G + warp) * DH;
+    const bf16* q0 = P.q + ((size_t)(n0 + min(t0, cnt - 1)) * P.Hq + head) * DH;
+    const bf16* q1 = P.q + ((size_t)(n0 + min(t1, cnt - 1)) * P.Hq + head) * DH;
 #pragma unroll
     for (int s = 0; s < DH / 16; ++s) {
       qf[s][0] = row0 ? *reinterpret_cast<const uint32_t*>(q0 + s * 16 + kk) : 0u;
@@ -790,7 +957,7 @@ attention_prefill_tma_kernel(const __grid_constant__ CUtensorMap map, const Attn
   }
   const float sc0 = P.scale_log2 * temperature(p0, P.attn_scale, P.floor_scale);
   const float sc1 = P.scale_log2 * temperature(p1, P.attn_scale, P.floor_scale);
-  const float slope = slope_log2(P, hk * G + warp, true);
+  const float slope = slope_log2(P, head, true);
   float m[2] = {NEG_BIG, NEG_BIG}, l[2] = {0.f, 0.f};
   float o[DH / 8][4];
 #pragma unroll
@@ -807,7 +974,7 @@ attention_prefill_tma_kernel(const __grid_constant__ CUtensorMap map, const Attn
       }
       break;
     }
-    const int tile_key = key_begin + t * KT;
+    const int tile_key = walk_key(t, n_kept, key_begin, KT);
     const uint32_t kt = base + st * STAGE_BYTES, vt = kt + HALVES * HALF_BYTES;
     // rows of this thread that see no key of the tile at all skip nothing: the masks below handle it
     const bool need_mask = tile_key + KT - 1 > p_first || tile_key < first_key(p_last, P.chunk, P.window) || cnt < 16;
@@ -835,7 +1002,8 @@ attention_prefill_tma_kernel(const __grid_constant__ CUtensorMap map, const Attn
         for (int e = 0; e < 4; ++e) {
           bool in = true;
           const int key = tile_key + half * 32 + nt * 8 + (lane & 3) * 2 + (e & 1);
-          if (need_mask) in = (e < 2) ? (row0 && key >= lo0 && key <= p0) : (row1 && key >= lo1 && key <= p1);
+          const bool kept = key < P.keep;
+          if (need_mask) in = (e < 2) ? (row0 && (kept || key >= lo0) && key <= p0) : (row1 && (kept || key >= lo1) && key <= p1);
           s[nt][e] = in ? fmaf(-slope, (float)(((e < 2) ? p0 : p1) - key), scaled_score(P, s[nt][e], (e < 2) ? sc0 : sc1)) : NEG_BIG;
           mx[e >> 1] = fmaxf(mx[e >> 1], s[nt][e]);
         }
@@ -884,16 +1052,21 @@ attention_prefill_tma_kernel(const __grid_constant__ CUtensorMap map, const Attn
     __syncthreads();  // every warp is done reading this stage
     if (threadIdx.x == 0 && t + PRE_STAGES < n_tiles) {
       asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
-      tma_issue_tile<DH>(&map, P, table, hk, key_begin + (t + PRE_STAGES) * KT, base + st * STAGE_BYTES,
+      tma_issue_tile<DH>(&map, P, table, hk, walk_key(t + PRE_STAGES, n_kept, key_begin, KT), base + st * STAGE_BYTES,
                          smem_u32(&full_bar[st]), box_rows);
     }
   }
   if (!ok) return;
-  {
+  const float i0 = inverse_sum_with_sink(m[0], l[0], P.sink, head), i1 = inverse_sum_with_sink(m[1], l[1], P.sink, head);
+  if (P.maps == 2) {
+    store_map_difference<DH>(P, reinterpret_cast<float*>(smem_raw + (base - smem_u32(smem_raw))), o, i0, i1, warp, lane, active, heads.h0,
+                             (size_t)n0, t0, t1, row0, row1);
+    return;
+  }
+  if (active) {
     const int col = (lane & 3) * 2;
-    const float i0 = inverse_sum_with_sink(m[0], l[0], P.sink, hk * G + warp), i1 = inverse_sum_with_sink(m[1], l[1], P.sink, hk * G + warp);
-    bf16* o0 = P.out + ((size_t)(n0 + t0) * P.Hq + hk * G + warp) * DH;
-    bf16* o1 = P.out + ((size_t)(n0 + t1) * P.Hq + hk * G + warp) * DH;
+    bf16* o0 = P.out + ((size_t)(n0 + t0) * P.Hq + head) * DH;
+    bf16* o1 = P.out + ((size_t)(n0 + t1) * P.Hq + head) * DH;
 #pragma unroll
     for (int i = 0; i < DH / 8; ++i) {
       if (row0) *reinterpret_cast<__nv_bfloat162*>(o0 + i * 8 + col) = __floats2bfloat162_rn(o[i][0] * i0, o[i][1] * i0);
@@ -906,7 +1079,7 @@ attention_prefill_tma_kernel(const __grid_constant__ CUtensorMap map, const Attn
 static int fill_params(AttnParams& P, const void* q, const void* pages, const int* block_table, int bt_stride,
                        const int* req_of_token, const int* positions, void* out, int Hq, int Hkv, int dh, int page_size,
                        int num_pages, float scale, int chunk, int window, float attn_scale, float floor_scale, const float* sink, const float* slopes,
-                       float softcap, int* status) {
+                       float softcap, int keep, const MapDifference* diff, int* status) {
   JLX_REQUIRE(Hq > 0 && Hkv > 0 && Hq % Hkv == 0, "attention: %d query heads are no multiple of %d KV heads", Hq, Hkv);
   JLX_REQUIRE(dh == 64 || dh == 128, "attention_mma: head size %d is not built (64 and 128 are); use the generic kernel", dh);
   JLX_REQUIRE(page_size > 0 && num_pages > 0 && bt_stride > 0, "attention: bad cache sizes");
@@ -922,6 +1095,17 @@ static int fill_params(AttnParams& P, const void* q, const void* pages, const in
   P.tiles = nullptr; P.part_o = nullptr; P.part_ml = nullptr; P.max_splits = 0; P.split_keys = SPLIT_UNIT; P.rows = nullptr;
   P.sink = sink;
   P.slopes = slopes;
+  JLX_REQUIRE(keep >= 0, "attention: the count of kept first keys is negative");
+  P.keep = keep;
+  P.maps = diff ? 2 : 1;
+  P.diff = MapDifference{};
+  if (diff) {
+    JLX_REQUIRE((Hq / Hkv) % 2 == 0, "attention: heads of two maps need an even number of query rows per KV head (got %d)", Hq / Hkv);
+    JLX_REQUIRE(diff->map_dim > 0 && 2 * diff->map_dim <= dh && diff->out_dim > 0 && diff->out_dim <= dh && diff->ld_out >= (long long)Hq / 2 * diff->out_dim,
+                "attention: two maps of %d entries and values of %d do not fit a head size of %d", diff->map_dim, diff->out_dim, dh);
+    JLX_REQUIRE(!sink, "attention: the difference of two maps takes no sink");
+    P.diff = *diff;
+  }
   return 0;
 }
 
@@ -957,9 +1141,8 @@ static int make_cache_map(CUtensorMap* map, const void* pages, long long rows, i
 }
 
 JLX_API int jlx_attention_mma_supported(int Hq, int Hkv, int dh, int decode) {
-  if (Hkv <= 0 || Hq % Hkv) return 0;
-  const int G = Hq / Hkv;
-  return (dh == 64 || dh == 128) && G <= (decode ? 16 : 8);
+  (void)decode;
+  return Hkv > 0 && Hq % Hkv == 0 && (dh == 64 || dh == 128);
 }
 
 // Multiprocessors of the current device (asked once per device).
@@ -1003,18 +1186,19 @@ JLX_API int jlx_attention_decode(const void* q, const void* pages, const int* bl
                                  const int* req_of_token, const int* positions, void* out, int N, int Hq, int Hkv, int dh,
                                  int page_size, int num_pages, float scale, int chunk, int window, float attn_scale,
                                  float floor_scale, float* part_o, float* part_ml, int max_splits, int split_keys,
-                                 const int* rows, const float* sink, const float* slopes, float softcap, int* status, cudaStream_t stream) {
+                                 const int* rows, const float* sink, const float* slopes, float softcap, int keep, const MapDifference* diff,
+                                 int* status, cudaStream_t stream) {
   AttnParams P;
   if (fill_params(P, q, pages, block_table, bt_stride, req_of_token, positions, out, Hq, Hkv, dh, page_size, num_pages,
-                  scale, chunk, window, attn_scale, floor_scale, sink, slopes, softcap, status)) return 1;
-  JLX_REQUIRE(Hq / Hkv <= 16, "attention_decode: %d query heads per KV head; up to 16 are supported", Hq / Hkv);
+                  scale, chunk, window, attn_scale, floor_scale, sink, slopes, softcap, keep, diff, status)) return 1;
   JLX_REQUIRE(part_o && part_ml && max_splits > 0, "attention_decode: scratch for the partial results is missing");
   JLX_REQUIRE(split_keys > 0 && split_keys % SPLIT_UNIT == 0, "attention_decode: split size %d is no multiple of %d", split_keys, SPLIT_UNIT);
-  JLX_REQUIRE(N <= 65535 && Hkv <= 65535, "attention_decode: too many rows");
+  const int head_blocks = Hkv * ((Hq / Hkv + DEC_MAX_G - 1) / DEC_MAX_G);
+  JLX_REQUIRE(N <= 65535 && head_blocks <= 65535, "attention_decode: too many rows");
   if (N == 0) return 0;
   P.part_o = part_o; P.part_ml = part_ml; P.max_splits = max_splits; P.split_keys = split_keys; P.rows = rows;
   const size_t smem = (size_t)2 * DEC_STAGES * KT * dh * 2;
-  dim3 grid(max_splits, Hkv, N);
+  dim3 grid(max_splits, head_blocks, N);
   // pages that hold whole 64-key tiles, or divide them, go through TMA; other page sizes through cp.async
   const bool tma = (page_size % KT == 0 || KT % page_size == 0) && page_size >= 8 &&
                    (long long)num_pages * 2 * Hkv * page_size < (1ll << 31);
@@ -1043,7 +1227,10 @@ JLX_API int jlx_attention_decode(const void* q, const void* pages, const int* bl
     attention_decode_kernel<64><<<grid, 128, smem, stream>>>(P);
     JLX_LAUNCH_CHECK("attention_decode");
   }
-  if (dh == 128) JLX_CUDA(jlx_launch_pdl(attention_combine_kernel<128>, dim3(N, Hq), dim3(128), 0, stream, P));
+  if (diff) {
+    if (dh == 128) JLX_CUDA(jlx_launch_pdl(attention_combine_maps_kernel<128>, dim3(N, Hq / 2), dim3(128), 0, stream, P));
+    else JLX_CUDA(jlx_launch_pdl(attention_combine_maps_kernel<64>, dim3(N, Hq / 2), dim3(64), 0, stream, P));
+  } else if (dh == 128) JLX_CUDA(jlx_launch_pdl(attention_combine_kernel<128>, dim3(N, Hq), dim3(128), 0, stream, P));
   else JLX_CUDA(jlx_launch_pdl(attention_combine_kernel<64>, dim3(N, Hq), dim3(64), 0, stream, P));
   JLX_LAUNCH_CHECK("attention_combine");
   return 0;
@@ -1053,19 +1240,17 @@ JLX_API int jlx_attention_decode(const void* q, const void* pages, const int* bl
 JLX_API int jlx_attention_prefill(const void* q, const void* pages, const int* block_table, int bt_stride,
                                   const int* req_of_token, const int* positions, void* out, const int* tiles, int n_tiles,
                                   int Hq, int Hkv, int dh, int page_size, int num_pages, float scale, int chunk, int window,
-                                  float attn_scale, float floor_scale, const float* sink, const float* slopes, float softcap, int* status,
-                                  cudaStream_t stream) {
+                                  float attn_scale, float floor_scale, const float* sink, const float* slopes, float softcap, int keep,
+                                  const MapDifference* diff, int* status, cudaStream_t stream) {
   AttnParams P;
   if (fill_params(P, q, pages, block_table, bt_stride, req_of_token, positions, out, Hq, Hkv, dh, page_size, num_pages,
-                  scale, chunk, window, attn_scale, floor_scale, sink, slopes, softcap, status)) return 1;
-  const int G = Hq / Hkv;
-  JLX_REQUIRE(G <= 8, "attention_prefill: %d query heads per KV head; up to 8 are supported", G);
-  JLX_REQUIRE(Hkv <= 65535, "attention_prefill: too many KV heads");
+                  scale, chunk, window, attn_scale, floor_scale, sink, slopes, softcap, keep, diff, status)) return 1;
+  const int G = Hq / Hkv < PRE_MAX_G ? Hq / Hkv : PRE_MAX_G;
   if (n_tiles == 0) return 0;
   P.tiles = tiles;
   // blocks are handed out by blockIdx.x first: every head of the list's first (heaviest) tile before lighter tiles
   JLX_REQUIRE(n_tiles <= 65535, "attention_prefill: %d tiles; up to 65535 are supported", n_tiles);
-  dim3 grid(Hkv, n_tiles);
+  dim3 grid(Hkv * ((Hq / Hkv + PRE_MAX_G - 1) / PRE_MAX_G), n_tiles);
   const bool tma = (page_size % KT == 0 || KT % page_size == 0) && page_size >= 8 &&
                    (long long)num_pages * 2 * Hkv * page_size < (1ll << 31);
   if (tma) {

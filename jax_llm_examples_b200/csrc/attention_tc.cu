@@ -22,10 +22,16 @@
 // window; scale dh^-0.5; 32-bit softmax), with the attention temperature on layers that have it.  The
 // reference sends prefill attention to a TPU library (model.py:842-864).
 //
+// Kept first keys and heads of two maps (attention_maps.cuh): an item's key tiles are then those of the kept keys and those
+// of the window; a head's two maps are two items in a row of one block, whose outputs lie in two accumulators, and the
+// second one's end takes the difference, norms it and stores the head (a map's score product runs over its own part of
+// the rows only).
+//
 // Every wait on a barrier is bounded; after a timeout the block raises JLX_STATUS_WAIT_TIMEOUT, waits
 // (bounded) for its own copies, frees its tensor memory and returns.
 #include <cuda.h>
 
+#include "attention_maps.cuh"
 #include "common.cuh"
 #include "mbarrier.cuh"
 #include "softcap.cuh"
@@ -180,6 +186,10 @@ struct TcParams {
   int* status;
   const float* sink;    // optional, [Hq]: one more term exp(sink[h]) in the softmax's denominator, without a value
   const float* slopes;  // optional, [Hq]: slopes[h] * (query position - key position) is taken off the scaled score
+  int keep;             // the sequence's first so many keys are visible besides the window's
+  int maps;             // 2: the heads are pairs of maps, `out` gets their differences; 1: plain heads
+  int vec_out;          // rows of `out` may be stored 16 bytes at a time
+  MapDifference diff;
 };
 
 __device__ __forceinline__ int first_key(int p, int chunk, int window) {
@@ -196,7 +206,7 @@ __device__ __forceinline__ int first_key(int p, int chunk, int window) {
 
 // A work item: one tile of up to 128 query tokens of one request, and one query head.
 struct Item {
-  int head, hk, n0, cnt, p_first, p_last, key_begin, n_kv;
+  int head, hk, n0, cnt, p_first, p_last, key_begin, n_kept, n_kv;
   const int* table;
 };
 
@@ -209,7 +219,7 @@ struct Item {
 // once per item; only the wait for the last product and the store of the output remain between two items.
 __global__ void __launch_bounds__(NTHREADS, 1)
 attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_kv, const TcParams P,
-                            int n_items) {
+                            int n_units) {
   JLX_TL(TL_ATTN_PREFILL);
   extern __shared__ __align__(1024) uint8_t smem_raw[];
   const uint32_t base = (smem_u32(smem_raw) + 1023u) & ~1023u;
@@ -240,18 +250,22 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
   auto item = [&](int i) {
     Item it;
     it.n_kv = 0;
-    const int rank = (i & 1) ? (int)gridDim.x - 1 - (int)blockIdx.x : (int)blockIdx.x;
-    const long long w = (long long)i * gridDim.x + rank;
-    if (w >= n_items) return it;
-    const int tile = (int)(w / P.Hq);
-    it.head = (int)(w % P.Hq);
+    // what is dealt out is a head: one item, or the two items of its maps, which a block runs one after the other
+    const int u = P.maps == 2 ? i >> 1 : i, heads = P.maps == 2 ? P.Hq >> 1 : P.Hq;
+    const int rank = (u & 1) ? (int)gridDim.x - 1 - (int)blockIdx.x : (int)blockIdx.x;
+    const long long w = (long long)u * gridDim.x + rank;
+    if (w >= n_units) return it;
+    const int tile = (int)(w / heads);
+    it.head = (int)(w % heads);
+    if (P.maps == 2) it.head = 2 * it.head + (i & 1);
     it.hk = it.head / G;
     it.n0 = P.tiles[2 * tile];
     it.cnt = P.tiles[2 * tile + 1];
     it.p_first = P.positions[it.n0];
     it.p_last = it.p_first + it.cnt - 1;
     it.key_begin = first_key(it.p_first, P.chunk, P.window) / BKV * BKV;
-    it.n_kv = (it.p_last - it.key_begin) / BKV + 1;
+    it.n_kept = P.keep > 0 ? kept_tiles(P.keep, it.key_begin, BKV) : 0;
+    it.n_kv = it.n_kept + (it.p_last - it.key_begin) / BKV + 1;
     it.table = P.block_table + (size_t)P.req_of_token[it.n0] * P.bt_stride;
     return it;
   };
@@ -263,7 +277,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
     failed = 0;
     asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
   }
-  if (warp == 1) tmem_alloc(smem_u32(&tmem_slot), 512);  // S0, S1 (128 columns each), O (128): 384 -> 512
+  if (warp == 1) tmem_alloc(smem_u32(&tmem_slot), 512);  // S0, S1 (128 columns each), O (128, two of them for two maps)
   tc_fence_before();
   __syncthreads();
   tc_fence_after();
@@ -291,7 +305,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
           const uint32_t dst = (which ? v_s : k_s) + st * TILE_BYTES;
           mbar_expect_tx(bar, TILE_BYTES);
           for (int b = 0; b < BKV / 64; ++b) {  // pages hold whole 64-key blocks
-            const int pos = it.key_begin + j * BKV + b * 64;
+            const int pos = walk_key(j, it.n_kept, it.key_begin, BKV) + b * 64;
             const int pi = pos / P.page_size;
             int page = pi < P.bt_stride ? it.table[pi] : -1;
             if (page >= P.num_pages) { atomicOr(P.status, JLX_STATUS_BAD_PAGE); page = 0; }
@@ -340,10 +354,17 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         if (!ok || *(volatile int*)&failed) { ok = false; return; }
         tc_fence_after();
         const uint32_t kb = k_s + st * TILE_BYTES;
+        // two maps: the rows' part that belongs to this item's map (the rest of the query row is zero)
+        int k_lo = 0, k_hi = DH / 16;
+        if (P.maps == 2) {
+          k_lo = (i & 1) * P.diff.map_dim / 16;
+          k_hi = (((i & 1) + 1) * P.diff.map_dim + 15) / 16;
+        }
 #pragma unroll
         for (int kk = 0; kk < DH / 16; ++kk) {
+          if (kk < k_lo || kk >= k_hi) continue;
           const uint32_t off = (kk >> 2) * HALF_BYTES + (kk & 3) * 32;  // 16 elements = 32 bytes along the row
-          umma_bf16(tm_s0 + st * 128, desc_k_major(q_s + off), desc_k_major(kb + off), idesc_qk, kk != 0);
+          umma_bf16(tm_s0 + st * 128, desc_k_major(q_s + off), desc_k_major(kb + off), idesc_qk, kk != k_lo);
         }
         umma_commit(BAR(B_SFULL + st));   // S is complete
         umma_commit(BAR(B_KEMPTY + st));  // K may be overwritten
@@ -364,10 +385,11 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
           if (!ok || *(volatile int*)&failed) { ok = false; break; }
           tc_fence_after();
           const uint32_t vb = v_s + st * TILE_BYTES;
+          const uint32_t tm_acc = tm_o + (P.maps == 2 && (i & 1) ? 128 : 0);
 #pragma unroll
           for (int kk = 0; kk < BKV / 16; ++kk) {
             // P: 16 keys = 8 columns of tensor memory; V: MN-major, 16 keys = 16 rows of 128 bytes
-            umma_bf16_a_tmem(tm_o, tm_s0 + st * 128 + kk * 8, desc_mn_major(vb + kk * 16 * 128, HALF_BYTES), idesc_pv, (j | kk) != 0);
+            umma_bf16_a_tmem(tm_acc, tm_s0 + st * 128 + kk * 8, desc_mn_major(vb + kk * 16 * 128, HALF_BYTES), idesc_pv, (j | kk) != 0);
           }
           umma_commit(BAR(B_VEMPTY + st));  // V may be overwritten
           umma_commit(BAR(B_ODONE));        // O holds the item's tiles up to this one
@@ -394,10 +416,12 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
     int g = 0;      // the tile's number in the block's stream
     int meets = 0;  // meetings of this quarter's threads so far (the phase of their barrier)
     Item upcoming = item(0);
+    float inv_first = 0.f;  // two maps: 1 / sum of the head's first map, kept until the second is done
     for (int i = 0; ok; ++i) {
       const Item it = upcoming;
       if (it.n_kv == 0) break;
       const bool live = row < it.cnt;
+      const uint32_t tm_acc = tm_o + (P.maps == 2 && (i & 1) ? 128 : 0);
       const int p_row = it.p_first + min(row, it.cnt - 1);
       const int lo_row = first_key(p_row, P.chunk, P.window);
       const int lo_last = first_key(it.p_last, P.chunk, P.window);
@@ -419,8 +443,8 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         ok = __all_sync(0xffffffffu, ok);
         if (!ok) break;
         tc_fence_after();
-        const int tile_key = it.key_begin + j * BKV + col0;
-        const bool need_mask = biased || it.key_begin + j * BKV + BKV - 1 > it.p_first || it.key_begin + j * BKV < lo_last;
+        const int tile0 = walk_key(j, it.n_kept, it.key_begin, BKV), tile_key = tile0 + col0;
+        const bool need_mask = biased || tile0 + BKV - 1 > it.p_first || tile0 < lo_last;
         const uint32_t s_addr = tm_s0 + st * 128 + lane_addr + col0;
         // this thread's raw scores of the row come into registers once
         uint32_t v[CP];
@@ -433,7 +457,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
 #pragma unroll
           for (int c = 0; c < CP; ++c) {
             const int key = tile_key + c;
-            const float sv = (key >= lo_row && key <= p_row) ? fmaf(-bias_raw, (float)(p_row - key), __uint_as_float(v[c])) : NEG_BIG;
+            const float sv = ((key >= lo_row || key < P.keep) && key <= p_row) ? fmaf(-bias_raw, (float)(p_row - key), __uint_as_float(v[c])) : NEG_BIG;
             v[c] = __float_as_uint(sv);
             mx4[c & 3] = fmaxf(mx4[c & 3], sv);
           }
@@ -507,11 +531,11 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
           uint32_t o[32];
 #pragma unroll 1
           for (int c0 = part * (DH / PARTS); c0 < (part + 1) * (DH / PARTS); c0 += 32) {
-            tmem_ld32(tm_o + lane_addr + c0, o);
+            tmem_ld32(tm_acc + lane_addr + c0, o);
             tmem_ld_wait();
 #pragma unroll
             for (int c = 0; c < 32; ++c) o[c] = __float_as_uint(__uint_as_float(o[c]) * corr);
-            tmem_st32(tm_o + lane_addr + c0, o);
+            tmem_st32(tm_acc + lane_addr + c0, o);
           }
         }
         tmem_st_wait();
@@ -542,6 +566,59 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         const float mm = fmaxf(m, sk);
         const float c = exp2f(m - mm);
         inv = c / (total * c + exp2f(sk - mm));
+      }
+      if (P.maps == 2) {
+        if (!(i & 1)) {  // the first map's rows stay in their accumulator
+          inv_first = inv;
+          tc_fence_before();
+          continue;
+        }
+        // o = a1 - weight * a2 for this thread's 32 columns, the row's sum of squares through shared memory, then the store
+        static_assert(DH / PARTS == 32, "a thread takes 32 of the output's columns");
+        const int c0 = part * 32;
+        uint32_t a[32], b[32];
+        tmem_ld32(tm_o + lane_addr + c0, a);
+        tmem_ld32(tm_o + 128 + lane_addr + c0, b);
+        tmem_ld_wait();
+        tc_fence_before();
+        const float w2 = P.diff.weight * inv;
+        float ss = 0.f;  // (columns beyond out_dim are zero, as the padded values are)
+#pragma unroll
+        for (int c = 0; c < 32; ++c) {
+          const float o = fmaf(__uint_as_float(a[c]), inv_first, -w2 * __uint_as_float(b[c]));
+          a[c] = __float_as_uint(o);
+          ss = fmaf(o, o, ss);
+        }
+        const int mq = meets & 1;
+        xsum[mq][part][row] = ss;
+        mbar_arrive(BAR(B_MEET + quarter));
+        ok = __all_sync(0xffffffffu, mbar_wait(BAR(B_MEET + quarter), mq));
+        ++meets;
+        if (!ok) break;
+        ss = 0.f;
+#pragma unroll
+        for (int q = 0; q < PARTS; ++q) ss += xsum[mq][q][row];
+        const float r = P.diff.mult / sqrtf(ss / (float)P.diff.out_dim + P.diff.eps);
+        bf16* dst = P.out + (size_t)(it.n0 + row) * P.diff.ld_out + (size_t)(it.head >> 1) * P.diff.out_dim + c0;
+        if (live) {
+#pragma unroll
+          for (int c = 0; c < 32; c += 8) {
+            if (P.vec_out) {
+              if (c0 + c < P.diff.out_dim) {
+                uint4 o;
+                __nv_bfloat162* op = reinterpret_cast<__nv_bfloat162*>(&o);
+#pragma unroll
+                for (int u = 0; u < 4; ++u) op[u] = __floats2bfloat162_rn(__uint_as_float(a[c + 2 * u]) * r, __uint_as_float(a[c + 2 * u + 1]) * r);
+                *reinterpret_cast<uint4*>(dst + c) = o;
+              }
+            } else {
+#pragma unroll
+              for (int u = 0; u < 8; ++u)
+                if (c0 + c + u < P.diff.out_dim) dst[c + u] = __float2bfloat16_rn(__uint_as_float(a[c + u]) * r);
+            }
+          }
+        }
+        continue;
       }
       bf16* dst = P.out + ((size_t)(it.n0 + row) * P.Hq + it.head) * DH;
       uint32_t v[32];
@@ -605,7 +682,7 @@ JLX_API int jlx_attention_prefill_tc(const void* q, const void* pages, const int
                                      const int* req_of_token, const int* positions, void* out, const int* tiles,
                                      int n_tiles, int N, int Hq, int Hkv, int dh, int page_size, int num_pages, float scale,
                                      int chunk, int window, float attn_scale, float floor_scale, const float* sink, const float* slopes,
-                                     float softcap, int* status, cudaStream_t stream) {
+                                     float softcap, int keep, const MapDifference* diff, int* status, cudaStream_t stream) {
   JLX_REQUIRE(jlx_attention_prefill_tc_supported(Hq, Hkv, dh, page_size),
               "attention_prefill_tc: needs head size 128 and pages of a multiple of 64 tokens (got %d, %d)", dh, page_size);
   JLX_REQUIRE(N > 0 && num_pages > 0 && bt_stride > 0, "attention_prefill_tc: bad sizes");
@@ -615,6 +692,13 @@ JLX_API int jlx_attention_prefill_tc(const void* q, const void* pages, const int
   JLX_REQUIRE(attn_scale == 0.f || floor_scale > 0.f, "attention: floor_scale must be positive");
   JLX_REQUIRE(Hq <= 65535, "attention_prefill_tc: too many heads");
   JLX_REQUIRE(softcap >= 0.f, "attention: the score cap must be positive (0: none)");
+  JLX_REQUIRE(keep >= 0, "attention: the count of kept first keys is negative");
+  if (diff) {
+    JLX_REQUIRE((Hq / Hkv) % 2 == 0 && diff->map_dim > 0 && 2 * diff->map_dim <= dh && diff->out_dim > 0 && diff->out_dim <= dh &&
+                diff->ld_out >= (long long)Hq / 2 * diff->out_dim,
+                "attention_prefill_tc: two maps of %d entries and values of %d do not fit %d query rows of %d", diff->map_dim, diff->out_dim, Hq, dh);
+    JLX_REQUIRE(!sink, "attention: the difference of two maps takes no sink");
+  }
   if (n_tiles == 0) return 0;
   EncodeTiledFn fn = encode_fn();
   JLX_REQUIRE(fn != nullptr, "attention_prefill_tc: the driver does not offer cuTensorMapEncodeTiled");
@@ -646,6 +730,10 @@ JLX_API int jlx_attention_prefill_tc(const void* q, const void* pages, const int
   P.cap_log2 = softcap > 0.f ? softcap * 1.4426950408889634f : 0.f;
   P.chunk = chunk; P.window = window; P.attn_scale = attn_scale;
   P.floor_scale = floor_scale; P.status = status; P.sink = sink; P.slopes = slopes;
+  P.keep = keep;
+  P.maps = diff ? 2 : 1;
+  P.diff = diff ? *diff : MapDifference{};
+  P.vec_out = diff && diff->out_dim % 8 == 0 && diff->ld_out % 8 == 0;
   const size_t smem = 5 * (size_t)TILE_BYTES + 1024;
   static bool cfg = false;
   if (!cfg) {
@@ -659,8 +747,8 @@ JLX_API int jlx_attention_prefill_tc(const void* q, const void* pages, const int
     JLX_CUDA(cudaGetDevice(&dev));
     JLX_CUDA(cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev));
   }
-  const int n_items = n_tiles * Hq;
-  attention_prefill_tc_kernel<<<dim3(n_items < sms ? n_items : sms), NTHREADS, smem, stream>>>(map_q, map_kv, P, n_items);
+  const int n_units = n_tiles * (Hq / P.maps);
+  attention_prefill_tc_kernel<<<dim3(n_units < sms ? n_units : sms), NTHREADS, smem, stream>>>(map_q, map_kv, P, n_units);
   JLX_LAUNCH_CHECK("attention_prefill_tc");
   return 0;
 }

@@ -147,13 +147,14 @@ __device__ __forceinline__ void router_topk(float* scores, int E, int k, size_t 
 // What a norm adds to the residual stream before it normalises: up to DELTA_MAX_TERMS terms, added in the order given.
 // A term is `splits` float32 partials [z][rows][D] (z ascending, `stride` elements apart), of which token r takes row
 // base + r, or, with `index`, the k rows index[r * k + j], j ascending (an expert layer's rows in expert order: the
-// norm then does the un-permute and the sum over a token's experts that a kernel of its own would do).
+// norm then does the un-permute and the sum over a token's experts that a kernel of its own would do), times `scale`.
 #define DELTA_MAX_TERMS 3
 struct DeltaTerm {
   const float* p;
   long long stride;
   const int* index;
   int splits, k, base;
+  float scale;
 };
 struct DeltaSpec {
   int n;
@@ -168,6 +169,7 @@ struct DeltaSpec {
 #define DELTA_CHUNK 8
 struct DeltaSources {
   const float* ptr[DELTA_MAX_STREAMS];
+  float scale[DELTA_MAX_STREAMS];
   int n;
 };
 // Called by every thread; thread 0 fills `src`, a barrier follows.
@@ -182,7 +184,10 @@ __device__ __forceinline__ void resolve_delta(DeltaSources& src, const DeltaSpec
       const int rows = t.index ? t.k : 1;
       for (int j = 0; j < rows; ++j) {
         const size_t row = t.index && real ? (size_t)t.index[r * t.k + j] : (size_t)t.base + r;
-        for (int z = 0; z < t.splits && n < DELTA_MAX_STREAMS; ++z) src.ptr[n++] = t.p + (size_t)z * t.stride + row * D;
+        for (int z = 0; z < t.splits && n < DELTA_MAX_STREAMS; ++z, ++n) {
+          src.ptr[n] = t.p + (size_t)z * t.stride + row * D;
+          src.scale[n] = t.scale;
+        }
       }
     }
     src.n = n;
@@ -201,16 +206,22 @@ __device__ __forceinline__ void add_streams4(float4& s, const DeltaSources& src,
     }
 #pragma unroll
     for (int u = 0; u < DELTA_CHUNK; ++u)
-      if (q0 + u < src.n) { s.x += v[u].x; s.y += v[u].y; s.z += v[u].z; s.w += v[u].w; }
+      if (q0 + u < src.n) {
+        const float c = src.scale[q0 + u];
+        s.x = fmaf(c, v[u].x, s.x); s.y = fmaf(c, v[u].y, s.y); s.z = fmaf(c, v[u].z, s.z); s.w = fmaf(c, v[u].w, s.w);
+      }
   }
 }
 
+// With `places` (int [N * copies]) row n of the norm goes to the rows places[n * copies + j] of `out` instead of row n: a routed
+// feed-forward whose pairs are sorted already gets its rows in expert order, and no kernel gathers them.
+#define NORM_MAX_COPIES 16
 template <typename TO>
 __global__ void __launch_bounds__(1024)
 add_rmsnorm_kernel(float* __restrict__ x, const DeltaSpec ds,
                    const float* __restrict__ gamma, float eps, TO* __restrict__ out, float* __restrict__ out32,
                    const int* __restrict__ row_index, int D, int row_in_smem, const float* __restrict__ w_router, int E,
-                   int k, int* __restrict__ topk_idx, float* __restrict__ topk_w) {
+                   int k, int* __restrict__ topk_idx, float* __restrict__ topk_w, const int* __restrict__ places, int copies) {
   JLX_TL(TL_NORM);
   extern __shared__ __align__(16) float rowbuf[];  // [D] when row_in_smem
   __shared__ float scratch[33];
@@ -237,7 +248,9 @@ add_rmsnorm_kernel(float* __restrict__ x, const DeltaSpec ds,
   pdl_wait();
   const size_t r = row_index ? (size_t)row_index[n] : (size_t)n;
   float* xr = x + r * D;
-  if (has_delta) resolve_delta(src, ds, r, D);
+  __shared__ size_t dst[NORM_MAX_COPIES];  // where the row goes: its first elements in `out`
+  if ((int)threadIdx.x < copies) dst[threadIdx.x] = (places ? (size_t)places[(size_t)n * copies + threadIdx.x] : (size_t)n) * D;
+  if (has_delta) resolve_delta(src, ds, r, D);  // (barriers behind it and in block_sum)
   JLX_TL_MARK(0);
   float ss = 0.f;
   if (vec) {
@@ -263,7 +276,8 @@ add_rmsnorm_kernel(float* __restrict__ x, const DeltaSpec ds,
       const float4 t = row4[i];
       const float4 g = turn == 0 ? g_ahead : (gamma ? g4[i] : make_float4(1.f, 1.f, 1.f, 1.f));
       const float4 v = make_float4(g.x * t.x / rms, g.y * t.y / rms, g.z * t.z / rms, g.w * t.w / rms);
-      if (out) store4<TO>(out + (size_t)n * D + 4 * i, v);
+      if (out)
+        for (int j = 0; j < copies; ++j) store4<TO>(out + dst[j] + 4 * i, v);
       if (out32) reinterpret_cast<float4*>(out32 + (size_t)n * D)[i] = v;
       row4[i] = v;
     }
@@ -271,7 +285,7 @@ add_rmsnorm_kernel(float* __restrict__ x, const DeltaSpec ds,
     for (int d = threadIdx.x; d < D; d += blockDim.x) {
       float s = xr[d];
       if (has_delta) {
-        for (int q = 0; q < src.n; ++q) s += src.ptr[q][d];
+        for (int q = 0; q < src.n; ++q) s = fmaf(src.scale[q], src.ptr[q][d], s);
         if (!row_index) xr[d] = s;
       }
       if (row_in_smem) rowbuf[d] = s;
@@ -286,10 +300,11 @@ add_rmsnorm_kernel(float* __restrict__ x, const DeltaSpec ds,
       } else {
         s = xr[d];
         if (has_delta && row_index)
-          for (int q = 0; q < src.n; ++q) s += src.ptr[q][d];
+          for (int q = 0; q < src.n; ++q) s = fmaf(src.scale[q], src.ptr[q][d], s);
       }
       const float v = (gamma ? gamma[d] * s : s) / rms;
-      if (out) out[(size_t)n * D + d] = from_f32<TO>(v);
+      if (out)
+        for (int j = 0; j < copies; ++j) out[dst[j] + d] = from_f32<TO>(v);
       if (out32) out32[(size_t)n * D + d] = v;
       if (row_in_smem) rowbuf[d] = v;
     }
@@ -342,7 +357,7 @@ add_rmsnorm_router_cluster_kernel(float* __restrict__ x, const DeltaSpec ds,
                                   const float* __restrict__ gamma, float eps, TO* __restrict__ out, float* __restrict__ out32, int D,
                                   int slice,
                                   const float* __restrict__ w_router, int E, int k, int* __restrict__ topk_idx,
-                                  float* __restrict__ topk_w, const DispatchArgs dp) {
+                                  float* __restrict__ topk_w, const DispatchArgs dp, const int* __restrict__ places, int copies) {
   JLX_TL(TL_NORM_ROUTER);
   namespace cg = cooperative_groups;
   cg::cluster_group cluster = cg::this_cluster();
@@ -363,6 +378,7 @@ add_rmsnorm_router_cluster_kernel(float* __restrict__ x, const DeltaSpec ds,
   float4* x4 = reinterpret_cast<float4*>(x + (size_t)n * D);
   float4* row4 = reinterpret_cast<float4*>(rowbuf);
   __shared__ DeltaSources src;
+  __shared__ size_t dst[NORM_MAX_COPIES];  // where the row goes (see add_rmsnorm_kernel)
   // this block's slices of the norm's and the router's weights have left L2 since the layer before: they are asked
   // back while the predecessor still runs.  (No rehearsal, see jlx_rehearses: the kernel follows a matrix product
   // whose blocks fill the GPU, its cluster starts only microseconds before that ends, and a rehearsal then still runs
@@ -385,6 +401,7 @@ add_rmsnorm_router_cluster_kernel(float* __restrict__ x, const DeltaSpec ds,
   for (int pass = ROUTER || gridDim.x > C ? 1 : 0; pass < 2; ++pass) {
   const bool real = pass == 1;
   if (real) pdl_wait();
+  if (real && (int)threadIdx.x < copies) dst[threadIdx.x] = (places ? (size_t)places[(size_t)n * copies + threadIdx.x] : (size_t)n) * D;
   if (ds.n > 0) resolve_delta(src, ds, (size_t)n, D, real);
   float ss = 0.f;
   for (int i = (lo >> 2) + threadIdx.x; i < (hi >> 2); i += blockDim.x) {
@@ -415,7 +432,8 @@ add_rmsnorm_router_cluster_kernel(float* __restrict__ x, const DeltaSpec ds,
     const float4 s = row4[i - (lo >> 2)];
     const float4 g = i == mine ? g_ahead : (gamma ? g4[i] : make_float4(1.f, 1.f, 1.f, 1.f));
     const float4 v = make_float4(g.x * s.x * inv_rms, g.y * s.y * inv_rms, g.z * s.z * inv_rms, g.w * s.w * inv_rms);
-    if (real) store4<TO>(out + (size_t)n * D + 4 * i, v);
+    if (real)
+      for (int j = 0; j < copies; ++j) store4<TO>(out + dst[j] + 4 * i, v);
     if (real && out32) reinterpret_cast<float4*>(out32 + (size_t)n * D)[i] = v;
     row4[i - (lo >> 2)] = v;
   }
@@ -515,10 +533,12 @@ add_rmsnorm_router_cluster_kernel(float* __restrict__ x, const DeltaSpec ds,
 JLX_API int jlx_add_rmsnorm(float* x, const DeltaSpec* delta, const float* gamma,
                             float eps, void* out, int out_dtype, float* out32, const int* row_index, int N, int D,
                             const float* w_router, int E, int k, int* topk_idx, float* topk_w, const DispatchArgs* dispatch,
-                            int* dispatched, cudaStream_t stream) {
+                            int* dispatched, const int* places, int copies, cudaStream_t stream) {
   if (dispatched) *dispatched = 0;
   JLX_REQUIRE(N >= 0 && D > 0, "add_rmsnorm: bad sizes N=%d D=%d", N, D);
   JLX_REQUIRE(eps > 0.f, "add_rmsnorm: eps must be positive");
+  JLX_REQUIRE(copies >= 1 && copies <= NORM_MAX_COPIES && (places || copies == 1) && !(places && (row_index || w_router)),
+              "add_rmsnorm: rows in %d places each (up to %d, without chosen rows and without a router)", copies, NORM_MAX_COPIES);
   DeltaSpec ds = {};
   if (delta) ds = *delta;
   JLX_REQUIRE(ds.n >= 0 && ds.n <= DELTA_MAX_TERMS, "add_rmsnorm: %d terms to add; up to %d are supported", ds.n, DELTA_MAX_TERMS);
@@ -572,10 +592,10 @@ JLX_API int jlx_add_rmsnorm(float* x, const DeltaSpec* delta, const float* gamma
     }
     if (w_router)
       JLX_CUDA(cudaLaunchKernelEx(&cfg, add_rmsnorm_router_cluster_kernel<bf16, true>, x, ds, gamma, eps,
-                                  (bf16*)out, out32, D, slice, w_router, E, k, topk_idx, topk_w, dp));
+                                  (bf16*)out, out32, D, slice, w_router, E, k, topk_idx, topk_w, dp, places, copies));
     else
       JLX_CUDA(cudaLaunchKernelEx(&cfg, add_rmsnorm_router_cluster_kernel<bf16, false>, x, ds, gamma, eps,
-                                  (bf16*)out, out32, D, slice, w_router, E, k, topk_idx, topk_w, dp));
+                                  (bf16*)out, out32, D, slice, w_router, E, k, topk_idx, topk_w, dp, places, copies));
     JLX_LAUNCH_CHECK("add_rmsnorm (cluster)");
     return 0;
   }
@@ -591,7 +611,7 @@ JLX_API int jlx_add_rmsnorm(float* x, const DeltaSpec* delta, const float* gamma
     const bool exact = out_dtype == JLX_F32;
     const int threads = (D >= 2048 && (exact || N <= 256)) ? 1024 : 256;
     JLX_CUDA(jlx_launch_pdl(add_rmsnorm_kernel<TO>, dim3(N), dim3(threads), smem, stream, x, ds,
-                            gamma, eps, (TO*)out, out32, row_index, D, row_in_smem, w_router, E, k, topk_idx, topk_w));
+                            gamma, eps, (TO*)out, out32, row_index, D, row_in_smem, w_router, E, k, topk_idx, topk_w, places, copies));
   });
   JLX_LAUNCH_CHECK("add_rmsnorm");
   return 0;
@@ -669,5 +689,29 @@ JLX_API int jlx_silu_mul(const void* gu, int in_dtype, int splits, long long spl
   JLX_DISPATCH_DTYPE(in_dtype, TI, JLX_DISPATCH_DTYPE(out_dtype, TO,
       (silu_mul_kernel<TI, TO><<<rows, 256, 0, stream>>>((const TI*)gu, splits, split_stride, (TO*)out, F, interleaved, form))));
   JLX_LAUNCH_CHECK("silu_mul");
+  return 0;
+}
+
+// x <- cap * tanh(x / cap), in place: a cap on the logits.  (The library's tanhf: the kernel is bound by memory.)
+__global__ void soft_cap_kernel(float* __restrict__ x, size_t n, float cap) {
+  JLX_TL(TL_OTHER);
+  pdl_launch_dependents();
+  pdl_wait();
+  const size_t step = (size_t)gridDim.x * blockDim.x, t = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+  float4* x4 = reinterpret_cast<float4*>(x);
+  for (size_t i = t; i < n / 4; i += step) {
+    float4 v = x4[i];
+    v.x = cap * tanhf(v.x / cap); v.y = cap * tanhf(v.y / cap); v.z = cap * tanhf(v.z / cap); v.w = cap * tanhf(v.w / cap);
+    x4[i] = v;
+  }
+  for (size_t i = n / 4 * 4 + t; i < n; i += step) x[i] = cap * tanhf(x[i] / cap);
+}
+
+JLX_API int jlx_soft_cap(float* x, long long n, float cap, cudaStream_t stream) {
+  JLX_REQUIRE(n >= 0 && cap > 0.f && ((uintptr_t)x & 15) == 0, "soft_cap: the cap must be positive and the rows 16-byte aligned");
+  if (n == 0) return 0;
+  const long long blocks = (n / 4 + 255) / 256;
+  JLX_CUDA(jlx_launch_pdl(soft_cap_kernel, dim3((unsigned)(blocks < 1 ? 1 : (blocks > 1184 ? 1184 : blocks))), dim3(256), 0, stream, x, (size_t)n, cap));
+  JLX_LAUNCH_CHECK("soft_cap");
   return 0;
 }

@@ -7,7 +7,8 @@
 // no check for running out of pages.  Here pages are handed out and taken back on the host:
 //
 //  * A *group* is a set of layers with the same need: all keys (kind 0), the keys of the current
-//    chunk of `size` positions (kind 1), or the last `size` keys (kind 2).  Each group has its own
+//    chunk of `size` positions (kind 1), or the last `size` keys (kind 2), the sequence's first `keep`
+//    keys besides where a group asks for that (their pages then live as long as the request).  Each group has its own
 //    pool of pages and its own block table; a page id means the same slot in every layer of the group.
 //  * A *slot* is a live request: its committed length, its reserved length and one block-table row
 //    per group (logical page index = position / page_size -> page id, -1 where nothing is held).
@@ -26,11 +27,12 @@ enum Kind { ALL = 0, CHUNK = 1, WINDOW = 2 };
 struct Group {
   int kind = ALL;
   int size = 0;
+  int kept_pages = 0;                   // a request's first so many pages are given back only with the request
   int num_pages = 0;
   std::vector<int32_t> free_stack;      // LIFO: a page given back is the next one handed out
   std::vector<uint8_t> held;            // 1 while a block table holds the page
   std::vector<int32_t> table;           // [max_slots][max_pages_per_req]
-  std::vector<int32_t> first_held;      // per slot: lowest logical page that may still be held
+  std::vector<int32_t> first_held;      // per slot: lowest logical page that may still be held (beyond the kept ones)
 };
 
 struct Slot {
@@ -72,12 +74,13 @@ API void* cm_create(int page_size, int max_slots, int max_pages_per_req) {
 
 API void cm_destroy(void* h) { delete static_cast<Manager*>(h); }
 
-API int cm_add_group(void* h, int kind, int size, int num_pages) {
+API int cm_add_group(void* h, int kind, int size, int keep, int num_pages) {
   Manager* m = static_cast<Manager*>(h);
-  if (kind < ALL || kind > WINDOW || num_pages <= 0 || (kind != ALL && size <= 0)) return -1;
+  if (kind < ALL || kind > WINDOW || num_pages <= 0 || keep < 0 || (kind != ALL && size <= 0)) return -1;
   Group g;
   g.kind = kind;
   g.size = size;
+  g.kept_pages = (int)ceil_div(keep, m->page_size);
   g.num_pages = num_pages;
   g.held.assign(num_pages, 0);
   for (int p = num_pages - 1; p >= 0; --p) g.free_stack.push_back(p);
@@ -149,7 +152,8 @@ API int cm_reserve(void* h, int s, long long new_len) {
 }
 
 // The step that filled positions [committed, new_len) has been launched.  Gives back, per group, the
-// pages wholly before the first position that the request's next query can read.  Returns the
+// pages wholly before the first position that the request's next query can read (but for the kept first
+// ones).  Returns the
 // number of pages given back, or a negative code for misuse.
 API int cm_commit(void* h, int s, long long new_len) {
   Manager* m = static_cast<Manager*>(h);
@@ -162,7 +166,7 @@ API int cm_commit(void* h, int s, long long new_len) {
     if (g.kind == ALL) continue;
     const int64_t dead_pages = first_needed(g, new_len) / m->page_size;  // pages [0, dead_pages) are dead
     int32_t* row = g.table.data() + (size_t)s * m->max_pages_per_req;
-    for (int64_t i = g.first_held[s]; i < dead_pages; ++i) {
+    for (int64_t i = g.first_held[s] > g.kept_pages ? g.first_held[s] : g.kept_pages; i < dead_pages; ++i) {
       const int32_t p = row[i];
       if (p >= 0) {
         g.held[p] = 0;
@@ -186,7 +190,7 @@ API int cm_release(void* h, int s) {
   int freed = 0;
   for (Group& g : m->groups) {
     int32_t* row = g.table.data() + (size_t)s * m->max_pages_per_req;
-    for (int64_t i = g.first_held[s]; i < hi; ++i) {
+    for (int64_t i = g.kept_pages > 0 ? 0 : g.first_held[s]; i < hi; ++i) {
       const int32_t p = row[i];
       if (p >= 0) {
         g.held[p] = 0;

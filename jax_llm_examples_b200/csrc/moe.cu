@@ -172,10 +172,31 @@ JLX_API int jlx_router(const float* h, const float* w_router, int* topk_idx, flo
 // With tile_rows > 0 it also lists the row tiles of the grouped products that follow: tile_list[t] =
 // (group, first row) for every tile of tile_rows rows that holds at least one row, and n_tiles[0] = how many,
 // so that a product's blocks find their work with one load instead of a walk over the offsets.
+// With `by.table` the choices are not given but looked up: token n's are row ids[n] of the table (and are written to
+// `by.chosen` if that is given); the sort then needs nothing but the step's token ids.
+struct TableChoice {
+  const int* ids;      // [N] token ids
+  const int* table;    // [V, k]
+  int* chosen;         // optional [N, k]
+  int V, k;
+};
+__device__ __forceinline__ int pair_choice(const int* topk_idx, const TableChoice& by, int i, int* status) {
+  if (!by.table) return topk_idx[i];
+  const int n = i / by.k;
+  int id = by.ids[n];
+  if (id < 0 || id >= by.V) {
+    atomicOr(status, JLX_STATUS_BAD_TOKEN);
+    id = 0;
+  }
+  const int e = by.table[(size_t)id * by.k + (i - n * by.k)];
+  if (by.chosen) by.chosen[i] = e;
+  return e;
+}
+
 __global__ void expert_sort_kernel(const int* __restrict__ topk_idx, int* __restrict__ offsets,
                                    int* __restrict__ sorted_pair, int* __restrict__ sorted_pos, int P, int E, int extra_rows,
                                    int tile_rows, int* __restrict__ tile_list, int* __restrict__ n_tiles, int* status,
-                                   int in_smem, int tile_groups) {
+                                   int in_smem, int tile_groups, const TableChoice by) {
   JLX_TL(TL_SORT);
   __shared__ int counts[ROUTER_MAX_E + 1];
   extern __shared__ int staged[];  // the choices, when `in_smem`: both passes below walk them once per expert
@@ -187,7 +208,7 @@ __global__ void expert_sort_kernel(const int* __restrict__ topk_idx, int* __rest
     const bool real = pass == 1;
     if (real) pdl_wait();
     if (in_smem) {
-      for (int i = threadIdx.x; i < P; i += blockDim.x) staged[i] = real ? topk_idx[i] : -1;
+      for (int i = threadIdx.x; i < P; i += blockDim.x) staged[i] = real ? pair_choice(topk_idx, by, i, status) : -1;
       __syncthreads();
     }
     if (real) JLX_TL_MARK(0);
@@ -232,7 +253,7 @@ __global__ void expert_sort_kernel(const int* __restrict__ topk_idx, int* __rest
 __global__ void __launch_bounds__(SORT_WARPS * 32)
 expert_sort_many_kernel(const int* __restrict__ topk_idx, int* __restrict__ offsets, int* __restrict__ sorted_pair,
                         int* __restrict__ sorted_pos, int P, int E, int extra_rows, int tile_rows, int* __restrict__ tile_list,
-                        int* __restrict__ n_tiles, int* status, int tile_groups) {
+                        int* __restrict__ n_tiles, int* status, int tile_groups, const TableChoice by) {
   JLX_TL(TL_SORT);
   __shared__ int counts[ROUTER_MAX_E + 1];
   extern __shared__ int held[];  // [SORT_WARPS][E]: a warp's pairs per expert, then its next place among them
@@ -246,7 +267,7 @@ expert_sort_many_kernel(const int* __restrict__ topk_idx, int* __restrict__ offs
   __syncwarp();
   for (int base = lo; base < hi; base += 32) {
     const int i = base + lane;
-    const int v = i < hi ? topk_idx[i] : -1;
+    const int v = i < hi ? pair_choice(topk_idx, by, i, status) : -1;
     const unsigned same = __match_any_sync(0xffffffffu, v);
     if (v >= 0 && v < E && (same & ((1u << lane) - 1u)) == 0) mine[v] += __popc(same);
     __syncwarp();
@@ -266,7 +287,7 @@ expert_sort_many_kernel(const int* __restrict__ topk_idx, int* __restrict__ offs
   __syncthreads();
   for (int base = lo; base < hi; base += 32) {
     const int i = base + lane;
-    const int v = i < hi ? topk_idx[i] : -1;
+    const int v = i < hi ? pair_choice(topk_idx, by, i, status) : -1;
     const unsigned same = __match_any_sync(0xffffffffu, v);
     const unsigned before = same & ((1u << lane) - 1u);
     const bool ok = v >= 0 && v < E;
@@ -285,19 +306,26 @@ expert_sort_many_kernel(const int* __restrict__ topk_idx, int* __restrict__ offs
 // tile_list: int [(ceil((P + extra_rows) / tile_rows) + groups) * 2]; n_tiles: int [1]; both unused if tile_rows == 0.
 JLX_API int jlx_expert_sort(const int* topk_idx, int* offsets, int* sorted_pair, int* sorted_pos, int P, int E,
                             int extra_rows, int tile_rows, int* tile_list, int* n_tiles, int* status, int tile_groups,
-                            cudaStream_t stream) {
+                            const TableChoice* table, cudaStream_t stream) {
   JLX_REQUIRE(tile_rows == 0 || (tile_list && n_tiles), "expert_sort: tile list outputs missing");
   JLX_REQUIRE(tile_groups >= 0 && (tile_groups == 0 || extra_rows == 0), "expert_sort: tiles for the first groups only, without an appended group");
   JLX_REQUIRE(P >= 0 && E >= 1 && E <= ROUTER_MAX_E && extra_rows >= 0, "expert_sort: bad sizes P=%d E=%d", P, E);
+  TableChoice by = {};
+  if (table) {
+    by = *table;
+    JLX_REQUIRE(by.ids && by.table && by.V > 0 && by.k > 0 && P % by.k == 0, "expert_sort: incomplete table of choices");
+  } else {
+    JLX_REQUIRE(topk_idx || P == 0, "expert_sort: no choices");
+  }
   if (P >= 1024) {
     JLX_CUDA(jlx_launch_pdl(expert_sort_many_kernel, dim3(1), dim3(SORT_WARPS * 32), (size_t)SORT_WARPS * E * sizeof(int), stream, topk_idx,
-                            offsets, sorted_pair, sorted_pos, P, E, extra_rows, tile_rows, tile_list, n_tiles, status, tile_groups));
+                            offsets, sorted_pair, sorted_pos, P, E, extra_rows, tile_rows, tile_list, n_tiles, status, tile_groups, by));
     return 0;
   }
   const int warps = E < 32 ? E : 32;
   const int in_smem = (size_t)P * sizeof(int) <= 40 * 1024;
   JLX_CUDA(jlx_launch_pdl(expert_sort_kernel, dim3(1), dim3(warps * 32), in_smem ? (size_t)P * sizeof(int) : 0, stream, topk_idx,
-                          offsets, sorted_pair, sorted_pos, P, E, extra_rows, tile_rows, tile_list, n_tiles, status, in_smem, tile_groups));
+                          offsets, sorted_pair, sorted_pos, P, E, extra_rows, tile_rows, tile_list, n_tiles, status, in_smem, tile_groups, by));
   return 0;
 }
 

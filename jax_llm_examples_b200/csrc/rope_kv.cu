@@ -394,6 +394,11 @@ JLX_API int jlx_kv_store(const void* k, const void* v, void* pages, int dtype, c
 // were projected).  q_out and the cache keep `dpad` entries per head: keys, queries and values are padded with zeros
 // up to it, so that one page layout and the attention kernels built for equal sizes serve keys of one size and values
 // of another.
+//
+// `bias` (float32, one number per projected column, or null) is added to the projected rows first.  With `maps` = 2 the q and
+// k heads are pairs of maps over the values of one head: Hq and Hkv count q rows and VALUE heads, the 2 Hkv keys of dk
+// entries lie head by head as [map 1, map 2] and go side by side into one cached row, and a query row holds its map's
+// entries at that map's place, zeros elsewhere (see attention_maps.cuh).
 enum { ROPE_PAIRS_HALVES = 0, ROPE_PAIRS_INTERLEAVED = 1 };
 // ROPE_NORM_WHOLE: before the rotation, over ALL heads of the projection at once: q / sqrt(mean over its Hq dk entries
 // + eps) * w, w: [Hq dk] ([Hkv dk] for k).
@@ -414,7 +419,7 @@ __global__ void rope_half_kv_store_kernel(RopeRowsView proj, int k_col, int v_co
                                           const float* __restrict__ k_norm_w, float eps, const float* __restrict__ inv_freq,
                                           int rot, int pairing, int norm_mode, int Hq, int Hkv, int dk, int dv, int dpad,
                                           int page_size, int num_pages, int store, int* status, float amplitude, const float* __restrict__ q_scale,
-                                          int v_norm) {
+                                          int v_norm, const float* __restrict__ bias, int maps) {
   JLX_TL(TL_ROPE);
   pdl_launch_dependents_if_small();
   __shared__ float whole_part[2][8];
@@ -446,16 +451,18 @@ __global__ void rope_half_kv_store_kernel(RopeRowsView proj, int k_col, int v_co
   }
   __syncthreads();
   pdl_wait();
-  const int heads = Hq + (store ? 2 * Hkv : 0);
+  const int n_k = maps * Hkv;  // keys that the token projects
+  const int heads = Hq + (store ? n_k + Hkv : 0);
   float whole_rms[2] = {1.f, 1.f};  // of all q entries, of all k entries
   if (norm_mode == ROPE_NORM_WHOLE) {
     // every block of the token makes both sums itself, in an order fixed by the block's size (the model's head count)
     for (int which = 0; which < (store ? 2 : 1); ++which) {
-      const int cnt = (which ? Hkv : Hq) * dk, col0 = which ? k_col : 0;
+      const int cnt = (which ? n_k : Hq) * dk, col0 = which ? k_col : 0;
       float ss = 0.f;
       for (int i = threadIdx.x; i < cnt; i += blockDim.x) {
         float v = 0.f;
         for (int z = 0; z < proj.splits; ++z) v += proj.p[(size_t)z * proj.split_stride + n * proj.ld + col0 + i];
+        if (bias) v += bias[col0 + i];
         ss = fmaf(v, v, ss);
       }
       ss = warp_sum(ss);
@@ -465,22 +472,35 @@ __global__ void rope_half_kv_store_kernel(RopeRowsView proj, int k_col, int v_co
     for (int which = 0; which < (store ? 2 : 1); ++which) {
       float ss = 0.f;
       for (int w = 0; w < nwarp; ++w) ss += whole_part[which][w];
-      whole_rms[which] = sqrtf(ss / (float)((which ? Hkv : Hq) * dk) + eps);
+      whole_rms[which] = sqrtf(ss / (float)((which ? n_k : Hq) * dk) + eps);
     }
   }
   for (int hh = blockIdx.y * nwarp + warp; hh < heads; hh += gridDim.y * nwarp) {
-    const bool is_q = hh < Hq, is_k = !is_q && hh < Hq + Hkv;
+    const bool is_q = hh < Hq, is_k = !is_q && hh < Hq + n_k;
     const bool qk = is_q || is_k;
     const int d = qk ? dk : dv;
-    const int col = is_q ? hh * dk : (is_k ? k_col + (hh - Hq) * dk : v_col + (hh - Hq - Hkv) * dv);
+    const int col = is_q ? hh * dk : (is_k ? k_col + (hh - Hq) * dk : v_col + (hh - Hq - n_k) * dv);
+    // where the head's entries go in its row of dpad, and which stretch of the row this warp writes
+    int at = 0, w_lo = 0, w_hi = dpad;
     T* dst;
-    if (is_q) dst = q_out + (n * Hq + hh) * dpad;
-    else if (!kdst) continue;
-    else dst = kdst + (size_t)((is_k ? hh - Hq : Hkv + hh - Hq - Hkv)) * page_size * dpad;
+    if (is_q) {
+      dst = q_out + (n * Hq + hh) * dpad;
+      at = (hh % maps) * dk;
+    } else if (!kdst) {
+      continue;
+    } else if (is_k) {
+      const int map = (hh - Hq) % maps;
+      dst = kdst + (size_t)((hh - Hq) / maps) * page_size * dpad;
+      at = w_lo = map * dk;
+      if (map + 1 < maps) w_hi = w_lo + dk;  // the last map's warp writes the padding
+    } else {
+      dst = kdst + (size_t)(Hkv + hh - Hq - n_k) * page_size * dpad;
+    }
     float ss = 0.f;
     for (int i = lane; i < d; i += 32) {
       float s = 0.f;
       for (int z = 0; z < proj.splits; ++z) s += proj.p[(size_t)z * proj.split_stride + n * proj.ld + col + i];
+      if (bias) s += bias[col + i];
       row[i] = s;
       ss = fmaf(s, s, ss);
     }
@@ -519,14 +539,15 @@ __global__ void rope_half_kv_store_kernel(RopeRowsView proj, int k_col, int v_co
     }
     __syncwarp();
     const float qs = is_q && q_scale ? q_scale[hh] : 1.f;
-    for (int i = lane; i < dpad; i += 32) {
+    for (int j = w_lo + lane; j < w_hi; j += 32) {
+      const int i = j - at;
       float y = 0.f;
-      if (i < d) {
+      if (i >= 0 && i < d) {
         y = turned[i];
         if (after) y = w ? y / rms_turned * w[i] : y / rms_turned;
         y *= qs;
       }
-      dst[i] = from_f32<T>(y);
+      dst[j] = from_f32<T>(y);
     }
     __syncwarp();
   }
@@ -541,16 +562,17 @@ JLX_API int jlx_rope_half_kv_store(const RopeRowsView* proj, int k_col, int v_co
                                    const float* q_norm_w, const float* k_norm_w, float eps, const float* inv_freq, int rot,
                                    int pairing, int norm_mode, int N, int Hq, int Hkv, int dk, int dv, int dpad, int page_size,
                                    int num_pages, int store, int* status, float amplitude, const float* q_scale, int v_norm,
-                                   cudaStream_t stream) {
+                                   const float* bias, int maps, cudaStream_t stream) {
   JLX_REQUIRE(N >= 0 && Hq > 0 && Hkv > 0 && dk > 0 && dv > 0, "rope_half: bad sizes");
-  JLX_REQUIRE(dpad >= dk && dpad >= dv, "rope_half: the padded head size %d is below the key or value size (%d, %d)", dpad, dk, dv);
+  JLX_REQUIRE(maps == 1 || (maps == 2 && Hq % 2 == 0 && norm_mode != ROPE_NORM_WHOLE && v_col != k_col), "rope_half: %d maps per head with %d query rows", maps, Hq);
+  JLX_REQUIRE(dpad >= maps * dk && dpad >= dv, "rope_half: the padded head size %d is below the key or value size (%d, %d)", dpad, dk, dv);
   JLX_REQUIRE(rot >= 0 && rot % 2 == 0 && rot <= dk, "rope_half: %d rotated entries of %d", rot, dk);
   JLX_REQUIRE(rot == 0 || inv_freq, "rope_half: frequencies missing");
   JLX_REQUIRE(pairing == ROPE_PAIRS_HALVES || pairing == ROPE_PAIRS_INTERLEAVED, "rope_half: unknown pairing %d", pairing);
   JLX_REQUIRE(norm_mode >= ROPE_NORM_NONE && norm_mode <= ROPE_NORM_WHOLE, "rope_half: unknown norm mode %d", norm_mode);
   JLX_REQUIRE(!store || (pages && block_table && page_size > 0 && num_pages > 0), "rope_half: cache missing");
   if (N == 0) return 0;
-  const int heads = Hq + (store ? 2 * Hkv : 0);
+  const int heads = Hq + (store ? (maps + 1) * Hkv : 0);
   const int nwarp = heads < 8 ? heads : 8;
   const int by = N >= 64 ? 1 : (heads + nwarp - 1) / nwarp;
   const size_t smem = sizeof(float) * (2 * (size_t)nwarp * (dk > dv ? dk : dv) + rot);
@@ -559,7 +581,7 @@ JLX_API int jlx_rope_half_kv_store(const RopeRowsView* proj, int k_col, int v_co
     JLX_CUDA(jlx_launch_pdl(rope_half_kv_store_kernel<T>, dim3(N, by), dim3(nwarp * 32), smem, stream, *proj, k_col, v_col,
                             (T*)q_out, (T*)pages, block_table, bt_stride, req_of_token, positions, q_norm_w, k_norm_w, eps,
                             inv_freq, rot, pairing, norm_mode, Hq, Hkv, dk, dv, dpad, page_size, num_pages, store, status, amplitude,
-                            q_scale, v_norm));
+                            q_scale, v_norm, bias, maps));
   });
   JLX_LAUNCH_CHECK("rope_half_kv_store");
   return 0;

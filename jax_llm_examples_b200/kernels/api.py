@@ -130,7 +130,8 @@ DISPATCH_MAX_ROWS, DISPATCH_MAX_PAIRS = 16, 64  # csrc/elementwise.cu
 
 
 class _DeltaTerm(ctypes.Structure):
-    _fields_ = [("p", c_void_p), ("stride", c_longlong), ("index", c_void_p), ("splits", c_int), ("k", c_int), ("base", c_int)]
+    _fields_ = [("p", c_void_p), ("stride", c_longlong), ("index", c_void_p), ("splits", c_int), ("k", c_int), ("base", c_int),
+                ("scale", c_float)]
 
 
 class _DeltaSpec(ctypes.Structure):
@@ -146,11 +147,12 @@ class _DispatchArgs(ctypes.Structure):  # DispatchArgs in csrc/elementwise.cu
 def add_rmsnorm(x: torch.Tensor, delta, gamma: torch.Tensor | None, eps: float,
                 out: torch.Tensor | None, out32: torch.Tensor | None = None, row_index: torch.Tensor | None = None,
                 delta_splits: int = 1, w_router: torch.Tensor | None = None, topk_idx: torch.Tensor | None = None,
-                topk_w: torch.Tensor | None = None, dispatch=None) -> bool:
+                topk_w: torch.Tensor | None = None, dispatch=None, places: torch.Tensor | None = None, copies: int = 1) -> bool:
     """x (+= delta); out = gamma * x / sqrt(mean(x^2) + eps).  ``delta``: a float32 tensor that may hold
     ``delta_splits`` split-K partials [splits, N, D], added in order; or a list of up to DELTA_MAX_TERMS terms
-    ``(data, splits, index, k, base)`` added in the order given: of the float32 partials ``data`` [splits, rows, D]
-    token r takes row ``base + r`` or, with ``index`` (int32 [N * k]), the k rows ``index[r * k + j]``.
+    ``(data, splits, index, k, base[, scale])`` added in the order given: of the float32 partials ``data`` [splits, rows, D]
+    token r takes row ``base + r`` or, with ``index`` (int32 [N * k]), the k rows ``index[r * k + j]``, times ``scale``.
+    ``places`` (int32 [N * copies]): the normed row n goes to the rows places[n * copies + j] of ``out`` instead of row n.
     With row_index, row n reads source row row_index[n] and x is not written back.  With w_router [E, D] the token
     is routed in the same kernel: topk_idx / topk_w [N, k].  ``dispatch`` (with w_router; an object with the tensors
     counter, offsets, sorted_pair, sorted_pos, a_sorted, status, the optional pair tiles = (tile_list, n_tiles) and
@@ -168,10 +170,14 @@ def add_rmsnorm(x: torch.Tensor, delta, gamma: torch.Tensor | None, eps: float,
         raise KernelError(f"add_rmsnorm: {len(terms)} terms to add; up to {DELTA_MAX_TERMS} are supported")
     spec = _DeltaSpec()
     spec.n = len(terms)
-    for q, (data, splits, index, k_rows, base) in enumerate(terms):
+    for q, (data, splits, index, k_rows, base, *scale) in enumerate(terms):
         sp, stride = _splits(data, splits)
         spec.t[q].p, spec.t[q].stride, spec.t[q].splits = data.data_ptr(), stride, sp
         spec.t[q].index, spec.t[q].k, spec.t[q].base = (index.data_ptr() if index is not None else None), k_rows, base
+        spec.t[q].scale = scale[0] if scale else 1.0
+    if places is not None and (places.dtype != torch.int32 or places.numel() != n * copies or out is None or out.numel() != n * copies * D):
+        raise KernelError(f"add_rmsnorm: {n} rows in {copies} places each need int32 places and an output of so many rows")
+    _contig(places)
     E = k = 0
     if w_router is not None:
         if w_router.dtype != torch.float32 or topk_idx is None or topk_w is None:
@@ -189,8 +195,16 @@ def add_rmsnorm(x: torch.Tensor, delta, gamma: torch.Tensor | None, eps: float,
     _run("elementwise", "jlx_add_rmsnorm", _ptr(x), ctypes.byref(spec) if terms else None, _ptr(gamma), c_float(eps),
          _ptr(out), c_int(code(out.dtype) if out is not None else F32), _ptr(out32), _ptr(row_index), c_int(n), c_int(D),
          _ptr(w_router), c_int(E), c_int(k), _ptr(topk_idx), _ptr(topk_w), ctypes.byref(dp) if dp is not None else None,
-         ctypes.byref(did), _stream())
+         ctypes.byref(did), _ptr(places), c_int(copies), _stream())
     return bool(did.value)
+
+
+def soft_cap(x: torch.Tensor, cap: float) -> None:
+    """x <- cap * tanh(x / cap), in place (float32)."""
+    _contig(x)
+    if x.dtype != torch.float32:
+        raise KernelError("soft_cap: float32 values are capped")
+    _run("elementwise", "jlx_soft_cap", _ptr(x), c_longlong(x.numel()), c_float(cap), _stream())
 
 
 SILU_GLU = (1.0, 0.0, 0.0)  # (alpha, limit, shift) of the gated activation: silu(gate) * up
@@ -697,7 +711,8 @@ def rope_norm_kv_store(proj: _RowsView, k_col: int, v_col: int, q_out: torch.Ten
                        q_norm_weight: torch.Tensor | None, k_norm_weight: torch.Tensor | None, eps: float,
                        inv_freq: torch.Tensor | None, rot_dims: int, Hq: int, Hkv: int, dk: int, dv: int, status: torch.Tensor,
                        pairing: str = "halves", norm: str = "before", amplitude: float = 1.0,
-                       q_head_scale: torch.Tensor | None = None, v_norm: bool = False) -> None:
+                       q_head_scale: torch.Tensor | None = None, v_norm: bool = False, bias: torch.Tensor | None = None,
+                       maps: int = 1) -> None:
     """From projected float32 rows (q heads from the view's first column, k heads from column k_col, v heads of dv
     entries from v_col; v_col = k_col stores the keys as projected as values): q and k RMS-normed over dk (``norm``:
     "none", "before" or "after" the rotation; with a weight where one is given), their first rot_dims entries rotated
@@ -705,7 +720,13 @@ def rope_norm_kv_store(proj: _RowsView, k_col: int, v_col: int, q_out: torch.Ten
     k and v into the token's cache row (pages [P, 2, Hkv, page_size, dpad]), all padded with zeros to dpad.
     ``norm`` "whole": before the rotation, over all heads of q (of k) at once, the weights [Hq dk] and [Hkv dk].
     ``amplitude`` multiplies both the cosine and the sine of every angle.  ``v_norm``: every value head is divided by its
-    root mean square over dv.  ``q_head_scale`` (float32 [Hq]): every query head is multiplied by its number, last."""
+    root mean square over dv.  ``q_head_scale`` (float32 [Hq]): every query head is multiplied by its number, last.
+    ``bias`` (float32, one number per projected column from the view's first one on) is added to the projected rows first.
+    ``maps`` 2: q and k heads are pairs of maps over one head's values: Hq query rows, Hkv value heads and 2 Hkv keys; a
+    cached key row holds both maps side by side, a query row its map's entries at that map's place (dpad >= 2 dk)."""
+    if bias is not None and (bias.dtype != torch.float32 or bias.numel() < v_col + Hkv * dv):
+        raise KernelError("rope_norm_kv_store: the bias must be float32 with a number for every projected column")
+    _contig(bias)
     if q_head_scale is not None and (q_head_scale.dtype != torch.float32 or q_head_scale.numel() != Hq):
         raise KernelError(f"rope_norm_kv_store: the queries' factors must be float32 [{Hq}]")
     _contig(q_head_scale)
@@ -721,7 +742,7 @@ def rope_norm_kv_store(proj: _RowsView, k_col: int, v_col: int, q_out: torch.Ten
          _ptr(positions), _ptr(q_norm_weight), _ptr(k_norm_weight), c_float(eps), _ptr(inv_freq), c_int(rot_dims),
          c_int(ROPE_PAIRINGS[pairing]), c_int(ROPE_NORMS[norm]), c_int(N), c_int(Hq), c_int(Hkv), c_int(dk), c_int(dv), c_int(dpad),
          c_int(pages.shape[3] if store else 0), c_int(pages.shape[0] if store else 0), c_int(int(store)), _ptr(status),
-         c_float(amplitude), _ptr(q_head_scale), c_int(int(v_norm)), _stream())
+         c_float(amplitude), _ptr(q_head_scale), c_int(int(v_norm)), _ptr(bias), c_int(maps), _stream())
 
 
 def rope_half_kv_store(proj: _RowsView, k_col: int, v_col: int, q_out: torch.Tensor, pages: torch.Tensor | None,
@@ -775,14 +796,46 @@ def kv_store(k: torch.Tensor, v: torch.Tensor, pages: torch.Tensor, block_table:
 
 
 # ---------------------------------------------------------------------------------- attention
+class MapDifference(ctypes.Structure):  # MapDifference in csrc/attention_maps.cuh
+    """Heads of two maps: query rows 2h and 2h + 1 are head h's maps; the attention kernels that take this write
+    o / sqrt(mean(o^2) + eps) * mult, o = a1 - weight * a2 over the head's ``out_dim`` values, at
+    out[n, h * out_dim + c] (``ld_out`` elements between tokens)."""
+
+    _fields_ = [("map_dim", c_int), ("out_dim", c_int), ("weight", c_float), ("mult", c_float), ("eps", c_float), ("pad_", c_int),
+                ("ld_out", c_longlong)]
+
+
+def map_difference_spec(map_dim: int, weight: float, mult: float, eps: float, out: torch.Tensor, heads: int) -> MapDifference:
+    """The difference written into ``out`` [N, heads * out_dim] (maybe a column range of wider rows)."""
+    if out.dim() != 2 or out.stride(1) != 1 or out.shape[1] % heads:
+        raise KernelError("the difference of two maps goes into rows [N, heads * values] of contiguous entries")
+    ld = out.stride(0) if out.shape[0] > 1 else out.shape[1]
+    return MapDifference(map_dim, out.shape[1] // heads, weight, mult, eps, 0, ld)
+
+
+def map_difference(attn: torch.Tensor, out: torch.Tensor, diff: MapDifference) -> None:
+    """The difference as a kernel of its own: attn float32 [N, 2 H, dpad] (``attention_generic`` with float32 output)."""
+    _contig(attn)
+    N, H2, dpad = attn.shape
+    if attn.dtype != torch.float32 or out.shape != (N, H2 // 2 * diff.out_dim):
+        raise KernelError("map_difference: float32 maps [N, 2 H, dpad] and rows [N, H * values]")
+    _run("attention_generic", "jlx_map_difference", _ptr(attn), _ptr(out), c_int(code(out.dtype)), ctypes.byref(diff), c_int(N), c_int(H2 // 2),
+         c_int(dpad), _stream())
+
+
+def _diff(diff: MapDifference | None):
+    return None if diff is None else ctypes.byref(diff)
+
+
 def attention_generic(q: torch.Tensor, pages: torch.Tensor, block_table: torch.Tensor, req_of_token: torch.Tensor,
                       positions: torch.Tensor, out: torch.Tensor, scale: float, chunk: int, window: int,
                       attn_scale: float, floor_scale: float, status: torch.Tensor, sink: torch.Tensor | None = None,
-                      slopes: torch.Tensor | None = None, softcap: float = 0.0) -> None:
-    """q: [N, Hq, dh]; pages: [P, 2, Hkv, page, dh]; out: [N, Hq, dh].  ``sink``: float32 [Hq] or None; with it the
+                      slopes: torch.Tensor | None = None, softcap: float = 0.0, keep: int = 0) -> None:
+    """q: [N, Hq, dh]; pages: [P, 2, Hkv, page, dh]; out: [N, Hq, dh] (float32 or bfloat16).  ``sink``: float32 [Hq] or None; with it the
     softmax's denominator has one more term exp(sink[h]) that carries no value.  ``slopes``: float32 [Hq] or None; with
     it slopes[h] * (query position - key position) is taken off every scaled score.  ``softcap`` > 0: a scaled score s
-    becomes softcap * tanh(s / softcap) first (all four attention kernels take all three)."""
+    becomes softcap * tanh(s / softcap) first.  ``keep``: the sequence's first so many keys are visible besides the window's
+    (all four attention kernels take all four; the other three also a ``diff``, see :class:`MapDifference`)."""
     _contig(q, pages, block_table, out)
     _check_sink(sink, q.shape[1])
     _check_sink(slopes, q.shape[1], "slopes")
@@ -791,8 +844,8 @@ def attention_generic(q: torch.Tensor, pages: torch.Tensor, block_table: torch.T
     if dh2 != dh or pages.dtype != q.dtype:
         raise KernelError("attention: cache pages and queries disagree in head size or element type")
     _run("attention_generic", "jlx_attention_generic", _ptr(q), _ptr(pages), c_int(code(q.dtype)), _ptr(block_table),
-         c_int(block_table.shape[1]), _ptr(req_of_token), _ptr(positions), _ptr(out), c_int(N), c_int(Hq), c_int(Hkv),
-         c_int(dh), c_int(page_size), c_int(P), c_float(scale), c_int(chunk), c_int(window), c_float(attn_scale),
+         c_int(block_table.shape[1]), _ptr(req_of_token), _ptr(positions), _ptr(out), c_int(code(out.dtype)), c_int(N), c_int(Hq), c_int(Hkv),
+         c_int(dh), c_int(page_size), c_int(P), c_float(scale), c_int(chunk), c_int(window), c_int(keep), c_float(attn_scale),
          c_float(floor_scale), _ptr(sink), _ptr(slopes), c_float(softcap), _ptr(status), _stream())
 
 
@@ -818,12 +871,13 @@ def attention_decode(q: torch.Tensor, pages: torch.Tensor, block_table: torch.Te
                      positions: torch.Tensor, out: torch.Tensor, scale: float, chunk: int, window: int, attn_scale: float,
                      floor_scale: float, part_o: torch.Tensor, part_ml: torch.Tensor, max_splits: int, split_keys: int,
                      status: torch.Tensor, rows: torch.Tensor | None = None, n_rows: int = 0,
-                     sink: torch.Tensor | None = None, slopes: torch.Tensor | None = None, softcap: float = 0.0) -> None:
+                     sink: torch.Tensor | None = None, slopes: torch.Tensor | None = None, softcap: float = 0.0, keep: int = 0,
+                     diff: MapDifference | None = None) -> None:
     """Split-KV attention for one query token per request (tensor cores, bfloat16).
     part_o: float32 [N * Hq * max_splits * dh]; part_ml: float32 [N * Hq * max_splits * 2].
     rows / n_rows: work on these token rows only (int32, the first n_rows entries): the single decoded tokens of
     a step that also holds prompt portions; N is then n_rows."""
-    _contig(q, pages, block_table, out, part_o, part_ml, rows)
+    _contig(q, pages, block_table, out if diff is None else None, part_o, part_ml, rows)
     N, Hq, dh = q.shape
     _check_sink(sink, Hq)
     _check_sink(slopes, Hq, "slopes")
@@ -836,16 +890,17 @@ def attention_decode(q: torch.Tensor, pages: torch.Tensor, block_table: torch.Te
          _ptr(req_of_token), _ptr(positions), _ptr(out), c_int(N), c_int(Hq), c_int(Hkv), c_int(dh), c_int(page_size),
          c_int(P), c_float(scale), c_int(chunk), c_int(window), c_float(attn_scale), c_float(floor_scale), _ptr(part_o),
          _ptr(part_ml), c_int(max_splits), c_int(split_keys), _ptr(rows), _ptr(sink), _ptr(slopes),
-         c_float(softcap), _ptr(status), _stream())
+         c_float(softcap), c_int(keep), _diff(diff), _ptr(status), _stream())
 
 
 def attention_prefill(q: torch.Tensor, pages: torch.Tensor, block_table: torch.Tensor, req_of_token: torch.Tensor,
                       positions: torch.Tensor, out: torch.Tensor, tiles: torch.Tensor, n_tiles: int, scale: float,
                       chunk: int, window: int, attn_scale: float, floor_scale: float, status: torch.Tensor,
-                      sink: torch.Tensor | None = None, slopes: torch.Tensor | None = None, softcap: float = 0.0) -> None:
+                      sink: torch.Tensor | None = None, slopes: torch.Tensor | None = None, softcap: float = 0.0, keep: int = 0,
+                     diff: MapDifference | None = None) -> None:
     """Flash attention over the paged cache for prompt portions (tensor cores, bfloat16).
     tiles: int32 [n_tiles, 2] = (first token row, count <= 16), each within one request."""
-    _contig(q, pages, block_table, out, tiles)
+    _contig(q, pages, block_table, out if diff is None else None, tiles)
     N, Hq, dh = q.shape
     _check_sink(sink, Hq)
     _check_sink(slopes, Hq, "slopes")
@@ -853,7 +908,7 @@ def attention_prefill(q: torch.Tensor, pages: torch.Tensor, block_table: torch.T
     _run("attention_mma", "jlx_attention_prefill", _ptr(q), _ptr(pages), _ptr(block_table), c_int(block_table.shape[1]),
          _ptr(req_of_token), _ptr(positions), _ptr(out), _ptr(tiles), c_int(n_tiles), c_int(Hq), c_int(Hkv), c_int(dh),
          c_int(page_size), c_int(P), c_float(scale), c_int(chunk), c_int(window), c_float(attn_scale),
-         c_float(floor_scale), _ptr(sink), _ptr(slopes), c_float(softcap), _ptr(status), _stream())
+         c_float(floor_scale), _ptr(sink), _ptr(slopes), c_float(softcap), c_int(keep), _diff(diff), _ptr(status), _stream())
 
 
 def attention_prefill_tc_supported(q_dtype: torch.dtype, Hq: int, Hkv: int, dh: int, page_size: int) -> bool:
@@ -865,11 +920,12 @@ def attention_prefill_tc_supported(q_dtype: torch.dtype, Hq: int, Hkv: int, dh: 
 def attention_prefill_tc(q: torch.Tensor, pages: torch.Tensor, block_table: torch.Tensor, req_of_token: torch.Tensor,
                          positions: torch.Tensor, out: torch.Tensor, tiles: torch.Tensor, n_tiles: int, scale: float,
                          chunk: int, window: int, attn_scale: float, floor_scale: float, status: torch.Tensor,
-                         sink: torch.Tensor | None = None, slopes: torch.Tensor | None = None, softcap: float = 0.0) -> None:
+                         sink: torch.Tensor | None = None, slopes: torch.Tensor | None = None, softcap: float = 0.0, keep: int = 0,
+                     diff: MapDifference | None = None) -> None:
     """Flash attention for prompt portions on tcgen05 (bfloat16, head size 128, pages of a multiple of 64).
     tiles: int32 [n_tiles, 2] = (first token row, count <= 128), each within one request; only the rows
     of these tiles are written."""
-    _contig(q, pages, block_table, out, tiles)
+    _contig(q, pages, block_table, out if diff is None else None, tiles)
     N, Hq, dh = q.shape
     _check_sink(sink, Hq)
     _check_sink(slopes, Hq, "slopes")
@@ -877,7 +933,7 @@ def attention_prefill_tc(q: torch.Tensor, pages: torch.Tensor, block_table: torc
     _run("attention_tc", "jlx_attention_prefill_tc", _ptr(q), _ptr(pages), _ptr(block_table), c_int(block_table.shape[1]),
          _ptr(req_of_token), _ptr(positions), _ptr(out), _ptr(tiles), c_int(n_tiles), c_int(N), c_int(Hq), c_int(Hkv),
          c_int(dh), c_int(page_size), c_int(P), c_float(scale), c_int(chunk), c_int(window), c_float(attn_scale),
-         c_float(floor_scale), _ptr(sink), _ptr(slopes), c_float(softcap), _ptr(status), _stream())
+         c_float(floor_scale), _ptr(sink), _ptr(slopes), c_float(softcap), c_int(keep), _diff(diff), _ptr(status), _stream())
 
 
 # ------------------------------------------------------------------------------------- GEMMs
@@ -979,23 +1035,39 @@ def router(h32: torch.Tensor, w_router: torch.Tensor, topk_idx: torch.Tensor, to
          c_int(int(weight_form == "softmax_normalized" if normalize is None else normalize)), _stream())
 
 
-def expert_sort(topk_idx: torch.Tensor, offsets: torch.Tensor, sorted_pair: torch.Tensor, sorted_pos: torch.Tensor,
+class _TableChoice(ctypes.Structure):  # TableChoice in csrc/moe.cu
+    _fields_ = [("ids", c_void_p), ("table", c_void_p), ("chosen", c_void_p), ("V", c_int), ("k", c_int)]
+
+
+def expert_sort(topk_idx: torch.Tensor | None, offsets: torch.Tensor, sorted_pair: torch.Tensor, sorted_pos: torch.Tensor,
                 E: int, status: torch.Tensor, extra_rows: int = 0, tile_rows: int = 0,
-                tile_list: torch.Tensor | None = None, n_tiles: torch.Tensor | None = None, tile_groups: int = 0) -> None:
+                tile_list: torch.Tensor | None = None, n_tiles: torch.Tensor | None = None, tile_groups: int = 0,
+                token_ids: torch.Tensor | None = None, table: torch.Tensor | None = None) -> None:
     """Counting sort of the (token, choice) pairs by expert.  offsets: [E + 1], or [E + 2] with extra_rows > 0:
     one more group of that many rows appended after the experts.  With tile_rows > 0 also the list of row
     tiles of that height that hold rows: tile_list int32 [(ceil(rows / tile_rows) + groups) * 2], n_tiles [1];
-    ``tile_groups`` > 0: tiles of the first so many groups only (the later ones are experts without weights)."""
-    _contig(topk_idx, offsets, sorted_pair, sorted_pos, tile_list, n_tiles)
+    ``tile_groups`` > 0: tiles of the first so many groups only (the later ones are experts without weights).
+    ``token_ids`` (int32 [N]) and ``table`` (int32 [V, k]): the choices are the table's rows of the step's tokens
+    (``topk_idx`` gets them if it is given)."""
+    _contig(topk_idx, offsets, sorted_pair, sorted_pos, tile_list, n_tiles, token_ids, table)
+    pairs = sorted_pair.numel()
+    by = None
+    if table is not None:
+        if table.dtype != torch.int32 or token_ids is None or token_ids.dtype != torch.int32 or token_ids.numel() * table.shape[1] != pairs \
+                or (topk_idx is not None and topk_idx.numel() != pairs):
+            raise KernelError("expert_sort: a table of choices is int32 [V, k], for int32 token ids, with places for every pair")
+        by = _TableChoice(token_ids.data_ptr(), table.data_ptr(), None if topk_idx is None else topk_idx.data_ptr(), table.shape[0], table.shape[1])
+    elif topk_idx is None or topk_idx.numel() != pairs:
+        raise KernelError("expert_sort: no choices to sort, or places for another number of pairs")
     if offsets.numel() < E + 1 + (extra_rows > 0):
         raise KernelError("expert_sort: offsets too short")
     if tile_rows > 0:
-        rows, groups = topk_idx.numel() + extra_rows, E + (extra_rows > 0)
+        rows, groups = pairs + extra_rows, E + (extra_rows > 0)
         if tile_list is None or n_tiles is None or tile_list.numel() < 2 * (-(-rows // tile_rows) + groups):
             raise KernelError("expert_sort: tile list too short")
     _run("moe", "jlx_expert_sort", _ptr(topk_idx), _ptr(offsets), _ptr(sorted_pair), _ptr(sorted_pos),
-         c_int(topk_idx.numel()), c_int(E), c_int(extra_rows), c_int(tile_rows), _ptr(tile_list), _ptr(n_tiles),
-         _ptr(status), c_int(tile_groups), _stream())
+         c_int(pairs), c_int(E), c_int(extra_rows), c_int(tile_rows), _ptr(tile_list), _ptr(n_tiles),
+         _ptr(status), c_int(tile_groups), None if by is None else ctypes.byref(by), _stream())
 
 
 def permute_scale(h32: torch.Tensor, sorted_pair: torch.Tensor, topk_w: torch.Tensor | None, a_sorted: torch.Tensor, k: int,

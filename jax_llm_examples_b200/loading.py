@@ -16,7 +16,7 @@ from .config.base import load_config_json
 from .config.registry import resolve
 from .parts.base import Runtime
 from .parts.decoder import DecoderModel
-from .weights.loader import check_tensors, load_tensors
+from .weights.loader import check_tensors, keep_precision, load_tensors
 from .weights.random_init import random_tensor
 
 _DTYPES = {"bfloat16": torch.bfloat16, "bf16": torch.bfloat16, "float32": torch.float32, "fp32": torch.float32,
@@ -93,6 +93,5 @@ def model_from_tensors(config_json: Mapping[str, Any], tensors: Mapping[str, tor
     arch = resolve(config_json)
     cfg = arch.parse_config(config_json)
     check_tensors(tensors, arch.tensor_specs(cfg))
-    conv = {n: (t.to(torch.float32) if dt == torch.float32 or t.dtype == torch.float32 else t.to(torch.bfloat16)).to(device)
-            for n, t in tensors.items()}
+    conv = {n: keep_precision(t, dt).to(device) for n, t in tensors.items()}
     return _built(arch.build(cfg, conv, Runtime(dt, torch.device(device))))

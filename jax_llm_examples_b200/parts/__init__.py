@@ -1,11 +1,11 @@
-from .attention import GatedPagedAttention, PagedAttention, plan_attention_tiles
-from .base import (Block, FeedForward, KVNeed, LayerCache, Mixer, Norm, Part, PositionEncoding, PostNormed, ProjectedMixer, Rows, RowSum, Runtime, Scaled, StateNeed,
+from .attention import DifferentialAttention, GatedPagedAttention, PagedAttention, plan_attention_tiles
+from .base import (Block, FeedForward, KVNeed, LayerCache, Mixer, Norm, Part, PositionEncoding, PostNormed, ProjectedMixer, RowPlaces, Rows, RowSum, Runtime, Scaled, StateNeed,
                    StepContext, StepShape, Workspace, as_rows, known_parts, make_part, register_part)
 from .block import EmbeddingReentryBlock, HyperConnectionBlock, PostNormBlock, PreNormBlock, ReinjectionBlock, SandwichNormBlock, ScaledPreNormBlock
 from .conv import ResidualShortConv
 from .decoder import CachePlan, DecoderModel, LayerRun
 from .delta_rule import GatedDeltaRule
-from .feedforward import DenseBiasedMLP, DenseSwiGLU, GroupLimitedGLUExperts, RoutedExperts, RoutedMLPExperts, SoftmaxRoutedMLPExperts
+from .feedforward import DenseBiasedMLP, DenseSwiGLU, GroupLimitedGLUExperts, RoutedExperts, RoutedMLPExperts, SoftmaxRoutedMLPExperts, TableRoutedGLUExperts
 from .latent_attention import LatentAttention, rotary_frequencies
 from .linear_attention import GatedLinearAttention, RetentionMixer, TimeMixWKV
 from .linear import grouped_linear, grouped_swiglu_linear, interleave_gate_up, linear, swiglu_linear
@@ -16,6 +16,7 @@ from .positions import (InterleavedRope, NoPositionWithTemperature, UnfusedEncod
                         wavelength_scaled_frequencies, yarn_frequencies)
 
 __all__ = [
+    "DifferentialAttention", "RowPlaces", "TableRoutedGLUExperts",
     "EmbeddingReentryBlock", "GatedDeltaRule", "wavelength_scaled_frequencies", "yarn_frequencies", "HyperConnectionBlock",
     "GroupLimitedGLUExperts", "PostNormBlock", "RetentionMixer", "RoutedMLPExperts", "StreamRMSNorm",
     "GatedLinearAttention", "GatedPagedAttention", "ParallelMixers", "ProjectedMixer", "Scaled", "ScaledPreNormBlock",

@@ -77,6 +77,7 @@ class PagedAttention(Mixer):
 
     sink: torch.Tensor | None = None
     softcap: float = 0.0  # > 0: a scaled score s becomes softcap * tanh(s / softcap)
+    keep_first: int = 0  # > 0, with a window: the sequence's first so many keys stay visible besides the window's
     slopes: torch.Tensor | None = None  # [Hq]: slopes[h] * (query position - key position) is taken off the scaled scores
 
     @staticmethod
@@ -107,7 +108,7 @@ class PagedAttention(Mixer):
         if self.chunk is not None and self.window is None:
             keep = Retention.chunk(self.chunk)
         elif self.window is not None and self.chunk is None:
-            keep = Retention.window(self.window)
+            keep = Retention.window(self.window, self.keep_first)
         else:
             keep = Retention.all()  # both limits at once: keep everything (correct, not minimal)
         return KVNeed(self.n_kv_heads, self.head_dim, keep)
@@ -125,7 +126,7 @@ class PagedAttention(Mixer):
         with scope("projection"):
             return linear(ctx, out.view(q.shape[0], -1), self.w_o, torch.float32, partials=True)
 
-    def _split_kv(self, ctx: StepContext, q, cache: LayerCache, out, attn_scale, floor_scale, rows, n_rows: int) -> None:
+    def _split_kv(self, ctx: StepContext, q, cache: LayerCache, out, attn_scale, floor_scale, rows, n_rows: int, diff=None) -> None:
         """Split-KV attention for requests that bring one token: all rows of q, or the listed ones."""
         chunk, window = self.chunk or 0, self.window or 0
         split_keys, splits = K.attention_decode_plan(ctx.max_kv_len, chunk, window, n_rows * self.n_kv_heads)
@@ -134,18 +135,19 @@ class PagedAttention(Mixer):
         part_ml = ctx.workspace.get("attn_part_ml", n * 2, torch.float32)
         K.attention_decode(q, cache.pages, cache.block_table, ctx.req_of_token, ctx.positions, out, self.scale,
                            chunk, window, attn_scale, floor_scale, part_o, part_ml, splits, split_keys, ctx.status,
-                           rows, n_rows, self.sink, self.slopes, self.softcap)
+                           rows, n_rows, self.sink, self.slopes, self.softcap, self.keep_first, diff)
 
-    def attend(self, ctx: StepContext, q, cache: LayerCache, out, attn_scale: float, floor_scale: float) -> None:
-        """Tensor-core kernels where they are built (bfloat16, head size 64 or 128, small groups): split-KV for
+    def attend(self, ctx: StepContext, q, cache: LayerCache, out, attn_scale: float, floor_scale: float, diff=None) -> None:
+        """Tensor-core kernels where they are built (bfloat16, head size 64 or 128): split-KV for
         requests that bring one token, flash tiles for the others (tcgen05 for long portions of head size 128);
-        the generic kernel where those are not built."""
+        the generic kernel where those are not built.  ``diff`` (``K.MapDifference``): query rows are pairs of maps and
+        ``out`` gets the heads' differences, which the tensor-core kernels take in their last lines."""
         chunk, window = self.chunk or 0, self.window or 0
         decode = ctx.max_q_len == 1
         if self.head_dim in self.MMA_HEAD_SIZES and K.attention_mma_supported(q.dtype, self.n_heads, self.n_kv_heads,
                                                                               self.head_dim, decode):
             if decode:
-                self._split_kv(ctx, q, cache, out, attn_scale, floor_scale, None, q.shape[0])
+                self._split_kv(ctx, q, cache, out, attn_scale, floor_scale, None, q.shape[0], diff)
                 return
             tiles_all = ctx.arrays.get("attn_tiles_all")
             if tiles_all is not None:
@@ -153,24 +155,28 @@ class PagedAttention(Mixer):
                 if count["attn_single_rows"]:
                     # the single decoded tokens of a mixed step go to the split-KV kernel, by their row list
                     self._split_kv(ctx, q, cache, out, attn_scale, floor_scale, ctx.arrays["attn_single_rows"],
-                                   count["attn_single_rows"])
+                                   count["attn_single_rows"], diff)
                 tiles, n_tiles = tiles_all, count["attn_tiles_all"]  # every request that brings more than one token
                 if count["attn_tiles_long"] and self.head_dim in self.TC_HEAD_SIZES and K.attention_prefill_tc_supported(
                         q.dtype, self.n_heads, self.n_kv_heads, self.head_dim, cache.pages.shape[3]):
                     # long portions on the tcgen05 kernel (128-token tiles), the short ones below
                     K.attention_prefill_tc(q, cache.pages, cache.block_table, ctx.req_of_token, ctx.positions, out,
                                            ctx.arrays["attn_tiles_long"], count["attn_tiles_long"], self.scale, chunk, window,
-                                           attn_scale, floor_scale, ctx.status, self.sink, self.slopes, self.softcap)
+                                           attn_scale, floor_scale, ctx.status, self.sink, self.slopes, self.softcap, self.keep_first, diff)
                     tiles, n_tiles = ctx.arrays["attn_tiles_short"], count["attn_tiles_short"]
                     kinds = ("tc", "flash" if n_tiles else "", "split_kv" if count["attn_single_rows"] else "")
                     ctx.scratch.setdefault("attention_kernels", set()).add(tuple(k for k in kinds if k))
                 if n_tiles:
                     K.attention_prefill(q, cache.pages, cache.block_table, ctx.req_of_token, ctx.positions, out, tiles,
                                         n_tiles, self.scale, chunk, window, attn_scale, floor_scale, ctx.status, self.sink, self.slopes,
-                                        self.softcap)
+                                        self.softcap, self.keep_first, diff)
                 return
-        K.attention_generic(q, cache.pages, cache.block_table, ctx.req_of_token, ctx.positions, out, self.scale,
-                            self.chunk or 0, self.window or 0, attn_scale, floor_scale, ctx.status, self.sink, self.slopes, self.softcap)
+        maps = out if diff is None else torch.empty(q.shape, dtype=torch.float32, device=q.device)
+        K.attention_generic(q, cache.pages, cache.block_table, ctx.req_of_token, ctx.positions, maps, self.scale,
+                            self.chunk or 0, self.window or 0, attn_scale, floor_scale, ctx.status, self.sink, self.slopes, self.softcap,
+                            self.keep_first)
+        if diff is not None:
+            K.map_difference(maps, out, diff)
 
 
 register_part("mixer", "paged_attention", PagedAttention)
@@ -198,8 +204,9 @@ class GatedPagedAttention(ProjectedMixer, PagedAttention):
     rounded).  ``softcap``: a scaled score s becomes softcap * tanh(s / softcap), before a bias and the sink.
     ``value_norm``: every value head is divided by its root mean square (no weight) before it is cached.
     ``keep_window``: pages are kept for a window of at least this many positions (a layer with a longer window
-    reads them; 0: for good).  ``window``: a query
-    sees itself and the window - 1 positions before it; ``chunk``: the positions of its own chunk.  Keys, queries and
+    reads them; 0: for good).  ``in_bias`` (one number per row of ``w_in``, gate rows excepted): added to the projected
+    rows.  ``window``: a query
+    sees itself and the window - 1 positions before it, with ``keep_first`` also the sequence's first so many; ``chunk``: the positions of its own chunk.  Keys, queries and
     values are kept at one padded size (``padded_dim`` >= max(dk, dv), zeros beyond their own): one page layout, and the
     attention kernels built for equal sizes, serve both.  It is a :class:`ProjectedMixer`: beside another mixer that
     reads the same input, both share their input and output products."""
@@ -214,7 +221,7 @@ class GatedPagedAttention(ProjectedMixer, PagedAttention):
                  norm: str | None = None, values_are_keys: bool = False, gate: str | None = None,
                  rot_amplitude: float = 1.0, slopes: torch.Tensor | None = None, query_temperature: tuple[float, float] | None = None,
                  projects_kv: bool = True, keep_window: int | None = None, head_temperature: torch.Tensor | None = None,
-                 softcap: float | None = None, value_norm: bool = False):
+                 softcap: float | None = None, value_norm: bool = False, keep_first: int = 0, in_bias: torch.Tensor | None = None):
         if n_heads % n_kv_heads:
             raise ValueError(f"{n_heads} query heads are no multiple of {n_kv_heads} KV heads")
         gate = ("head" if gated else "none") if gate is None else gate
@@ -266,12 +273,21 @@ class GatedPagedAttention(ProjectedMixer, PagedAttention):
         if self.softcap < 0:
             raise ValueError("the score cap must be positive")
         self.position, self.qk_norm_eps = None, None
+        self.keep_first, self.in_bias = self._kept_keys(keep_first, window, chunk), f32(in_bias)
+        if in_bias is not None and in_bias.numel() != n_heads * head_dim + kv_rows:
+            raise ValueError(f"the projections' bias has {in_bias.numel()} entries for {n_heads * head_dim + kv_rows} rows")
+
+    @staticmethod
+    def _kept_keys(keep_first: int, window: int | None, chunk: int | None) -> int:
+        if keep_first < 0 or (keep_first and chunk is not None):
+            raise ValueError(f"{keep_first} kept first keys: a window can keep them, not a chunk")
+        return int(keep_first) if window is not None else 0  # without a window every key is visible anyway
 
     def kv_need(self) -> KVNeed:
         need = PagedAttention.kv_need(self)
         if self.keep_window is not None and self.window is not None and self.chunk is None:
             # another layer reads these pages through a longer window (0: without one): keep them that long
-            keep = Retention.all() if self.keep_window == 0 else Retention.window(max(self.window, self.keep_window))
+            keep = Retention.all() if self.keep_window == 0 else Retention.window(max(self.window, self.keep_window), self.keep_first)
             need = KVNeed(need.num_kv_heads, need.head_dim, keep)
         return need
 
@@ -303,7 +319,7 @@ class GatedPagedAttention(ProjectedMixer, PagedAttention):
                                  cache.pages if cache.writes else None, cache.block_table if cache.writes else None,
                                  ctx.req_of_token, ctx.positions, self.q_norm_weight, self.k_norm_weight, self.eps,
                                  self.inv_freq, self.rot_dims, Hq, Hkv, dk, dv, ctx.status, self.pairing, self.norm,
-                                 self.rot_amplitude, self.head_temperature, self.value_norm)
+                                 self.rot_amplitude, self.head_temperature, self.value_norm, self.in_bias)
         attn = torch.empty_like(q)
         with scope("attention"):
             self.attend(ctx, q, cache, attn, *self.q_temperature)
@@ -333,3 +349,82 @@ class GatedPagedAttention(ProjectedMixer, PagedAttention):
 
 
 register_part("mixer", "gated_paged_attention", GatedPagedAttention)
+
+
+class DifferentialAttention(ProjectedMixer, PagedAttention):
+    """Attention whose every head is the difference of two maps over the same values (grouped queries; key/value head g serves
+    the query heads g H/G .. (g + 1) H/G - 1):
+
+        a_m = softmax(scale * rot(q_m) rot(k_m)^T) v,  m = 1, 2;   o = a_1 - map_weight * a_2;
+        out = W_o [ (1 - diff) * o / sqrt(mean(o^2) + eps)  for every head ].
+
+    ``w_in``: q (head by head [map 1, map 2], 2 H dk rows), k (the same, 2 G dk) and v (G dv) stacked, ``in_bias``: a number per
+    row of it or None.  The first ``rot_dims`` entries of every map turn by the position ("halves": entry i with i +
+    rot_dims / 2), cosine and sine times ``rot_amplitude``.  ``map_weight``: one number for the layer (:func:`map_weight_of`
+    makes it from its vectors).  ``window`` / ``keep_first``: a query sees itself and the window - 1 positions before it, and
+    the sequence's first ``keep_first``.
+
+    One cached key row per key/value head holds both maps' keys side by side, its value row the head's values, both padded
+    to one size; a map's query is zero outside its own part.  The two maps are so two query rows of a plain grouped
+    attention over one copy of keys and values, and every attention kernel serves them; the tensor-core kernels take the
+    difference, its norm and the store in their own last lines, from 32-bit sums."""
+
+    kernel_libraries = ("attention_generic", "gemm_simt", "rope_kv")
+    kernel_libraries_bf16 = ("attention_mma", "attention_tc", "gemm_stream")
+
+    def __init__(self, w_in: torch.Tensor, w_o: torch.Tensor, heads: int, kv_heads: int, dim: int, value_dim: int, scale: float, eps: float,
+                 map_weight: float, diff: float, in_bias: torch.Tensor | None = None, inv_freq: torch.Tensor | None = None, rot_dims: int = 0,
+                 rot_amplitude: float = 1.0, window: int | None = None, keep_first: int = 0, padded_dim: int | None = None):
+        if heads % kv_heads:
+            raise ValueError(f"{heads} query heads are no multiple of {kv_heads} KV heads")
+        rows = 2 * heads * dim + 2 * kv_heads * dim + kv_heads * value_dim
+        if w_in.shape[0] != rows or w_o.shape[1] != heads * value_dim or w_o.shape[0] != w_in.shape[1]:
+            raise ValueError(f"attention weights do not fit: w_in {tuple(w_in.shape)}, w_o {tuple(w_o.shape)} for {heads}/{kv_heads} heads of two "
+                             f"maps of {dim} (values {value_dim})")
+        if in_bias is not None and in_bias.numel() != rows:
+            raise ValueError(f"the projections' bias has {in_bias.numel()} entries for {rows} rows")
+        if rot_dims % 2 or not 0 <= rot_dims <= dim or (rot_dims and (inv_freq is None or inv_freq.numel() != rot_dims // 2)):
+            raise ValueError(f"{rot_dims} rotated entries of {dim} need {rot_dims // 2} frequencies")
+        f32 = lambda t: None if t is None else t.to(torch.float32).contiguous()  # noqa: E731
+        self.w_in, self.w_o, self.in_bias, self.inv_freq = w_in, w_o, f32(in_bias), f32(inv_freq)
+        self.heads, self.map_dim, self.value_dim = heads, dim, value_dim
+        self.n_heads, self.n_kv_heads = 2 * heads, kv_heads  # what the attention kernels see: a query row per map
+        self.head_dim = max(2 * dim, value_dim) if padded_dim is None else int(padded_dim)
+        if self.head_dim < max(2 * dim, value_dim):
+            raise ValueError(f"padded size {self.head_dim} is below that of two maps' keys or of the values")
+        self.rot_dims, self.rot_amplitude, self.scale, self.eps = int(rot_dims), float(rot_amplitude), float(scale), float(eps)
+        self.map_weight, self.diff = float(map_weight), float(diff)
+        self.chunk, self.window = None, window
+        self.keep_first = GatedPagedAttention._kept_keys(keep_first, window, None)
+        self.position, self.qk_norm_eps = None, None
+
+    @staticmethod
+    def map_weight_of(q1: torch.Tensor, k1: torch.Tensor, q2: torch.Tensor, k2: torch.Tensor, diff: float) -> float:
+        """exp(q1 . k1) - exp(q2 . k2) + diff: what the second map counts for."""
+        dot = lambda a, b: torch.exp((a.to(torch.float64) * b.to(torch.float64)).sum())  # noqa: E731
+        return float(dot(q1, k1) - dot(q2, k2)) + float(diff)
+
+    @staticmethod
+    def padded_size(dim: int, value_dim: int, dtype: torch.dtype) -> int:
+        return GatedPagedAttention.padded_size(2 * dim, value_dim, dtype)
+
+    def sub_parts(self):
+        return ()
+
+    def core(self, ctx: StepContext, h, proj: Rows, col: int, cache: LayerCache, out: torch.Tensor, mult: float) -> None:
+        if not cache.writes:
+            raise RuntimeError("an attention layer with key and value projections was scheduled to read another layer's cache")
+        n, dk = proj.data.shape[-2], self.map_dim
+        k_col = self.n_heads * dk
+        v_col = k_col + 2 * self.n_kv_heads * dk
+        q = torch.empty((n, self.n_heads, self.head_dim), dtype=ctx.runtime.dtype, device=proj.data.device)
+        with scope("rope"):
+            K.rope_norm_kv_store(K.rows_view(proj.data, proj.splits, col), k_col, v_col, q, cache.pages, cache.block_table, ctx.req_of_token,
+                                 ctx.positions, None, None, self.eps, self.inv_freq, self.rot_dims, self.n_heads, self.n_kv_heads, dk,
+                                 self.value_dim, ctx.status, "halves", "none", self.rot_amplitude, bias=self.in_bias, maps=2)
+        with scope("attention"):
+            diff = K.map_difference_spec(dk, self.map_weight, (1.0 - self.diff) * mult, self.eps, out, self.heads)
+            self.attend(ctx, q, cache, out, 0.0, 1.0, diff)
+
+
+register_part("mixer", "differential_attention", DifferentialAttention)

@@ -65,7 +65,7 @@ class Rows:
 
     As a term of a :class:`RowSum` the rows may also lie elsewhere in ``data``: token r's row is ``base + r``, or,
     with ``index`` (int32 [N * k]), the sum of the k rows ``index[r * k + j]``, j ascending, each times
-    ``weights[r, j]`` (float32 [N, k]) if there are weights."""
+    ``weights[r, j]`` (float32 [N, k]) if there are weights, all of them times the number ``scale``."""
 
     data: torch.Tensor
     splits: int = 1
@@ -73,6 +73,7 @@ class Rows:
     k: int = 1
     base: int = 0
     weights: torch.Tensor | None = None
+    scale: float = 1.0
 
 
 @dataclasses.dataclass
@@ -266,6 +267,8 @@ class Part:
 
     kernel_libraries: tuple[str, ...] = ()
     kernel_libraries_bf16: tuple[str, ...] = ()
+    # True: the part has work that needs only the step's tokens: ``begin_step(ctx)`` is called before the first block runs.
+    begins_steps: bool = False
     # False: forward() reads the step's host copies (``ctx.host_*``) or otherwise does work that a captured
     # CUDA graph would freeze; a model with such a part is never replayed from a graph.
     capturable: bool = True
@@ -284,6 +287,11 @@ class Part:
         function (parts of the same kind share it, so it runs once however many layers use it) and must return
         the same names with the same sizes for steps of the same shape when it wants to be replayed from a graph."""
         return ()
+
+    def begin_step(self, ctx: "StepContext") -> None:
+        """Work of a step that needs nothing but its description (token ids, positions), called once per step and part
+        before the first block, if ``begins_steps``: a part may put it on the second stream, beside the first layers, and
+        leave what it made in ``ctx.scratch``."""
 
     def sub_parts(self) -> "tuple[Part, ...]":
         """Parts inside this one (a block's norms, mixer and feed-forward; an attention's position encoding)."""
@@ -332,8 +340,17 @@ class CorrectedRouter:
     dispatch: Callable[["StepContext", int], Dispatch]
 
 
+@dataclasses.dataclass
+class RowPlaces:
+    """Where a feed-forward wants its input rows: row n at the rows ``index[n * copies + j]`` of [N * copies, D] (int32)."""
+
+    index: torch.Tensor
+    copies: int
+
+
 class Norm(Part):
     fuses_router: bool = False  # True: forward(router=...) also routes the tokens in its kernel
+    places_rows: bool = False  # True: forward(places=RowPlaces) writes its rounded rows where they are wanted
 
     def forward(self, ctx: StepContext, x: torch.Tensor, delta: "torch.Tensor | Rows | None", *, out_dtype: torch.dtype,
                 want_f32: bool = False, row_index: torch.Tensor | None = None, router=None):
@@ -421,6 +438,11 @@ class FeedForward(Part):
     def router_request(self):
         """(w_router, top_k) if the preceding norm may route the tokens for this part, else None; optionally a third
         element, see Norm.forward."""
+        return None
+
+    def row_places(self, ctx: StepContext, n: int) -> "RowPlaces | None":
+        """Where this part wants the preceding norm to write its n rows, if it knows that before it sees them and the
+        norm can (``Norm.places_rows``); forward() then gets rows in that order, no ``h32``, and the places as ``routing``."""
         return None
 
     def corrected_router(self) -> "CorrectedRouter | None":

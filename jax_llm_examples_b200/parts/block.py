@@ -31,6 +31,13 @@ class PreNormBlock(Block):
         if self.feed_forward is None:
             return a
         want32 = self.feed_forward.needs_f32_input
+        if self.norm2.places_rows:
+            places = self.feed_forward.row_places(ctx, x.shape[0])
+            if places is not None:  # the experts are known before the row is: the norm writes it where they read it
+                with scope("attn_post_norm"):
+                    h = self.norm2.forward(ctx, x, a, out_dtype=dt, places=places)[0]
+                with scope("ffn"):
+                    return self.feed_forward.forward(ctx, h, None, places)
         router = self.feed_forward.router_request() if self.norm2.fuses_router else None
         with scope("attn_post_norm"):
             h, h32, routing = self.norm2.forward(ctx, x, a, out_dtype=dt, want_f32=want32, router=router)
@@ -153,7 +160,8 @@ class PostNormBlock(Block):
     def _closing(norm: Norm, y, bias=None):
         from .base import PostNormed, RowSum, as_rows
 
-        if isinstance(y, RowSum) and len(y.terms) == 1 and y.terms[0].base == 0 and y.terms[0].data.dtype == torch.float32:
+        if isinstance(y, RowSum) and len(y.terms) == 1 and y.terms[0].base == 0 and y.terms[0].scale == 1.0 \
+                and y.terms[0].data.dtype == torch.float32:
             rows = y.terms[0]
         else:
             rows = as_rows(y)

@@ -42,13 +42,16 @@ class DecoderModel:
 
     def __init__(self, runtime: Runtime, embedding: torch.Tensor, blocks: list[Block], final_norm: Norm,
                  lm_head: torch.Tensor, schedule: list[LayerRun] | None = None, config=None, embedding_scale: float = 1.0,
-                 residual_streams: int | None = None):
+                 residual_streams: int | None = None, logit_softcap: float | None = None):
         self.runtime, self.embedding, self.blocks = runtime, embedding, blocks
         # None: one residual row per token.  A number S: every token carries S rows (x is [N, S * D]), all equal to
         # the embedding's output at the start; the blocks' and the final norms are the kind that keeps streams.
         self.residual_streams = residual_streams
         self.final_norm, self.lm_head, self.config = final_norm, lm_head, config
         self.embedding_scale = float(embedding_scale)  # the residual stream starts as scale * embedding row
+        if logit_softcap is not None and logit_softcap <= 0:
+            raise ValueError("the cap on the logits must be positive")
+        self.logit_softcap = logit_softcap  # logits <- cap * tanh(logits / cap)
         self.vocab_size, self.hidden_size = embedding.shape
         if schedule is None:
             schedule = self.schedule_of([(i,) for i in range(len(blocks))], blocks)
@@ -56,6 +59,7 @@ class DecoderModel:
         self.plan = self._make_plan()
         # a block that wants the embedding's output later on (to feed it in again) gets a copy of it in
         # ``ctx.scratch["embedding_output"]``
+        self._step_openers = tuple(p for p in self.parts() if p.begins_steps)
         self.keeps_embedding_output = any(getattr(b, "wants_embedding_output", False) for b in blocks)
 
     @staticmethod
@@ -101,7 +105,8 @@ class DecoderModel:
                     if w.retention != need.retention:
                         # the reader must not need keys that the writer's group gives back: the writer keeps everything,
                         # or both look back over a window and the writer's is at least as long
-                        wide = w.retention.kind == need.retention.kind == Retention.window(1).kind and w.retention.size >= need.retention.size
+                        wide = w.retention.kind == need.retention.kind == Retention.window(1).kind and w.retention.size >= need.retention.size \
+                            and w.retention.keep >= need.retention.keep
                         if w.retention != Retention.all() and not wide:
                             raise ValueError(f"schedule entry {pos}: reads a cache whose pages are released by another rule")
             needs = mixer.state_needs()
@@ -167,6 +172,8 @@ class DecoderModel:
                 block_tables: list[torch.Tensor]) -> torch.Tensor:
         """Runs the step's tokens through the schedule; returns float32 logits [M, V] at ctx.logit_rows."""
         rt = self.runtime
+        for part in self._step_openers:
+            part.begin_step(ctx)
         x = torch.empty((ctx.n_tokens, self.hidden_size), dtype=torch.float32, device=rt.device)
         K.embed(ctx.token_ids, self.embedding, x, ctx.status, self.embedding_scale)
         if self.keeps_embedding_output:
@@ -187,4 +194,7 @@ class DecoderModel:
         if ctx.n_logit_rows == 0:
             return torch.empty((0, self.vocab_size), dtype=torch.float32, device=rt.device)
         h = self.final_norm.forward(ctx, x, delta, out_dtype=rt.dtype, row_index=ctx.logit_rows)[0]
-        return linear(ctx, h, self.lm_head, torch.float32)
+        logits = linear(ctx, h, self.lm_head, torch.float32)
+        if self.logit_softcap is not None:
+            K.soft_cap(logits, self.logit_softcap)
+        return logits

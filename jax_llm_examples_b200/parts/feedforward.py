@@ -7,7 +7,7 @@ import torch
 from ..kernels import api as K
 from ..tracing import active as tracing_active
 from ..tracing import scope
-from .base import CorrectedRouter, Dispatch, FeedForward, Rows, RowSum, StepContext, as_rows, register_part
+from .base import CorrectedRouter, Dispatch, FeedForward, RowPlaces, Rows, RowSum, StepContext, as_rows, register_part
 from .linear import (STREAM_MAX_ROWS, group_rows_hint, grouped_act_linear, grouped_linear, grouped_swiglu_linear, grouped_swiglu_streams,
                      interleave_gate_up, linear,
                      swiglu_linear)
@@ -456,3 +456,111 @@ class GroupLimitedGLUExperts(FeedForward):
 
 
 register_part("feed_forward", "group_limited_glu_experts", GroupLimitedGLUExperts)
+
+
+class TableRoutedGLUExperts(FeedForward):
+    """Gated experts without a router: a table gives every token id its experts, whose outputs count alike,
+
+        out = (1 / k) * sum_j expert_(table[token, j])(h).
+
+    ``table``: int32 [vocab, k], the entries of a row differ; ``we_gate_up``: [E, 2F, D] (gate rows then up rows); ``we_down``:
+    [E, D, F]; ``glu``: the gated activation (``K.glu_form``).
+
+    Which rows go where depends on the step's token ids alone.  The sort of the (token, expert) pairs therefore runs ahead of
+    the layers, on the second stream beside whatever comes first (``begin_step``), once per step however many layer runs
+    share this part; and the norm in front of it writes its rows straight to their places in expert order
+    (``row_places``), so that neither a router, nor a sort, nor a gather stands between the norm and the experts' products.
+    The result is a :class:`RowSum` of one scaled term, the rows still in expert order."""
+
+    kernel_libraries = ("moe", "elementwise", "gemm_simt")
+    kernel_libraries_bf16 = ("gemm_stream",)
+    begins_steps = True
+    needs_f32_input = True  # behind a norm that does not place its rows
+    MAX_COPIES = 16  # places per row that the norm's kernel takes (csrc/elementwise.cu)
+
+    def __init__(self, table: torch.Tensor, we_gate_up: torch.Tensor, we_down: torch.Tensor, glu=K.SILU_GLU):
+        E = we_gate_up.shape[0]
+        if we_down.shape[0] != E or we_gate_up.shape[1] != 2 * we_down.shape[2] or we_gate_up.shape[2] != we_down.shape[1]:
+            raise ValueError(f"expert weights do not fit: gate_up {tuple(we_gate_up.shape)}, down {tuple(we_down.shape)}")
+        if table.dim() != 2 or table.is_floating_point() or not 1 <= table.shape[1] <= E:
+            raise ValueError(f"a table of experts is integers [vocab, k] with k of at most {E} experts, not {table.dtype} {tuple(table.shape)}")
+        if int(table.min()) < 0 or int(table.max()) >= E:
+            raise ValueError(f"the table names experts {int(table.min())}..{int(table.max())}; there are {E}")
+        ordered = table.sort(dim=1).values
+        if bool((ordered[:, 1:] == ordered[:, :-1]).any()):
+            raise ValueError("a row of the table names an expert twice")
+        self.table = table.to(torch.int32).contiguous()
+        self.interleaved = _can_interleave(we_gate_up)
+        self.we_gate_up = interleave_gate_up(we_gate_up) if self.interleaved else we_gate_up.contiguous()
+        self.we_down = we_down.contiguous()
+        self.top_k, self.num_experts, self.glu = table.shape[1], E, tuple(glu)
+
+    def begin_step(self, ctx: StepContext) -> None:
+        n, k, E, dev = ctx.n_tokens, self.top_k, self.num_experts, self.table.device
+        i32 = lambda size: torch.empty(size, dtype=torch.int32, device=dev)  # noqa: E731
+        tiles, tile_rows = None, 0
+        if self.we_gate_up.dtype == torch.bfloat16 and ctx.runtime.dtype == torch.bfloat16:
+            tile_rows = K.gemm_stream_token_tile(group_rows_hint(n * k, E))
+            tiles = (i32(2 * (-(-n * k // tile_rows) + E)), i32(1))
+        chosen = i32(n * k) if "record_routing" in ctx.scratch else None
+        routing = {"offsets": i32(E + 1), "pair": i32(n * k), "pos": i32(n * k), "tiles": tiles, "chosen": chosen, "ready": None}
+
+        def sort():
+            with scope("permute"):
+                K.expert_sort(chosen, routing["offsets"], routing["pair"], routing["pos"], E, ctx.status, 0,
+                              *((tile_rows, *tiles) if tiles is not None else ()), token_ids=ctx.token_ids, table=self.table)
+
+        if ctx.workspace is None:
+            sort()
+        else:  # the buffers were made on the step's own stream, which joins the second one before they are read or freed
+            main, side = torch.cuda.current_stream(), ctx.workspace.side_stream()
+            side.wait_stream(main)
+            with torch.cuda.stream(side):
+                sort()
+                routing["ready"] = side.record_event()
+        ctx.scratch[("table_routing", id(self))] = routing
+
+    def _routing(self, ctx: StepContext) -> dict:
+        key = ("table_routing", id(self))
+        if key not in ctx.scratch:
+            self.begin_step(ctx)
+        routing = ctx.scratch[key]
+        if routing["ready"] is not None:
+            torch.cuda.current_stream().wait_event(routing["ready"])
+            routing["ready"] = None
+        return routing
+
+    def row_places(self, ctx: StepContext, n: int) -> RowPlaces | None:
+        return RowPlaces(self._routing(ctx)["pos"], self.top_k) if self.top_k <= self.MAX_COPIES else None
+
+    def forward(self, ctx: StepContext, h, h32, routing=None):
+        rt, k, E = ctx.runtime, self.top_k, self.num_experts
+        r = self._routing(ctx)
+        offsets, pos, tiles = r["offsets"], r["pos"], r["tiles"]
+        n, D = ctx.n_tokens, self.we_down.shape[1]
+        if "record_routing" in ctx.scratch:
+            ctx.scratch["record_routing"].append(r["chosen"].view(n, k))
+        with scope("moe_routed_expert"):
+            if isinstance(routing, RowPlaces):
+                a_sorted = h
+            else:
+                a_sorted = torch.empty((n * k, D), dtype=rt.dtype, device=h32.device)
+                K.permute_scale(h32, r["pair"], None, a_sorted, k)
+            with scope("we_gate_up"):
+                one_product = grouped_swiglu_streams(a_sorted, self.we_gate_up, self.interleaved)
+                act = grouped_swiglu_linear(ctx, a_sorted, self.we_gate_up, offsets, self.interleaved, rt.dtype, 0, tiles, self.glu)
+            with scope("we_down"):
+                y = as_rows(grouped_linear(ctx, act, self.we_down, offsets, torch.float32, partials=True, tiles=tiles,
+                                           after_grouped=one_product and not tracing_active()))
+
+        def combine() -> torch.Tensor:
+            delta = torch.empty((n, D), dtype=torch.float32, device=y.data.device)
+            with scope("unpermute"):
+                K.moe_combine(y.data, None, pos, delta, k, 1, y.splits, -1,
+                              pair_weights=torch.full((n, k), 1.0 / k, dtype=torch.float32, device=y.data.device))
+            return delta
+
+        return RowSum([Rows(y.data, y.splits, pos, k, 0, None, 1.0 / k)], combine)
+
+
+register_part("feed_forward", "table_routed_glu_experts", TableRoutedGLUExperts)

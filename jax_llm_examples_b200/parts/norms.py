@@ -15,22 +15,25 @@ class RMSNorm(Norm):
 
     kernel_libraries = ("elementwise",)
     fuses_router = True
+    places_rows = True
     FUSED_ROUTER_MAX_ROWS = 64  # above this many rows (bfloat16) the router runs as its own many-rows kernel
 
     def __init__(self, weight: torch.Tensor | None, eps: float):
         self.weight = None if weight is None else weight.to(torch.float32).contiguous()
         self.eps = float(eps)
 
-    def forward(self, ctx: StepContext, x, delta, *, out_dtype, want_f32=False, row_index=None, router=None):
+    def forward(self, ctx: StepContext, x, delta, *, out_dtype, want_f32=False, row_index=None, router=None, places=None):
+        """``places`` (:class:`RowPlaces`): the rounded rows come out in the order that names, several times each."""
         n = x.shape[0] if row_index is None else row_index.numel()
         dev = x.device
-        out = torch.empty((n, x.shape[1]), dtype=out_dtype, device=dev)
+        copies = 1 if places is None else places.copies
+        out = torch.empty((n * copies, x.shape[1]), dtype=out_dtype, device=dev)
         out32 = torch.empty((n, x.shape[1]), dtype=torch.float32, device=dev) if want_f32 else None
         # a sum of terms (an expert layer's rows still in expert order) is added term by term in the kernel
         # (the kernel takes so many terms, rows per token and partials; beyond that the sum is made by its producer)
         if isinstance(delta, RowSum) and len(delta.terms) <= K.DELTA_MAX_TERMS and all(t.k <= 16 and t.weights is None for t in delta.terms) and \
                 sum((t.k if t.index is not None else 1) * t.splits for t in delta.terms) <= K.DELTA_MAX_STREAMS:
-            terms = [(t.data, t.splits, t.index, t.k, t.base) for t in delta.terms]
+            terms = [(t.data, t.splits, t.index, t.k, t.base, t.scale) for t in delta.terms]
         else:
             d = as_rows(delta)
             terms = None if d is None else [(d.data, d.splits, None, 1, 0)]
@@ -54,7 +57,7 @@ class RMSNorm(Norm):
                 and out_dtype == torch.bfloat16 and n <= K.DISPATCH_MAX_ROWS and n * k <= K.DISPATCH_MAX_PAIRS:
             dispatch = offer[0](ctx, n)
         did = K.add_rmsnorm(x, terms, self.weight, self.eps, out, out32, row_index, 1, None if unfused else w_router, idx, wt,
-                            dispatch)
+                            dispatch, None if places is None else places.index, copies)
         if did:
             routing = (idx, wt, dispatch)
         if unfused:

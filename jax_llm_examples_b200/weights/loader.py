@@ -27,8 +27,9 @@ import torch
 class TensorSpec:
     name: str
     shape: tuple[int, ...]  # an entry of -1: a size that only the stored tensor gives (any size fits)
-    init: str = "normal"  # "normal": N(0, std); "norm": 1 + N(0, norm_noise); "bias": N(0, 1/4); "unit": in (0, 1); "identity": I + N(0, norm_noise)
+    init: str = "normal"  # "normal": N(0, std); "norm": 1 + N(0, norm_noise); "bias": N(0, 1/4); "unit": in (0, 1); "identity": I + N(0, norm_noise); "choices": integer rows of distinct entries in [0, high)
     optional: bool = False
+    high: int = 0
 
 
 class WeightError(ValueError):
@@ -64,7 +65,7 @@ def _shard_files(model_dir: Path) -> list[Path]:
     return files
 
 
-def _keep_precision(t: torch.Tensor, dtype: torch.dtype) -> torch.Tensor:
+def keep_precision(t: torch.Tensor, dtype: torch.dtype) -> torch.Tensor:
     if t.dtype in (torch.int8, torch.int16, torch.int32, torch.int64, torch.uint8, torch.bool):
         return t.to(torch.int32)
     if dtype == torch.float32:
@@ -109,7 +110,7 @@ def load_tensors(
                     wrong.append(f"{file_name}: expected {list(specs[name].shape)}, found {list(shape)}")
                     found[name] = None  # type: ignore[assignment]
                     continue
-                found[name] = _keep_precision(f.get_tensor(file_name), dtype)
+                found[name] = keep_precision(f.get_tensor(file_name), dtype)
     missing = [n for n, s in specs.items() if n not in found and not s.optional]
     if missing or unexpected or wrong:
         raise WeightError(str(model_dir), missing, sorted(unexpected), wrong)

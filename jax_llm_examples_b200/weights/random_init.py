@@ -35,6 +35,8 @@ def random_tensor(spec: TensorSpec, seed: int, dtype: torch.dtype, device: str |
             raise ValueError(f"tensor {spec.name}: a size that only a stored tensor gives cannot be drawn at random "
                              "(the configuration must name it)")
         n *= s
+    if spec.init == "choices":  # a table: every row holds shape[1] different numbers below `high`
+        return torch.rand((spec.shape[0], spec.high), generator=g, device=device).argsort(dim=1)[:, :spec.shape[1]].to(torch.int32).contiguous()
     if n <= (1 << 28):
         t = torch.randn(spec.shape, generator=g, dtype=torch.float32, device=device)
         if spec.init == "norm":
