@@ -484,12 +484,15 @@ def run_compare(args) -> dict:
     --compare marinex: the same for Marinex (16 experts in every layer) beside the three models that have its mechanisms'
     nearest relatives: Koduzen with 16 experts (group-limited experts, attention behind a weighted norm and a rotation),
     Tebivik (latent attention, norms on the sublayers' outputs) and a dense Llama-4-style decoder (attention over all
-    earlier positions), at equal width, depth, head count and feed-forward size."""
+    earlier positions), at equal width, depth, head count and feed-forward size.
+    --compare samerax: the same for Samerax beside Koduzen with one residual row (the closest: windowed attention with
+    YaRN-scaled rotation, gated experts, the same norm kernel), both with a dense feed-forward and with 16 experts in every
+    second layer, at equal width, depth, head count and feed-forward size."""
     import torch
 
     import jax_llm_examples_b200 as J
     from jax_llm_examples_b200 import tracing
-    from jax_llm_examples_b200.config.presets import dense_llama_sized, koduzen_sized, makisun_sized, marinex_sized, tebivik_sized, vofusun_sized
+    from jax_llm_examples_b200.config.presets import dense_llama_sized, koduzen_sized, makisun_sized, marinex_sized, samerax_sized, tebivik_sized, vofusun_sized
 
     peaks, peak_src = _peaks()
     hbm, tflops = peaks["hbm_gbs"] * 1e9, peaks["bf16_tflops"] * 1e12
@@ -501,7 +504,8 @@ def run_compare(args) -> dict:
         sizes = [(w, args.layers, h, f) for w, _, h, f in sizes]
     what = {"tebivik": "Tebivik beside a dense Llama-4-style decoder", "makisun": "Makisun beside Tebivik",
             "vofusun": "Vofusun beside Makisun", "koduzen": "Koduzen beside Makisun",
-            "marinex": "Marinex beside Koduzen, Tebivik and a dense Llama-4-style decoder"}[args.compare]
+            "marinex": "Marinex beside Koduzen, Tebivik and a dense Llama-4-style decoder",
+            "samerax": "Samerax beside Koduzen"}[args.compare]
     out = {"metric": "prefill and decode throughput, " + what, "unit": "tok/s", "n_gpus": 1,
            "dtype": "bf16", "data": "synthetic (random weights and tokens)", "peaks": peaks, "peaks_source": peak_src,
            "config": {"prefill_tokens": P, "decode_batch": B, "decode_context": C, "l2": "a 256 MiB buffer is written between timed steps"},
@@ -722,6 +726,55 @@ def run_compare(args) -> dict:
         }
         out["sizes"].append({"width": width, "layers": layers, "heads": heads, "ff": ff, "marinex": x, "koduzen_16_experts": k, "tebivik": t,
                              "dense_llama": l, "fraction_of_measured_roofline": roof})
+    for width, layers, heads, ff in sizes if args.compare == "samerax" else ():
+        x, xe = measure(samerax_sized(width, layers, heads, ff)), measure(samerax_sized(width, layers, heads, ff, experts=16))
+        k, ke = measure(koduzen_sized(width, layers, heads, ff, streams=0)), measure(koduzen_sized(width, layers, heads, ff, experts=16, streams=0))
+        k_ret = sum(1 for i in range(layers) if i % 4 == 2)
+        k_own, k_att = sum(1 for i in range(layers) if i % 4 in (0, 3)), layers - k_ret
+        dim, dh, hkv, window, kept, fe, moe = 64, 128, max(heads // 4, 1), 1024, 16, ff // 4, layers // 2
+        seen_w = sum(min(i + 1, window) for i in range(P))
+        seen_x = sum(min(i + 1, window + kept) for i in range(P))
+        keys_x, keys_k = min(C, window + kept), min(C, window)
+        # a head of Samerax: two score products over 64 entries and two products with 128 values per visible key
+        norm = lambda n: (2 * layers + 1) * n * width * 14
+        norm_e = lambda n: norm(n) + moe * n * width * (2 + 4)  # the rows of two experts are written, and read back, instead of one
+        rope = lambda n, full, q_only: n * (full * (heads + 2 * hkv) + q_only * heads) * dh * 6
+        # experts that B tokens' choices touch, on average (two of Koduzen's 18 choices have no weights)
+        idle_x, idle_k = 16 * (1 - 2 / 16) ** B, 16 * (1 - 2 / 18) ** B
+        pm = lambda m, name: m["prefill_kernels_ms"].get(name, 0)  # noqa: E731
+        dm = lambda m, name: m["decode_kernels_ms"].get(name, 0)  # noqa: E731
+        streamed = lambda m, head_gb, idle: m["weights_gb"] * 1e9 - head_gb - idle * 3 * width * fe * 2
+        emb = 32768 * width * 2
+        roof = {
+            "decode": {
+                "samerax attention_decode": frac(dm(x, "jlx_attention_decode"), layers * B * keys_x * 2 * hkv * dh * 2),
+                "koduzen attention_decode": frac(dm(k, "jlx_attention_decode"), k_att * B * keys_k * 2 * hkv * dh * 2),
+                "samerax add_rmsnorm": frac(dm(x, "jlx_add_rmsnorm"), norm(B)),
+                "samerax add_rmsnorm (rows to the experts)": frac(dm(xe, "jlx_add_rmsnorm"), norm_e(B)),
+                "koduzen add_rmsnorm": frac(dm(k, "jlx_add_rmsnorm"), norm(B)),
+                "samerax rope_half_kv_store": frac(dm(x, "jlx_rope_half_kv_store"), rope(B, layers, 0)),
+                "koduzen rope_half_kv_store": frac(dm(k, "jlx_rope_half_kv_store"), rope(B, k_own, k_att - k_own)),
+                "samerax gemm_stream (all weights of the step)": frac(dm(x, "jlx_gemm_stream"), streamed(x, emb, 0)),
+                "koduzen gemm_stream (all weights of the step)": frac(dm(k, "jlx_gemm_stream"), streamed(k, 0, 0)),
+                "samerax, 16 experts: gemm_stream": frac(dm(xe, "jlx_gemm_stream"), streamed(xe, emb, moe * idle_x)),
+                "koduzen, 16 experts: gemm_stream": frac(dm(ke, "jlx_gemm_stream"), streamed(ke, 0, moe * idle_k)),
+            },
+            "prefill": {
+                "samerax attention_prefill_tc": frac(pm(x, "jlx_attention_prefill_tc"), 0, layers * heads * seen_x * 2 * 2 * (dim + dh)),
+                "koduzen attention_prefill_tc": frac(pm(k, "jlx_attention_prefill_tc"), 0, k_att * heads * seen_w * 4 * dh),
+                "samerax add_rmsnorm": frac(pm(x, "jlx_add_rmsnorm"), norm(P)),
+                "samerax add_rmsnorm (rows to the experts)": frac(pm(xe, "jlx_add_rmsnorm"), norm_e(P)),
+                "koduzen add_rmsnorm": frac(pm(k, "jlx_add_rmsnorm"), norm(P)),
+                "samerax rope_half_kv_store": frac(pm(x, "jlx_rope_half_kv_store"), rope(P, layers, 0)),
+                "koduzen rope_half_kv_store": frac(pm(k, "jlx_rope_half_kv_store"), rope(P, k_own, k_att - k_own)),
+                "samerax experts gemm_stream": frac(pm(xe, "jlx_gemm_stream"), 0, moe * P * 2 * 3 * width * fe * 2),
+                "koduzen experts gemm_stream": frac(pm(ke, "jlx_gemm_stream"), 0, moe * P * 2 * 16 / 18 * 3 * width * fe * 2),
+                "samerax expert_sort (us per layer)": round(pm(xe, "jlx_expert_sort") * 1e3 / moe, 2),
+                "koduzen expert_sort (us per layer)": round(pm(ke, "jlx_expert_sort") * 1e3 / moe, 2),
+            },
+        }
+        out["sizes"].append({"width": width, "layers": layers, "heads": heads, "ff": ff, "samerax": x, "samerax_16_experts": xe, "koduzen": k,
+                             "koduzen_16_experts": ke, "fraction_of_measured_roofline": roof})
     for width, layers, heads, ff in sizes if args.compare == "makisun" else ():
         m, t = measure(makisun_sized(width, layers, heads, ff)), measure(tebivik_sized(width, layers, heads, ff))
         routed = measure(makisun_sized(width, layers, heads, ff, experts=16))
@@ -805,7 +858,7 @@ def main() -> int:
     ap.add_argument("--long-tokens", type=int, default=32768)
     ap.add_argument("--skip-e2e", action="store_true", help="skip the end-to-end run (for profiling captures)")
     ap.add_argument("--skip-prefill", action="store_true", help="skip the prefill measurement (for profiling captures)")
-    ap.add_argument("--compare", default=None, choices=["tebivik", "makisun", "vofusun", "koduzen", "marinex"],
+    ap.add_argument("--compare", default=None, choices=["tebivik", "makisun", "vofusun", "koduzen", "marinex", "samerax"],
                     help="instead of the benchmark: throughput of this architecture at real layer sizes beside the closest "
                     "model the framework had before (with --prefill-tokens, --batch, --context up to 4096, --layers)")
     args = ap.parse_args()

@@ -227,6 +227,34 @@ PRESETS["marinex_tiny"] = {
          "mixer": {"heads": 2, "kv_heads": 1, "dim": 32, "vdim": 32, "rot": {"base": 500.0, "dims": 32}, "scale": 0.2, "softcap": 12.0}},
     ],
 }
+def samerax_sized(width: int, layers: int, heads: int, ff: int, vocab: int = 32768, experts: int = 0) -> dict[str, Any]:
+    """A Samerax configuration at the layer sizes of a real model: every head the difference of two maps of 64 over values of
+    128, four query heads per key head, a window of 1024 that keeps the first 16 keys, the whole map rotated with
+    YaRN-scaled frequencies; a dense feed-forward in every layer, or with ``experts`` > 0 a mixture that a table of token
+    ids chooses from (top 2, each expert a quarter of ``ff``) in every second layer."""
+    dense = {"kind": "dense", "ff": ff}
+    routed = {"kind": "moe", "expert": {"ff": ff // 4}, "router": {"experts": experts, "top": 2}}
+    att = {"heads": heads, "kv_heads": max(heads // 4, 1), "dim": 64, "vdim": 128, "mask": {"size": 1024, "keep_first": 16}, "scale": 0.125, "diff": 0.5,
+           "rot": {"base": 250000.0, "dims": 64, "scaling": {"factor": 4.0, "original": 8192, "fast": 16.0, "slow": 2.0}}}
+    return {"architecture": "Samerax", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "embedding": {"scale": 1.0}, "logit_softcap": 30.0,
+            "layers": [{"type": "attention", "mixer": dict(att), "mlp": routed if experts and i % 2 else dense} for i in range(layers)]}
+
+
+_SAMERAX_TINY = [
+    {"type": "attention", "mlp": {"kind": "moe", "expert": {"ff": 24}, "router": {"experts": 5, "top": 2}},
+     "mixer": {"heads": 4, "kv_heads": 2, "dim": 16, "vdim": 24, "scale": 0.25, "diff": 0.3, "mask": {"size": 20, "keep_first": 3},
+               "rot": {"base": 10000.0, "dims": 8, "scaling": {"factor": 4.0, "original": 64, "fast": 8.0, "slow": 1.0}}}},
+    {"type": "attention", "mlp": {"kind": "dense", "ff": 96},
+     "mixer": {"heads": 2, "kv_heads": 1, "dim": 24, "vdim": 40, "scale": 0.2, "diff": 0.7, "mask": {"size": 33, "keep_first": 1},
+               "rot": {"base": 500.0, "dims": 24}}},
+]
+# Samerax, tiny: two layers, the first one run again with a cache of its own, a layer without a feed-forward.
+PRESETS["samerax_tiny"] = {
+    "architecture": "Samerax", "vocab": 256, "width": 64, "norm": {"eps": 1e-6}, "embedding": {"scale": 2.0}, "logit_softcap": 20.0,
+    "layers": [*_SAMERAX_TINY, dict(_SAMERAX_TINY[0], weights_of=0), dict(_SAMERAX_TINY[1], mlp=None)],
+}
+PRESETS["samerax_2k"] = samerax_sized(2048, 8, 16, 8192, experts=16)
+PRESETS["samerax_4k"] = samerax_sized(4096, 8, 32, 14336, experts=16)
 PRESETS["marinex_2k"] = marinex_sized(2048, 8, 16, 8192)
 PRESETS["marinex_4k"] = marinex_sized(4096, 8, 32, 14336)
 PRESETS["koduzen_2k"] = koduzen_sized(2048, 8, 16, 8192)

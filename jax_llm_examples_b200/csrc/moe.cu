@@ -253,12 +253,19 @@ __global__ void expert_sort_kernel(const int* __restrict__ topk_idx, int* __rest
 __global__ void __launch_bounds__(SORT_WARPS * 32)
 expert_sort_many_kernel(const int* __restrict__ topk_idx, int* __restrict__ offsets, int* __restrict__ sorted_pair,
                         int* __restrict__ sorted_pos, int P, int E, int extra_rows, int tile_rows, int* __restrict__ tile_list,
-                        int* __restrict__ n_tiles, int* status, int tile_groups, const TableChoice by) {
+                        int* __restrict__ n_tiles, int* status, int tile_groups, const TableChoice by, int staging) {
   JLX_TL(TL_SORT);
   __shared__ int counts[ROUTER_MAX_E + 1];
   extern __shared__ int held[];  // [SORT_WARPS][E]: a warp's pairs per expert, then its next place among them
+  int* staged = held + SORT_WARPS * E;  // [P] with `staging`: choices that take two loads to find are looked up once, all at a time
   pdl_launch_dependents();
   pdl_wait();
+  if (staging) {
+#pragma unroll 4
+    for (int i = threadIdx.x; i < P; i += SORT_WARPS * 32) staged[i] = pair_choice(topk_idx, by, i, status);
+    __syncthreads();
+  }
+  auto choice = [&](int i) { return staging ? staged[i] : pair_choice(topk_idx, by, i, status); };
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int per = ((P + SORT_WARPS - 1) / SORT_WARPS + 31) & ~31;
   const int lo = min(P, warp * per), hi = min(P, lo + per);
@@ -267,7 +274,7 @@ expert_sort_many_kernel(const int* __restrict__ topk_idx, int* __restrict__ offs
   __syncwarp();
   for (int base = lo; base < hi; base += 32) {
     const int i = base + lane;
-    const int v = i < hi ? pair_choice(topk_idx, by, i, status) : -1;
+    const int v = i < hi ? choice(i) : -1;
     const unsigned same = __match_any_sync(0xffffffffu, v);
     if (v >= 0 && v < E && (same & ((1u << lane) - 1u)) == 0) mine[v] += __popc(same);
     __syncwarp();
@@ -287,7 +294,7 @@ expert_sort_many_kernel(const int* __restrict__ topk_idx, int* __restrict__ offs
   __syncthreads();
   for (int base = lo; base < hi; base += 32) {
     const int i = base + lane;
-    const int v = i < hi ? pair_choice(topk_idx, by, i, status) : -1;
+    const int v = i < hi ? choice(i) : -1;
     const unsigned same = __match_any_sync(0xffffffffu, v);
     const unsigned before = same & ((1u << lane) - 1u);
     const bool ok = v >= 0 && v < E;
@@ -318,8 +325,10 @@ JLX_API int jlx_expert_sort(const int* topk_idx, int* offsets, int* sorted_pair,
     JLX_REQUIRE(topk_idx || P == 0, "expert_sort: no choices");
   }
   if (P >= 1024) {
-    JLX_CUDA(jlx_launch_pdl(expert_sort_many_kernel, dim3(1), dim3(SORT_WARPS * 32), (size_t)SORT_WARPS * E * sizeof(int), stream, topk_idx,
-                            offsets, sorted_pair, sorted_pos, P, E, extra_rows, tile_rows, tile_list, n_tiles, status, tile_groups, by));
+    const size_t held = (size_t)SORT_WARPS * E * sizeof(int), with_pairs = held + (size_t)P * sizeof(int);
+    const int staging = table && with_pairs <= 44 * 1024;
+    JLX_CUDA(jlx_launch_pdl(expert_sort_many_kernel, dim3(1), dim3(SORT_WARPS * 32), staging ? with_pairs : held, stream, topk_idx,
+                            offsets, sorted_pair, sorted_pos, P, E, extra_rows, tile_rows, tile_list, n_tiles, status, tile_groups, by, staging));
     return 0;
   }
   const int warps = E < 32 ? E : 32;

@@ -553,6 +553,94 @@ __global__ void rope_half_kv_store_kernel(RopeRowsView proj, int k_col, int v_co
   }
 }
 
+// The same for many tokens (a prompt portion) in bfloat16 without a norm, rotated in halves or not at all: one block per token,
+// four neighbouring entries of a head's row per thread and access (16 bytes in, 8 out), so that a token's angles are made once
+// and nothing passes through shared memory but them.  Needs sizes, columns and the half of the rotation in fours.
+__global__ void __launch_bounds__(256)
+rope_half_rows_kernel(RopeRowsView proj, int k_col, int v_col, bf16* __restrict__ q_out, bf16* __restrict__ pages, const int* __restrict__ block_table,
+                      int bt_stride, const int* __restrict__ req_of_token, const int* __restrict__ positions, const float* __restrict__ inv_freq, int rot,
+                      int Hq, int Hkv, int dk, int dv, int dpad, int page_size, int num_pages, int store, int* status, float amplitude,
+                      const float* __restrict__ q_scale, const float* __restrict__ bias, int maps) {
+  JLX_TL(TL_ROPE);
+  pdl_launch_dependents_if_small();
+  extern __shared__ __align__(16) float angles_s[];  // [2][rot / 2]: sines, then cosines, of this token's angles
+  const size_t n = blockIdx.x;
+  const int pos = positions[n], half = rot >> 1;
+  float* sn = angles_s;
+  float* cs = angles_s + half;
+  for (int i = threadIdx.x; i < half; i += blockDim.x) {
+    float s, c;
+    sincosf((float)pos * inv_freq[i], &s, &c);
+    sn[i] = s * amplitude;
+    cs[i] = c * amplitude;
+  }
+  bf16* kdst = nullptr;
+  if (store) {
+    const int page = block_table[(size_t)req_of_token[n] * bt_stride + pos / page_size];
+    if (page < 0 || page >= num_pages) {
+      if (threadIdx.x == 0) atomicOr(status, JLX_STATUS_BAD_PAGE);
+    } else {
+      kdst = pages + ((size_t)page * 2 * Hkv * page_size + (size_t)(pos % page_size)) * dpad;
+    }
+  }
+  __syncthreads();
+  pdl_wait();
+  const float* row = proj.p + n * proj.ld;
+  const int quads = dpad >> 2, rows = Hq + (kdst ? 2 * Hkv : 0);
+  auto fetch = [&](int col) {  // four projected entries: partial sums added in order, then the bias
+    float4 v = *reinterpret_cast<const float4*>(row + col);
+    for (int z = 1; z < proj.splits; ++z) {
+      const float4 w = *reinterpret_cast<const float4*>(row + (size_t)z * proj.split_stride + col);
+      v.x += w.x; v.y += w.y; v.z += w.z; v.w += w.w;
+    }
+    if (bias) {
+      const float4 b = *reinterpret_cast<const float4*>(bias + col);
+      v.x += b.x; v.y += b.y; v.z += b.z; v.w += b.w;
+    }
+    return v;
+  };
+  for (int idx = threadIdx.x; idx < rows * quads; idx += blockDim.x) {
+    const int r = idx / quads, j = (idx - r * quads) * 4;  // output row (a query row, a cached key row, a value row), first entry
+    float4 y = make_float4(0.f, 0.f, 0.f, 0.f);
+    bf16* dst;
+    int col = -1, i = j;  // column of the entries, and their place in their map
+    if (r < Hq) {
+      dst = q_out + (n * Hq + r) * dpad;
+      i = j - (r % maps) * dk;
+      if (i >= 0 && i < dk) col = r * dk + i;
+    } else if (r < Hq + Hkv) {
+      dst = kdst + (size_t)(r - Hq) * page_size * dpad;
+      if (j < maps * dk) {
+        col = k_col + (r - Hq) * maps * dk + j;
+        i = j % dk;
+      }
+    } else {
+      dst = kdst + (size_t)(r - Hq) * page_size * dpad;
+      if (j < dv) col = v_col + (r - Hq - Hkv) * dv + j;
+      i = rot;  // values do not turn
+    }
+    if (col >= 0) {
+      y = fetch(col);
+      if (i < rot) {
+        const bool first = i < half;
+        const int f = first ? i : i - half;
+        const float4 w = fetch(first ? col + half : col - half);
+        const float4 s = *reinterpret_cast<const float4*>(sn + f), c = *reinterpret_cast<const float4*>(cs + f);
+        const float g = first ? -1.f : 1.f;
+        y = make_float4(y.x * c.x + g * w.x * s.x, y.y * c.y + g * w.y * s.y, y.z * c.z + g * w.z * s.z, y.w * c.w + g * w.w * s.w);
+      }
+      if (r < Hq && q_scale) {
+        const float m = q_scale[r];
+        y.x *= m; y.y *= m; y.z *= m; y.w *= m;
+      }
+    }
+    uint2 o;
+    *reinterpret_cast<__nv_bfloat162*>(&o.x) = __floats2bfloat162_rn(y.x, y.y);
+    *reinterpret_cast<__nv_bfloat162*>(&o.y) = __floats2bfloat162_rn(y.z, y.w);
+    *reinterpret_cast<uint2*>(dst + j) = o;
+  }
+}
+
 // proj: float32 rows (see RopeRowsView; p points at the first q column).  pages: [P, 2, Hkv, page_size, dpad] or null.
 // pairing: which entries turn together; norm_mode: no q/k norm, before the rotation, or after it (a null weight: the
 // norm without one).  v_norm: each value head is divided by its root mean square over dv (no weight).  q_scale [Hq] (or
@@ -572,6 +660,16 @@ JLX_API int jlx_rope_half_kv_store(const RopeRowsView* proj, int k_col, int v_co
   JLX_REQUIRE(norm_mode >= ROPE_NORM_NONE && norm_mode <= ROPE_NORM_WHOLE, "rope_half: unknown norm mode %d", norm_mode);
   JLX_REQUIRE(!store || (pages && block_table && page_size > 0 && num_pages > 0), "rope_half: cache missing");
   if (N == 0) return 0;
+  const bool in_fours = dk % 4 == 0 && dv % 4 == 0 && dpad % 4 == 0 && k_col % 4 == 0 && v_col % 4 == 0 && rot % 8 == 0 && proj->ld % 4 == 0 &&
+                        proj->split_stride % 4 == 0 &&
+                        (((uintptr_t)proj->p | (uintptr_t)q_out | (uintptr_t)pages | (uintptr_t)bias) & 15) == 0;
+  if (N >= 64 && dtype == JLX_BF16 && norm_mode == ROPE_NORM_NONE && !v_norm && (pairing == ROPE_PAIRS_HALVES || rot == 0) && in_fours && rot <= 4096) {
+    JLX_CUDA(jlx_launch_pdl(rope_half_rows_kernel, dim3(N), dim3(256), (size_t)rot * sizeof(float), stream, *proj, k_col, v_col, (bf16*)q_out, (bf16*)pages,
+                            block_table, bt_stride, req_of_token, positions, inv_freq, rot, Hq, Hkv, dk, dv, dpad, page_size, num_pages, store, status,
+                            amplitude, q_scale, bias, maps));
+    JLX_LAUNCH_CHECK("rope_half_rows");
+    return 0;
+  }
   const int heads = Hq + (store ? (maps + 1) * Hkv : 0);
   const int nwarp = heads < 8 ? heads : 8;
   const int by = N >= 64 ? 1 : (heads + nwarp - 1) / nwarp;

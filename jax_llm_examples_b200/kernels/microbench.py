@@ -57,21 +57,33 @@ def attention_decode(a) -> dict:
     pos = torch.full((a.batch,), a.context - 1, device=dev, dtype=torch.int32)
     req = torch.arange(a.batch, device=dev, dtype=torch.int32)
     status = torch.zeros(1, device=dev, dtype=torch.int32)
-    keys, splits = K.attention_decode_plan(a.context, a.chunk, 0, a.batch * a.kv_heads)
+    keys, splits = K.attention_decode_plan(a.context, a.chunk, a.window, a.batch * a.kv_heads)
     if a.split_keys:
         keys, splits = a.split_keys, -(-a.context // a.split_keys) + 1
     part_o = torch.empty(a.batch * a.heads * splits * a.head_dim, device=dev)
     part_ml = torch.empty(a.batch * a.heads * splits * 2, device=dev)
 
     def run():
-        K.attention_decode(q, pages, table, req, pos, out, a.head_dim ** -0.5, a.chunk, 0, 0.0, 1.0, part_o, part_ml, splits,
-                           keys, status, softcap=a.softcap)
+        K.attention_decode(q, pages, table, req, pos, out, a.head_dim ** -0.5, a.chunk, a.window, 0.0, 1.0, part_o, part_ml, splits,
+                           keys, status, softcap=a.softcap, keep=a.keep, diff=diff)
 
+    diff, out = _maps(a, q, out)
     t = _time(run, a.reps, _flush(a))
-    nbytes = a.batch * a.context * 2 * a.kv_heads * a.head_dim * 2
+    nbytes = a.batch * min(a.context, (a.window or a.context) + a.keep) * 2 * a.kv_heads * a.head_dim * 2
     assert int(status) == 0
     return {"kernel": "attention_decode", "batch": a.batch, "context": a.context, "split_keys": keys, "splits": splits,
             "us": round(t * 1e6, 1), "GB": round(nbytes / 1e9, 3), "GB/s": round(nbytes / t / 1e9, 1)}
+
+
+def _maps(a, q, out):
+    """With --maps: the query heads are pairs of maps of half the head size each, and the kernel ends in their difference."""
+    if not a.maps:
+        return None, out
+    half = a.head_dim // 2
+    q[:, 0::2, half:] = 0
+    q[:, 1::2, :half] = 0
+    out = torch.empty(q.shape[0], a.heads // 2 * a.head_dim, device="cuda", dtype=torch.bfloat16)
+    return K.map_difference_spec(half, 0.7, 0.5, 1e-6, out, a.heads // 2), out
 
 
 def attention_prefill(a) -> dict:
@@ -88,13 +100,39 @@ def attention_prefill(a) -> dict:
     fn = K.attention_prefill_tc if a.tc else K.attention_prefill
 
     def run():
-        fn(q, pages, table, req, pos, out, tiles, tiles.shape[0], a.head_dim ** -0.5, a.chunk, 0, 0.0, 1.0, status, softcap=a.softcap)
+        fn(q, pages, table, req, pos, out, tiles, tiles.shape[0], a.head_dim ** -0.5, a.chunk, a.window, 0.0, 1.0, status, softcap=a.softcap, keep=a.keep,
+           diff=diff)
 
+    diff, out = _maps(a, q, out)
     t = _time(run, a.reps, _flush(a))
-    flops = 4 * a.heads * a.head_dim * T * (T + 1) / 2
+    seen = sum(min(i + 1, (a.window or T) + a.keep) for i in range(T))
+    flops = (3 if a.maps else 4) * a.heads * a.head_dim * seen
     assert int(status) == 0
     return {"kernel": "attention_prefill_tc" if a.tc else "attention_prefill", "tokens": T, "us": round(t * 1e6, 1), "TFLOP": round(flops / 1e12, 4),
             "TFLOP/s": round(flops / t / 1e12, 1)}
+
+
+def expert_sort(a) -> dict:
+    """The sort of a step's (token, expert) pairs, from given choices or (--table) from a table of token ids."""
+    dev, V = "cuda", 32768
+    P = a.tokens * a.top
+    table = torch.rand(V, a.experts, device=dev).argsort(1)[:, :a.top].to(torch.int32).contiguous()
+    ids = torch.randint(0, V, (a.tokens,), device=dev, dtype=torch.int32)
+    i32 = lambda n: torch.empty(n, device=dev, dtype=torch.int32)  # noqa: E731
+    tile_rows = K.gemm_stream_token_tile(max(P // a.experts, 1))
+    out = (i32(a.experts + 1), i32(P), i32(P))
+    status, tiles = torch.zeros(1, device=dev, dtype=torch.int32), (i32(2 * (-(-P // tile_rows) + a.experts)), i32(1))
+    choice = table[ids.long()].contiguous()
+
+    def run():
+        if a.table:
+            K.expert_sort(None, *out, a.experts, status, 0, tile_rows, *tiles, token_ids=ids, table=table)
+        else:
+            K.expert_sort(choice, *out, a.experts, status, 0, tile_rows, *tiles)
+
+    t = _time(run, a.reps, _flush(a))
+    assert int(status) == 0
+    return {"kernel": "expert_sort", "tokens": a.tokens, "experts": a.experts, "table": a.table, "us": round(t * 1e6, 1)}
 
 
 def gemm(a) -> dict:
@@ -289,7 +327,7 @@ def main(argv=None) -> int:
     ap = argparse.ArgumentParser(description=__doc__.split("\n\n")[0])
     sub = ap.add_subparsers(dest="what", required=True)
     for name in ("attention_decode", "attention_prefill", "gemm", "decay_scan", "delta_scan", "conv_unit_prep", "stream_mix_norm",
-                 "latent_decode", "close_route"):
+                 "latent_decode", "close_route", "expert_sort"):
         p = sub.add_parser(name)
         p.add_argument("--reps", type=int, default=10)
         p.add_argument("--no-flush", action="store_true", help="do not flush L2 between launches")
@@ -320,6 +358,10 @@ def main(argv=None) -> int:
             for flag, value in (("rows", 8), ("width", 2048), ("experts", 16), ("top", 2), ("splits", 4)):
                 p.add_argument(f"--{flag}", type=int, default=value)
             p.add_argument("--unfused", action="store_true")
+        if name == "expert_sort":
+            for flag, value in (("tokens", 2048), ("experts", 16), ("top", 2)):
+                p.add_argument(f"--{flag}", type=int, default=value)
+            p.add_argument("--table", action="store_true", help="the choices are looked up by token id")
         if name.startswith("attention"):
             p.add_argument("--softcap", type=float, default=0.0, help="cap * tanh(score / cap)")
             p.add_argument("--heads", type=int, default=40)
@@ -327,6 +369,9 @@ def main(argv=None) -> int:
             p.add_argument("--head-dim", type=int, default=128)
             p.add_argument("--page-size", type=int, default=64)
             p.add_argument("--chunk", type=int, default=0)
+            p.add_argument("--window", type=int, default=0)
+            p.add_argument("--keep", type=int, default=0, help="first keys that the window keeps")
+            p.add_argument("--maps", action="store_true", help="the query heads are pairs of maps of half the head size, taken off one another at the end")
         if name == "attention_decode":
             p.add_argument("--batch", type=int, default=8)
             p.add_argument("--context", type=int, default=8192)
@@ -345,7 +390,7 @@ def main(argv=None) -> int:
     a = ap.parse_args(argv)
     print(json.dumps({"attention_decode": attention_decode, "attention_prefill": attention_prefill, "gemm": gemm, "decay_scan": decay_scan,
                       "delta_scan": delta_scan, "conv_unit_prep": conv_unit_prep, "stream_mix_norm": stream_mix_norm,
-                      "latent_decode": latent_decode, "close_route": close_route}[a.what](a)))
+                      "latent_decode": latent_decode, "close_route": close_route, "expert_sort": expert_sort}[a.what](a)))
     return 0
 
 

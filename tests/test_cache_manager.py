@@ -65,6 +65,31 @@ def test_window_group_releases_behind_the_window():
     m.check()
 
 
+@pytest.mark.parametrize("keep, kept", [(1, 1), (16, 1), (17, 2), (40, 3)])
+def test_a_window_that_keeps_the_first_tokens_keeps_their_pages(keep, kept):
+    """Pages of 16: those of the first `keep` tokens stay until the request ends, the window's old ones go."""
+    m = CacheManager(16, 2, 32)
+    g = m.add_group(Retention.window(20, keep), 12)
+    a, b = m.alloc_slot(), m.alloc_slot()
+    for n in (15, 37, 100, 180):
+        m.reserve(a, n)
+        m.commit(a, n)
+        m.check()
+        first = max(0, n - 19) // 16
+        want = set(range(min(kept, -(-n // 16)))) | set(range(first, -(-n // 16)))
+        assert {i for i in range(32) if m.table(g)[a][i] >= 0} == want
+    m.reserve(b, 16)
+    held = [int(m.table(g)[a][i]) for i in range(kept)]
+    m.release(a)
+    assert m.free_pages(g) == 11 and (m.table(g)[a] < 0).all()
+    m.check()
+    m.reserve(b, 16 * 12)  # the kept pages are handed out again
+    assert set(held) <= set(int(p) for p in m.table(g)[b][:12])
+    m.release(b)
+    m.check()
+    assert m.free_pages(g) == 12
+
+
 def test_out_of_pages_takes_nothing_and_pages_are_reused_lifo():
     m = _manager(pages=4)
     a, b = m.alloc_slot(), m.alloc_slot()
@@ -112,6 +137,7 @@ def test_random_orders_keep_the_invariants(seed):
     m.add_group(Retention.all(), pages)
     m.add_group(Retention.chunk(chunk), pages)
     m.add_group(Retention.window(rng.choice([5, 40])), pages)
+    m.add_group(Retention.window(rng.choice([3, 30]), rng.choice([1, 16, 50])), pages)
     live: dict[int, int] = {}
     for _ in range(600):
         op = rng.random()
@@ -139,12 +165,13 @@ def test_random_orders_keep_the_invariants(seed):
                 for g, r in enumerate(m.groups):
                     first = 0 if r.kind == 0 else ((live[s] // r.size) * r.size if r.kind == 1 else max(0, live[s] - r.size + 1))
                     row = m.table(g)[s]
+                    assert all(row[i] >= 0 for i in range((min(r.keep, live[s]) + page - 1) // page))
                     assert all(row[i] >= 0 for i in range(first // page, (live[s] + page - 1) // page))
         m.check()
     for s in list(live):
         m.release(s)
     m.check()
-    assert all(m.free_pages(g) == pages for g in range(3)) and m.free_slots() == 5
+    assert all(m.free_pages(g) == pages for g in range(4)) and m.free_slots() == 5
 
 
 def test_pack_step_layout():
