@@ -326,7 +326,8 @@ __global__ void __launch_bounds__(128) attention_decode_kernel(const AttnParams 
 // stage: no per-lane copy instructions, so the load/store units stay free and the queue stays deep.
 // Rows of keys outside [lo, p] are copied too (from page 0 where the block table has no page); their
 // scores are masked, and their values are finite numbers written by this engine, so 0 * value = 0.
-template <int DH>
+// GENERAL: with kept first keys, or groups of more query heads than a block takes (the plain case is leaner without them).
+template <int DH, bool GENERAL>
 __global__ void __launch_bounds__(128)
 attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map, const AttnParams P, int box_rows) {
   JLX_TL(TL_ATTN_DECODE);
@@ -340,7 +341,7 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map, const AttnP
   // Until pdl_wait() below, only what no kernel of this step writes is read: the step's description (rows,
   // positions, requests, block table: on the device before the step began) and keys and values of earlier steps.
   const int slot = blockIdx.z, n = P.rows ? P.rows[slot] : slot, split = blockIdx.x;
-  const BlockHeads heads = block_heads(P, blockIdx.y, DEC_MAX_G);
+  const BlockHeads heads = GENERAL ? block_heads(P, blockIdx.y, DEC_MAX_G) : BlockHeads{(int)blockIdx.y, (int)blockIdx.y * (P.Hq / P.Hkv), P.Hq / P.Hkv};
   const int hk = heads.hk, h0 = heads.h0, G = heads.G;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int p = P.positions[n], r = P.req_of_token[n];
@@ -350,13 +351,13 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map, const AttnP
   const int key_end = min(p + 1, key_begin + P.split_keys);
   // the splits share the tiles of the kept first keys between them, each walks its own before its stretch of the window
   int kept_lo = 0, n_kept = 0;
-  if (P.keep > 0) {
+  if (GENERAL && P.keep > 0) {
     const int kept = kept_tiles(P.keep, first_split * P.split_keys, KT), n_splits = p / P.split_keys - first_split + 1;
     kept_lo = split * kept / n_splits;
     n_kept = (split + 1) * kept / n_splits - kept_lo;
   }
   const int n_tiles = n_kept + (key_end - key_begin + KT - 1) / KT;
-  auto tile_first_key = [&](int t) { return t < n_kept ? (kept_lo + t) * KT : key_begin + (t - n_kept) * KT; };
+  auto tile_first_key = [&](int t) { return GENERAL && t < n_kept ? (kept_lo + t) * KT : key_begin + (t - n_kept) * KT; };
   const int* table = P.block_table + (size_t)r * P.bt_stride;
 
   if (threadIdx.x == 0) {
@@ -373,7 +374,8 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map, const AttnP
   const bool cached = n_boxes <= DEC_MAX_BOXES;
   if (cached) {
     for (int b = threadIdx.x; b < n_boxes; b += blockDim.x) {
-      const int pi = (tile_first_key(b / boxes_per_tile) + (b % boxes_per_tile) * box_rows) / P.page_size;
+      const int pos = GENERAL ? tile_first_key(b / boxes_per_tile) + (b % boxes_per_tile) * box_rows : key_begin + b * box_rows;
+      const int pi = pos / P.page_size;
       page_of_box[b] = pi < P.bt_stride ? table[pi] : -1;
     }
     __syncthreads();
@@ -461,7 +463,7 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map, const AttnP
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         const int key = tile_key + warp * 16 + nt * 8 + (lane & 3) * 2 + (e & 1);
-        const bool in = (key >= lo || key < P.keep) && key <= p;
+        const bool in = (key >= lo || (GENERAL && key < P.keep)) && key <= p;
         s[nt][e] = in ? fmaf(-sl[e >> 1], (float)(p - key), scaled_score(P, s[nt][e], sc)) : NEG_BIG;
         mx[e >> 1] = fmaxf(mx[e >> 1], s[nt][e]);
       }
@@ -1206,15 +1208,21 @@ JLX_API int jlx_attention_decode(const void* q, const void* pages, const int* bl
     CUtensorMap map;
     const int box_rows = page_size < KT ? page_size : KT;
     if (make_cache_map(&map, pages, (long long)num_pages * 2 * Hkv * page_size, dh, box_rows)) return 1;
-    if (dh == 128) {
-      static bool cfg = false;
-      if (!cfg) { JLX_CUDA(cudaFuncSetAttribute(attention_decode_tma_kernel<128>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem + 1024)); cfg = true; }
-      JLX_CUDA(jlx_launch_pdl(attention_decode_tma_kernel<128>, grid, dim3(128), smem + 1024, stream, map, P, box_rows));
-    } else {
-      static bool cfg = false;
-      if (!cfg) { JLX_CUDA(cudaFuncSetAttribute(attention_decode_tma_kernel<64>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem + 1024)); cfg = true; }
-      JLX_CUDA(jlx_launch_pdl(attention_decode_tma_kernel<64>, grid, dim3(128), smem + 1024, stream, map, P, box_rows));
-    }
+#define DECODE_TMA(DHV, GEN)                                                                                               \
+    do {                                                                                                                   \
+      static bool cfg = false;                                                                                             \
+      if (!cfg) {                                                                                                          \
+        JLX_CUDA(cudaFuncSetAttribute(attention_decode_tma_kernel<DHV, GEN>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem + 1024)); \
+        cfg = true;                                                                                                        \
+      }                                                                                                                    \
+      JLX_CUDA(jlx_launch_pdl(attention_decode_tma_kernel<DHV, GEN>, grid, dim3(128), smem + 1024, stream, map, P, box_rows)); \
+    } while (0)
+    const bool general = keep > 0 || head_blocks != Hkv;
+    if (dh == 128 && general) DECODE_TMA(128, true);
+    else if (dh == 128) DECODE_TMA(128, false);
+    else if (general) DECODE_TMA(64, true);
+    else DECODE_TMA(64, false);
+#undef DECODE_TMA
     JLX_LAUNCH_CHECK("attention_decode_tma");
   } else if (dh == 128) {
     static bool cfg = false;

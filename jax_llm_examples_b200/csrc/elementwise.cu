@@ -147,17 +147,18 @@ __device__ __forceinline__ void router_topk(float* scores, int E, int k, size_t 
 // What a norm adds to the residual stream before it normalises: up to DELTA_MAX_TERMS terms, added in the order given.
 // A term is `splits` float32 partials [z][rows][D] (z ascending, `stride` elements apart), of which token r takes row
 // base + r, or, with `index`, the k rows index[r * k + j], j ascending (an expert layer's rows in expert order: the
-// norm then does the un-permute and the sum over a token's experts that a kernel of its own would do), times `scale`.
+// norm then does the un-permute and the sum over a token's experts that a kernel of its own would do).  Every row of every
+// term is multiplied by `scale` as it is added.
 #define DELTA_MAX_TERMS 3
 struct DeltaTerm {
   const float* p;
   long long stride;
   const int* index;
   int splits, k, base;
-  float scale;
 };
 struct DeltaSpec {
   int n;
+  float scale;
   DeltaTerm t[DELTA_MAX_TERMS];
 };
 
@@ -169,7 +170,6 @@ struct DeltaSpec {
 #define DELTA_CHUNK 8
 struct DeltaSources {
   const float* ptr[DELTA_MAX_STREAMS];
-  float scale[DELTA_MAX_STREAMS];
   int n;
 };
 // Called by every thread; thread 0 fills `src`, a barrier follows.
@@ -184,10 +184,7 @@ __device__ __forceinline__ void resolve_delta(DeltaSources& src, const DeltaSpec
       const int rows = t.index ? t.k : 1;
       for (int j = 0; j < rows; ++j) {
         const size_t row = t.index && real ? (size_t)t.index[r * t.k + j] : (size_t)t.base + r;
-        for (int z = 0; z < t.splits && n < DELTA_MAX_STREAMS; ++z, ++n) {
-          src.ptr[n] = t.p + (size_t)z * t.stride + row * D;
-          src.scale[n] = t.scale;
-        }
+        for (int z = 0; z < t.splits && n < DELTA_MAX_STREAMS; ++z) src.ptr[n++] = t.p + (size_t)z * t.stride + row * D;
       }
     }
     src.n = n;
@@ -195,8 +192,8 @@ __device__ __forceinline__ void resolve_delta(DeltaSources& src, const DeltaSpec
   __syncthreads();
 }
 
-// s += the streams' 16-byte element i, in stream order; a chunk of streams is in flight at once.
-__device__ __forceinline__ void add_streams4(float4& s, const DeltaSources& src, int i, bool real = true) {
+// s += c * the streams' 16-byte element i, in stream order; a chunk of streams is in flight at once.
+__device__ __forceinline__ void add_streams4(float4& s, const DeltaSources& src, float c, int i, bool real = true) {
   for (int q0 = 0; q0 < src.n; q0 += DELTA_CHUNK) {
     float4 v[DELTA_CHUNK];
 #pragma unroll
@@ -207,7 +204,6 @@ __device__ __forceinline__ void add_streams4(float4& s, const DeltaSources& src,
 #pragma unroll
     for (int u = 0; u < DELTA_CHUNK; ++u)
       if (q0 + u < src.n) {
-        const float c = src.scale[q0 + u];
         s.x = fmaf(c, v[u].x, s.x); s.y = fmaf(c, v[u].y, s.y); s.z = fmaf(c, v[u].z, s.z); s.w = fmaf(c, v[u].w, s.w);
       }
   }
@@ -249,7 +245,7 @@ add_rmsnorm_kernel(float* __restrict__ x, const DeltaSpec ds,
   const size_t r = row_index ? (size_t)row_index[n] : (size_t)n;
   float* xr = x + r * D;
   __shared__ size_t dst[NORM_MAX_COPIES];  // where the row goes: its first elements in `out`
-  if ((int)threadIdx.x < copies) dst[threadIdx.x] = (places ? (size_t)places[(size_t)n * copies + threadIdx.x] : (size_t)n) * D;
+  if (places && (int)threadIdx.x < copies) dst[threadIdx.x] = (size_t)places[(size_t)n * copies + threadIdx.x] * D;
   if (has_delta) resolve_delta(src, ds, r, D);  // (barriers behind it and in block_sum)
   JLX_TL_MARK(0);
   float ss = 0.f;
@@ -260,7 +256,7 @@ add_rmsnorm_kernel(float* __restrict__ x, const DeltaSpec ds,
     for (int i = threadIdx.x; i < D4; i += blockDim.x) {
       float4 t = x4[i];  // in flight together with the first chunk of streams
       if (has_delta) {
-        add_streams4(t, src, i);
+        add_streams4(t, src, ds.scale, i);
         if (!row_index) x4[i] = t;
       }
       row4[i] = t;
@@ -276,8 +272,11 @@ add_rmsnorm_kernel(float* __restrict__ x, const DeltaSpec ds,
       const float4 t = row4[i];
       const float4 g = turn == 0 ? g_ahead : (gamma ? g4[i] : make_float4(1.f, 1.f, 1.f, 1.f));
       const float4 v = make_float4(g.x * t.x / rms, g.y * t.y / rms, g.z * t.z / rms, g.w * t.w / rms);
-      if (out)
+      if (places) {
         for (int j = 0; j < copies; ++j) store4<TO>(out + dst[j] + 4 * i, v);
+      } else if (out) {
+        store4<TO>(out + (size_t)n * D + 4 * i, v);
+      }
       if (out32) reinterpret_cast<float4*>(out32 + (size_t)n * D)[i] = v;
       row4[i] = v;
     }
@@ -285,7 +284,7 @@ add_rmsnorm_kernel(float* __restrict__ x, const DeltaSpec ds,
     for (int d = threadIdx.x; d < D; d += blockDim.x) {
       float s = xr[d];
       if (has_delta) {
-        for (int q = 0; q < src.n; ++q) s = fmaf(src.scale[q], src.ptr[q][d], s);
+        for (int q = 0; q < src.n; ++q) s = fmaf(ds.scale, src.ptr[q][d], s);
         if (!row_index) xr[d] = s;
       }
       if (row_in_smem) rowbuf[d] = s;
@@ -300,11 +299,14 @@ add_rmsnorm_kernel(float* __restrict__ x, const DeltaSpec ds,
       } else {
         s = xr[d];
         if (has_delta && row_index)
-          for (int q = 0; q < src.n; ++q) s = fmaf(src.scale[q], src.ptr[q][d], s);
+          for (int q = 0; q < src.n; ++q) s = fmaf(ds.scale, src.ptr[q][d], s);
       }
       const float v = (gamma ? gamma[d] * s : s) / rms;
-      if (out)
+      if (places) {
         for (int j = 0; j < copies; ++j) out[dst[j] + d] = from_f32<TO>(v);
+      } else if (out) {
+        out[(size_t)n * D + d] = from_f32<TO>(v);
+      }
       if (out32) out32[(size_t)n * D + d] = v;
       if (row_in_smem) rowbuf[d] = v;
     }
@@ -401,14 +403,14 @@ add_rmsnorm_router_cluster_kernel(float* __restrict__ x, const DeltaSpec ds,
   for (int pass = ROUTER || gridDim.x > C ? 1 : 0; pass < 2; ++pass) {
   const bool real = pass == 1;
   if (real) pdl_wait();
-  if (real && (int)threadIdx.x < copies) dst[threadIdx.x] = (places ? (size_t)places[(size_t)n * copies + threadIdx.x] : (size_t)n) * D;
+  if (!ROUTER && real && places && (int)threadIdx.x < copies) dst[threadIdx.x] = (size_t)places[(size_t)n * copies + threadIdx.x] * D;
   if (ds.n > 0) resolve_delta(src, ds, (size_t)n, D, real);
   float ss = 0.f;
   for (int i = (lo >> 2) + threadIdx.x; i < (hi >> 2); i += blockDim.x) {
     float4 s = make_float4(1.f, 1.f, 1.f, 1.f);
     if (real) s = x4[i];
     if (ds.n > 0) {
-      add_streams4(s, src, i, real);
+      add_streams4(s, src, ds.scale, i, real);
       if (real) x4[i] = s;
     }
     row4[i - (lo >> 2)] = s;
@@ -432,8 +434,12 @@ add_rmsnorm_router_cluster_kernel(float* __restrict__ x, const DeltaSpec ds,
     const float4 s = row4[i - (lo >> 2)];
     const float4 g = i == mine ? g_ahead : (gamma ? g4[i] : make_float4(1.f, 1.f, 1.f, 1.f));
     const float4 v = make_float4(g.x * s.x * inv_rms, g.y * s.y * inv_rms, g.z * s.z * inv_rms, g.w * s.w * inv_rms);
-    if (real)
-      for (int j = 0; j < copies; ++j) store4<TO>(out + dst[j] + 4 * i, v);
+    if (!ROUTER && places) {
+      if (real)
+        for (int j = 0; j < copies; ++j) store4<TO>(out + dst[j] + 4 * i, v);
+    } else if (real) {
+      store4<TO>(out + (size_t)n * D + 4 * i, v);
+    }
     if (real && out32) reinterpret_cast<float4*>(out32 + (size_t)n * D)[i] = v;
     row4[i - (lo >> 2)] = v;
   }

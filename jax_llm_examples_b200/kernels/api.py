@@ -130,12 +130,11 @@ DISPATCH_MAX_ROWS, DISPATCH_MAX_PAIRS = 16, 64  # csrc/elementwise.cu
 
 
 class _DeltaTerm(ctypes.Structure):
-    _fields_ = [("p", c_void_p), ("stride", c_longlong), ("index", c_void_p), ("splits", c_int), ("k", c_int), ("base", c_int),
-                ("scale", c_float)]
+    _fields_ = [("p", c_void_p), ("stride", c_longlong), ("index", c_void_p), ("splits", c_int), ("k", c_int), ("base", c_int)]
 
 
 class _DeltaSpec(ctypes.Structure):
-    _fields_ = [("n", c_int), ("t", _DeltaTerm * DELTA_MAX_TERMS)]
+    _fields_ = [("n", c_int), ("scale", c_float), ("t", _DeltaTerm * DELTA_MAX_TERMS)]
 
 
 class _DispatchArgs(ctypes.Structure):  # DispatchArgs in csrc/elementwise.cu
@@ -147,11 +146,13 @@ class _DispatchArgs(ctypes.Structure):  # DispatchArgs in csrc/elementwise.cu
 def add_rmsnorm(x: torch.Tensor, delta, gamma: torch.Tensor | None, eps: float,
                 out: torch.Tensor | None, out32: torch.Tensor | None = None, row_index: torch.Tensor | None = None,
                 delta_splits: int = 1, w_router: torch.Tensor | None = None, topk_idx: torch.Tensor | None = None,
-                topk_w: torch.Tensor | None = None, dispatch=None, places: torch.Tensor | None = None, copies: int = 1) -> bool:
+                topk_w: torch.Tensor | None = None, dispatch=None, places: torch.Tensor | None = None, copies: int = 1,
+                delta_scale: float = 1.0) -> bool:
     """x (+= delta); out = gamma * x / sqrt(mean(x^2) + eps).  ``delta``: a float32 tensor that may hold
     ``delta_splits`` split-K partials [splits, N, D], added in order; or a list of up to DELTA_MAX_TERMS terms
-    ``(data, splits, index, k, base[, scale])`` added in the order given: of the float32 partials ``data`` [splits, rows, D]
-    token r takes row ``base + r`` or, with ``index`` (int32 [N * k]), the k rows ``index[r * k + j]``, times ``scale``.
+    ``(data, splits, index, k, base)`` added in the order given: of the float32 partials ``data`` [splits, rows, D]
+    token r takes row ``base + r`` or, with ``index`` (int32 [N * k]), the k rows ``index[r * k + j]``; all of
+    them times ``delta_scale``.
     ``places`` (int32 [N * copies]): the normed row n goes to the rows places[n * copies + j] of ``out`` instead of row n.
     With row_index, row n reads source row row_index[n] and x is not written back.  With w_router [E, D] the token
     is routed in the same kernel: topk_idx / topk_w [N, k].  ``dispatch`` (with w_router; an object with the tensors
@@ -170,11 +171,11 @@ def add_rmsnorm(x: torch.Tensor, delta, gamma: torch.Tensor | None, eps: float,
         raise KernelError(f"add_rmsnorm: {len(terms)} terms to add; up to {DELTA_MAX_TERMS} are supported")
     spec = _DeltaSpec()
     spec.n = len(terms)
-    for q, (data, splits, index, k_rows, base, *scale) in enumerate(terms):
+    spec.scale = delta_scale
+    for q, (data, splits, index, k_rows, base) in enumerate(terms):
         sp, stride = _splits(data, splits)
         spec.t[q].p, spec.t[q].stride, spec.t[q].splits = data.data_ptr(), stride, sp
         spec.t[q].index, spec.t[q].k, spec.t[q].base = (index.data_ptr() if index is not None else None), k_rows, base
-        spec.t[q].scale = scale[0] if scale else 1.0
     if places is not None and (places.dtype != torch.int32 or places.numel() != n * copies or out is None or out.numel() != n * copies * D):
         raise KernelError(f"add_rmsnorm: {n} rows in {copies} places each need int32 places and an output of so many rows")
     _contig(places)

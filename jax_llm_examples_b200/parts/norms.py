@@ -32,10 +32,11 @@ class RMSNorm(Norm):
         # a sum of terms (an expert layer's rows still in expert order) is added term by term in the kernel
         # (the kernel takes so many terms, rows per token and partials; beyond that the sum is made by its producer)
         if isinstance(delta, RowSum) and len(delta.terms) <= K.DELTA_MAX_TERMS and all(t.k <= 16 and t.weights is None for t in delta.terms) and \
+                len({t.scale for t in delta.terms}) <= 1 and \
                 sum((t.k if t.index is not None else 1) * t.splits for t in delta.terms) <= K.DELTA_MAX_STREAMS:
-            terms = [(t.data, t.splits, t.index, t.k, t.base, t.scale) for t in delta.terms]
+            terms, scale = [(t.data, t.splits, t.index, t.k, t.base) for t in delta.terms], delta.terms[0].scale if delta.terms else 1.0
         else:
-            d = as_rows(delta)
+            d, scale = as_rows(delta), 1.0
             terms = None if d is None else [(d.data, d.splits, None, 1, 0)]
         routing = None
         w_router = idx = wt = None
@@ -57,7 +58,7 @@ class RMSNorm(Norm):
                 and out_dtype == torch.bfloat16 and n <= K.DISPATCH_MAX_ROWS and n * k <= K.DISPATCH_MAX_PAIRS:
             dispatch = offer[0](ctx, n)
         did = K.add_rmsnorm(x, terms, self.weight, self.eps, out, out32, row_index, 1, None if unfused else w_router, idx, wt,
-                            dispatch, None if places is None else places.index, copies)
+                            dispatch, None if places is None else places.index, copies, scale)
         if did:
             routing = (idx, wt, dispatch)
         if unfused:

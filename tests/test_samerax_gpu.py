@@ -205,7 +205,7 @@ def test_biased_projections_turned_and_laid_side_by_side(dtype, H_, G, d, dv, dp
 @pytest.mark.parametrize("out_dtype", [torch.float32, torch.bfloat16])
 @pytest.mark.parametrize("N, D, copies, k, splits", [(3, 36, 2, 3, 1), (5, 2048, 4, 2, 3), (40, 1024, 1, 1, 2), (17, 200, 16, 4, 1), (2, 30, 3, 5, 2), (70, 4096, 2, 2, 1)])
 def test_the_norm_writes_its_rows_where_they_are_wanted(out_dtype, N, D, copies, k, splits):
-    """x += scale * (the sum of a token's rows in expert order) + a second term; the normed row goes to all its places, in the
+    """x += scale * (the sum of a token's rows in expert order + a second term); the normed row goes to all its places, in the
     one-block kernel and in the cluster kernel of a decode step."""
     from jax_llm_examples_b200.kernels import api as K
 
@@ -213,8 +213,8 @@ def test_the_norm_writes_its_rows_where_they_are_wanted(out_dtype, N, D, copies,
     x, y, z = torch.randn(N, D, device=DEV), torch.randn(splits, N * k, D, device=DEV), torch.randn(N, D, device=DEV)
     idx, places = (torch.randperm(N * m).to(torch.int32).to(DEV) for m in (k, copies))
     w, out = torch.randn(D, device=DEV), torch.full((N * copies, D), float("nan"), device=DEV, dtype=out_dtype)
-    ref = x.double() + y.double().sum(0)[idx.long()].view(N, k, D).sum(1) / k + z.double()
-    K.add_rmsnorm(x, [(y, splits, idx, k, 0, 1.0 / k), (z, 1, None, 1, 0)], w, 1e-5, out, places=places, copies=copies)
+    ref = x.double() + y.double().sum(0)[idx.long()].view(N, k, D).sum(1) / k + z.double() / k
+    K.add_rmsnorm(x, [(y, splits, idx, k, 0), (z, 1, None, 1, 0)], w, 1e-5, out, places=places, copies=copies, delta_scale=1.0 / k)
     _close(x, ref, 2e-6, "residual")
     normed = plain.rms_norm(ref, w.double(), 1e-5)
     _close(out[places.long()].view(N, copies, D), normed[:, None].expand(N, copies, D), 2e-6 if out_dtype == torch.float32 else 5e-3, "rows")
